@@ -7,10 +7,11 @@ from .mefepel import MefepelConfig
 from .zebovik import ZebovikConfig
 from .rarevik import RarevikConfig
 from .gatosun import GatosunConfig
+from .dapupel import DapupelConfig
 from .presets import preset_config, preset_dict, preset_names
 
 __all__ = [
     "resolve_dtype", "ModelConfig", "config_class_for", "config_from_dict", "load_config", "register_architecture",
-    "registered_architectures", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen2Config", "MefepelConfig", "ZebovikConfig", "RarevikConfig", "GatosunConfig",
+    "registered_architectures", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen2Config", "MefepelConfig", "ZebovikConfig", "RarevikConfig", "GatosunConfig", "DapupelConfig",
     "preset_config", "preset_dict", "preset_names",
 ]

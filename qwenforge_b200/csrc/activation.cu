@@ -132,6 +132,73 @@ QF_EXPORT int qf_scaled_swiglu(int is_bf16, const void* gu, const float* row_sca
     return (int)launch_pdl(scaled_swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, row_scale, (float*)out, inter, total);
 }
 
+// The clamped gate on rows whose input was to be scaled: both halves of the UNSCALED rows' product times s_r, then clamped.
+template <typename T>
+__global__ void scaled_clamped_glu_kernel(const T* __restrict__ gu, const float* __restrict__ row_scale, T* __restrict__ out, int inter,
+                                          size_t total, float limit, float alpha) {
+    grid_chain_entry();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / inter, c = i % inter;
+        const float s = row_scale[t];
+        const float g = fminf(s * Num<T>::to_f(gu[t * 2 * inter + c]), limit);
+        const float u = fminf(fmaxf(s * Num<T>::to_f(gu[t * 2 * inter + inter + c]), -limit), limit);
+        out[i] = Num<T>::from_f(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+    }
+}
+
+QF_EXPORT int qf_scaled_clamped_glu(int is_bf16, const void* gu, const float* row_scale, void* out, int rows, int inter, float limit,
+                                    float alpha, cudaStream_t stream) {
+    const size_t total = (size_t)rows * inter;
+    if (total == 0) return 0;
+    const size_t most = (size_t)(qf_sm_count() > 0 ? qf_sm_count() : 1) * 16;
+    const int blocks = (int)((total + 255) / 256 < most ? (total + 255) / 256 : most);
+    if (is_bf16)
+        return (int)launch_pdl(scaled_clamped_glu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, row_scale, (bf16*)out,
+                               inter, total, limit, alpha);
+    return (int)launch_pdl(scaled_clamped_glu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, row_scale, (float*)out,
+                           inter, total, limit, alpha);
+}
+
+// A gate per element, in place: x[t][c] *= sigmoid(gate[t][c]). Rows of x are contiguous, rows of the gate may be strided.
+template <typename T>
+__global__ void sigmoid_gate_kernel(T* __restrict__ x, const T* __restrict__ gate, long long gate_stride, int width, size_t total) {
+    grid_chain_entry();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = Num<T>::from_f(Num<T>::to_f(x[i]) / (1.0f + expf(-Num<T>::to_f(gate[i / width * gate_stride + i % width]))));
+}
+
+// Eight bf16 elements per thread: width and gate_stride multiples of 8, 16-byte aligned bases.
+__global__ void sigmoid_gate_bf16x8_kernel(bf16* __restrict__ x, const bf16* __restrict__ gate, long long gate_stride, int width, size_t total8) {
+    grid_chain_entry();
+    const int per_row = width / 8;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total8; i += (size_t)gridDim.x * blockDim.x) {
+        uint4 x4 = *reinterpret_cast<const uint4*>(x + i * 8);
+        const uint4 g4 = *reinterpret_cast<const uint4*>(gate + i / per_row * gate_stride + i % per_row * 8);
+        __nv_bfloat162* x2 = reinterpret_cast<__nv_bfloat162*>(&x4);
+        const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&g4);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 v = __bfloat1622float2(x2[j]), g = __bfloat1622float2(g2[j]);
+            x2[j] = __floats2bfloat162_rn(v.x / (1.0f + expf(-g.x)), v.y / (1.0f + expf(-g.y)));
+        }
+        *reinterpret_cast<uint4*>(x + i * 8) = x4;
+    }
+}
+
+QF_EXPORT int qf_sigmoid_gate(int is_bf16, void* x, const void* gate, long long gate_stride, int rows, int width, cudaStream_t stream) {
+    const size_t total = (size_t)rows * width;
+    if (total == 0) return 0;
+    const size_t most = (size_t)(qf_sm_count() > 0 ? qf_sm_count() : 1) * 16;
+    if (is_bf16 && width % 8 == 0 && gate_stride % 8 == 0 && ((uintptr_t)x | (uintptr_t)gate) % 16 == 0) {
+        const size_t want = (total / 8 + 255) / 256;
+        return (int)launch_pdl(sigmoid_gate_bf16x8_kernel, dim3((unsigned)(want < most ? want : most)), dim3(256), 0, stream, (bf16*)x,
+                               (const bf16*)gate, gate_stride, width, total / 8);
+    }
+    const dim3 grid((unsigned)((total + 255) / 256 < most ? (total + 255) / 256 : most));
+    if (is_bf16) return (int)launch_pdl(sigmoid_gate_kernel<bf16>, grid, dim3(256), 0, stream, (bf16*)x, (const bf16*)gate, gate_stride, width, total);
+    return (int)launch_pdl(sigmoid_gate_kernel<float>, grid, dim3(256), 0, stream, (float*)x, (const float*)gate, gate_stride, width, total);
+}
+
 // out = act(x + bias): the first half of a feed-forward without a gate. kind 0: the square of relu, 1: tanh-GELU,
 // 2: silu, 3: relu, 4: GELU in its exact form, z Phi(z) through erf, 5: tanh. Float32 inside; bias may be null.
 

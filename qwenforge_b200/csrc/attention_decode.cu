@@ -22,6 +22,8 @@
 // no value; it is added where a row's runs come together (not with fold_later: the caller's fold knows no sinks).
 // `shared_values`: the values are the keys themselves (pages of one plane, as a latent attention keeps them): half a
 // page is fetched once and read as both.
+// `bias_scale`, `bias_rate` (float32 per query head, or null): after the cap a score of the key `far` positions back loses
+// bias_scale[h] * ln(1 + bias_rate[h] * far), with the hardware's base-2 logarithm; compiled as a variant of its own.
 #include <algorithm>
 
 #include "tma.cuh"
@@ -103,13 +105,14 @@ decode_plan_kernel(const int* __restrict__ cu_q, const int* __restrict__ tok_pos
     for (int j = before + lane; j < n_pairs; j += 32) plan[j] = make_int4(-1, 0, 0, -1);
 }
 
-template <int D, int WARPS, bool TMA>
+template <int D, int WARPS, bool TMA, bool BIASED>
 __global__ void __launch_bounds__(WARPS * 32)
 decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __restrict__ q, bf16* __restrict__ out,
                     const int* __restrict__ cu_q, const int4* __restrict__ plan, KvSite<bf16> site, int n_heads, int chunks, float scale_log2,
                     int window, int mask_block, float cap_in, float cap_out, int max_splits, int n_seqs, int fold_later, float* __restrict__ part_o,
                     float* __restrict__ part_ml, int* __restrict__ counters, int* err, unsigned long long* stamps,
-                    const float* __restrict__ sinks, int shared_values) {
+                    const float* __restrict__ sinks, int shared_values, const float* __restrict__ bias_scale,
+                    const float* __restrict__ bias_rate) {
     constexpr int DEC_WARPS = WARPS, DEC_THREADS = WARPS * 32;
     // measuring aid: if `stamps` is given, thread 0 leaves nanosecond time stamps of the block's phases in stamps[block][8]
     auto stamp = [&](int phase) {
@@ -166,7 +169,16 @@ decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __re
     int lo = window > 0 ? max(0, L - window) : 0;
     if (mask_block > 0) lo = max(lo, (L - 1) / mask_block * mask_block);   // the new token's block of the mask
     // capped scores: s <- cap * tanh(s * scale / cap) in base-2 units (cap_in = scale / cap, cap_out = cap * log2(e))
-    const float sl2 = cap_out > 0.f ? 1.f : scale_log2;
+    const float sl2 = cap_out > 0.f || BIASED ? 1.f : scale_log2;
+    float by[2] = {0.f, 0.f}, rate[2] = {0.f, 0.f};   // the distance bias of this lane's two heads (weights: no wait needed)
+    if constexpr (BIASED) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int row = (threadIdx.x & 31) / 4 + 8 * r;
+            by[r] = row < n_g ? bias_scale[head0 + row] : 0.f;
+            rate[r] = row < n_g ? bias_rate[head0 + row] : 0.f;
+        }
+    }
     const int first_page = lo / QF_PAGE, last_page = (L - 1) / QF_PAGE;
     const int pps = (last_page - first_page + n_splits) / n_splits;  // ceil(pages / splits)
     const int p_begin = first_page + split * pps, p_end = min(p_begin + pps, last_page + 1);
@@ -308,6 +320,16 @@ decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __re
                         float y;
                         asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(s[t][e] * cap_in));
                         s[t][e] = cap_out * y;
+                    }
+            }
+            if constexpr (BIASED) {
+                const float raw = cap_out > 0.f ? 1.f : scale_log2;
+#pragma unroll
+                for (int t = 0; t < 4; ++t)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float far = (float)(L - 1 - (key0 + 8 * t + 2 * (lane & 3) + (e & 1)));
+                        s[t][e] = fmaf(-by[e >> 1], __log2f(fmaf(rate[e >> 1], fmaxf(far, 0.f), 1.f)), s[t][e] * raw);
                     }
             }
             const bool full = key0 >= lo && key0 + HALF <= L;  // every key of the half is visible
@@ -560,7 +582,7 @@ template <int D>
 static int resident_blocks() {
     static int held = -1;
     if (held < 0) {
-        auto kernel = decode_split_kernel<D, decode_warps(D), decode_tma(D)>;
+        auto kernel = decode_split_kernel<D, decode_warps(D), decode_tma(D), false>;
         int n = 0;
         if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(D)) != cudaSuccess ||
             cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, kernel, decode_warps(D) * 32, decode_smem(D)) != cudaSuccess)
@@ -596,17 +618,17 @@ QF_EXPORT int qf_attention_decode_warps(int head_dim) {
     return head_dim == 32 || head_dim == 64 || head_dim == 96 || head_dim == 128 ? decode_warps(head_dim) : 0;
 }
 
-template <int D>
+template <int D, bool BIASED>
 static int launch(const void* q, void* out, const int* cu_q, const int4* plan, void* base, const int* table,
                   long long page_elems, int table_stride, int kv_heads, int n_heads, int n_seqs, float scale, int window,
                   int n_splits, int fold_later, float* part_o, float* part_ml, int* counters, int* err,
                   unsigned long long* stamps, const float* sinks, int shared_values, int mask_block, float softcap,
-                  cudaStream_t stream) {
+                  const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
     constexpr int WARPS = decode_warps(D);
     constexpr bool TMA = decode_tma(D);
     const int G = n_heads / kv_heads, chunks = (G + 15) / 16;
     const size_t smem = decode_smem(D);
-    cudaError_t e = cudaFuncSetAttribute(decode_split_kernel<D, WARPS, TMA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(decode_split_kernel<D, WARPS, TMA, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     KvSite<bf16> site{(bf16*)base, table, page_elems, table_stride, kv_heads, D};
     CUtensorMap kv_map = {};
@@ -616,10 +638,10 @@ static int launch(const void* q, void* out, const int* cu_q, const int4* plan, v
         if (!qf_make_map_bf16(&kv_map, base, 1ll << 31, D, D, QF_PAGE / 2)) return (int)cudaErrorNotSupported;
     }
     dim3 grid((unsigned)(plan_pairs(n_seqs, kv_heads, n_heads, D, n_splits) * kv_heads * chunks));
-    return (int)launch_pdl(decode_split_kernel<D, WARPS, TMA>, grid, dim3(WARPS * 32), smem, stream, kv_map, (const bf16*)q,
+    return (int)launch_pdl(decode_split_kernel<D, WARPS, TMA, BIASED>, grid, dim3(WARPS * 32), smem, stream, kv_map, (const bf16*)q,
                            (bf16*)out, cu_q, plan, site, n_heads, chunks, scale * 1.4426950408889634f, window, mask_block,
                            softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, n_splits,
-                           n_seqs, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values);
+                           n_seqs, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values, bias_scale, bias_rate);
 }
 
 // How many 16-byte units a plan of this shape holds (what qf_attention_decode_plan writes and qf_attention_decode
@@ -657,15 +679,16 @@ static int decode_run(const void* q, void* out, const int* cu_q, const void* pla
                       long long page_elems, int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
                       float scale, int window, int n_splits, int fold_later, float* part_o, float* part_ml, int* counters,
                       int* err, unsigned long long* stamps, const float* sinks, int shared_values, cudaStream_t stream,
-                      int mask_block = 0, float softcap = 0.f) {
+                      int mask_block = 0, float softcap = 0.f, const float* bias_scale = nullptr, const float* bias_rate = nullptr) {
     if (n_seqs <= 0) return 0;
     if (kv_heads <= 0 || n_heads % kv_heads || n_splits < 1 || !plan || (fold_later && sinks)) return (int)cudaErrorInvalidValue;
     if (fold_later ? (!part_o || !part_ml) : !out) return (int)cudaErrorInvalidValue;
-#define QF_CASE(DIM)                                                                                                   \
-    case DIM:                                                                                                          \
-        return launch<DIM>(q, out, cu_q, (const int4*)plan, base, table, page_elems, table_stride, kv_heads, n_heads, \
-                           n_seqs, scale, window, n_splits, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values,   \
-                           mask_block, softcap, stream);
+#define QF_DECODE_ARGS q, out, cu_q, (const int4*)plan, base, table, page_elems, table_stride, kv_heads, n_heads, n_seqs, scale, window, \
+                       n_splits, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values, mask_block, softcap,       \
+                       bias_scale, bias_rate, stream
+#define QF_CASE(DIM) \
+    case DIM:        \
+        return bias_scale ? launch<DIM, true>(QF_DECODE_ARGS) : launch<DIM, false>(QF_DECODE_ARGS);
     switch (head_dim) {
         QF_CASE(32)
         QF_CASE(64)
@@ -675,6 +698,7 @@ static int decode_run(const void* q, void* out, const int* cu_q, const void* pla
             return (int)cudaErrorInvalidValue;
     }
 #undef QF_CASE
+#undef QF_DECODE_ARGS
 }
 
 QF_EXPORT int qf_attention_decode(const void* q, void* out, const int* cu_q, const void* plan, void* base,
@@ -706,6 +730,19 @@ QF_EXPORT int qf_attention_decode_masked(const void* q, void* out, const int* cu
     return decode_run(q, out, cu_q, plan, base, table, page_elems, table_stride, kv_heads, head_dim, n_heads, n_seqs, scale,
                       window, n_splits, fold_later, part_o, part_ml, counters, err, nullptr, sinks, shared_values, stream,
                       mask_block, softcap);
+}
+
+// And with a distance bias: bias_scale, bias_rate float32 [n_heads] each, both or neither (see the top of the file).
+QF_EXPORT int qf_attention_decode_biased(const void* q, void* out, const int* cu_q, const void* plan, void* base,
+                                         const int* table, long long page_elems, int table_stride, int kv_heads, int head_dim,
+                                         int n_heads, int n_seqs, float scale, int window, int n_splits, int fold_later,
+                                         float* part_o, float* part_ml, int* counters, int* err, const float* sinks,
+                                         int shared_values, int mask_block, float softcap, const float* bias_scale,
+                                         const float* bias_rate, cudaStream_t stream) {
+    if (!bias_scale != !bias_rate) return (int)cudaErrorInvalidValue;
+    return decode_run(q, out, cu_q, plan, base, table, page_elems, table_stride, kv_heads, head_dim, n_heads, n_seqs, scale,
+                      window, n_splits, fold_later, part_o, part_ml, counters, err, nullptr, sinks, shared_values, stream,
+                      mask_block, softcap, bias_scale, bias_rate);
 }
 
 // A measuring aid: the same launch, with every block's thread 0 writing nanosecond time stamps to stamps[block][8]:

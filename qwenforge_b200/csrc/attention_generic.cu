@@ -24,6 +24,9 @@
 // they come from a second cache that holds one row per block (`blocks`), are walked first, in tiles of 32 rows from row
 // 0, and share the softmax with the window's keys.
 //
+// A fourth: a distance bias (`bias_scale`, `bias_rate`: float32, one per query head, or null). After the cap a score of key j
+// under query i loses bias_scale[h] * ln(1 + bias_rate[h] * (i - j)).
+//
 // Steps of one token per sequence (decoding) give only sequences x kv heads blocks, each walking a whole sequence. For
 // them the keys are cut into chunks of GEN_CHUNK positions at absolute multiples of GEN_CHUNK: a block per (sequence,
 // kv head, chunk) leaves its rows' maximum, sum and unnormalised output in scratch, and a second kernel folds a row's
@@ -60,7 +63,8 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const int
                          const int* __restrict__ tok_pos, const int* __restrict__ slots, KvSite<T> site, int n_heads,
                          int group_chunk, int tokens_per_tile, float scale, int window, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int* err, const float* __restrict__ sinks, int shared_values, int mask_block,
-                         float softcap, KvSite<T> blocks, int pool) {
+                         float softcap, KvSite<T> blocks, int pool, const float* __restrict__ bias_scale,
+                         const float* __restrict__ bias_rate) {
     extern __shared__ float smem[];
     const int D = site.head_dim, G = n_heads / site.kv_heads;
     const int chunks = (G + group_chunk - 1) / group_chunk;
@@ -162,6 +166,10 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const int
             for (int d = 0; d < D; ++d) s = fmaf(qr[d], kr[d], s);
             s *= scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            if (bias_scale && kj <= row_pos[i]) {
+                const int h = kvh * G + g0 + r % n_g;
+                s -= bias_scale[h] * log1pf(bias_rate[h] * (float)(row_pos[i] - kj));
+            }
             const bool visible = kj <= hi && kj >= lo;
             s = visible ? s : -FLT_MAX;
             const float m_new = fmaxf(m[i], warp_max(s));
@@ -254,9 +262,9 @@ static int launch(const void* q, void* out, const int* cu_q, const int* tok_pos,
                   const int* table, long long page_elems, int table_stride, int kv_heads, int head_dim, int n_heads,
                   int n_seqs, int max_q_len, float scale, int window, int* err, const float* sinks, int shared_values,
                   int chunk, float softcap, void* blocks_base, const int* blocks_table, long long blocks_page_elems,
-                  int blocks_table_stride, int pool, cudaStream_t stream) {
+                  int blocks_table_stride, int pool, const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
-    if (pool > 0 && (!blocks_base || !blocks_table || window <= 0 || shared_values)) return (int)cudaErrorInvalidValue;
+    if (pool > 0 && (!blocks_base || !blocks_table || window <= 0 || shared_values || bias_scale)) return (int)cudaErrorInvalidValue;
     if (head_dim > 32 * MAX_DPL || kv_heads <= 0 || n_heads % kv_heads) return (int)cudaErrorInvalidValue;
     const int G = n_heads / kv_heads;
     const int group_chunk = G < MAX_ROWS ? G : MAX_ROWS;
@@ -272,7 +280,7 @@ static int launch(const void* q, void* out, const int* cu_q, const int* tok_pos,
     attention_generic_kernel<T, false, MAX_DPL><<<grid, WARPS * 32, smem, stream>>>(
         (const T*)q, (T*)out, cu_q, tok_pos, slots, site, n_heads, group_chunk, tokens_per_tile, scale, window, nullptr, nullptr,
         err, sinks, shared_values, chunk, softcap,
-        KvSite<T>{(T*)blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, kv_heads, head_dim}, pool);
+        KvSite<T>{(T*)blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, kv_heads, head_dim}, pool, bias_scale, bias_rate);
     return (int)cudaGetLastError();
 }
 
@@ -280,7 +288,8 @@ template <typename T, int MAX_DPL>
 static int launch_decode(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots, void* base,
                          const int* table, long long page_elems, int table_stride, int kv_heads, int head_dim, int n_heads,
                          int n_seqs, int max_kv_len, float scale, int window, float* part_o, float* part_ml, int* err,
-                         const float* sinks, int shared_values, int chunk, float softcap, cudaStream_t stream) {
+                         const float* sinks, int shared_values, int chunk, float softcap, const float* bias_scale,
+                         const float* bias_rate, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (head_dim > 32 * MAX_DPL || kv_heads <= 0 || n_heads % kv_heads || max_kv_len <= 0) return (int)cudaErrorInvalidValue;
     const int G = n_heads / kv_heads;
@@ -294,7 +303,7 @@ static int launch_decode(const void* q, void* out, const int* cu_q, const int* t
     KvSite<T> site{(T*)base, table, page_elems, table_stride, kv_heads, head_dim};
     attention_generic_kernel<T, true, MAX_DPL><<<dim3(n_chunks, kv_heads * chunks, n_seqs), WARPS * 32, smem, stream>>>(
         (const T*)q, (T*)out, cu_q, tok_pos, slots, site, n_heads, group_chunk, 1, scale, window, part_o, part_ml, err, nullptr,
-        shared_values, chunk, softcap, KvSite<T>{nullptr, nullptr, 0, 0, kv_heads, head_dim}, 0);
+        shared_values, chunk, softcap, KvSite<T>{nullptr, nullptr, 0, 0, kv_heads, head_dim}, 0, bias_scale, bias_rate);
     e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     attention_generic_fold_kernel<T><<<dim3(n_heads, n_seqs), 64, 0, stream>>>((T*)out, cu_q, tok_pos, slots, n_heads, head_dim,
@@ -313,6 +322,20 @@ static int launch_decode(const void* q, void* out, const int* cu_q, const int* t
 // chunk: > 0 limits a query to the keys of its own block of that many positions; softcap: > 0 caps the scores.
 // pool > 0: rows of whole blocks of `pool` positions, kept in a second cache of the same head shape (blocks_*), join the
 // window's keys (see the top of the file).
+// bias_scale, bias_rate: the distance bias, float32 [n_heads] each, both or neither (not with rows of whole blocks).
+QF_EXPORT int qf_attention_generic_biased(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,
+                                          const int* slots, void* base, const int* table, long long page_elems,
+                                          int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
+                                          int max_q_len, float scale, int window, int* err, const float* sinks,
+                                          int shared_values, int chunk, float softcap, void* blocks_base,
+                                          const int* blocks_table, long long blocks_page_elems, int blocks_table_stride, int pool,
+                                          const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
+    if (!bias_scale != !bias_rate) return (int)cudaErrorInvalidValue;
+    QF_GENERIC_DISPATCH(launch, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, head_dim,
+                        n_heads, n_seqs, max_q_len, scale, window, err, sinks, shared_values, chunk, softcap, blocks_base,
+                        blocks_table, blocks_page_elems, blocks_table_stride, pool, bias_scale, bias_rate, stream)
+}
+
 QF_EXPORT int qf_attention_generic_pooled(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,
                                           const int* slots, void* base, const int* table, long long page_elems,
                                           int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
@@ -320,9 +343,9 @@ QF_EXPORT int qf_attention_generic_pooled(int is_bf16, const void* q, void* out,
                                           int shared_values, int chunk, float softcap, void* blocks_base,
                                           const int* blocks_table, long long blocks_page_elems, int blocks_table_stride, int pool,
                                           cudaStream_t stream) {
-    QF_GENERIC_DISPATCH(launch, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, head_dim,
-                        n_heads, n_seqs, max_q_len, scale, window, err, sinks, shared_values, chunk, softcap, blocks_base,
-                        blocks_table, blocks_page_elems, blocks_table_stride, pool, stream)
+    return qf_attention_generic_biased(is_bf16, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads,
+                                       head_dim, n_heads, n_seqs, max_q_len, scale, window, err, sinks, shared_values, chunk, softcap,
+                                       blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, pool, nullptr, nullptr, stream);
 }
 
 QF_EXPORT int qf_attention_generic_masked(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,
@@ -355,14 +378,27 @@ QF_EXPORT int qf_attention_generic(int is_bf16, const void* q, void* out, const 
 // The same for a step of ONE token per sequence, cut into chunks of keys (see the top of the file). `max_kv_len`: an
 // upper bound of any sequence's length after the step; scratch: part_o float32 [n_seqs * n_heads * n_chunks * head_dim],
 // part_ml float32 [n_seqs * n_heads * n_chunks * 2] with n_chunks = ceil(max_kv_len / 256).
+QF_EXPORT int qf_attention_generic_decode_biased(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,
+                                                 const int* slots, void* base, const int* table, long long page_elems,
+                                                 int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
+                                                 int max_kv_len, float scale, int window, float* part_o, float* part_ml, int* err,
+                                                 const float* sinks, int shared_values, int chunk, float softcap,
+                                                 const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
+    if (!bias_scale != !bias_rate) return (int)cudaErrorInvalidValue;
+    QF_GENERIC_DISPATCH(launch_decode, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, head_dim,
+                        n_heads, n_seqs, max_kv_len, scale, window, part_o, part_ml, err, sinks, shared_values, chunk, softcap, bias_scale,
+                        bias_rate, stream)
+}
+
 QF_EXPORT int qf_attention_generic_decode_masked(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,
                                                  const int* slots, void* base, const int* table, long long page_elems,
                                                  int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
                                                  int max_kv_len, float scale, int window, float* part_o, float* part_ml, int* err,
                                                  const float* sinks, int shared_values, int chunk, float softcap,
                                                  cudaStream_t stream) {
-    QF_GENERIC_DISPATCH(launch_decode, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, head_dim,
-                        n_heads, n_seqs, max_kv_len, scale, window, part_o, part_ml, err, sinks, shared_values, chunk, softcap, stream)
+    return qf_attention_generic_decode_biased(is_bf16, q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads,
+                                              head_dim, n_heads, n_seqs, max_kv_len, scale, window, part_o, part_ml, err, sinks,
+                                              shared_values, chunk, softcap, nullptr, nullptr, stream);
 }
 
 QF_EXPORT int qf_attention_generic_decode_ex(int is_bf16, const void* q, void* out, const int* cu_q, const int* tok_pos,

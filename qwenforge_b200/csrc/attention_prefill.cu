@@ -18,6 +18,9 @@
 // positions that lies wholly before its window (blocks b with b * pool + pool - 1 <= p - window). Those rows live in a
 // second cache of the same head shape, one row per block (`blocks`); its pages are walked first, by the same loop and the
 // same buffers, masked by how many blocks each row sees, and share the softmax with the window's keys.
+// `bias_scale`, `bias_rate` (float32 per query head, or null): after the cap a score of key j under query i loses
+// bias_scale[h] * ln(1 + bias_rate[h] * (i - j)), with the hardware's base-2 logarithm on the float32 argument; compiled as a
+// variant of its own.
 #include "mma.cuh"
 
 #define PF_WARPS 4
@@ -30,13 +33,13 @@ __device__ __forceinline__ float fast_tanh(float x) {
     return y;
 }
 
-template <int D, int G, bool POOLED>
+template <int D, int G, bool POOLED, bool BIASED>
 __global__ void __launch_bounds__(PF_THREADS * G, (D <= 64 ? 4 : 2) / G)
 prefill_flash_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, const int* __restrict__ cu_q,
                      const int* __restrict__ tok_pos, const int* __restrict__ slots, KvSite<bf16> site, int n_heads,
                      int n_seqs, int n_tiles, int wave, float scale_log2, int window, int* err,
                      const float* __restrict__ sinks, int shared_values, int mask_block, float cap_in, float cap_out,
-                     KvSite<bf16> blocks, int pool) {
+                     KvSite<bf16> blocks, int pool, const float* __restrict__ bias_scale, const float* __restrict__ bias_rate) {
     grid_chain_entry();
     auto seen_of = [&](int pos) -> int {   // blocks of `pool` positions wholly before the window of a query at `pos`
         const int past = pos - window + 1;
@@ -44,7 +47,7 @@ prefill_flash_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, const i
     };
     // capped scores: s <- cap * tanh(s * scale / cap) in base-2 units, cap_in = scale / cap, cap_out = cap * log2(e); the
     // capped score then needs no further scale
-    const float sl2 = cap_out > 0.f ? 1.f : scale_log2;
+    const float sl2 = cap_out > 0.f || BIASED ? 1.f : scale_log2;
     auto lo_of = [&](int pos) -> int {   // lowest position a query at `pos` sees: its window and its block of the mask
         int lo = window > 0 ? max(0, pos - window + 1) : 0;
         if (mask_block > 0) lo = max(lo, pos / mask_block * mask_block);
@@ -176,6 +179,16 @@ prefill_flash_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, const i
                 for (int t = 0; t < 8; ++t)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) s[t][e] = cap_out * fast_tanh(s[t][e] * cap_in);
+            }
+            if (BIASED) {   // in base-2 units: the factor log2(e) turns the natural logarithm into the base-2 one
+                const float by = bias_scale[head], rate = bias_rate[head], raw = cap_out > 0.f ? 1.f : scale_log2;
+#pragma unroll
+                for (int t = 0; t < 8; ++t)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float far = (float)(row_pos[e >> 1] - (key0 + 8 * t + 2 * (lane & 3) + (e & 1)));
+                        s[t][e] = fmaf(-by, __log2f(fmaf(rate, fmaxf(far, 0.f), 1.f)), s[t][e] * raw);
+                    }
             }
             const bool full = rows ? key0 + QF_PAGE <= seen_of(warp_first)
                                    : key0 + QF_PAGE - 1 <= warp_first && key0 >= lo_of(warp_last);
@@ -327,22 +340,24 @@ prefill_flash_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, const i
     }
 }
 
-template <int D, int G, bool POOLED>
+template <int D, int G, bool POOLED, bool BIASED>
 static int launch_groups(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots, KvSite<bf16> site,
                          int n_heads, int n_seqs, int max_q_len, float scale, int window, int* err, const float* sinks,
-                         int shared_values, int mask_block, float softcap, KvSite<bf16> block_rows, int pool, cudaStream_t stream) {
+                         int shared_values, int mask_block, float softcap, KvSite<bf16> block_rows, int pool,
+                         const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
     size_t smem = (size_t)4 * G * QF_PAGE * (D + 8) * sizeof(bf16);
     const size_t merge = (size_t)(G - 1) * PF_WARPS * (D / 8 * 4 + 4) * 32 * sizeof(float);
     if (smem < merge) smem = merge;
-    cudaError_t e = cudaFuncSetAttribute(prefill_flash_kernel<D, G, POOLED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_flash_kernel<D, G, POOLED, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     const int n_tiles = (max_q_len + PF_BM - 1) / PF_BM;
     const long long blocks = (long long)n_tiles * n_heads * n_seqs;
     if (blocks > 0x7fffffffll) return (int)cudaErrorInvalidValue;
-    return (int)launch_pdl(prefill_flash_kernel<D, G, POOLED>, dim3((unsigned)blocks), dim3(PF_THREADS * G), smem, stream, (const bf16*)q,
+    return (int)launch_pdl(prefill_flash_kernel<D, G, POOLED, BIASED>, dim3((unsigned)blocks), dim3(PF_THREADS * G), smem, stream, (const bf16*)q,
                            (bf16*)out, cu_q, tok_pos, slots, site, n_heads, n_seqs, n_tiles, qf_sm_count(),
                            scale * 1.4426950408889634f, window, err, sinks, shared_values, mask_block,
-                           softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, block_rows, pool);
+                           softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, block_rows, pool,
+                           bias_scale, bias_rate);
 }
 
 template <int D>
@@ -350,7 +365,8 @@ static int launch(const void* q, void* out, const int* cu_q, const int* tok_pos,
                   const int* table, long long page_elems, int table_stride, int kv_heads, int n_heads, int n_seqs,
                   int n_tokens, int max_q_len, int max_kv_len, float scale, int window, int* err, const float* sinks,
                   int shared_values, int mask_block, float softcap, void* blocks_base, const int* blocks_table,
-                  long long blocks_page_elems, int blocks_table_stride, int pool, cudaStream_t stream) {
+                  long long blocks_page_elems, int blocks_table_stride, int pool, const float* bias_scale,
+                  const float* bias_rate, cudaStream_t stream) {
     KvSite<bf16> site{(bf16*)base, table, page_elems, table_stride, kv_heads, D};
     KvSite<bf16> blocks{(bf16*)blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, kv_heads, D};
     // Two groups of warps per tile when tiles walk many pages and all tiles find room on the SMs at once (a short
@@ -365,9 +381,10 @@ static int launch(const void* q, void* out, const int* cu_q, const int* tok_pos,
     if (pool > 0) span += max_kv_len / pool;                      // the rows of the blocks before the window
     const bool split = span >= 8 * QF_PAGE && tiles < (long long)qf_sm_count() * (D <= 64 ? 4 : 2);
 #define QF_GROUPS_ARGS q, out, cu_q, tok_pos, slots, site, n_heads, n_seqs, max_q_len, scale, window, err, sinks, shared_values, mask_block, \
-                       softcap, blocks, pool, stream
-    if (pool > 0) return split ? launch_groups<D, 2, true>(QF_GROUPS_ARGS) : launch_groups<D, 1, true>(QF_GROUPS_ARGS);
-    return split ? launch_groups<D, 2, false>(QF_GROUPS_ARGS) : launch_groups<D, 1, false>(QF_GROUPS_ARGS);
+                       softcap, blocks, pool, bias_scale, bias_rate, stream
+    if (pool > 0) return split ? launch_groups<D, 2, true, false>(QF_GROUPS_ARGS) : launch_groups<D, 1, true, false>(QF_GROUPS_ARGS);
+    if (bias_scale) return split ? launch_groups<D, 2, false, true>(QF_GROUPS_ARGS) : launch_groups<D, 1, false, true>(QF_GROUPS_ARGS);
+    return split ? launch_groups<D, 2, false, false>(QF_GROUPS_ARGS) : launch_groups<D, 1, false, false>(QF_GROUPS_ARGS);
 #undef QF_GROUPS_ARGS
 }
 
@@ -379,20 +396,23 @@ static int launch(const void* q, void* out, const int* cu_q, const int* tok_pos,
 // scale) becomes softcap * tanh(s / softcap), with the hardware's approximate tanh.
 // pool > 0: the rows of whole blocks of `pool` positions, kept in a second cache of the same head shape (blocks_*), join
 // the window's keys (see the top of the file).
-QF_EXPORT int qf_attention_prefill_pooled(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots,
+// bias_scale, bias_rate: the distance bias, float32 [n_heads] each, both or neither (not with rows of whole blocks).
+QF_EXPORT int qf_attention_prefill_biased(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots,
                                           void* base, const int* table, long long page_elems, int table_stride, int kv_heads,
                                           int head_dim, int n_heads, int n_seqs, int n_tokens, int max_q_len, int max_kv_len,
                                           float scale, int window, int* err, const float* sinks, int shared_values,
                                           int mask_block, float softcap, void* blocks_base, const int* blocks_table,
-                                          long long blocks_page_elems, int blocks_table_stride, int pool, cudaStream_t stream) {
+                                          long long blocks_page_elems, int blocks_table_stride, int pool, const float* bias_scale,
+                                          const float* bias_rate, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
+    if (!bias_scale != !bias_rate || (pool > 0 && bias_scale)) return (int)cudaErrorInvalidValue;
     if (kv_heads <= 0 || n_heads % kv_heads) return (int)cudaErrorInvalidValue;
     if (pool > 0 && (!blocks_base || !blocks_table || window <= 0 || shared_values)) return (int)cudaErrorInvalidValue;
 #define QF_CASE(DIM)                                                                                                 \
     case DIM:                                                                                                        \
         return launch<DIM>(q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, n_heads,  \
                            n_seqs, n_tokens, max_q_len, max_kv_len, scale, window, err, sinks, shared_values, mask_block, softcap, \
-                           blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, pool, stream);
+                           blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, pool, bias_scale, bias_rate, stream);
     switch (head_dim) {
         QF_CASE(32)
         QF_CASE(64)
@@ -402,6 +422,18 @@ QF_EXPORT int qf_attention_prefill_pooled(const void* q, void* out, const int* c
             return (int)cudaErrorInvalidValue;
     }
 #undef QF_CASE
+}
+
+QF_EXPORT int qf_attention_prefill_pooled(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots,
+                                          void* base, const int* table, long long page_elems, int table_stride, int kv_heads,
+                                          int head_dim, int n_heads, int n_seqs, int n_tokens, int max_q_len, int max_kv_len,
+                                          float scale, int window, int* err, const float* sinks, int shared_values,
+                                          int mask_block, float softcap, void* blocks_base, const int* blocks_table,
+                                          long long blocks_page_elems, int blocks_table_stride, int pool, cudaStream_t stream) {
+    return qf_attention_prefill_biased(q, out, cu_q, tok_pos, slots, base, table, page_elems, table_stride, kv_heads, head_dim,
+                                       n_heads, n_seqs, n_tokens, max_q_len, max_kv_len, scale, window, err, sinks, shared_values,
+                                       mask_block, softcap, blocks_base, blocks_table, blocks_page_elems, blocks_table_stride, pool,
+                                       nullptr, nullptr, stream);
 }
 
 QF_EXPORT int qf_attention_prefill_masked(const void* q, void* out, const int* cu_q, const int* tok_pos, const int* slots,

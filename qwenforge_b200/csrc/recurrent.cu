@@ -629,14 +629,37 @@ QF_EXPORT int qf_gated_group_norm(int is_bf16, const float* y, const void* gate,
 // the step's last taps - 1 inputs into the state, a thread per (sequence, channel), reading all it needs before it writes.
 // In a step of ONE token per sequence (`single`) a channel's kept inputs have one reader, the thread of that token and
 // channel, which then moves them itself: no second kernel.
+// CACHED: channels from `tail` on are keys (and values): they are not stored beside the others but written to the token's own
+// position in the paged cache, head after head (keys, then values where the pages hold both); `out` then has rows of `tail`
+// channels. What a layer without norm and rotation has between its projections and its attention is this one launch.
 #define CONV_MAX_TAPS 16
 
+template <typename T> struct ConvCache {
+    KvSite<T> site;
+    const int* tok_pos;
+    int tail;
+    int* err;
+};
+
+// Where channel c (>= tail) of a token belongs; nullptr where nothing is to be written.
 template <typename T>
+__device__ __forceinline__ T* conv_cache_place(const ConvCache<T>& cache, int slot, int t, int c) {
+    if (slot < 0) return nullptr;
+    const int head = (c - cache.tail) / cache.site.head_dim, d = (c - cache.tail) % cache.site.head_dim;
+    T* row = kv_row(cache.site, slot, cache.tok_pos[t], head, 0);
+    if (!row) {
+        atomicOr(cache.err, QF_ERR_NO_PAGE);
+        return nullptr;
+    }
+    return row + d;
+}
+
+template <typename T, bool CACHED>
 __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ weight,
                                         const float* __restrict__ bias, const int* __restrict__ cu_q,
                                         const int* __restrict__ tok_seq, const int* __restrict__ slots,
                                         float* __restrict__ state, long long slot_stride, long long offset, int taps,
-                                        int n_tokens, int channels, T* __restrict__ out, int plain, int single) {
+                                        int n_tokens, int channels, T* __restrict__ out, int plain, int single, ConvCache<T> cache) {
     grid_chain_entry();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)n_tokens * channels) return;
@@ -654,7 +677,9 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, c
         if (single && before && back >= 1 && back < taps - 1) before[(size_t)(taps - 2 - back) * channels + c] = u;
     }
     if (single && before && taps > 1) before[(size_t)(taps - 2) * channels + c] = Num<T>::to_f(x[(size_t)t * x_stride + c]);
-    out[(size_t)t * channels + c] = Num<T>::from_f(plain ? z : z / (1.f + expf(-z)));
+    T* dst = out + (size_t)t * channels + c;
+    if (CACHED) dst = c < cache.tail ? out + (size_t)t * cache.tail + c : conv_cache_place(cache, slot, t, c);
+    if (!CACHED || dst) *dst = Num<T>::from_f(plain ? z : z / (1.f + expf(-z)));
 }
 
 // The same convolution for long steps: a thread takes 16 bytes of channels and a run of CONV_RUN(TAPS) consecutive tokens, keeps
@@ -664,12 +689,12 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, c
 // tokens of a run: the more taps, the more a longer run saves (taps - 1 inputs are fetched again at the start of every run)
 #define CONV_RUN(TAPS) ((TAPS) >= 4 ? 8 : 4)
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool CACHED>
 __global__ void __launch_bounds__(128)
 causal_conv_run_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ weight, const float* __restrict__ bias,
                        const int* __restrict__ cu_q, const int* __restrict__ tok_seq, const int* __restrict__ slots,
                        const float* __restrict__ state, long long slot_stride, long long offset, int n_tokens, int channels,
-                       T* __restrict__ out, int plain) {
+                       T* __restrict__ out, int plain, ConvCache<T> cache) {
     constexpr int V = 16 / (int)sizeof(T);
     constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
     grid_chain_entry();
@@ -723,7 +748,9 @@ causal_conv_run_kernel(const T* __restrict__ x, int x_stride, const float* __res
             for (int r = 0; r + 1 < TAPS - 1; ++r) hist[r][v] = hist[r + 1][v];
             if (TAPS > 1) hist[H - 1][v] = u;
         }
-        *reinterpret_cast<uint4*>(out + (size_t)t * channels + c0) = *reinterpret_cast<const uint4*>(res);
+        T* dst = out + (size_t)t * channels + c0;
+        if (CACHED) dst = c0 < cache.tail ? out + (size_t)t * cache.tail + c0 : conv_cache_place(cache, slots[seq], t, c0);
+        if (!CACHED || dst) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(res);
     }
 }
 
@@ -746,27 +773,28 @@ __global__ void conv_state_kernel(const T* __restrict__ x, int x_stride, const i
     for (int r = 0; r < taps - 1; ++r) kept[(size_t)r * channels + c] = next[r];
 }
 
-template <typename T>
+template <typename T, bool CACHED>
 static int launch_conv(const void* x, int x_stride, const float* weight, const float* bias, const int* cu_q, const int* tok_seq,
                        const int* slots, int n_seqs, float* state, long long slot_stride, long long offset, int taps,
-                       int n_tokens, int channels, void* out, int plain, int single, cudaStream_t stream) {
+                       int n_tokens, int channels, void* out, int plain, int single, ConvCache<T> cache, cudaStream_t stream) {
     const long long total = (long long)n_tokens * channels;
     constexpr int V = 16 / (int)sizeof(T);
     const bool runs = !single && n_tokens >= 32 && (taps == 2 || taps == 3 || taps == 4) && channels % V == 0 &&
-                      x_stride % V == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+                      x_stride % V == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0 &&
+                      (!CACHED || (cache.tail % V == 0 && cache.site.head_dim % V == 0 && ((uintptr_t)cache.site.base & 15) == 0));
     cudaError_t e;
     if (runs) {
         const int run = CONV_RUN(taps);
         const long long items = (long long)((n_tokens + run - 1) / run) * (channels / V);
         const dim3 grid((unsigned)((items + 127) / 128)), block(128);
-#define QF_CONV_RUN(TAPS) launch_pdl(causal_conv_run_kernel<T, TAPS>, grid, block, 0, stream, (const T*)x, x_stride, weight, bias, \
-                                     cu_q, tok_seq, slots, (const float*)state, slot_stride, offset, n_tokens, channels, (T*)out, plain)
+#define QF_CONV_RUN(TAPS) launch_pdl(causal_conv_run_kernel<T, TAPS, CACHED>, grid, block, 0, stream, (const T*)x, x_stride, weight, bias, \
+                                     cu_q, tok_seq, slots, (const float*)state, slot_stride, offset, n_tokens, channels, (T*)out, plain, cache)
         e = taps == 2 ? QF_CONV_RUN(2) : taps == 3 ? QF_CONV_RUN(3) : QF_CONV_RUN(4);
 #undef QF_CONV_RUN
     } else {
-        e = launch_pdl(causal_conv_silu_kernel<T>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream,
+        e = launch_pdl(causal_conv_silu_kernel<T, CACHED>, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream,
                        (const T*)x, x_stride, weight, bias, cu_q, tok_seq, slots, state, slot_stride, offset,
-                       taps, n_tokens, channels, (T*)out, plain, single);
+                       taps, n_tokens, channels, (T*)out, plain, single, cache);
     }
     if (e != cudaSuccess || taps <= 1 || single) return (int)e;
     const long long pairs = (long long)n_seqs * channels;
@@ -785,10 +813,33 @@ QF_EXPORT int qf_causal_conv(int is_bf16, const void* x, int x_stride, const flo
     if (single && n_tokens != n_seqs) return (int)cudaErrorInvalidValue;
     if (n_tokens <= 0 || channels <= 0) return 0;
     if (taps < 1 || taps > CONV_MAX_TAPS) return (int)cudaErrorInvalidValue;
-    return is_bf16 ? launch_conv<bf16>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps,
-                                       n_tokens, channels, out, plain, single, stream)
-                   : launch_conv<float>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps,
-                                        n_tokens, channels, out, plain, single, stream);
+    return is_bf16 ? launch_conv<bf16, false>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps,
+                                              n_tokens, channels, out, plain, single, ConvCache<bf16>{}, stream)
+                   : launch_conv<float, false>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps,
+                                               n_tokens, channels, out, plain, single, ConvCache<float>{}, stream);
+}
+
+// The convolution whose channels from `tail` on go to the paged cache: heads of head_dim channels, kv_heads of keys and, with
+// pages of two planes, as many of values behind them (page_elems = planes * kv_heads * QF_PAGE * head_dim). out: [T][tail].
+QF_EXPORT int qf_causal_conv_cached(int is_bf16, const void* x, int x_stride, const float* weight, const float* bias,
+                                    const int* cu_q, const int* tok_seq, const int* slots, int n_seqs, float* state,
+                                    long long slot_stride, long long offset, int taps, int n_tokens, int channels, void* out, int plain,
+                                    int single, const int* tok_pos, void* base, const int* table, long long page_elems,
+                                    int table_stride, int kv_heads, int head_dim, int tail, int* err, cudaStream_t stream) {
+    if (single && n_tokens != n_seqs) return (int)cudaErrorInvalidValue;
+    if (n_tokens <= 0 || channels <= 0) return 0;
+    if (taps < 1 || taps > CONV_MAX_TAPS || tail < 0 || kv_heads <= 0 || head_dim <= 0 || (channels - tail) % (kv_heads * head_dim) ||
+        channels <= tail || (long long)(channels - tail) * QF_PAGE > page_elems)
+        return (int)cudaErrorInvalidValue;
+    if (is_bf16)
+        return launch_conv<bf16, true>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps, n_tokens,
+                                       channels, out, plain, single,
+                                       ConvCache<bf16>{KvSite<bf16>{(bf16*)base, table, page_elems, table_stride, kv_heads, head_dim}, tok_pos, tail, err},
+                                       stream);
+    return launch_conv<float, true>(x, x_stride, weight, bias, cu_q, tok_seq, slots, n_seqs, state, slot_stride, offset, taps, n_tokens,
+                                    channels, out, plain, single,
+                                    ConvCache<float>{KvSite<float>{(float*)base, table, page_elems, table_stride, kv_heads, head_dim}, tok_pos, tail, err},
+                                    stream);
 }
 
 QF_EXPORT int qf_causal_conv_silu(int is_bf16, const void* x, int x_stride, const float* weight, const float* bias,

@@ -17,7 +17,7 @@ from ..cache import SequenceCache
 from ..config import ModelConfig, ModelSpec, load_config, resolve_dtype
 from ..csrc import prepare
 from ..parts import build_block, build_part
-from ..parts.base import Pending, PendingNormed
+from ..parts.base import Pending, PendingNormed, PendingStreams
 from ..weights import load_weights, random_state_on_device
 from .step import StepContext, context_of, pack_step
 
@@ -149,10 +149,16 @@ class Model:
                 delta = None
             delta = block.forward(hidden, delta, ctx, site, own)
             if self.observer is not None:
-                self.observer(index + 1, hidden, delta.value() if isinstance(delta, Pending) else delta)
+                if isinstance(delta, PendingStreams):   # the streams' sum stands in the stream's place
+                    self.observer(index + 1, delta.total(), None)
+                else:
+                    self.observer(index + 1, hidden, delta.value() if isinstance(delta, Pending) else delta)
         if ctx.want_rows is None:
             return None
         if isinstance(delta, Pending):
+            normed = delta.normed_rows(ctx.want_rows, self.final_norm, ctx.err)
+            if normed is not None:
+                return self.head.forward(normed)
             delta.add_to(hidden)
             delta = None
         shape = (ctx.want_rows.numel(), hidden.shape[1])

@@ -269,8 +269,11 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, to
                       window: int, err: torch.Tensor, scratch: Optional["DecodeScratch"] = None,
                       max_kv_len: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
                       shared_values: bool = False, chunk: int = 0, softcap: float = 0.0,
-                      blocks: Optional[KvSiteArgs] = None, pool: int = 0) -> None:
+                      blocks: Optional[KvSiteArgs] = None, pool: int = 0,
+                      distance_bias: Optional[tuple] = None) -> None:
     """Causal grouped-query attention of the step's queries over each sequence's cache (any sizes, SIMT float32 math).
+    `distance_bias` = (scale, rate), float32 [n_heads] each: after the cap, a score of key j under query i loses
+    scale[h] * ln(1 + rate[h] * (i - j)).
     `pool` > 0 with `blocks` (a second cache of the same head shape that holds one row per block of `pool` positions) and a
     window: a query also sees the row of every block that lies wholly before its window, in the same softmax.
     `chunk` > 0: a query sees only the keys of its own block of `chunk` positions (blocks counted from position 0 of the
@@ -292,6 +295,7 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, to
         _dev("sinks", sinks, torch.float32)
         if sinks.numel() != n_heads:
             raise KernelError("attention_generic: sinks must hold one float32 per query head")
+    by, rate = _distance_bias("attention_generic", distance_bias, n_heads, pool)
     if pool > 0:
         if blocks is None or window <= 0 or shared_values or (blocks.kv_heads, blocks.head_dim) != (site.kv_heads, d):
             raise KernelError("attention_generic: rows of whole blocks need a window and a second cache of the same head shape")
@@ -300,19 +304,32 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, to
             and max_kv_len > GENERIC_DECODE_CHUNK):
         n_chunks = -(-int(max_kv_len) // GENERIC_DECODE_CHUNK)
         scratch.ensure(n_seqs, n_heads, n_chunks, d, 0)
-        _check(library("attention_generic").qf_attention_generic_decode_masked(
+        _check(library("attention_generic").qf_attention_generic_decode_biased(
             _I(_is_bf16(q.dtype)), _ptr(q), _ptr(out), _ptr(cu_q), _ptr(tok_pos), _ptr(slots), _ptr(site.storage),
             _ptr(site.table), _LL(site.page_elems), _I(site.table_stride), _I(site.kv_heads), _I(d), _I(n_heads),
             _I(n_seqs), _I(int(max_kv_len)), _F(scale), _I(window), _ptr(scratch.part_o), _ptr(scratch.part_ml), _ptr(err),
-            _ptr(sinks), _I(int(bool(shared_values))), _I(int(chunk)), _F(softcap), _stream()), "attention_generic")
+            _ptr(sinks), _I(int(bool(shared_values))), _I(int(chunk)), _F(softcap), _ptr(by), _ptr(rate), _stream()), "attention_generic")
         return
-    _check(library("attention_generic").qf_attention_generic_pooled(
+    _check(library("attention_generic").qf_attention_generic_biased(
         _I(_is_bf16(q.dtype)), _ptr(q), _ptr(out), _ptr(cu_q), _ptr(tok_pos), _ptr(slots), _ptr(site.storage),
         _ptr(site.table), _LL(site.page_elems), _I(site.table_stride), _I(site.kv_heads), _I(d), _I(n_heads),
         _I(n_seqs), _I(max_q_len), _F(scale), _I(window), _ptr(err), _ptr(sinks), _I(int(bool(shared_values))),
         _I(int(chunk)), _F(softcap), _ptr(blocks.storage if pool > 0 else None), _ptr(blocks.table if pool > 0 else None),
-        _LL(blocks.page_elems if pool > 0 else 0), _I(blocks.table_stride if pool > 0 else 0), _I(int(pool)), _stream()),
-        "attention_generic")
+        _LL(blocks.page_elems if pool > 0 else 0), _I(blocks.table_stride if pool > 0 else 0), _I(int(pool)), _ptr(by), _ptr(rate),
+        _stream()), "attention_generic")
+
+
+def _distance_bias(what: str, pair, n_heads: int, pool: int = 0):
+    """(scale, rate) of a distance bias, checked; (None, None) without one."""
+    if pair is None:
+        return None, None
+    for name, t in zip(("scale", "rate"), pair):
+        _dev("the distance bias's " + name, t, torch.float32)
+        if t.numel() != n_heads:
+            raise KernelError(f"{what}: the distance bias holds one float32 per query head")
+    if pool > 0:
+        raise KernelError(f"{what}: a distance bias does not go with rows of whole blocks")
+    return pair
 
 
 FAST_ATTENTION_HEAD_DIMS = (32, 64, 96, 128)
@@ -322,10 +339,11 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, to
                       slots: torch.Tensor, site: KvSiteArgs, n_heads: int, n_seqs: int, max_q_len: int, scale: float,
                       window: int, err: torch.Tensor, max_kv_len: Optional[int] = None,
                       sinks: Optional[torch.Tensor] = None, shared_values: bool = False, chunk: int = 0,
-                      softcap: float = 0.0, blocks: Optional[KvSiteArgs] = None, pool: int = 0) -> None:
+                      softcap: float = 0.0, blocks: Optional[KvSiteArgs] = None, pool: int = 0,
+                      distance_bias: Optional[tuple] = None) -> None:
     """Tensor-core flash attention of spans of new tokens over the cache: bfloat16, head sizes 32/64/96/128.
-    `sinks`, `shared_values`, `chunk`, `softcap`, `blocks` and `pool`: as in `attention_generic` (the cap with the hardware's
-    approximate tanh).
+    `sinks`, `shared_values`, `chunk`, `softcap`, `blocks`, `pool` and `distance_bias`: as in `attention_generic` (the cap with the
+    hardware's approximate tanh, the bias with its base-2 logarithm).
     `max_kv_len`: an upper bound of any sequence's length after the step (None: unknown, taken as long); it only
     steers whether a tile of rows shares its pages among two groups of warps."""
     _dev("q", q, torch.bfloat16)
@@ -345,13 +363,14 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, to
         if blocks is None or window <= 0 or shared_values or (blocks.kv_heads, blocks.head_dim) != (site.kv_heads, d):
             raise KernelError("attention_prefill: rows of whole blocks need a window and a second cache of the same head shape")
         _dev("block rows", blocks.storage, torch.bfloat16)
-    _check(library("attention_prefill").qf_attention_prefill_pooled(
+    by, rate = _distance_bias("attention_prefill", distance_bias, n_heads, pool)
+    _check(library("attention_prefill").qf_attention_prefill_biased(
         _ptr(q), _ptr(out), _ptr(cu_q), _ptr(tok_pos), _ptr(slots), _ptr(site.storage), _ptr(site.table),
         _LL(site.page_elems), _I(site.table_stride), _I(site.kv_heads), _I(d), _I(n_heads), _I(n_seqs), _I(q.shape[0]),
         _I(max_q_len), _I(1 << 30 if max_kv_len is None else int(max_kv_len)), _F(scale), _I(window), _ptr(err),
         _ptr(sinks), _I(int(bool(shared_values))), _I(int(chunk)), _F(softcap), _ptr(blocks.storage if pool > 0 else None),
         _ptr(blocks.table if pool > 0 else None), _LL(blocks.page_elems if pool > 0 else 0),
-        _I(blocks.table_stride if pool > 0 else 0), _I(int(pool)), _stream()), "attention_prefill")
+        _I(blocks.table_stride if pool > 0 else 0), _I(int(pool)), _ptr(by), _ptr(rate), _stream()), "attention_prefill")
 
 
 TC_ATTENTION_HEAD_DIMS = (64, 128)
@@ -448,12 +467,12 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok
                      slots: torch.Tensor, site: KvSiteArgs, n_heads: int, n_seqs: int, scale: float, window: int,
                      n_splits: int, scratch: DecodeScratch, err: torch.Tensor, plan: Optional[torch.Tensor] = None,
                      fold_later: bool = False, sinks: Optional[torch.Tensor] = None, shared_values: bool = False,
-                     chunk: int = 0, softcap: float = 0.0) -> None:
+                     chunk: int = 0, softcap: float = 0.0, distance_bias: Optional[tuple] = None) -> None:
     """Split-K flash decoding: ONE new token per sequence over its cache; bfloat16, head sizes 32/64/96/128.
     `n_splits` is the most blocks that share one (sequence, kv head); `plan` (attention_decode_plan with the same
     shape, made in this step; made here when absent) says how many of them each sequence gets. With `fold_later` the
     kernel stops at the runs' partial results in `scratch` and writes no `out` (which may be None): `fold_project`
-    folds them on its way into the output projection. `sinks`, `shared_values`, `chunk`, `softcap`: as in
+    folds them on its way into the output projection. `sinks`, `shared_values`, `chunk`, `softcap`, `distance_bias`: as in
     `attention_generic` (sinks not with `fold_later`; a given `plan` must have been made with the same `chunk`; the cap
     with the hardware's approximate tanh)."""
     _dev("q", q, torch.bfloat16)
@@ -479,12 +498,13 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok
     partials = n_splits > 1 or fold_later
     if partials:
         scratch.ensure(n_seqs, n_heads, n_splits, d, n_counters)
-    _check(library("attention_decode").qf_attention_decode_masked(
+    by, rate = _distance_bias("attention_decode", distance_bias, n_heads)
+    _check(library("attention_decode").qf_attention_decode_biased(
         _ptr(q), _ptr(None if fold_later else out), _ptr(cu_q), _ptr(plan), _ptr(site.storage), _ptr(site.table),
         _LL(site.page_elems), _I(site.table_stride), _I(site.kv_heads), _I(d), _I(n_heads), _I(n_seqs), _F(scale),
         _I(window), _I(n_splits), _I(1 if fold_later else 0), _ptr(scratch.part_o if partials else None),
         _ptr(scratch.part_ml if partials else None), _ptr(scratch.counters if partials else None), _ptr(err),
-        _ptr(sinks), _I(int(bool(shared_values))), _I(int(chunk)), _F(softcap), _stream()), "attention_decode")
+        _ptr(sinks), _I(int(bool(shared_values))), _I(int(chunk)), _F(softcap), _ptr(by), _ptr(rate), _stream()), "attention_decode")
 
 
 class _FoldProjectArgs(ctypes.Structure):
@@ -1036,6 +1056,16 @@ def head_gate(x: torch.Tensor, gate: torch.Tensor, n_heads: int) -> None:
                                               _I(width // n_heads), _stream()), "head_gate")
 
 
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> None:
+    """x *= sigmoid(gate), element by element, in place: x [T, C] contiguous, gate [T, C] (rows may be strided), activation dtype."""
+    _dev("x", x)
+    _rows("gate", gate, x.dtype)
+    if gate.shape != x.shape:
+        raise KernelError("sigmoid_gate: x and gate differ in shape")
+    _check(library("activation").qf_sigmoid_gate(_I(_is_bf16(x.dtype)), _ptr(x), _ptr(gate), _LL(gate.stride(0)), _I(x.shape[0]),
+                                                 _I(x.shape[1]), _stream()), "sigmoid_gate")
+
+
 def pool_cache_write(cu_q: torch.Tensor, tok_pos: torch.Tensor, slots: torch.Tensor, site: KvSiteArgs, blocks: KvSiteArgs,
                      pool: int, max_q_len: int, err: torch.Tensor) -> None:
     """For every block of `pool` positions that this step completed (its last position is among the step's tokens, whose
@@ -1199,13 +1229,21 @@ def sandwich_norm(hidden: torch.Tensor, y: torch.Tensor, post_weight: torch.Tens
                                             _ptr(row_weight if dest is not None else None), _stream()), "sandwich_norm")
 
 
-def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, out: torch.Tensor) -> None:
-    """out[t, i] = g * sigmoid(alpha * g) * (u + 1) with g = min(gate_up[t, i], limit), u = clamp(gate_up[t, I + i], -limit, limit)."""
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, out: torch.Tensor, row_scale: Optional[torch.Tensor] = None) -> None:
+    """out[t, i] = g * sigmoid(alpha * g) * (u + 1) with g = min(gate_up[t, i], limit), u = clamp(gate_up[t, I + i], -limit, limit).
+    `row_scale` (float32 [rows]) multiplies both halves before they are clamped: rows whose input was to be scaled."""
     _dev("gate_up", gate_up)
     _dev("out", out, gate_up.dtype)
     rows, two_i = gate_up.shape
     if two_i % 2 or out.shape != (rows, two_i // 2):
         raise KernelError("clamped_glu: out must be [rows, width / 2]")
+    if row_scale is not None:
+        _dev("row_scale", row_scale, torch.float32)
+        if row_scale.numel() != rows:
+            raise KernelError("clamped_glu: row_scale must hold one float32 per row")
+        _check(library("activation").qf_scaled_clamped_glu(_I(_is_bf16(gate_up.dtype)), _ptr(gate_up), _ptr(row_scale), _ptr(out),
+                                                           _I(rows), _I(two_i // 2), _F(limit), _F(alpha), _stream()), "clamped_glu")
+        return
     _check(library("activation").qf_clamped_glu(_I(_is_bf16(gate_up.dtype)), _ptr(gate_up), _ptr(out), _I(rows),
                                                 _I(two_i // 2), _F(limit), _F(alpha), _stream()), "clamped_glu")
 
@@ -1213,19 +1251,28 @@ def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float, out: torch.Te
 def latent_norm_cache(down: torch.Tensor, q_rank: int, q_norm: Optional[torch.Tensor], kv_norm: torch.Tensor, eps: float,
                       tok_seq: torch.Tensor, tok_pos: torch.Tensor, slots: torch.Tensor, q_latent: Optional[torch.Tensor],
                       site: KvSiteArgs, write_cache: bool, err: torch.Tensor,
-                      latent_out: Optional[torch.Tensor] = None) -> None:
+                      latent_out: Optional[torch.Tensor] = None, rotated: Optional[tuple] = None) -> None:
     """The two latents of a latent attention from their fused down-projection `down` (float32 [T, q_rank + kv_rank]):
     q_latent [T, q_rank] = rmsnorm(down[:, :q_rank]) * q_norm, and rmsnorm(down[:, q_rank:]) * kv_norm written to each
     token's own position in a one-plane cache of a single head of kv_rank elements (`site`; and to `latent_out` in token
-    order, if given). q_rank 0: no query latent."""
+    order, if given). q_rank 0: no query latent.
+    `rotated` = (inv_freq float32 [R / 2], amplitude): `down` has R columns more, one key part that all heads share; its
+    neighbours (2i, 2i + 1) are turned by position * inv_freq[i] (cosine and sine times the amplitude) and kept behind the latent
+    in the same cache row, which then has site.head_dim >= kv_rank + R elements."""
     _dev("down", down, torch.float32, contiguous=False)
     _dev("kv_norm", kv_norm)
     _dev("cache", site.storage, kv_norm.dtype)
     for name, t in (("tok_seq", tok_seq), ("tok_pos", tok_pos), ("slots", slots)):
         _dev(name, t, torch.int32)
-    n, kv_rank = down.shape[0], site.head_dim
-    if down.stride(1) != 1 or down.shape[1] != q_rank + kv_rank or site.kv_heads != 1 or kv_norm.numel() != kv_rank:
-        raise KernelError("latent_norm_cache: down must be [tokens, q_rank + kv_rank] and the cache hold one head of kv_rank")
+    n, kv_rank = down.shape[0], kv_norm.numel()
+    inv_freq, amplitude = rotated if rotated is not None else (None, 1.0)
+    rot = 0
+    if inv_freq is not None:
+        _dev("inv_freq", inv_freq, torch.float32)
+        rot = 2 * inv_freq.numel()
+    if down.stride(1) != 1 or down.shape[1] != q_rank + kv_rank + rot or site.kv_heads != 1 or site.head_dim < kv_rank + rot:
+        raise KernelError("latent_norm_cache: down must be [tokens, q_rank + kv_rank + rotated] and the cache hold one head of "
+                          "kv_rank + rotated elements or more")
     if q_rank:
         _dev("q_norm", q_norm, kv_norm.dtype)
         _dev("q_latent", q_latent, kv_norm.dtype)
@@ -1235,11 +1282,31 @@ def latent_norm_cache(down: torch.Tensor, q_rank: int, q_norm: Optional[torch.Te
         _dev("latent_out", latent_out, kv_norm.dtype)
         if latent_out.shape != (n, kv_rank):
             raise KernelError("latent_norm_cache: latent_out must be [tokens, kv_rank]")
-    _check(library("latent_cache").qf_latent_norm_cache(
+    _check(library("latent_cache").qf_latent_norm_cache_turned(
         _I(_is_bf16(kv_norm.dtype)), _ptr(down), _I(down.stride(0)), _I(q_rank), _I(kv_rank), _ptr(q_norm if q_rank else None),
         _ptr(kv_norm), _F(eps), _ptr(tok_seq), _ptr(tok_pos), _ptr(slots), _ptr(q_latent if q_rank else None),
         _ptr(latent_out), _ptr(site.storage), _ptr(site.table), _LL(site.page_elems), _I(site.table_stride),
-        _I(1 if write_cache else 0), _I(n), _ptr(err), _stream()), "latent_norm_cache")
+        _I(1 if write_cache else 0), _I(n), _ptr(err), _I(site.head_dim), _I(rot), _ptr(inv_freq), _F(amplitude), _stream()),
+        "latent_norm_cache")
+
+
+def rotate_heads(x: torch.Tensor, x_pitch: int, x_first: int, out: torch.Tensor, out_pitch: int, out_first: int,
+                 inv_freq: torch.Tensor, amplitude: float, tok_pos: torch.Tensor, n_heads: int) -> None:
+    """The rotated part of every head's query, to its place in another layout: of head h's columns in x [T, H * x_pitch] those from
+    x_first on (R = 2 * inv_freq.numel() of them) are turned by the token's position, neighbours (2i, 2i + 1) by the angle
+    position * inv_freq[i] with cosine and sine times `amplitude`, and written to out [T, H * out_pitch] from out_first on, with
+    zeros from there to the end of the head's piece. x and out: activation dtype, rows may be strided."""
+    _rows("x", x)
+    _rows("out", out, x.dtype)
+    _dev("inv_freq", inv_freq, torch.float32)
+    _dev("tok_pos", tok_pos, torch.int32)
+    rot = 2 * inv_freq.numel()
+    if x.shape[1] < n_heads * x_pitch or out.shape[1] < n_heads * out_pitch or out.shape[0] != x.shape[0] or tok_pos.numel() != x.shape[0] \
+            or x_first + rot > x_pitch or out_first + rot > out_pitch:
+        raise KernelError("rotate_heads: the heads' rotated columns do not fit the rows")
+    _check(library("latent_cache").qf_rotate_heads(
+        _I(_is_bf16(x.dtype)), _ptr(x), _LL(x.stride(0)), _I(x_pitch), _I(x_first), _ptr(out), _LL(out.stride(0)), _I(out_pitch),
+        _I(out_first), _I(rot), _ptr(inv_freq), _F(amplitude), _ptr(tok_pos), _I(n_heads), _I(x.shape[0]), _stream()), "rotate_heads")
 
 
 def _grouped(x, weight, out, a_group_cols, c_group_cols, rows, plan, a_rows=None, gated=False, row_scale=None, clamp=None,
@@ -1263,16 +1330,19 @@ def _grouped(x, weight, out, a_group_cols, c_group_cols, rows, plan, a_rows=None
     _check(code, "grouped_gemm")
 
 
-def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> None:
+def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, x_pitch: int = 0, out_pitch: int = 0) -> None:
     """A product per head in one launch: out[:, g*N:(g+1)*N] = x[:, g*K:(g+1)*K] @ weight[g].T for weight [G, N, K],
-    x [T, G*K], out [T, G*N], all of the activation dtype."""
+    x [T, G*K], out [T, G*N], all of the activation dtype. With `x_pitch` (`out_pitch`) the heads' pieces of x (out) start that
+    many columns apart: head g reads columns g * x_pitch .. + K and writes g * out_pitch .. + N."""
     _dev("x", x, None, contiguous=False)
     _dev("weight", weight, x.dtype, contiguous=False)
     _dev("out", out, x.dtype, contiguous=False)
     groups, n, k = weight.shape
-    if x.shape[1] != groups * k or out.shape != (x.shape[0], groups * n) or weight.stride(2) != 1 or x.stride(1) != 1 or out.stride(1) != 1:
+    px, po = x_pitch or k, out_pitch or n
+    if px < k or po < n or x.shape[1] != groups * px or out.shape != (x.shape[0], groups * po) or weight.stride(2) != 1 \
+            or x.stride(1) != 1 or out.stride(1) != 1:
         raise KernelError(f"head_linear: shapes {tuple(x.shape)} x {tuple(weight.shape)} -> {tuple(out.shape)} do not agree")
-    _grouped(x, weight, out, k, n, x.shape[0], None)
+    _grouped(x, weight, out, px, po, x.shape[0], None)
 
 
 GROUP_TILE_ROWS = 64          # rows of a tile of the grouped products (QF_GROUP_BM in csrc/common.cuh)
@@ -1728,6 +1798,183 @@ def causal_conv_silu(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch
 def causal_conv(x, weight, bias, cu_q, tok_seq, slots, state, offset, out, single: bool = False) -> None:
     """`causal_conv_silu` without the activation."""
     causal_conv_silu(x, weight, bias, cu_q, tok_seq, slots, state, offset, out, activation="none", single=single)
+
+
+def causal_conv_cached(x: torch.Tensor, weight: torch.Tensor, cu_q: torch.Tensor, tok_seq: torch.Tensor, tok_pos: torch.Tensor,
+                       slots: torch.Tensor, state: torch.Tensor, offset: int, out: torch.Tensor, site: KvSiteArgs,
+                       err: torch.Tensor, single: bool = False) -> None:
+    """`causal_conv` over a layer's projections [q | k (| v)] whose keys (and values) go to the paged cache at the token's own
+    position instead of beside the queries: out [T, q width] takes the first columns, the rest are kv_heads * head_dim keys and, where
+    the cache's pages hold two planes, as many values."""
+    _rows("x", x)
+    _dev("out", out, x.dtype)
+    _dev("weight", weight, torch.float32)
+    _dev("cache", site.storage, x.dtype)
+    for name, t in (("tok_seq", tok_seq), ("tok_pos", tok_pos), ("slots", slots)):
+        _dev(name, t, torch.int32)
+    n, c = x.shape
+    taps, tail = weight.shape[1], out.shape[1]
+    planes = site.storage.shape[1]
+    if weight.shape[0] != c or out.shape[0] != n or not 1 <= taps <= CONV_MAX_TAPS or c - tail != planes * site.kv_heads * site.head_dim:
+        raise KernelError("causal_conv_cached: weight must be [C, taps], out [T, q width], and C - q width the cache's columns per position")
+    _state(state, (offset, (taps - 1) * c))
+    _check(library("recurrent").qf_causal_conv_cached(
+        _I(_is_bf16(x.dtype)), _ptr(x), _I(x.stride(0)), _ptr(weight), _ptr(None), _ptr(cu_q), _ptr(tok_seq), _ptr(slots),
+        _I(cu_q.numel() - 1), _ptr(state), _LL(state.stride(0)), _LL(offset), _I(taps), _I(n), _I(c), _ptr(out), _I(1),
+        _I(1 if single and n == cu_q.numel() - 1 else 0), _ptr(tok_pos), _ptr(site.storage), _ptr(site.table), _LL(site.page_elems),
+        _I(site.table_stride), _I(site.kv_heads), _I(site.head_dim), _I(tail), _ptr(err), _stream()), "causal_conv_cached")
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# The gated delta rule (csrc/delta_rule.cu)
+def _delta_args(what, q, k, v, z, bias, rate_log, logit, state, s_offset, n_heads, n_groups, dim, vdim):
+    for name, t in (("q", q), ("k", k), ("v", v)):
+        _rows(name, t, q.dtype)
+    _is_bf16(q.dtype)
+    n = q.shape[0]
+    if n_groups <= 0 or n_heads % n_groups or q.shape[1] != n_groups * dim or k.shape != q.shape or v.shape != (n, n_heads * vdim):
+        raise KernelError(f"{what}: q, k must be [T, groups * dim], v [T, heads * vdim]")
+    if not 1 <= dim <= OUTER_STATE_MAX_DIM:
+        raise KernelError(f"{what}: a state of {dim} rows per head exceeds the kernel's {OUTER_STATE_MAX_DIM}")
+    _rows("z", z, torch.float32)
+    _rows("logit", logit, torch.float32)
+    _dev("bias", bias, torch.float32)
+    _dev("rate_log", rate_log, torch.float32)
+    if z.shape != (n, n_heads * dim) or logit.shape != (n, n_heads) or bias.numel() != n_heads * dim or rate_log.numel() != n_heads:
+        raise KernelError(f"{what}: z must be float32 [T, heads * dim], logit [T, heads], bias [heads * dim], rate_log [heads]")
+    _state(state, (s_offset, n_heads * dim * vdim))
+    return (_I(_is_bf16(q.dtype)), _ptr(q), _I(q.stride(0)), _ptr(k), _I(k.stride(0)), _ptr(v), _I(v.stride(0)), _ptr(z), _I(z.stride(0)),
+            _ptr(bias), _ptr(rate_log), _ptr(logit), _I(logit.stride(0)))
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, rate_log: torch.Tensor,
+               logit: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_heads: int,
+               n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor) -> None:
+    """The gated delta rule with a decay per head and key channel, token after token of every sequence, float32 inside:
+        q, k <- x / sqrt(sum(x^2) + 1e-6) per head (q also times q_scale);  g = exp(-exp(rate_log_h) softplus(z + bias));
+        beta = sigmoid(logit);  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  y = S^T q.
+    q, k: [T, groups * dim] (head h reads group h // (heads / groups)), v: [T, heads * vdim] in the activation dtype; z float32
+    [T, heads * dim], logit float32 [T, heads]; rows may be strided; bias float32 [heads * dim], rate_log float32 [heads]; y float32
+    [T, heads * vdim]; S (dim x vdim per head) in `state` at s_offset as [heads, dim, vdim]."""
+    args = _delta_args("delta_scan", q, k, v, z, bias, rate_log, logit, state, s_offset, n_heads, n_groups, dim, vdim)
+    n = q.shape[0]
+    _dev("y", y, torch.float32)
+    if y.shape != (n, n_heads * vdim):
+        raise KernelError("delta_scan: y must be float32 [T, heads * vdim]")
+    lib = library("delta_rule")
+    padded = int(lib.qf_delta_padded(_I(dim)))
+    packed = torch.empty(n_heads * n * (3 * padded + 1), dtype=torch.float32, device=q.device)
+    _check(lib.qf_delta_scan(*args, _ptr(cu_q), _ptr(slots), _I(cu_q.numel() - 1), _ptr(state), _LL(state.stride(0)), _LL(s_offset), _I(n),
+                             _I(n_heads), _I(n_groups), _I(dim), _I(vdim), _F(q_scale), _ptr(packed),
+                             _ptr(packed[n_heads * n * 3 * padded:]), _ptr(y), _stream()), "delta_scan")
+
+
+DELTA_FUSED_MAX_VDIM = 128   # value sizes up to which a single token's norm and gate ride on `delta_token`
+
+
+def delta_token(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, rate_log: torch.Tensor,
+                logit: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_heads: int,
+                n_groups: int, dim: int, vdim: int, q_scale: float, y: Optional[torch.Tensor] = None,
+                norm: Optional[torch.Tensor] = None, eps: float = 0.0, gate: Optional[torch.Tensor] = None,
+                out: Optional[torch.Tensor] = None) -> None:
+    """`delta_scan` for a step of ONE token per sequence. Instead of y (or beside it), for vdim <= DELTA_FUSED_MAX_VDIM, `out`
+    [T, heads * vdim] in the activation dtype takes what follows the recurrence: y / rms(y) per head (eps inside the root) times
+    norm [vdim] times sigmoid(gate [T, heads * vdim])."""
+    args = _delta_args("delta_token", q, k, v, z, bias, rate_log, logit, state, s_offset, n_heads, n_groups, dim, vdim)
+    n = q.shape[0]
+    if n != cu_q.numel() - 1 or (y is None and out is None):
+        raise KernelError("delta_token: one token per sequence, and somewhere to put the result")
+    if y is not None:
+        _dev("y", y, torch.float32)
+        if y.shape != (n, n_heads * vdim):
+            raise KernelError("delta_token: y must be float32 [T, heads * vdim]")
+    if out is not None:
+        _dev("out", out, q.dtype)
+        _dev("norm", norm, q.dtype)
+        _rows("gate", gate, q.dtype)
+        if out.shape != (n, n_heads * vdim) or gate.shape != out.shape or norm.numel() != vdim or vdim > DELTA_FUSED_MAX_VDIM:
+            raise KernelError(f"delta_token: out and gate must be [T, heads * vdim], norm [vdim], vdim at most {DELTA_FUSED_MAX_VDIM}")
+    _check(library("delta_rule").qf_delta_token(
+        *args, _ptr(cu_q), _ptr(slots), _I(n), _ptr(state), _LL(state.stride(0)), _LL(s_offset), _I(n_heads), _I(n_groups), _I(dim), _I(vdim),
+        _F(q_scale), _ptr(y), _ptr(norm), _F(eps), _ptr(gate), _I(gate.stride(0) if gate is not None else 0), _ptr(out), _stream()),
+        "delta_token")
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Several residual streams (csrc/streams.cu)
+STREAMS_MAX = 8
+
+
+def streams_norm(source: torch.Tensor, n_streams: int, coefficients: Optional[tuple], y, in_weight: Optional[torch.Tensor],
+                 new: Optional[torch.Tensor] = None, norm: Optional[tuple] = None, out: Optional[torch.Tensor] = None,
+                 conv: Optional[tuple] = None, rows: Optional[torch.Tensor] = None, err: Optional[torch.Tensor] = None,
+                 y_rows: Optional[tuple] = None) -> None:
+    """What stands between one sublayer and the next where a token carries n_streams float32 rows X, in one launch:
+        Y[r] = sum_s mix[s, r] X[s] + out_w[r] y;   u = sum_r in_weight[r] Y[r];   h = tanh(alpha u) * weight + bias;
+        z_t = h_t + sum_j taps[:, j] h_(t - n_taps + 1 + j)
+    source: float32 [T, W] (one row that stands for every stream) or [T, n_streams, W]. y: the sublayer's output [T, W] with
+    coefficients = (mix [n, n], out_w [n]) float32, or None (X passes as it is). y_rows = (dest int32 [T * top], top, row_weight
+    float32 or None): token t's output is the sum of the rows y[dest[t * top + k]] (times their weights). in_weight float32 [n];
+    None: ones. new: float32 [T, n_streams, W] takes Y (not the source's memory), or None.
+    norm = (weight, bias, alpha); None: u itself goes to `out`, float32. out: [T, W] in the activation dtype.
+    conv = (taps float32 [W, n_taps], cu_q, slots, max_q_len, state, offset): h before the step's first token comes from the slot's state
+    (float32 [n_taps - 1, W] at `offset`, zeros at a sequence's start), which then takes the sequence's last values of h.
+    rows (int32 [R]): only these tokens, out [R, W]; `err` takes an index outside the step."""
+    _dev("source", source, torch.float32)
+    n_tokens, width = source.shape[0], source.shape[-1]
+    if source.dim() not in (2, 3) or (source.dim() == 3 and source.shape[1] != n_streams) or not 1 <= n_streams <= STREAMS_MAX:
+        raise KernelError(f"streams_norm: source must be float32 [T, W] or [T, streams, W] with 1 to {STREAMS_MAX} streams")
+    mix, out_w = coefficients if coefficients is not None else (None, None)
+    dest, top, row_weight = y_rows if y_rows is not None else (None, 1, None)
+    weight, bias, alpha = norm if norm is not None else (None, None, 0.0)
+    dtype = weight.dtype if weight is not None else (y.dtype if y is not None else torch.float32)
+    for name, t, count in (("mix", mix, n_streams * n_streams), ("out_w", out_w, n_streams), ("in_weight", in_weight, n_streams)):
+        if t is not None:
+            _dev(name, t, torch.float32)
+            if t.numel() != count:
+                raise KernelError(f"streams_norm: {name} must hold {count} float32")
+    if y is not None:
+        _dev("y", y, dtype)
+        if mix is None or y.dim() != 2 or y.shape[1] != width or (dest is None and y.shape[0] != n_tokens):
+            raise KernelError("streams_norm: y must be [T, W] (or rows to be summed) and comes with its coefficients")
+        if dest is not None:
+            _dev("dest", dest, torch.int32)
+            if dest.numel() != n_tokens * top:
+                raise KernelError("streams_norm: dest must name `top` rows per token")
+    if new is not None:
+        _dev("new", new, torch.float32)
+        if new.shape != (n_tokens, n_streams, width) or rows is not None:
+            raise KernelError("streams_norm: new must be float32 [T, streams, W], for all of the step's tokens")
+    n_rows = n_tokens
+    if rows is not None:
+        _dev("rows", rows, torch.int32)
+        if err is None or conv is not None:
+            raise KernelError("streams_norm: named rows need the error word and do not go with a convolution")
+        n_rows = rows.numel()
+    _dev("out", out, dtype if norm is not None else torch.float32)
+    if out.shape != (n_rows, width):
+        raise KernelError("streams_norm: out must be [rows, W]")
+    if norm is not None:
+        _dev("weight", weight)
+        _dev("bias", bias, dtype)
+        if weight.numel() != width or bias.numel() != width:
+            raise KernelError("streams_norm: the norm's weight and bias must be [W]")
+    taps, cu_q, slots, max_q_len, state, offset = conv if conv is not None else (None, None, None, 0, None, 0)
+    n_taps = 0
+    if taps is not None:
+        _dev("taps", taps, torch.float32)
+        _dev("cu_q", cu_q, torch.int32)
+        _dev("slots", slots, torch.int32)
+        n_taps = taps.shape[1]
+        if taps.shape[0] != width or not 1 <= n_taps <= CONV_MAX_TAPS or norm is None:
+            raise KernelError(f"streams_norm: taps must be float32 [W, 1 to {CONV_MAX_TAPS}] behind a norm")
+        _state(state, (offset, (n_taps - 1) * width))
+    _check(library("streams").qf_streams_norm(
+        _I(_is_bf16(dtype)), _ptr(source), _LL(source.stride(0)), _LL(source.stride(1) if source.dim() == 3 else 0), _ptr(new), _ptr(y),
+        _ptr(dest), _I(top), _ptr(row_weight), _ptr(mix), _ptr(out_w), _ptr(in_weight), _ptr(weight), _ptr(bias), _F(alpha),
+        _ptr(out if norm is not None else None), _ptr(None if norm is not None else out), _ptr(rows), _I(n_rows if rows is not None else 0),
+        _I(n_tokens), _ptr(taps), _I(n_taps), _ptr(cu_q), _ptr(slots), _I(slots.numel() if slots is not None else 0), _I(max_q_len), _ptr(state),
+        _LL(state.stride(0) if state is not None else 0), _LL(offset), _I(n_streams), _I(width), _ptr(err), _stream()), "streams_norm")
 
 
 # ---------------------------------------------------------------------------------------------------------------------

@@ -37,6 +37,11 @@ Options that other designs switch on, each a parameter of the spec (all off for 
   value_mix      {"role": "source" | "mix", "key": name}: the layers that share a key form a chain through one step. The
                  source keeps its values (after the bias) for the others; a "mix" layer replaces its own by
                  (1 - l) v + l v_source of the same token, l a learned number (`value_mix`), and caches the mixed values
+  shared_values  the values are the keys as they leave the convolution: no value projection, and the cache keeps one plane
+  distance_bias  after the cap, a score of key j under query i loses r1_h * ln(1 + r2_h * (i - j)), two numbers per head from the
+                 weight files (`bias_scale`, `bias_rate`)
+  out_gate       the concatenated heads are multiplied element by element with sigmoid(G h), a projection [heads * value_dim,
+                 hidden] of the same input whose columns follow those of q, k, v in the one product
 The position part may pair components 2j and 2j + 1 (`rotary_interleaved`) instead of j and j + R/2.
 """
 from __future__ import annotations
@@ -82,6 +87,18 @@ class GqaAttention(Mixer):
         self.gated = bool(p.get("head_gate", False))
         self.row_norm_eps = None if p.get("row_norm_eps") is None else float(p["row_norm_eps"])
         self.value_mix = dict(p["value_mix"]) if p.get("value_mix") else None
+        self.shared_values = bool(p.get("shared_values", False))
+        self.distance_bias = bool(p.get("distance_bias", False))
+        self.out_gate = bool(p.get("out_gate", False))
+        if self.shared_values and (self.value_dim != self.key_dim or p.get("position") is not None or p.get("qkv_bias") or self.pool > 0
+                                   or self.conv_taps <= 0 or not self.own_kv or self.qk_norm_eps is not None
+                                   or self.unit_norm_eps is not None or self.row_norm_eps is not None or self.value_mix is not None):
+            raise ValueError("gqa_attention: values that are the keys go with keys that come straight out of a short convolution "
+                             "(no rotation, norm, bias or pooled rows) and have their size")
+        if self.out_gate and (self.gated or self.value_dim != self.head_dim):
+            raise ValueError("gqa_attention: a gate per element goes with values as wide as the kernels' heads, without a gate per head")
+        if self.distance_bias and self.pool > 0:
+            raise ValueError("gqa_attention: a distance bias does not go with pooled blocks")
         if self.value_mix is not None and (self.value_mix.get("role") not in ("source", "mix") or not p.get("own_kv", True)):
             raise ValueError("gqa_attention: value_mix has the role 'source' or 'mix' and goes with values of the layer's own")
         if self.row_norm_eps is not None and (p.get("qk_norm_eps") is not None or int(p.get("conv_taps") or 0) > 0 or not p.get("own_kv", True)):
@@ -101,7 +118,7 @@ class GqaAttention(Mixer):
         self.plain = (self.value_dim == self.key_dim and self.unit_norm_eps is None and self.softcap == 0.0 and self.chunk == 0
                       and self.sink == "none" and self.own_kv and self.conv_taps == 0 and self.qk_norm_eps is None
                       and self.pool == 0 and not self.gated and not self.interleaved and self.row_norm_eps is None
-                      and self.value_mix is None)
+                      and self.value_mix is None and not self.shared_values and not self.distance_bias and not self.out_gate)
         self.qkv_bias = bool(p.get("qkv_bias", False))
         self.out_bias = bool(p.get("out_bias", False))
         self.scale = float(p.get("scale") or self.key_dim ** -0.5)
@@ -111,9 +128,13 @@ class GqaAttention(Mixer):
         if self.head_dim > 256:
             raise ValueError(f"gqa_attention: head_dim {self.head_dim} > 256 is not supported by the attention kernels")
         self.position = build_part("position", p["position"]) if p.get("position") is not None else None
+        if getattr(self.position, "amplitude", 1.0) != 1.0:
+            raise ValueError("gqa_attention: its rotation kernels take no factor on cosine and sine")
         self.q_width = self.n_heads * self.head_dim
         self.kv_width = self.n_kv * self.head_dim
-        self.qkv_width = self.q_width + (2 * self.kv_width if self.own_kv else 0)   # the gates' columns follow
+        # (the gates' columns follow)
+        self.qkv_width = self.q_width + ((1 if self.shared_values else 2) * self.kv_width if self.own_kv else 0)
+        self.bias_pair = None
         self.qkv_weight = self.qkv_bias_t = self.o_weight = self.o_bias_t = self.sinks = None
         self.conv_weight = self.q_norm = self.k_norm = self.q_row_norm = self.k_row_norm = None
         self.mix_weight = 0.0
@@ -125,8 +146,9 @@ class GqaAttention(Mixer):
         kd, vd = self.key_dim, self.value_dim
         specs = [TensorSpec(self.file_name("q_weight"), (self.n_heads * kd, self.hidden))]
         if self.own_kv:
-            specs += [TensorSpec(self.file_name("k_weight"), (self.n_kv * kd, self.hidden)),
-                      TensorSpec(self.file_name("v_weight"), (self.n_kv * vd, self.hidden))]
+            specs.append(TensorSpec(self.file_name("k_weight"), (self.n_kv * kd, self.hidden)))
+            if not self.shared_values:
+                specs.append(TensorSpec(self.file_name("v_weight"), (self.n_kv * vd, self.hidden)))
         specs.append(TensorSpec(self.file_name("o_weight"), (self.hidden, self.n_heads * vd)))
         if self.qkv_bias:
             specs.append(TensorSpec(self.file_name("q_bias"), (self.n_heads * kd,), init="bias"))
@@ -137,14 +159,20 @@ class GqaAttention(Mixer):
             specs.append(TensorSpec(self.file_name("o_bias"), (self.hidden,), init="bias"))
         if self.conv_taps > 0:
             specs += [TensorSpec(self.file_name("q_conv"), (self.n_heads * kd, self.conv_taps), init="conv", keep="float32"),
-                      TensorSpec(self.file_name("k_conv"), (self.n_kv * kd, self.conv_taps), init="conv", keep="float32"),
-                      TensorSpec(self.file_name("v_conv"), (self.n_kv * vd, self.conv_taps), init="conv", keep="float32")]
+                      TensorSpec(self.file_name("k_conv"), (self.n_kv * kd, self.conv_taps), init="conv", keep="float32")]
+            if not self.shared_values:
+                specs.append(TensorSpec(self.file_name("v_conv"), (self.n_kv * vd, self.conv_taps), init="conv", keep="float32"))
         if self.qk_norm_eps is not None:
             specs += [TensorSpec(self.file_name("q_norm"), (kd,), init="norm"), TensorSpec(self.file_name("k_norm"), (kd,), init="norm")]
         if self.sink == "learned":
             specs.append(TensorSpec(self.file_name("sink"), (self.n_heads,), init="logit", keep="float32"))
         if self.gated:
             specs.append(TensorSpec(self.file_name("g_weight"), (self.n_heads, self.hidden)))
+        if self.out_gate:
+            specs.append(TensorSpec(self.file_name("g_weight"), (self.n_heads * vd, self.hidden)))
+        if self.distance_bias:
+            specs += [TensorSpec(self.file_name("bias_scale"), (self.n_heads,), init="positive", keep="float32"),
+                      TensorSpec(self.file_name("bias_rate"), (self.n_heads,), init="positive", keep="float32")]
         if self.row_norm_eps is not None:
             specs += [TensorSpec(self.file_name("q_row_norm"), (self.n_heads * kd,), init="norm"),
                       TensorSpec(self.file_name("k_row_norm"), (self.n_kv * kd,), init="norm")]
@@ -154,7 +182,7 @@ class GqaAttention(Mixer):
 
     def kernel_libraries(self, dtype):
         libs = {"rope_cache", "attention_generic"} | ({"recurrent"} if self.conv_taps > 0 else set()) \
-            | ({"activation"} if self.gated else set()) | ({"norm"} if self.row_norm_eps is not None or self.value_mix else set())
+            | ({"activation"} if self.gated or self.out_gate else set()) | ({"norm"} if self.row_norm_eps is not None or self.value_mix else set())
         if dtype == torch.float32:
             libs.add("gemm_f32")
         elif not self.plain and self.head_dim in ops.FAST_ATTENTION_HEAD_DIMS:
@@ -166,7 +194,7 @@ class GqaAttention(Mixer):
         return libs
 
     def cache_need(self):
-        kv = KvNeed(self.n_kv, self.head_dim, self.window, chunk=self.chunk, pool=self.pool)
+        kv = KvNeed(self.n_kv, self.head_dim, self.window, planes=1 if self.shared_values else 2, chunk=self.chunk, pool=self.pool)
         if self.pool <= 0 and self.conv_taps <= 0:
             return kv
         items = [("kv", kv)]
@@ -189,16 +217,22 @@ class GqaAttention(Mixer):
         kd, vd = self.key_dim, self.value_dim
         pieces = [self._padded(t("q_weight"), self.n_heads, kd)]
         if self.own_kv:
-            pieces += [self._padded(t("k_weight"), self.n_kv, kd), self._padded(t("v_weight"), self.n_kv, vd)]
-        if self.gated:   # the gates' logits are further columns of the one product
+            pieces.append(self._padded(t("k_weight"), self.n_kv, kd))
+            if not self.shared_values:
+                pieces.append(self._padded(t("v_weight"), self.n_kv, vd))
+        if self.gated or self.out_gate:   # the gates' logits are further columns of the one product
             pieces.append(t("g_weight"))
             rows = sum(p.shape[0] for p in pieces)
             if rows % 8:   # zero rows up to a row pitch of whole 16 bytes: the library's products choose their kernels by it
                 pieces.append(pieces[0].new_zeros((8 - rows % 8, pieces[0].shape[1])))
         self.qkv_weight = torch.cat(pieces, dim=0).contiguous()
         if self.conv_taps > 0:   # zero taps under the padding: what is zero stays zero
-            self.conv_weight = torch.cat((self._padded(t("q_conv"), self.n_heads, kd), self._padded(t("k_conv"), self.n_kv, kd),
-                                          self._padded(t("v_conv"), self.n_kv, vd)), dim=0).to(torch.float32).contiguous()
+            taps = [self._padded(t("q_conv"), self.n_heads, kd), self._padded(t("k_conv"), self.n_kv, kd)]
+            if not self.shared_values:
+                taps.append(self._padded(t("v_conv"), self.n_kv, vd))
+            self.conv_weight = torch.cat(taps, dim=0).to(torch.float32).contiguous()
+        if self.distance_bias:
+            self.bias_pair = tuple(t(k).to(torch.float32).contiguous() for k in ("bias_scale", "bias_rate"))
         if self.qk_norm_eps is not None:
             self.q_norm, self.k_norm = t("q_norm").contiguous(), t("k_norm").contiguous()
         if self.row_norm_eps is not None:   # (zero weights under the padding, where the rows hold zeros anyway)
@@ -289,19 +323,25 @@ class GqaAttention(Mixer):
             self._prepare_rows(qkv, ctx)
         else:
             qkv = ops.linear_rows(x, self.qkv_weight)           # [T, q | k | v (| gates)]
-        gates = qkv[:, self.qkv_width:self.qkv_width + self.n_heads] if self.gated else None
-        if self.conv_taps > 0:
+        gates = qkv[:, self.qkv_width:self.qkv_width + (self.n_heads if self.gated else self.q_width)] if self.gated or self.out_gate else None
+        q = torch.empty((n, self.q_width), dtype=x.dtype, device=x.device)
+        args = ops.KvSiteArgs(kv_site.storage, kv_site.table, self.n_kv, self.head_dim)
+        # nothing stands between the convolution and the attention: it writes queries and cache itself
+        straight = self.conv_taps > 0 and self.position is None and self.qk_norm_eps is None and self.unit_norm_eps is None
+        if straight:
+            ops.causal_conv_cached(qkv[:, :self.qkv_width], self.conv_weight, ctx.cu_q, ctx.tok_seq, ctx.tok_pos, ctx.slots,
+                                   site["conv"].storage, 0, q, args, ctx.err, single=ctx.is_decode and n == ctx.n_seqs)
+        elif self.conv_taps > 0:
             mixed = torch.empty((n, self.qkv_width), dtype=x.dtype, device=x.device)
             ops.causal_conv(qkv[:, :self.qkv_width], self.conv_weight, None, ctx.cu_q, ctx.tok_seq, ctx.slots, site["conv"].storage,
                             0, mixed, single=ctx.is_decode and n == ctx.n_seqs)
             qkv = mixed
-        q = torch.empty((n, self.q_width), dtype=x.dtype, device=x.device)
-        args = ops.KvSiteArgs(kv_site.storage, kv_site.table, self.n_kv, self.head_dim)
         norm_first = self.qk_norm_eps is not None
-        ops.rope_cache_write(qkv, ctx.tok_seq, ctx.tok_pos, ctx.slots, inv_freq, rot_dim, self.n_heads, q, args, writes_cache,
-                             ctx.err, bias=late_bias, unit_norm_eps=self.qk_norm_eps if norm_first else self.unit_norm_eps,
-                             norm_dim=self.key_dim, has_kv=self.own_kv, interleaved=self.interleaved, norm_first=norm_first,
-                             q_norm=self.q_norm, k_norm=self.k_norm)
+        if not straight:
+            ops.rope_cache_write(qkv, ctx.tok_seq, ctx.tok_pos, ctx.slots, inv_freq, rot_dim, self.n_heads, q, args, writes_cache,
+                                 ctx.err, bias=late_bias, unit_norm_eps=self.qk_norm_eps if norm_first else self.unit_norm_eps,
+                                 norm_dim=self.key_dim, has_kv=self.own_kv, interleaved=self.interleaved, norm_first=norm_first,
+                                 q_norm=self.q_norm, k_norm=self.k_norm)
         blocks = None
         if self.pool > 0:
             blocks = ops.KvSiteArgs(site["blocks"].storage, site["blocks"].table, self.n_kv, self.head_dim)
@@ -310,21 +350,28 @@ class GqaAttention(Mixer):
         fast = ctx.attention == "auto" and x.dtype == torch.bfloat16 and self.head_dim in ops.FAST_ATTENTION_HEAD_DIMS
         # (pooled rows: single tokens run on the kernel of portions too. What a token reads there is bounded by its window
         # and a row per block before it, a few pages that need no cut into runs; the split-K kernel does not take the rows.)
+        more = {}   # what only this kind of attention asks for
+        if self.shared_values:
+            more["shared_values"] = True
+        if self.bias_pair is not None:
+            more["distance_bias"] = self.bias_pair
         if fast and ctx.is_decode and n == ctx.n_seqs and self.pool == 0:
             n_splits = self.decode_splits(ctx)
             ops.attention_decode(q, attended, ctx.cu_q, ctx.tok_pos, ctx.slots, args, self.n_heads, ctx.n_seqs, self.scale,
                                  self.window, n_splits, ctx.decode_scratch, ctx.err, self.decode_plan(ctx), sinks=self.sinks,
-                                 chunk=self.chunk, softcap=self.softcap)
+                                 chunk=self.chunk, softcap=self.softcap, **more)
         elif fast:
             ops.attention_prefill(q, attended, ctx.cu_q, ctx.tok_pos, ctx.slots, args, self.n_heads, ctx.n_seqs, ctx.max_q_len,
                                   self.scale, self.window, ctx.err, max_kv_len=ctx.max_kv_len, sinks=self.sinks,
-                                  chunk=self.chunk, softcap=self.softcap, blocks=blocks, pool=self.pool)
+                                  chunk=self.chunk, softcap=self.softcap, blocks=blocks, pool=self.pool, **more)
         else:
             ops.attention_generic(q, attended, ctx.cu_q, ctx.tok_pos, ctx.slots, args, self.n_heads, ctx.n_seqs, ctx.max_q_len,
                                   self.scale, self.window, ctx.err, scratch=ctx.decode_scratch, max_kv_len=ctx.max_kv_len,
-                                  sinks=self.sinks, chunk=self.chunk, softcap=self.softcap, blocks=blocks, pool=self.pool)
+                                  sinks=self.sinks, chunk=self.chunk, softcap=self.softcap, blocks=blocks, pool=self.pool, **more)
         if self.gated:
             ops.head_gate(attended, gates, self.n_heads)
+        elif self.out_gate:
+            ops.sigmoid_gate(attended, gates)
         return ops.linear(attended, self.o_weight, self.o_bias_t) if self.o_bias_t is not None else ops.linear_rows(attended, self.o_weight)
 
     def _prepare_rows(self, qkv, ctx) -> None:

@@ -45,7 +45,7 @@ class TensorSpec:
 
     init  how the random-weights mode draws it: "matrix" N(0, 0.02), "bias" N(0, 0.02), "norm" 1 + N(0, 0.1),
           "logit" N(0, 1), "conv" (1 + N(0, 0.5)) / sqrt(taps), "fraction" sigmoid(N(0, 1)), "rate" N(-1, 1),
-          "low_rank" N(0, 0.5)
+          "low_rank" N(0, 0.5), "share" 1/n + N(0, 0.1), "identity" the unit matrix + N(0, 0.1/n), "positive" |N(0, 1)|
     shape an extent of -1 takes whatever size the file holds (the part reads it from the tensor it is bound to)
     keep  "compute": kept in the activation dtype (bfloat16, or float32 on the 32-bit path)
           "stored":  kept as the file stores it if that is a 32-bit float, else as "compute"
@@ -148,6 +148,11 @@ class Pending:
         """The float32 tensor that will be added (for diagnosis; not on the product path)."""
         raise NotImplementedError
 
+    def normed_rows(self, rows: torch.Tensor, norm: "Norm", err: torch.Tensor):
+        """The named tokens' rows of the finished stream under `norm`, where this can be had without resolving the whole
+        stream (what an output head reads); None otherwise."""
+        return None
+
 
 class PendingPair(Pending):
     """The outputs of two sublayers that read the same input (a parallel layer): their sum goes into the stream, summed
@@ -222,6 +227,61 @@ class PendingNormed(Pending):
                 y = y * r.row_weight[:, None]
             y = y[r.dest.long()].view(-1, r.top, y.shape[1]).sum(1)
         return y * torch.rsqrt(y.square().mean(-1, keepdim=True) + self.eps) * self.weight.to(torch.float32)
+
+
+class PendingStreams(Pending):
+    """Several residual streams under way: the float32 rows as the sublayer before last left them (`source`: [T, n, W], or [T, W] for
+    one row that stands for all n), the last sublayer's output y (a tensor, a `RowSum`, or None where nothing is pending) and the
+    part that says how y enters (`mix`: its `mix`, `out_weight`). The single stream `hidden` of the model is what they start from
+    and, at the end, their sum."""
+    __slots__ = ("source", "n", "y", "rows", "mix")
+
+    def __init__(self, source: torch.Tensor, n: int, y=None, mix=None):
+        self.source, self.n, self.mix = source, n, mix
+        self.rows = (y.dest, y.top, y.row_weight) if isinstance(y, RowSum) else None
+        self.y = y.rows if isinstance(y, RowSum) else y
+
+    @property
+    def coefficients(self):
+        return None if self.y is None else (self.mix.mix, self.mix.out_weight)
+
+    def enter(self, into, norm, convolution, ctx, site) -> tuple:
+        """(what the next sublayer reads, the streams as they stand then). `into`: the next sublayer's part of role "streams";
+        `norm` its norm, `convolution` the filter in front of it (or None) with its state at `site`."""
+        from .. import ops
+        new = None if self.y is None else torch.empty((self.source.shape[0], self.n, self.source.shape[-1]), dtype=torch.float32,
+                                                      device=self.source.device)
+        after = self.source if new is None else new
+        fused = norm.elementwise() if hasattr(norm, "elementwise") else None
+        if fused is None:   # a norm that sums over the row reads u as a row of its own
+            u = torch.empty((self.source.shape[0], self.source.shape[-1]), dtype=torch.float32, device=self.source.device)
+            ops.streams_norm(self.source, self.n, self.coefficients, self.y, into.in_weight, new, None, u, y_rows=self.rows)
+            h = norm.forward(u, None)
+            return (h if convolution is None else convolution.forward(h, ctx, site)), after
+        h = torch.empty((self.source.shape[0], self.source.shape[-1]), dtype=fused[0].dtype, device=self.source.device)
+        conv = None if convolution is None else convolution.on_norm(ctx, site)
+        ops.streams_norm(self.source, self.n, self.coefficients, self.y, into.in_weight, new, fused, h, conv=conv, y_rows=self.rows)
+        return h, after
+
+    def total(self) -> torch.Tensor:
+        """The sum of the streams, float32 [T, W]."""
+        from .. import ops
+        out = torch.empty((self.source.shape[0], self.source.shape[-1]), dtype=torch.float32, device=self.source.device)
+        ops.streams_norm(self.source, self.n, self.coefficients, self.y, None, None, None, out, y_rows=self.rows)
+        return out
+
+    def add_to(self, hidden: torch.Tensor) -> None:
+        hidden.copy_(self.total())
+
+
+    def normed_rows(self, rows, norm, err):
+        fused = norm.elementwise() if hasattr(norm, "elementwise") else None
+        if fused is None:
+            return None
+        from .. import ops
+        out = torch.empty((rows.numel(), self.source.shape[-1]), dtype=fused[0].dtype, device=self.source.device)
+        ops.streams_norm(self.source, self.n, self.coefficients, self.y, None, None, fused, out, rows=rows, err=err, y_rows=self.rows)
+        return out
 
 
 class RowSum:

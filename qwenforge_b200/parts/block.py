@@ -8,7 +8,7 @@ from __future__ import annotations
 import torch
 
 from ..cache import BundleNeed
-from .base import Norm, Part, PendingNormed, PendingPair, PendingScaled
+from .base import Norm, Part, Pending, PendingNormed, PendingPair, PendingScaled, PendingStreams
 from .registry import build_part, register_part
 
 
@@ -168,6 +168,64 @@ class ParallelBlock(Part):
         return PendingPair(mixed, self.feed_forward.forward(h, ctx) if self.feed_forward is not None else None)
 
 
+class StreamsBlock(Part):
+    """Several residual streams (hyper-connections): with X[0..n-1] the streams, all equal to the embedding's output at the start,
+        u = sum_s a[s] X[s];   y = sublayer(filter(norm(u)));   X[r] <- sum_s M[s, r] X[s] + b[r] y
+    for the mixer and then, if the layer has one, for the feed-forward, each with coefficients of its own. Reads the layer spec's
+    parts `mixer_streams`, `mixer_norm`, `mixer` (and `mixer_input`, the filter, if there is one), and `feed_forward_streams`,
+    `feed_forward_norm`, `feed_forward` (and `feed_forward_input`). What a sublayer leaves stays pending with its coefficients
+    (`PendingStreams`): entering the streams, the next read, its norm and its filter are one kernel. The streams live between
+    the blocks in the pending object; the model's `hidden` is the row they start from and receives their sum at the end."""
+
+    accepts_pending = (PendingStreams,)
+
+    def __init__(self, layer_spec):
+        self.kind = "streams"
+        part = lambda role, name: build_part(role, layer_spec.part(name)) if name in layer_spec.parts else None
+        self.sublayers = []
+        for name, role in (("mixer", "mixer"), ("feed_forward", "feed_forward")):
+            if name in layer_spec.parts:
+                self.sublayers.append((name, build_part("streams", layer_spec.part(name + "_streams")),
+                                       build_part("norm", layer_spec.part(name + "_norm")), part("mixer_input", name + "_input"),
+                                       build_part(role, layer_spec.part(name))))
+        self.n = self.sublayers[0][1].streams
+        if self.sublayers[0][0] != "mixer" or any(s[1].streams != self.n for s in self.sublayers):
+            raise ValueError("streams: a layer has a mixer, and its sublayers work on as many streams")
+
+    def sub_parts(self):
+        return [p for _, *parts in self.sublayers for p in parts if p is not None]
+
+    def cache_need(self):
+        items = []
+        for name, _, _, filter_, sublayer in self.sublayers:
+            if filter_ is not None and filter_.cache_need() is not None:
+                items.append((name + "_input", filter_.cache_need()))
+            if name == "mixer" and sublayer.cache_need() is not None:
+                items.append(("mixer", sublayer.cache_need()))
+        return BundleNeed(tuple(items)) if items else None
+
+    def forward(self, hidden, delta, ctx, site, writes_cache):
+        if not writes_cache:
+            raise ValueError("streams: a layer whose inputs keep a state cannot read another entry's cache")
+        if not isinstance(delta, PendingStreams):
+            if isinstance(delta, Pending):
+                delta.add_to(hidden)
+            elif delta is not None:
+                from .. import ops
+                ops.residual_add(hidden, delta)
+            delta = PendingStreams(hidden, self.n)
+        at = lambda name: site.get(name) if site is not None else None
+        for name, streams, norm, filter_, sublayer in self.sublayers:
+            x, source = delta.enter(streams, norm, filter_, ctx, at(name + "_input"))
+            if name == "mixer":
+                y = sublayer.forward(x, ctx, at("mixer"), True)
+            else:   # a feed-forward that leaves several rows per token hands them over unsummed
+                y = (getattr(sublayer, "forward_rows", None) or sublayer.forward)(x, ctx)
+            delta = PendingStreams(source, self.n, y, streams)
+        return delta
+
+
+register_part("block", "streams", StreamsBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "sandwich_norm", SandwichBlock)

@@ -11,7 +11,7 @@
 Options, each a parameter of the spec:
   router_bias  z = R h + r, a float32 bias per expert, added before the choice
   gate         "clamped": expert(v) = D_e (g * sigmoid(alpha g) * (u + 1)) with g = min(G_e v, limit), u = clamp(U_e v, -limit, limit)
-               (`limit`, `alpha`) instead of the SwiGLU; the weight is then on the output
+               (`limit`, `alpha`) instead of the SwiGLU (a weight on the input multiplies both halves before they are clamped)
   shared       one more expert of the same form with sizes of its own (`size`, `limit`) that every token gets, added to the
                chosen experts' sum; with `gated` it is multiplied by sigmoid(s . h), one number per token
   gate         "none": the experts have no gate, expert(v) = D_e act(U_e v) with `activation` one of the library's (the square
@@ -56,8 +56,8 @@ class RoutedExperts(FeedForward):
         self.router_bias = bool(p.get("router_bias", False))
         self.gate = str(p.get("gate", "swiglu"))
         self.limit, self.alpha = float(p.get("limit") or 0.0), float(p.get("alpha") or 0.0)
-        if self.gate not in ("swiglu", "clamped", "none") or (self.gate == "clamped" and (self.weight_on != "output" or self.limit <= 0)):
-            raise ValueError("routed_experts: gate is 'swiglu', 'clamped' or 'none'; the clamped gate takes a positive limit and the weight on the output")
+        if self.gate not in ("swiglu", "clamped", "none") or (self.gate == "clamped" and self.limit <= 0):
+            raise ValueError("routed_experts: gate is 'swiglu', 'clamped' or 'none'; the clamped gate takes a positive limit")
         self.activation = str(p.get("activation") or "relu2")
         if self.gate == "none" and (self.weight_on != "output" or self.activation not in ops.ACTIVATIONS):
             raise ValueError("routed_experts: experts without a gate take one of the library's activations and the weight on the output")
@@ -186,6 +186,10 @@ class RoutedExperts(FeedForward):
             ops.expert_linear(x, self.gate_up, plan, act, gather=True, activation=self.activation)
             ops.expert_linear(act, self.down, plan, rows)
             return RowSum(rows, plan.dest, self.top, plan.sorted_weight)
+        # A weight on the expert's input moves behind its first product (G (w h) = w (G h), and the same for U), where it
+        # meets float32 sums.
+        on_input = self.weight_on == "input"
+        scale, row_weight = (plan.sorted_weight, None) if on_input else (None, plan.sorted_weight)
         if self.gate == "clamped":
             act = torch.empty((plan.pairs, self.inter), dtype=x.dtype, device=x.device)
             rows = torch.empty((plan.pairs, self.hidden), dtype=x.dtype, device=x.device)
@@ -193,23 +197,20 @@ class RoutedExperts(FeedForward):
                     and ops.tc_gemm_grouped_takes(act, self.down, plan):
                 # long steps: both products on the tcgen05 tensor cores, the clamped gate in the first one's epilogue
                 ops.moe_gather(x, plan, rows, False)
-                ops.tc_gemm_grouped(ops.TC_SWIGLU, rows, self.gate_up, plan, act, None, ctx.err, clamp=(self.limit, self.alpha))
+                ops.tc_gemm_grouped(ops.TC_SWIGLU, rows, self.gate_up, plan, act, scale, ctx.err, clamp=(self.limit, self.alpha))
                 y = torch.empty_like(rows)
                 ops.tc_gemm_grouped(ops.TC_PLAIN, act, self.down, plan, y, None, ctx.err)
-                return RowSum(y, plan.dest, self.top, plan.sorted_weight)
+                return RowSum(y, plan.dest, self.top, row_weight)
             # otherwise the rows are read through the plan's row map: the clamped gate in the product's epilogue where the small
             # tensor-core tile takes the operands, else both halves in one product and the gate behind it
             if self.limit > 0 and ops.expert_gate_takes(x, self.gate_up, plan):
-                ops.expert_gate_up(x, self.gate_up, plan, act, None, gather=True, clamp=(self.limit, self.alpha))
+                ops.expert_gate_up(x, self.gate_up, plan, act, scale, gather=True, clamp=(self.limit, self.alpha))
             else:
                 gate_up = torch.empty((plan.pairs, 2 * self.inter), dtype=x.dtype, device=x.device)
                 ops.expert_linear(x, self.gate_up, plan, gate_up, gather=True)
-                ops.clamped_glu(gate_up, self.limit, self.alpha, act)
+                ops.clamped_glu(gate_up, self.limit, self.alpha, act, **({"row_scale": scale} if on_input else {}))
             ops.expert_linear(act, self.down, plan, rows)
-            return RowSum(rows, plan.dest, self.top, plan.sorted_weight)
-        # A weight on the expert's input moves behind its first product (G (w h) = w (G h), and the same for U), where it
-        # meets float32 sums.
-        on_input = self.weight_on == "input"
+            return RowSum(rows, plan.dest, self.top, row_weight)
         act = torch.empty((plan.pairs, self.inter), dtype=x.dtype, device=x.device)
         rows = torch.empty((plan.pairs, self.hidden), dtype=x.dtype, device=x.device)
         if tile_rows == ops.kernels.GROUP_LARGE_TILE_ROWS and ops.tc_gemm_grouped_takes(rows, self.gate_up, plan, ops.TC_SWIGLU) \
@@ -217,13 +218,13 @@ class RoutedExperts(FeedForward):
             # long steps: both products on the tcgen05 tensor cores, the gate in the first one's epilogue (its tiled copies
             # want the sorted rows in memory, so they are gathered first)
             ops.moe_gather(x, plan, rows, False)
-            ops.tc_gemm_grouped(ops.TC_SWIGLU, rows, self.gate_up, plan, act, plan.sorted_weight if on_input else None, ctx.err)
+            ops.tc_gemm_grouped(ops.TC_SWIGLU, rows, self.gate_up, plan, act, scale, ctx.err)
             y = torch.empty_like(rows)
             ops.tc_gemm_grouped(ops.TC_PLAIN, act, self.down, plan, y, None, ctx.err)
-            return RowSum(y, plan.dest, self.top, None if on_input else plan.sorted_weight)
+            return RowSum(y, plan.dest, self.top, row_weight)
         # otherwise the sorted rows are read through the plan's row map and never stored
         if ops.expert_gate_takes(x, self.gate_up, plan):   # the gate in the product's epilogue
-            ops.expert_gate_up(x, self.gate_up, plan, act, plan.sorted_weight if on_input else None, gather=True)
+            ops.expert_gate_up(x, self.gate_up, plan, act, scale, gather=True)
         else:
             gate_up = torch.empty((plan.pairs, 2 * self.inter), dtype=x.dtype, device=x.device)
             ops.expert_linear(x, self.gate_up, plan, gate_up, gather=True)
@@ -232,7 +233,7 @@ class RoutedExperts(FeedForward):
             else:
                 ops.swiglu(gate_up, act)
         ops.expert_linear(act, self.down, plan, rows)
-        return RowSum(rows, plan.dest, self.top, None if on_input else plan.sorted_weight)
+        return RowSum(rows, plan.dest, self.top, row_weight)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

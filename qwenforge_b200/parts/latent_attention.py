@@ -1,4 +1,4 @@
-"""Latent attention without positions: queries and keys/values both go through a low-rank latent, and the key/value
+"""Latent attention: queries and keys/values both go through a low-rank latent, and the key/value
 latent is all that is kept per position.
 
   a = rmsnorm(Dq h) * nq,   q = Uq a            queries, `heads` heads of `dim`
@@ -11,10 +11,17 @@ latent is all that is kept per position.
   w_ij = exp(score_ij) / (exp(sink_head) + sum_{j' <= i} exp(score_ij'))  a learned sink per head joins the denominator
   result = O concat_heads(out_i)
 
+With a rotated part (`rot_dim`, `position`) every head's query has rot_dim components more, the position's rotation applied to
+them, and Dkv h has rot_dim rows more: ONE rotated key part e_j, shared by all heads and not normed, cached behind the latent:
+      score_ij = scale * ((Uk^T q_i) . c_j + qr_i . e_j) = scale * [Uk^T q_i | qr_i] . [c_j | e_j]
+  which is the same attention over rows of kv_rank + rot_dim numbers; of the weighted sum only the first kv_rank are read on.
+  Where that size lies under one that the tensor-core kernels have, rows are filled up to it with zeros.
+
 Dq and Dkv run as one product (float32 out: both norms read 32-bit sums); the two norms and the cache write are one
 kernel (`ops.latent_norm_cache`); the per-head maps into and out of the latent space are one grouped launch each
 (`ops.head_linear`). Nothing here knows a model: ranks, head sizes, scale and eps come from the spec, `q_rank` 0 means
-queries straight from h, `sinks` false means a plain softmax, `window` limits the keys like any attention's.
+queries straight from h, `sinks` false means a plain softmax, `window` limits the keys like any attention's, `rot_dim` 0 means no
+positions at all.
 """
 from __future__ import annotations
 
@@ -24,12 +31,14 @@ from .. import ops
 from ..cache import PAGE_TOKENS, KvNeed
 from .attention import TC_PREFILL_MIN_TOKENS
 from .base import Mixer, TensorSpec
-from .registry import register_part
+from .registry import build_part, register_part
 
 
 class LatentAttention(Mixer):
-    """params: hidden_size, num_heads, head_dim, value_dim, kv_rank, q_rank, scale, eps, sinks (bool), window.
-    tensors: q_down [q_rank, W], q_norm [q_rank], q_up [H*dim, q_rank] (q_rank 0: q_up [H*dim, W] alone), kv_down [kv_rank, W],
+    """params: hidden_size, num_heads, head_dim, value_dim, kv_rank, q_rank, scale, eps, sinks (bool), window, rot_dim, position
+    (PartSpec of a rotation of neighbours over rot_dim components, with rot_dim only).
+    tensors: q_down [q_rank, W], q_norm [q_rank], q_up [H*(dim+rot_dim), q_rank], head by head [dim | rot_dim] (q_rank 0: q_up
+    [.., W] alone), kv_down [kv_rank + rot_dim, W],
     kv_norm [kv_rank], k_up [H*dim, kv_rank], v_up [H*vdim, kv_rank], sink [H], o_weight [W, H*vdim]."""
 
     def __init__(self, spec):
@@ -45,20 +54,31 @@ class LatentAttention(Mixer):
         self.eps = float(p["eps"])
         self.has_sinks = bool(p.get("sinks", False))
         self.window = int(p.get("window") or 0)
-        if self.kv_rank > ops.GENERIC_MAX_HEAD_DIM:
-            raise ValueError(f"latent_attention: kv_rank {self.kv_rank} > {ops.GENERIC_MAX_HEAD_DIM} is not supported by the attention kernels")
+        self.rot_dim = int(p.get("rot_dim") or 0)
+        self.position = build_part("position", p["position"]) if self.rot_dim else None
+        if self.rot_dim and (not self.position.interleaved or self.position.rotary_dim != self.rot_dim):
+            raise ValueError("latent_attention: the rotated part is turned whole, neighbours paired")
+        # what a cache row holds: the latent, the rotated key part, and zeros up to a size that the tensor-core kernels have
+        held = self.kv_rank + self.rot_dim
+        self.row_dim = min((d for d in ops.FAST_ATTENTION_HEAD_DIMS if d >= held), default=held) if self.rot_dim else held
+        if self.row_dim > ops.GENERIC_MAX_HEAD_DIM:
+            raise ValueError(f"latent_attention: rows of {self.row_dim} > {ops.GENERIC_MAX_HEAD_DIM} are not supported by the attention kernels")
         self.down_weight = self.q_norm = self.kv_norm = self.q_up = self.k_absorb = self.v_up = self.sinks = self.o_weight = None
+
+    def sub_parts(self):
+        return [self.position] if self.position is not None else []
 
     def tensor_specs(self):
         h, d, v, r, q, w = self.n_heads, self.head_dim, self.value_dim, self.kv_rank, self.q_rank, self.hidden
-        specs = [TensorSpec(self.file_name("kv_down"), (r, w)), TensorSpec(self.file_name("kv_norm"), (r,), init="norm"),
+        qd = d + self.rot_dim
+        specs = [TensorSpec(self.file_name("kv_down"), (r + self.rot_dim, w)), TensorSpec(self.file_name("kv_norm"), (r,), init="norm"),
                  TensorSpec(self.file_name("k_up"), (h * d, r)), TensorSpec(self.file_name("v_up"), (h * v, r)),
                  TensorSpec(self.file_name("o_weight"), (w, h * v))]
         if q:
             specs += [TensorSpec(self.file_name("q_down"), (q, w)), TensorSpec(self.file_name("q_norm"), (q,), init="norm"),
-                      TensorSpec(self.file_name("q_up"), (h * d, q))]
+                      TensorSpec(self.file_name("q_up"), (h * qd, q))]
         else:
-            specs.append(TensorSpec(self.file_name("q_up"), (h * d, w)))
+            specs.append(TensorSpec(self.file_name("q_up"), (h * qd, w)))
         if self.has_sinks:
             specs.append(TensorSpec(self.file_name("sink"), (h,), init="logit", keep="float32"))
         return specs
@@ -67,14 +87,14 @@ class LatentAttention(Mixer):
         libs = {"latent_cache", "attention_generic", "grouped_gemm"}
         if dtype == torch.float32:
             libs.add("gemm_f32")
-        elif self.kv_rank in ops.FAST_ATTENTION_HEAD_DIMS:
+        elif self.row_dim in ops.FAST_ATTENTION_HEAD_DIMS:
             libs |= {"attention_decode", "attention_prefill", "skinny_gemm"}
-            if self.kv_rank in ops.TC_ATTENTION_HEAD_DIMS:
+            if self.row_dim in ops.TC_ATTENTION_HEAD_DIMS:
                 libs.add("attention_prefill_tc")
         return libs
 
     def cache_need(self):
-        return KvNeed(1, self.kv_rank, self.window, planes=1)
+        return KvNeed(1, self.row_dim, self.window, planes=1)
 
     def bind(self, tensors, dtype, device):
         t = lambda logical: tensors[self.file_name(logical)]
@@ -99,22 +119,29 @@ class LatentAttention(Mixer):
     def _latents(self, x, ctx, args, writes_cache):
         """The queries of the step's tokens, [T, H * dim], after the key/value latents went into the cache."""
         n = x.shape[0]
+        turned = {} if self.position is None else {"rotated": (self.position.fused_rotary()[0], self.position.amplitude)}
         down = ops.linear_rows(x, self.down_weight, out_dtype=torch.float32)
         if not self.q_rank:
             ops.latent_norm_cache(down, 0, None, self.kv_norm, self.eps, ctx.tok_seq, ctx.tok_pos, ctx.slots, None, args,
-                                  writes_cache, ctx.err)
+                                  writes_cache, ctx.err, **turned)
             return ops.linear_rows(x, self.q_up)
         q_latent = torch.empty((n, self.q_rank), dtype=x.dtype, device=x.device)
         ops.latent_norm_cache(down, self.q_rank, self.q_norm, self.kv_norm, self.eps, ctx.tok_seq, ctx.tok_pos, ctx.slots,
-                              q_latent, args, writes_cache, ctx.err)
+                              q_latent, args, writes_cache, ctx.err, **turned)
         return ops.linear_rows(q_latent, self.q_up)
 
     def forward(self, x, ctx, site, writes_cache):
-        n, h, r = x.shape[0], self.n_heads, self.kv_rank
+        n, h, r = x.shape[0], self.n_heads, self.row_dim
         args = ops.KvSiteArgs(site.storage, site.table, 1, r)
         q = self._latents(x, ctx, args, writes_cache)
         q_in_latent = torch.empty((n, h * r), dtype=x.dtype, device=x.device)
-        ops.head_linear(q, self.k_absorb, q_in_latent)
+        if self.position is None:
+            ops.head_linear(q, self.k_absorb, q_in_latent)
+        else:
+            qd = self.head_dim + self.rot_dim
+            ops.rotate_heads(q, qd, self.head_dim, q_in_latent, r, self.kv_rank, self.position.fused_rotary()[0], self.position.amplitude,
+                             ctx.tok_pos, h)
+            ops.head_linear(q, self.k_absorb, q_in_latent, x_pitch=qd, out_pitch=r)
         attended = torch.empty_like(q_in_latent)
         fast = ctx.attention == "auto" and x.dtype == torch.bfloat16 and r in ops.FAST_ATTENTION_HEAD_DIMS
         if fast and ctx.is_decode and n == ctx.n_seqs:
@@ -135,16 +162,19 @@ class LatentAttention(Mixer):
                                   self.scale, self.window, ctx.err, scratch=ctx.decode_scratch, max_kv_len=ctx.max_kv_len,
                                   sinks=self.sinks, shared_values=True)
         values = torch.empty((n, h * self.value_dim), dtype=x.dtype, device=x.device)
-        ops.head_linear(attended, self.v_up, values)
+        if r == self.kv_rank:
+            ops.head_linear(attended, self.v_up, values)
+        else:
+            ops.head_linear(attended, self.v_up, values, x_pitch=r)
         return ops.linear_rows(values, self.o_weight)
 
     def decode_plan(self, ctx, n_splits: int) -> torch.Tensor:
         """The decode attention's plan of this step, shared through the step's memo by every layer of this shape."""
-        key = ("latent_attention.decode_plan", self.n_heads, self.kv_rank, self.window, n_splits)
+        key = ("latent_attention.decode_plan", self.n_heads, self.row_dim, self.window, n_splits)
         memo = ctx.step_memo if ctx.step_memo is not None else {}
         plan = memo.get(key)
         if plan is None:
-            plan = memo[key] = ops.attention_decode_plan(ctx.cu_q, ctx.tok_pos, ctx.slots, 1, self.kv_rank, self.n_heads,
+            plan = memo[key] = ops.attention_decode_plan(ctx.cu_q, ctx.tok_pos, ctx.slots, 1, self.row_dim, self.n_heads,
                                                          ctx.n_seqs, self.window, n_splits, ctx.decode_scratch)
         return plan
 
@@ -152,7 +182,7 @@ class LatentAttention(Mixer):
         """The most blocks that may share one sequence's latents (see `GqaAttention.decode_splits`)."""
         span = ctx.max_kv_len if self.window <= 0 else min(ctx.max_kv_len, self.window + PAGE_TOKENS)
         pages = max(1, -(-span // PAGE_TOKENS))
-        warps = ops.attention_decode_warps(self.kv_rank)
+        warps = ops.attention_decode_warps(self.row_dim)
         return max(1, min(-(-pages // warps), 64))
 
 

@@ -86,6 +86,10 @@ class DynamicTanh(Norm):
         ops.add_dyt_norm_shift(hidden, delta, second, self.weight, self.bias, self.alpha, out, shift[0], shift[1], shift[2], shifted)
         return out, shifted
 
+    def elementwise(self):
+        """(weight, bias, alpha): this norm needs nothing but the element itself, so any kernel that has it may apply it."""
+        return self.weight, self.bias, self.alpha
+
     def step_weights(self):
         return [self.weight, self.bias]
 

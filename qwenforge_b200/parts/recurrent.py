@@ -26,9 +26,18 @@ Two more kinds decay every ROW of S by a number of its own (a decay per head and
       S <- diag(a_t) S + k_t v_t^T;  y_t = S^T q_t (AFTER the token);  out = Wo (rms_per_head(y; n) * silu(Wg h)),
       the norm's weight [vdim] shared by the heads
 
+And one corrects what the state already says about a key before it adds to it:
+
+  channel_delta (the gated delta rule with a decay per head and key channel, `ops.delta_scan`, `ops.delta_token`)
+      q, k, v = silu(causal_conv(W h)) in heads (a group of heads may share one q and k), q and k divided by their lengths,
+      q / sqrt(dim);  beta = sigmoid(Wb h) per head;  g = exp(-exp(A) softplus(A2 A1 h + b)) per head and key channel;
+      S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  y = S^T q (AFTER the token);
+      out = Wo (rms_per_head(y; n) * sigmoid(G2 G1 h)), the norm's weight [vdim] shared by the heads
+
 The state lives in the sequence cache as ONE float32 row per sequence and schedule entry (`StateNeed`), zeroed when a
 sequence starts: [S | n | m] for the matrix memory, [S | the convolution's last taps - 1 inputs] for the state space,
-[S | the last token's h] for the time mixing, [S] for the gated linear attention.
+[S | the last token's h] for the time mixing, [S] for the gated linear attention, [S | the convolution's last inputs] for the
+delta rule.
 The gates' pre-activations are products with float32 results, and everything from there to the scan's output is
 float32 in both precisions; the other projections and the convolution carry the activation dtype.
 """
@@ -331,6 +340,114 @@ class GatedLinearAttention(Mixer):
         return ops.linear_rows(out, self.o_weight)
 
 
+class ChannelDelta(Mixer):
+    """params: hidden_size, num_heads, num_kv_heads (heads of q and k), head_dim, value_dim, conv_taps, eps, and optionally rank and
+    gate_rank (of the decay's and the gate's low-rank pairs; read from the tensors where absent).
+    tensors: q_weight, k_weight [G*dim, W], v_weight [H*vdim, W], q_conv, k_conv, v_conv [.., taps], b_weight [H, W], rate_log [H],
+    a1 [rank, W], a2 [H*dim, rank], dt_bias [H*dim], g1 [gate_rank, W], g2 [H*vdim, gate_rank], norm [vdim], o_weight [W, H*vdim]."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.hidden, self.n_heads, self.groups = int(p["hidden_size"]), int(p["num_heads"]), int(p["num_kv_heads"])
+        self.dim, self.vdim, self.taps = int(p["head_dim"]), int(p["value_dim"]), int(p["conv_taps"])
+        self.eps, self.rank, self.gate_rank = float(p["eps"]), _rank_of(p), _rank_of(p, "gate_rank")
+        if self.n_heads % self.groups:
+            raise ValueError(f"channel_delta: {self.n_heads} heads are not divisible by {self.groups} heads of q and k")
+        if self.dim > ops.OUTER_STATE_MAX_DIM or not 1 <= self.taps <= ops.CONV_MAX_TAPS:
+            raise ValueError(f"channel_delta: head_dim up to {ops.OUTER_STATE_MAX_DIM} and 1 to {ops.CONV_MAX_TAPS} taps are supported")
+        self.qk_width, self.v_width = self.groups * self.dim, self.n_heads * self.vdim
+        self.channels = 2 * self.qk_width + self.v_width
+        self.conv_offset = -(-(self.n_heads * self.dim * self.vdim) // 4) * 4     # (16-byte rows for the convolution's kernels)
+        self.state_floats = -(-(self.conv_offset + (self.taps - 1) * self.channels) // 4) * 4
+        self.proj_weight = self.conv_weight = self.b_weight = self.rate_log = self.a2 = self.dt_bias = self.g2 = self.norm = None
+        self.norm_heads = self.o_weight = None
+
+    def tensor_specs(self):
+        f, h, d, v, w = self.file_name, self.n_heads, self.dim, self.vdim, self.hidden
+        qk = self.qk_width
+        specs = [TensorSpec(f("q_weight"), (qk, w)), TensorSpec(f("k_weight"), (qk, w)), TensorSpec(f("v_weight"), (h * v, w))]
+        specs += [TensorSpec(f(n + "_conv"), (rows, self.taps), init="conv", keep="float32") for n, rows in (("q", qk), ("k", qk), ("v", h * v))]
+        return specs + [TensorSpec(f("b_weight"), (h, w)), TensorSpec(f("rate_log"), (h,), init="rate", keep="float32"),
+                        TensorSpec(f("a1"), (self.rank, w)), TensorSpec(f("a2"), (h * d, self.rank), init="low_rank"),
+                        TensorSpec(f("dt_bias"), (h * d,), init="rate", keep="float32"), TensorSpec(f("g1"), (self.gate_rank, w)),
+                        TensorSpec(f("g2"), (h * v, self.gate_rank), init="low_rank"), TensorSpec(f("norm"), (v,), init="norm"),
+                        TensorSpec(f("o_weight"), (w, h * v))]
+
+    def kernel_libraries(self, dtype):
+        return {"recurrent", "delta_rule"} | ({"gemm_f32"} if dtype == torch.float32 else {"skinny_gemm"})
+
+    def cache_need(self):
+        return StateNeed((self.state_floats,), torch.float32)
+
+    def bind(self, tensors, dtype, device):
+        t = lambda logical: tensors[self.file_name(logical)]
+        self.rank, self.gate_rank = int(t("a1").shape[0]), int(t("g1").shape[0])
+        # one product for everything that reads h and is kept in the activation dtype, each low-rank middle filled up to whole 16 bytes
+        filled = lambda m: m if m.shape[0] % 8 == 0 else torch.cat((m, m.new_zeros((8 - m.shape[0] % 8, m.shape[1]))), dim=0)
+        pieces = [t("q_weight"), t("k_weight"), t("v_weight")]
+        if self.channels % 8:
+            pieces.append(pieces[0].new_zeros((8 - self.channels % 8, self.hidden)))
+        self.a_first = sum(p.shape[0] for p in pieces)
+        pieces.append(filled(t("a1")))
+        self.g_first = self.a_first + pieces[-1].shape[0]
+        pieces.append(filled(t("g1")))
+        self.proj_weight = torch.cat(pieces, dim=0).contiguous()
+        self.conv_weight = torch.cat((t("q_conv"), t("k_conv"), t("v_conv")), dim=0).to(torch.float32).contiguous()
+        self.b_weight, self.a2, self.g2 = t("b_weight").contiguous(), t("a2").contiguous(), t("g2").contiguous()
+        self.rate_log, self.dt_bias = (t(k).to(torch.float32).contiguous() for k in ("rate_log", "dt_bias"))
+        self.norm, self.o_weight = t("norm").contiguous(), t("o_weight")
+        self.norm_heads = self.norm.repeat(self.n_heads).contiguous()      # the one weight [vdim] under every head
+
+    def step_weights(self):
+        return [self.proj_weight, self.conv_weight, self.b_weight, self.a2, self.g2, self.rate_log, self.dt_bias, self.norm, self.o_weight]
+
+    def _gates(self, x, proj):
+        """The decays' pre-activations and beta's logits (float32 sums), and the output gate's logits."""
+        z = ops.linear_rows(proj[:, self.a_first:self.a_first + self.rank], self.a2, out_dtype=torch.float32)
+        gate = ops.linear_rows(proj[:, self.g_first:self.g_first + self.gate_rank], self.g2)
+        return z, gate
+
+    def forward(self, x, ctx, site, writes_cache):
+        if not writes_cache:
+            raise ValueError("channel_delta: a recurrent state cannot be read from another schedule entry")
+        n, h, d, v, qk = x.shape[0], self.n_heads, self.dim, self.vdim, self.qk_width
+        single = ctx.is_decode and n == ctx.n_seqs
+        mixed = torch.empty((n, self.channels), dtype=x.dtype, device=x.device)
+        conv = lambda: ops.causal_conv_silu(proj[:, :self.channels], self.conv_weight, None, ctx.cu_q, ctx.tok_seq, ctx.slots, site.storage,
+                                            self.conv_offset, mixed, single=single)
+        if runs_side_by_side(x):   # few rows: beta's product beside the one that feeds everything, the gates' beside the convolution
+            main, side = fork(x)
+            with torch.cuda.stream(side):
+                logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)
+            proj = ops.linear_rows(x, self.proj_weight)
+            join(main, side, logit)
+            main, side = fork(proj)
+            with torch.cuda.stream(side):
+                z, gate = self._gates(x, proj)
+            conv()
+            join(main, side, z, gate)
+        else:
+            logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)
+            proj = ops.linear_rows(x, self.proj_weight)                                  # [T, q | k | v | A1 h | G1 h]
+            z, gate = self._gates(x, proj)
+            conv()
+        q, k, value = mixed[:, :qk], mixed[:, qk:2 * qk], mixed[:, 2 * qk:]
+        args = (q, k, value, z, self.dt_bias, self.rate_log, logit, ctx.cu_q, ctx.slots, site.storage, 0, h, self.groups, d, v, d ** -0.5)
+        out = torch.empty((n, h * v), dtype=x.dtype, device=x.device)
+        if single and v <= ops.DELTA_FUSED_MAX_VDIM:
+            ops.delta_token(*args, norm=self.norm, eps=self.eps, gate=gate, out=out)
+            return ops.linear_rows(out, self.o_weight)
+        y = torch.empty((n, h * v), dtype=torch.float32, device=x.device)
+        if single:
+            ops.delta_token(*args, y=y)
+        else:
+            ops.delta_scan(*args, y)
+        ops.gated_group_norm(y, gate, self.norm_heads, self.eps, out, h, h, "sigmoid", False)
+        return ops.linear_rows(out, self.o_weight)
+
+
+register_part("mixer", "channel_delta", ChannelDelta)
 register_part("mixer", "matrix_memory", MatrixMemory)
 register_part("mixer", "time_mix", TimeMix)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)

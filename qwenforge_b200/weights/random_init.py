@@ -17,6 +17,18 @@ from .loader import merge_specs
 from .safetensors_io import save_safetensors
 
 
+_MIXING = ("share", "identity", "positive")
+
+
+def _mixing(spec: TensorSpec, noise: torch.Tensor) -> torch.Tensor:
+    """Coefficients of several streams (what they are read and passed on with), and numbers that are to be positive."""
+    if spec.init == "share":
+        return 1.0 / spec.shape[0] + 0.1 * noise
+    if spec.init == "identity":
+        return torch.eye(*spec.shape, device=noise.device) + 0.1 / spec.shape[0] * noise
+    return noise.abs()
+
+
 def draw_tensor(spec: TensorSpec, generator: torch.Generator, store_dtype: torch.dtype) -> torch.Tensor:
     if any(int(extent) < 0 for extent in spec.shape):
         raise ValueError(f"tensor {spec.name!r}: an extent that only a weight file gives cannot be drawn at random; "
@@ -38,6 +50,8 @@ def draw_tensor(spec: TensorSpec, generator: torch.Generator, store_dtype: torch
         value = noise - 1.0
     elif spec.init == "low_rank":    # the second matrix of a low-rank pair that sets a gate: wide enough to move it
         value = 0.5 * noise
+    elif spec.init in _MIXING:
+        value = _mixing(spec, noise)
     else:
         raise ValueError(f"tensor {spec.name!r}: unknown init {spec.init!r}")
     return value if spec.keep == "stored" else value.to(store_dtype)
@@ -57,6 +71,10 @@ def random_state_on_device(specs, seed: int, dtype: torch.dtype, device) -> dict
     for name, spec in merge_specs(specs).items():
         if spec.keep == "int32":
             out[name] = torch.zeros(spec.shape, dtype=torch.int32, device=device)
+            continue
+        if spec.init in _MIXING:   # (a few numbers each)
+            kept = torch.float32 if spec.keep in ("stored", "float32") else dtype
+            out[name] = _mixing(spec, torch.randn(spec.shape, generator=generator, dtype=torch.float32, device=device)).to(kept)
             continue
         if spec.init not in ("norm", "matrix", "bias", "logit", "conv", "fraction", "rate", "low_rank"):
             raise ValueError(f"tensor {spec.name!r}: unknown init {spec.init!r}")

@@ -140,7 +140,7 @@ def gather_keys(site, slot, lo, hi):
 
 
 def attention_generic(q, out, cu_q, tok_pos, slots, site, n_heads, n_seqs, max_q_len, scale, window, err, scratch=None, max_kv_len=None,
-                      sinks=None, shared_values=False, chunk=0, softcap=0.0, blocks=None, pool=0):
+                      sinks=None, shared_values=False, chunk=0, softcap=0.0, blocks=None, pool=0, distance_bias=None):
     d, kvh = site.head_dim, site.kv_heads
     groups = n_heads // kvh
     for s in range(n_seqs):
@@ -167,6 +167,9 @@ def attention_generic(q, out, cu_q, tok_pos, slots, site, n_heads, n_seqs, max_q
             scores = torch.einsum("hd,hjd->hj", qt, k) * scale
             if softcap > 0:
                 scores = softcap * torch.tanh(scores / softcap)
+            if distance_bias is not None:
+                far = torch.arange(p - lo, -1, -1, device=q.device, dtype=torch.float64)
+                scores = scores - _f(distance_bias[0])[:, None] * torch.log1p(_f(distance_bias[1])[:, None] * far[None, :])
             if sinks is not None:   # one more term in the denominator, with no value
                 weights = torch.softmax(torch.cat((scores, _f(sinks)[:, None]), dim=-1), -1)[:, :-1]
             else:
@@ -207,17 +210,21 @@ def sandwich_norm(hidden, y, post_weight, post_eps, next_weight=None, next_eps=0
         out.copy_(_rms(hidden, next_weight, next_eps).to(out.dtype))
 
 
-def clamped_glu(gate_up, limit, alpha, out):
+def clamped_glu(gate_up, limit, alpha, out, row_scale=None):
     inter = gate_up.shape[1] // 2
-    g = _f(gate_up[:, :inter]).clamp(max=limit)
-    u = _f(gate_up[:, inter:]).clamp(min=-limit, max=limit)
+    s = 1.0 if row_scale is None else _f(row_scale)[:, None]
+    g = (s * _f(gate_up[:, :inter])).clamp(max=limit)
+    u = (s * _f(gate_up[:, inter:])).clamp(min=-limit, max=limit)
     out.copy_((g * torch.sigmoid(alpha * g) * (u + 1)).to(out.dtype))
 
 
-def latent_norm_cache(down, q_rank, q_norm, kv_norm, eps, tok_seq, tok_pos, slots, q_latent, site, write_cache, err, latent_out=None):
+def latent_norm_cache(down, q_rank, q_norm, kv_norm, eps, tok_seq, tok_pos, slots, q_latent, site, write_cache, err, latent_out=None, rotated=None):
     if q_rank:
         q_latent.copy_(_rms(down[:, :q_rank], q_norm, eps).to(q_latent.dtype))
-    c = _rms(down[:, q_rank:], kv_norm, eps)
+    r = kv_norm.numel()
+    c = _rms(down[:, q_rank:q_rank + r], kv_norm, eps)
+    if rotated is not None:
+        turned = _turn_pairs(_f(down[:, q_rank + r:]), tok_pos, *rotated)
     if latent_out is not None:
         latent_out.copy_(c.to(latent_out.dtype))
     if not write_cache:
@@ -229,13 +236,32 @@ def latent_norm_cache(down, q_rank, q_norm, kv_norm, eps, tok_seq, tok_pos, slot
         pos = int(tok_pos[t])
         page = int(site.table[slot, pos // PAGE])
         assert page >= 0, "reference: write to a page that is not held"
-        site.storage[page, 0, 0, pos % PAGE, :] = c[t].to(site.storage.dtype)
+        site.storage[page, 0, 0, pos % PAGE, :r] = c[t].to(site.storage.dtype)
+        if rotated is not None:
+            site.storage[page, 0, 0, pos % PAGE, r:r + turned.shape[1]] = turned[t].to(site.storage.dtype)
 
 
-def head_linear(x, weight, out):
+def _turn_pairs(x, tok_pos, inv_freq, amplitude):
+    """x [T, ..., R]: neighbours turned by position * inv_freq, cosine and sine times the amplitude."""
+    angle = (tok_pos.to(torch.float32).unsqueeze(-1) * inv_freq.to(torch.float32)).to(torch.float64)
+    angle = angle.view((x.shape[0],) + (1,) * (x.dim() - 2) + (inv_freq.numel(),))
+    cos, sin = angle.cos() * amplitude, angle.sin() * amplitude
+    a, b = x[..., 0::2], x[..., 1::2]
+    return torch.stack((a * cos - b * sin, b * cos + a * sin), dim=-1).reshape(x.shape)
+
+
+def rotate_heads(x, x_pitch, x_first, out, out_pitch, out_first, inv_freq, amplitude, tok_pos, n_heads):
+    rot, n = 2 * inv_freq.numel(), x.shape[0]
+    part = _f(x).view(n, n_heads, x_pitch)[:, :, x_first:x_first + rot]
+    to = out.view(n, n_heads, out_pitch)
+    to[:, :, out_first:out_first + rot] = _turn_pairs(part, tok_pos, inv_freq, amplitude).to(out.dtype)
+    to[:, :, out_first + rot:] = 0
+
+
+def head_linear(x, weight, out, x_pitch=0, out_pitch=0):
     groups, n, k = weight.shape
-    y = torch.einsum("tgk,gnk->tgn", _f(x).view(x.shape[0], groups, k), _f(weight))
-    out.copy_(y.reshape(x.shape[0], groups * n).to(out.dtype))
+    y = torch.einsum("tgk,gnk->tgn", _f(x).view(x.shape[0], groups, x_pitch or k)[:, :, :k], _f(weight))
+    out.view(x.shape[0], groups, out_pitch or n)[:, :, :n] = y.to(out.dtype)
 
 
 class _Routing:
@@ -536,6 +562,102 @@ def causal_conv(x, weight, bias, cu_q, tok_seq, slots, state, offset, out, singl
     causal_conv_silu(x, weight, bias, cu_q, tok_seq, slots, state, offset, out, activation="none")
 
 
+def causal_conv_cached(x, weight, cu_q, tok_seq, tok_pos, slots, state, offset, out, site, err, single=False):
+    whole = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    causal_conv(x, weight, None, cu_q, tok_seq, slots, state, offset, whole)
+    width = out.shape[1]
+    out.copy_(whole[:, :width])
+    planes = site.storage.shape[1]
+    rows = whole[:, width:].reshape(x.shape[0], planes, site.kv_heads, site.head_dim)
+    for t in range(x.shape[0]):
+        slot = int(slots[int(tok_seq[t])])
+        if slot < 0:
+            continue
+        pos = int(tok_pos[t])
+        page = int(site.table[slot, pos // PAGE])
+        assert page >= 0, "reference: write to a page that is not held"
+        site.storage[page, :, :, pos % PAGE, :] = rows[t]
+
+
+def sigmoid_gate(x, gate):
+    x.copy_((_f(x) * torch.sigmoid(_f(gate))).to(x.dtype))
+
+
+def delta_scan(q, k, v, z, bias, rate_log, logit, cu_q, slots, state, s_offset, n_heads, n_groups, dim, vdim, q_scale, y):
+    per, size = n_heads // n_groups, n_heads * dim * vdim
+    unit = lambda x: x / torch.sqrt(x.square().sum(-1, keepdim=True) + 1e-6)
+    spread = lambda x: unit(_f(x).view(x.shape[0], n_groups, dim)).repeat_interleave(per, dim=1)
+    qs, ks, vs = spread(q) * q_scale, spread(k), _f(v).view(v.shape[0], n_heads, vdim)
+    rate = torch.nn.functional.softplus(_f(z) + _f(bias)).view(-1, n_heads, dim)
+    g = torch.exp(-torch.exp(_f(rate_log))[None, :, None] * rate)
+    beta = torch.sigmoid(_f(logit))
+    for s in range(cu_q.numel() - 1):
+        slot = int(slots[s])
+        S = torch.zeros(n_heads, dim, vdim, dtype=torch.float64, device=q.device)
+        if slot >= 0:
+            S = _f(state[slot, s_offset:s_offset + size]).view(n_heads, dim, vdim).clone()
+        for t in range(int(cu_q[s]), int(cu_q[s + 1])):
+            S = g[t][:, :, None] * S
+            u = beta[t][:, None] * (vs[t] - torch.einsum("hdv,hd->hv", S, ks[t]))
+            S = S + ks[t][:, :, None] * u[:, None, :]
+            y[t] = torch.einsum("hdv,hd->hv", S, qs[t]).reshape(-1).float()
+        if slot >= 0:
+            state[slot, s_offset:s_offset + size] = S.reshape(-1).float()
+
+
+def delta_token(q, k, v, z, bias, rate_log, logit, cu_q, slots, state, s_offset, n_heads, n_groups, dim, vdim, q_scale, y=None,
+                norm=None, eps=0.0, gate=None, out=None):
+    made = torch.empty(q.shape[0], n_heads * vdim, dtype=torch.float32, device=q.device)
+    delta_scan(q, k, v, z, bias, rate_log, logit, cu_q, slots, state, s_offset, n_heads, n_groups, dim, vdim, q_scale, made)
+    if y is not None:
+        y.copy_(made)
+    if out is not None:
+        r = _f(made).view(-1, n_heads, vdim)
+        r = r / torch.sqrt(r.square().mean(-1, keepdim=True) + eps) * _f(norm)
+        out.copy_((r.reshape(made.shape) * torch.sigmoid(_f(gate))).to(out.dtype))
+
+
+def streams_norm(source, n_streams, coefficients, y, in_weight, new=None, norm=None, out=None, conv=None, rows=None, err=None,
+                 y_rows=None):
+    X = _f(source)
+    if X.dim() == 2:
+        X = X[:, None, :].expand(-1, n_streams, -1)
+    Y = X
+    if y is not None:
+        mix, out_w = coefficients
+        y = _f(y)
+        if y_rows is not None:
+            dest, top, row_weight = y_rows
+            if row_weight is not None:
+                y = y * _f(row_weight)[:, None]
+            y = y[dest.long()].view(-1, top, y.shape[1]).sum(1)
+        Y = torch.einsum("sr,tsw->trw", _f(mix), X) + _f(out_w)[None, :, None] * y[:, None, :]
+    if new is not None:
+        new.copy_(Y.to(torch.float32))
+    u = Y.sum(1) if in_weight is None else torch.einsum("s,tsw->tw", _f(in_weight), Y)
+    if rows is not None:
+        u = u[rows.long()]
+    if norm is None:
+        out.copy_(u.to(out.dtype))
+        return
+    h = torch.tanh(norm[2] * u) * _f(norm[0]) + _f(norm[1])
+    if conv is not None:
+        taps, cu_q, slots, _, state, offset = conv
+        n, c = taps.shape[1], taps.shape[0]
+        filtered = torch.empty_like(h)
+        for s in range(cu_q.numel() - 1):
+            b, e, slot = int(cu_q[s]), int(cu_q[s + 1]), int(slots[s])
+            before = torch.zeros(n - 1, c, dtype=torch.float64, device=h.device)
+            if slot >= 0:
+                before = _f(state[slot, offset:offset + (n - 1) * c]).view(n - 1, c)
+            padded = torch.cat((before, h[b:e]))
+            filtered[b:e] = h[b:e] + sum(padded[j:j + e - b] * _f(taps)[:, j] for j in range(n))
+            if slot >= 0 and n > 1 and e > b:
+                state[slot, offset:offset + (n - 1) * c] = padded[padded.shape[0] - (n - 1):].reshape(-1).float()
+        h = filtered
+    out.copy_(h.to(out.dtype))
+
+
 def add_dyt_norm(hidden, a, b, weight, bias, alpha, out):
     if a is not None or b is not None:
         hidden += ((0 if a is None else _f(a)) + (0 if b is None else _f(b))).to(hidden.dtype)
@@ -582,7 +704,8 @@ def pool_cache_write(cu_q, tok_pos, slots, site, blocks, pool, max_q_len, err):
             blocks.storage[page, 1, :, block % PAGE, :] = v.mean(1).to(blocks.storage.dtype)
 
 
-ALL = dict(rows_prepare=rows_prepare, bias_glu=bias_glu, add_rms_norm_scaled=add_rms_norm_scaled, residual_add_scaled=residual_add_scaled, rms_norm_cols=rms_norm_cols,
+ALL = dict(causal_conv_cached=causal_conv_cached, sigmoid_gate=sigmoid_gate, delta_scan=delta_scan, delta_token=delta_token, streams_norm=streams_norm,
+           rotate_heads=rotate_heads, rows_prepare=rows_prepare, bias_glu=bias_glu, add_rms_norm_scaled=add_rms_norm_scaled, residual_add_scaled=residual_add_scaled, rms_norm_cols=rms_norm_cols,
            mix_rows=mix_rows, shift_mix=shift_mix, channel_decay=channel_decay, outer_state_scan_rows=outer_state_scan_rows,
            gated_rows=gated_rows, causal_conv=causal_conv, add_dyt_norm=add_dyt_norm, add_dyt_norm_shift=add_dyt_norm_shift, residual_add_pair=residual_add_pair, stream_pair=stream_pair,
            head_gate=head_gate, pool_cache_write=pool_cache_write, bias_act=bias_act, softcap_=softcap_, stabilized_gates=stabilized_gates, decay_gates=decay_gates,
