@@ -6,6 +6,7 @@ decode at batch 1 and 64, and the same decode rate end to end through the Python
     python bench.py --design mefepel     # instead: the Mefepel presets beside the Qwen2 presets of equal layer sizes
     python bench.py --design zebovik     # the same for the Zebovik presets (attention in blocks, mLSTM and Mamba-2 layers)
     python bench.py --design rarevik     # the same for the Rarevik presets (parallel layers, windows with pooled blocks, routed experts)
+    python bench.py --design dapupel     # the Dapupel presets (several streams, latent attention, delta rule, experts) beside Rarevik's and Qwen2's
     python bench.py --design gatosun     # the same for the Gatosun presets (window attention beside time mixing, gated linear attention, experts in groups)
                                          # (prompt and decode rates, device times by kind of kernel), as one JSON line
 
@@ -46,7 +47,7 @@ def parse():
     p.add_argument("--workload", default=None, choices=sorted(WORKLOADS),
                    help="run only this named workload (3B: 16 unequal prompts then 256 steps; 7B: batch 64 to context "
                         "8192 at temperature 0.7) and print its line")
-    p.add_argument("--design", default=None, choices=["mefepel", "zebovik", "rarevik", "gatosun"],
+    p.add_argument("--design", default=None, choices=["mefepel", "zebovik", "rarevik", "gatosun", "dapupel"],
                    help="measure another design's prefill and decode beside the Qwen2 model of equal size (kernel by "
                         "kernel), instead of the default workload")
     p.add_argument("--no-workloads", action="store_true", help="leave the 3B and 7B workloads out of the default run's points")
@@ -361,9 +362,13 @@ class _StubTokenizer:
 DESIGN_PAIRS = {"mefepel": [("mefepel-0.5b", "qwen2.5-0.5b", None), ("mefepel-3b", "qwen2.5-3b", None)],
                 "zebovik": [("zebovik-0.5b", "qwen2.5-0.5b", None), ("zebovik-3b", "qwen2.5-3b", None)],
                 "rarevik": [("rarevik-0.5b", "qwen2.5-0.5b", None), ("rarevik-3b", "qwen2.5-3b", None)],
-                "gatosun": [("gatosun-0.5b", "qwen2.5-0.5b", None), ("gatosun-3b", "qwen2.5-3b", None)]}
+                "gatosun": [("gatosun-0.5b", "qwen2.5-0.5b", None), ("gatosun-3b", "qwen2.5-3b", None)],
+                "dapupel": [("dapupel-0.5b", "rarevik-0.5b", None), ("dapupel-0.5b", "qwen2.5-0.5b", None),
+                            ("dapupel-3b", "rarevik-3b", None), ("dapupel-3b", "qwen2.5-3b", None)]}
 # what a kernel's label (ops/timing.py) counts as, so that like is laid beside like
-KERNEL_KINDS = (("attention_prefill", "attention (prompt)"), ("attention_decode", "attention (decode)"),
+KERNEL_KINDS = (("streams_norm", "streams + norm + filter"), ("rotate_heads", "rotation of queries"), ("delta_", "recurrent scan"),
+                ("sigmoid_gate", "gates"), ("causal_conv_cached", "convolution + cache write"),
+                ("attention_prefill", "attention (prompt)"), ("attention_decode", "attention (decode)"),
                 ("attention_generic", "attention (plain)"), ("head_linear", "per-head products"),
                 ("expert_linear", "expert products"), ("tc_gemm_grouped", "expert products"), ("scaled_swiglu", "gates"),
                 ("linear_rows", "products of the step's rows"), ("moe_", "routing"), ("linear", "library products"),
@@ -452,9 +457,14 @@ def design_point(preset, layers, args, pk, torch):
 
 def run_design(args, pk, torch):
     points = []
+    made = {}   # (a preset that stands in several pairs is measured once)
     with torch.inference_mode():
+        def point(preset, layers):
+            if (preset, layers) not in made:
+                made[preset, layers] = design_point(preset, layers, args, pk, torch)
+            return made[preset, layers]
         for ours, theirs, layers in DESIGN_PAIRS[args.design]:
-            points.append({"design": design_point(ours, layers, args, pk, torch), "beside": design_point(theirs, layers, args, pk, torch)})
+            points.append({"design": point(ours, layers), "beside": point(theirs, layers)})
     first = points[0]["design"]
     line = {"metric": f"decode tokens/s ({args.design}, {first['preset']}, batch {first['decode_batch']}, context {first['decode_context']})",
             "value": first["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3),

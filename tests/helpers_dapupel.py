@@ -82,3 +82,26 @@ def make_model_dir(cfg: dict, seed: int, folder=None, store_dtype=torch.float32,
     (folder / "config.json").write_text(json.dumps(cfg))
     save_safetensors(folder / "model.safetensors", {k: v.to(store_dtype) for k, v in weights.items()})
     return folder, weights
+
+
+def steady(cfg: dict, weights: dict, seed: int = 0) -> dict:
+    """The same weights with routers that choose by clear margins, so that bfloat16 rounding flips (next to) no choice: a few channels
+    carry a large number of either sign per token, no sublayer writes to them, the norms saturate there, and the routers read
+    nothing else. The logits do not see those channels."""
+    gen = torch.Generator().manual_seed(seed)
+    n, width = 8, int(cfg["width"])
+    w = {k: v.clone() for k, v in weights.items()}
+    w["final.norm"][:n] = 0
+    w["final.norm.b"][:n] = 0
+    sign = lambda *shape: torch.randint(0, 2, shape, generator=gen).float() * 2 - 1
+    w["embed"][:, :n] = 16.0 * sign(int(cfg["vocab"]), n)
+    for name in list(w):
+        if name.endswith("mix.o") or name.endswith(".down"):
+            w[name][:n] = 0
+        elif name.endswith(".router"):
+            experts = w[name].shape[0]
+            w[name].zero_()
+            w[name][:, :n] = (3.0 * sign(experts, n) * (1.0 + torch.rand(experts, n, generator=gen))).to(torch.bfloat16).float()
+        elif name.endswith("canon2"):
+            w[name][:n, :-1] *= 0.25
+    return w

@@ -272,8 +272,8 @@ def random_weights(cfg, seed):
         last = name.rsplit(".", 1)[-1]
         normal = lambda std, mean=0.0: torch.randn(shape, generator=gen) * std + mean
         if ".hc" in name:
-            t = normal(0.3, 1.0 / n) if last == "in" else normal(0.3, 1.0) if last == "out" else \
-                normal(0.3 / n) + 0.8 * torch.eye(n)
+            t = normal(0.3, 1.0 / n) if last == "in" else normal(0.15, 0.4) if last == "out" else \
+                normal(0.3 / n) + 0.9 * torch.eye(n)
         elif last == "alpha":
             t = normal(0.1, 0.7)
         elif ".norm" in name and last != "b":
@@ -293,7 +293,7 @@ def random_weights(cfg, seed):
         elif last == "b":
             t = normal(2.0 * shape[-1] ** -0.5)
         elif last in ("gate", "up"):
-            t = normal(3.0 * shape[-1] ** -0.5)
+            t = normal(2.0 * shape[-1] ** -0.5)
         elif last == "router":
             t = normal(2.0 * shape[-1] ** -0.5)
         elif name == "embed":
