@@ -6,15 +6,23 @@
 // q and k of head / (heads / groups). Everything from q, k, v (activation dtype) on is float32. A sequence whose slot is -1 (a
 // padding entry) runs from a zero state and stores nothing.
 //
-// Steps of many tokens take two kernels. `delta_prepare` works out, a warp per (token, head), what does not depend on the state:
-// the unit vectors, the decays and beta, packed for the scan as rows [g | k | q] of `padded` floats each. `delta_scan` then walks
-// every sequence's tokens in order. Eight lanes share a column of S, the rows dealt out in fours, so a warp has four columns
-// and a block of four warps sixteen; a lane's part of S stays in registers from the sequence's first token of the step to its
-// last. A token costs a lane four multiply-adds per row of its part (decay, S^T k, update, S^T q) and three shuffles
-// whose latency the chain waits for (u_t needs the whole column's S^T k); the shuffles of S^T q are put off and shared by
-// eight tokens, one lane ending up with one token's sum. Tokens are staged through shared memory DS_TOKENS at a time by
-// asynchronous copies, the next tile under way while one is worked on. The order of operations per token does not depend on
-// the cut of the sequence.
+// Steps of many tokens take two kernels. Token by token, every token's u would wait for a sum over the whole column of S
+// before the next token's could begin. So four tokens go together: with S the state before the four, G_i = g_1 .. g_i and
+// G_(i,j) = g_(j+1) .. g_i (products of numbers between 0 and 1, no quotients),
+//
+//   u_i = beta_i (v_i - S^T (G_i k_i) - sum_(j<i) c_ij u_j),   c_ij = k_i . G_(i,j) k_j
+//   y_i = S^T (G_i q_i) + sum_(j<=i) d_ij u_j,                 d_ij = q_i . G_(i,j) k_j
+//   S  <- diag(G_4) S + sum_j (G_(4,j) k_j) u_j^T
+//
+// which is the same recurrence, written out. `delta_prepare` works out all that does not depend on the state, a warp per
+// (head, four tokens): the unit vectors, the decays and their products, c, d and beta, packed as one record. `delta_scan` walks
+// every sequence's records in order. Eight lanes share two columns of S, the rows dealt out in fours, so a warp has eight columns
+// and a block of two warps sixteen (what a lane reads from shared memory serves both its columns: the shared memory's pace is
+// what bounds a block); a lane's part of S stays in registers, two rows to a register pair and one instruction, from the
+// sequence's first token of the step to its last. A column's eight sums (four for u, four for y) are formed together and reduced
+// together, each lane ending up with one of them. Records are staged through shared memory DS_TOKENS tokens at a time by asynchronous copies, the next
+// ones under way while these are worked on. Fours are counted from a sequence's first token of the step; the last one is
+// filled up with tokens that do nothing (g = 1, k = q = 0).
 //
 // Steps of one token per sequence take one kernel, `delta_token`: a block per (sequence, head, up to 128 columns) that does all of
 // it: unit vectors, decays, both products with the old state in one pass over S (y = (g S)^T q + (k . q) u), the update, and,
@@ -22,215 +30,362 @@
 #include "mma.cuh"
 
 #define DS_LANES 8
-#define DS_WARPS 4
-#define DS_COLS (DS_WARPS * 32 / DS_LANES)   // columns of S per block
+#define DS_WARPS 2
+#define DS_EACH 2                                       // columns of S per lane
+#define DS_COLS (DS_WARPS * 32 / DS_LANES * DS_EACH)    // and per block
 #define DELTA_LENGTH_EPS 1e-6f               // under the root of the unit vectors' length
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float channel_decay_of(float z, float rate_exp) { return expf(-rate_exp * softplus(z)); }
 
-// packed: [heads][n_tokens][3][padded] (g, k, q; zeros beyond dim); beta: [heads][n_tokens]
-template <typename T>
-__global__ void __launch_bounds__(256)
+// Two float32 in one register pair, worked on by one instruction, each half rounded as by fmaf and __fmul_rn.
+__device__ __forceinline__ unsigned long long pair_of(float lo, float hi) {
+    unsigned long long p;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(lo), "f"(hi));
+    return p;
+}
+__device__ __forceinline__ float2 unpair(unsigned long long p) {
+    float2 v;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(v.x), "=f"(v.y) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ float sum_of_pair(unsigned long long p) {
+    const float2 v = unpair(p);
+    return v.x + v.y;
+}
+__device__ __forceinline__ unsigned long long fma_pair(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ unsigned long long mul_pair(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+
+// A record of four tokens: [Gk 4][Gq 4][Gk' 4][G] rows of `padded` floats (zeros beyond dim; the four in this order: G_i k_i, G_i q_i,
+// G_(4,j) k_j and G_4), then c (8: c_21, c_31, c_32, c_41, c_42, c_43, two unused), d (16: row i, column j), beta (4), four unused.
+#define DS_GROUP 4
+#define DS_ROWS 13
+#define DS_SCALARS 32
+__host__ __device__ constexpr long long record_floats(int padded) { return (long long)DS_ROWS * padded + DS_SCALARS; }
+// The record of a sequence's first four tokens of the step (records of sequences do not overlap: see ops.delta_scan).
+__device__ __forceinline__ int first_record(int begin, int seq) { return begin / DS_GROUP + seq; }
+
+template <typename T, int NI>
+__global__ void __launch_bounds__(128)
 delta_prepare_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_stride, const float* __restrict__ z,
                      int z_stride, const float* __restrict__ bias, const float* __restrict__ rate_log, const float* __restrict__ logit,
-                     int logit_stride, int n_tokens, int heads, int groups, int dim, int padded, float q_scale,
-                     float* __restrict__ packed, float* __restrict__ beta) {
+                     int logit_stride, const int* __restrict__ cu_q, int n_records, int heads, int groups, int dim, float q_scale,
+                     float* __restrict__ packed) {
     grid_chain_entry();
-    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (item >= (long long)n_tokens * heads) return;
-    const int lane = threadIdx.x & 31, t = (int)(item / heads), head = (int)(item % heads), group = head / (heads / groups);
-    const T* qt = q + (size_t)t * q_stride + group * dim;
-    const T* kt = k + (size_t)t * k_stride + group * dim;
-    const float* zt = z + (size_t)t * z_stride + (size_t)head * dim;
-    float qv[8], kv[8], zv[8], qs = 0.f, ks = 0.f;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {   // dim <= 256
-        const int d = lane + 32 * i;
-        qv[i] = d < dim ? Num<T>::to_f(qt[d]) : 0.f;
-        kv[i] = d < dim ? Num<T>::to_f(kt[d]) : 0.f;
-        zv[i] = d < dim ? zt[d] + bias[(size_t)head * dim + d] : 0.f;
-        qs = fmaf(qv[i], qv[i], qs);
-        ks = fmaf(kv[i], kv[i], ks);
-    }
-    const float q_inv = q_scale / sqrtf(warp_sum(qs) + DELTA_LENGTH_EPS), k_inv = 1.f / sqrtf(warp_sum(ks) + DELTA_LENGTH_EPS);
+    constexpr int P = 32 * NI;
+    const int lane = threadIdx.x & 31, item = blockIdx.x * 4 + (threadIdx.x >> 5), seq = blockIdx.y;
+    const int head = item % heads, four = item / heads, group = head / (heads / groups);
+    const int begin = cu_q[seq], len = cu_q[seq + 1] - begin, t0 = four * DS_GROUP;
+    if (t0 >= len) return;
+    float qv[4][NI], kv[4][NI], g[4][NI];
     const float rate = expf(rate_log[head]);
-    float* row = packed + ((size_t)head * n_tokens + t) * 3 * padded;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int d = lane + 32 * i;
-        if (d >= padded) break;
-        row[d] = d < dim ? channel_decay_of(zv[i], rate) : 0.f;
-        row[padded + d] = kv[i] * k_inv;
-        row[2 * padded + d] = qv[i] * q_inv;
+    for (int j = 0; j < 4; ++j) {
+        const bool there = t0 + j < len;
+        const size_t t = begin + t0 + j;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int d = lane + 32 * i;
+            const bool in = there && d < dim;
+            qv[j][i] = in ? Num<T>::to_f(q[t * q_stride + group * dim + d]) : 0.f;
+            kv[j][i] = in ? Num<T>::to_f(k[t * k_stride + group * dim + d]) : 0.f;
+            g[j][i] = in ? z[t * z_stride + (size_t)head * dim + d] : 0.f;
+        }
     }
-    if (lane == 0) beta[(size_t)head * n_tokens + t] = 1.f / (1.f + expf(-logit[(size_t)t * logit_stride + head]));
+    float raw_beta = 0.f;
+    if (lane < 4 && t0 + lane < len) raw_beta = logit[(size_t)(begin + t0 + lane) * logit_stride + head];
+    float b[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) b[i] = lane + 32 * i < dim ? bias[(size_t)head * dim + lane + 32 * i] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        float qs = 0.f, ks = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            qs = fmaf(qv[j][i], qv[j][i], qs);
+            ks = fmaf(kv[j][i], kv[j][i], ks);
+        }
+        const float q_inv = q_scale / sqrtf(warp_sum(qs) + DELTA_LENGTH_EPS), k_inv = 1.f / sqrtf(warp_sum(ks) + DELTA_LENGTH_EPS);
+        const bool there = t0 + j < len;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            qv[j][i] *= q_inv;
+            kv[j][i] *= k_inv;
+            g[j][i] = there ? channel_decay_of(g[j][i] + b[i], rate) : 1.f;
+        }
+    }
+    float* rec = packed + ((size_t)head * n_records + first_record(begin, seq) + four) * record_floats(P);
+    float sums[16];   // c and d, this lane's parts: d_jj, then for i > j c_ij and d_ij
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int d = lane + 32 * i;
+        float run = 1.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            run *= g[j][i];
+            rec[j * P + d] = run * kv[j][i];
+            rec[(4 + j) * P + d] = run * qv[j][i];
+        }
+        rec[12 * P + d] = d < dim ? run : 0.f;
+    }
+    int at = 0;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        float w[NI], part = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            w[i] = kv[j][i];
+            part = fmaf(qv[j][i], w[i], part);
+        }
+        sums[at++] = part;
+#pragma unroll
+        for (int m = j + 1; m < 4; ++m) {
+            float pc = 0.f, pd = 0.f;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                w[i] *= g[m][i];
+                pc = fmaf(kv[m][i], w[i], pc);
+                pd = fmaf(qv[m][i], w[i], pd);
+            }
+            sums[at++] = pc;
+            sums[at++] = pd;
+        }
+#pragma unroll
+        for (int i = 0; i < NI; ++i) rec[(8 + j) * P + lane + 32 * i] = w[i];
+    }
+    // sixteen sums over the warp, halving the sums with the lanes: lane l ends with sum l / 2
+#pragma unroll
+    for (int o = 16, n = 8; n > 0; o >>= 1, n >>= 1) {
+        const bool upper = lane & o;
+#pragma unroll
+        for (int j = 0; j < n; ++j) {
+            const float mine = upper ? sums[j + n] : sums[j], theirs = upper ? sums[j] : sums[j + n];
+            sums[j] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
+        }
+    }
+    const float total = sums[0] + __shfl_xor_sync(0xffffffffu, sums[0], 1);
+    float* tail = rec + DS_ROWS * P;
+    if (!(lane & 1)) {
+        // order of the sums: d00 c10 d10 c20 d20 c30 d30 | d11 c21 d21 c31 d31 | d22 c32 d32 | d33
+        constexpr signed char place[16] = {8 + 0, 0, 8 + 4, 1, 8 + 8, 3, 8 + 12, 8 + 5, 2, 8 + 9, 4, 8 + 13, 8 + 10, 5, 8 + 14, 8 + 15};
+        int to = 0;
+#pragma unroll
+        for (int x = 0; x < 16; ++x) to = x == lane / 2 ? place[x] : to;
+        tail[to] = total;
+    } else if (lane < 12) {   // the upper triangle of d
+        constexpr signed char zero[6] = {8 + 1, 8 + 2, 8 + 3, 8 + 6, 8 + 7, 8 + 11};
+        int to = 0;
+#pragma unroll
+        for (int x = 0; x < 6; ++x) to = x == lane / 2 ? zero[x] : to;
+        tail[to] = 0.f;
+    }
+    if (lane < 4) tail[24 + lane] = t0 + lane < len ? 1.f / (1.f + expf(-raw_beta)) : 0.f;
 }
 
 // R rows of S per lane (a multiple of 4): padded = 8 * R. Lane l of a column has rows 4 * (l + 8 * i) .. + 3.
 template <typename T, int R, int TOKENS>
 __global__ void __launch_bounds__(DS_WARPS * 32)
-delta_scan_kernel(const float* __restrict__ packed, const float* __restrict__ beta, const T* __restrict__ v, int v_stride,
-                  const int* __restrict__ cu_q, const int* __restrict__ slots, float* __restrict__ state, long long slot_stride,
-                  long long s_offset, int n_tokens, int heads, int dim, int vdim, float* __restrict__ y) {
-    grid_chain_entry();
-    constexpr int P = DS_LANES * R, ROW = 3 * P, Q4 = R / 4, THREADS = DS_WARPS * 32;
+delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int v_stride, const int* __restrict__ cu_q,
+                  const int* __restrict__ slots, float* __restrict__ state, long long slot_stride, long long s_offset, int n_records,
+                  int heads, int dim, int vdim, float* __restrict__ y) {
+    constexpr int P = DS_LANES * R, Q4 = R / 4, THREADS = DS_WARPS * 32, FOURS = TOKENS / DS_GROUP;
+    constexpr int REC = (int)record_floats(P);
     extern __shared__ __align__(16) float ds_smem[];
-    float* rows_s = ds_smem;                               // [2][TOKENS][ROW]
-    float* v_s = rows_s + 2 * TOKENS * ROW;                // [2][TOKENS][DS_COLS]
-    float* beta_s = v_s + 2 * TOKENS * DS_COLS;            // [2][TOKENS]
+    float* rec_s = ds_smem;                                // [2][FOURS][REC]
+    float* v_s = rec_s + 2 * FOURS * REC;                  // [2][TOKENS][DS_COLS]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, head = blockIdx.y, seq = blockIdx.z;
-    const int part = lane & (DS_LANES - 1), col_in = warp * (32 / DS_LANES) + lane / DS_LANES, col = blockIdx.x * DS_COLS + col_in;
-    const int begin = cu_q[seq], end = cu_q[seq + 1], slot = slots[seq];
-    if (begin >= end) return;
-    float* column = (slot >= 0 && col < vdim) ? state + slot * slot_stride + s_offset + (long long)head * dim * vdim + col : nullptr;
-    float s[R];
+    const int part = lane & (DS_LANES - 1), col_in = (warp * (32 / DS_LANES) + lane / DS_LANES) * DS_EACH, col = blockIdx.x * DS_COLS + col_in;
+    const int begin = cu_q[seq], len = cu_q[seq + 1] - begin, slot = slots[seq];
+    if (len <= 0) return;
+    float* column = slot >= 0 ? state + slot * slot_stride + s_offset + (long long)head * dim * vdim + col : nullptr;
+    unsigned long long s[DS_EACH][R / 2];   // rows in pairs
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-        const int d = 4 * (part + DS_LANES * (i / 4)) + i % 4;
-        s[i] = (column && d < dim) ? column[(size_t)d * vdim] : 0.f;
-    }
-    constexpr int V_EACH = (TOKENS * DS_COLS + THREADS - 1) / THREADS;
-    float v_next[V_EACH], beta_next = 0.f;
-    // a tile's rows go straight to shared memory; its values and betas pass through registers
-    auto fetch = [&](int t0, int buf) {
-        const int n_here = min(TOKENS, end - t0);
-        const float* from = packed + ((size_t)head * n_tokens + t0) * ROW;
-        float* to = rows_s + buf * TOKENS * ROW;
-        for (int i = threadIdx.x; i < n_here * (ROW / 4); i += THREADS) cp_async_16(to + 4 * i, from + 4 * i, true);
+    for (int c = 0; c < DS_EACH; ++c)
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) {
+            const int d = 4 * (part + DS_LANES * (i / 2)) + 2 * (i % 2);
+            const bool there = column && col + c < vdim;
+            s[c][i] = pair_of(there && d < dim ? column[(size_t)d * vdim + c] : 0.f, there && d + 1 < dim ? column[(size_t)(d + 1) * vdim + c] : 0.f);
+        }
+    constexpr int V_EACH = TOKENS * DS_COLS / THREADS;
+    T v_next[V_EACH];
+    const float* records = packed + ((size_t)head * n_records + first_record(begin, seq)) * REC;
+    auto fetch = [&](int t0, int buf) {   // the records straight to shared memory, the values through registers
+        const int fours = min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP);
+        const float* from = records + (size_t)(t0 / DS_GROUP) * REC;
+        float* to = rec_s + buf * FOURS * REC;
+        for (int i = threadIdx.x; i < fours * (REC / 4); i += THREADS) cp_async_16(to + 4 * i, from + 4 * i, true);
         cp_async_commit();
 #pragma unroll
         for (int u = 0; u < V_EACH; ++u) {
-            const int i = threadIdx.x + u * THREADS, j = i / DS_COLS, c = blockIdx.x * DS_COLS + i % DS_COLS;
-            v_next[u] = (j < n_here && c < vdim) ? Num<T>::to_f(v[(size_t)(t0 + j) * v_stride + (size_t)head * vdim + c]) : 0.f;
+            const int i = threadIdx.x + u * THREADS, j = t0 + i / DS_COLS, c = blockIdx.x * DS_COLS + i % DS_COLS;
+            v_next[u] = (j < len && c < vdim) ? v[(size_t)(begin + j) * v_stride + (size_t)head * vdim + c] : Num<T>::from_f(0.f);
         }
-        if (threadIdx.x < n_here) beta_next = beta[(size_t)head * n_tokens + t0 + threadIdx.x];
     };
     auto stash = [&](int buf) {
 #pragma unroll
-        for (int u = 0; u < V_EACH; ++u) {
-            const int i = threadIdx.x + u * THREADS;
-            if (i < TOKENS * DS_COLS) v_s[buf * TOKENS * DS_COLS + i] = v_next[u];
-        }
-        if (threadIdx.x < TOKENS) beta_s[buf * TOKENS + threadIdx.x] = beta_next;
+        for (int u = 0; u < V_EACH; ++u) v_s[buf * TOKENS * DS_COLS + threadIdx.x + u * THREADS] = Num<T>::to_f(v_next[u]);
     };
-    fetch(begin, 0);
+    fetch(0, 0);
     stash(0);
-    for (int t0 = begin, turn = 0; t0 < end; t0 += TOKENS, ++turn) {
-        const int buf = turn & 1, n_here = min(TOKENS, end - t0);
+    for (int t0 = 0, turn = 0; t0 < len; t0 += TOKENS, ++turn) {
+        const int buf = turn & 1, fours = min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP);
         cp_async_wait<0>();
-        __syncthreads();   // this tile has arrived for everyone, and everyone is done with the other buffer
-        const bool more = t0 + TOKENS < end;
+        __syncthreads();   // these records have arrived for everyone, and everyone is done with the other buffer
+        const bool more = t0 + TOKENS < len;
         if (more) fetch(t0 + TOKENS, buf ^ 1);
-        const float* rows = rows_s + buf * TOKENS * ROW;
         const float* vs = v_s + buf * TOKENS * DS_COLS + col_in;
-        const float* bs = beta_s + buf * TOKENS;
-        auto token = [&](int j) -> float {   // this lane's part of y
-            const float4* g4 = reinterpret_cast<const float4*>(rows + j * ROW) + part;
-            const float4* k4 = reinterpret_cast<const float4*>(rows + j * ROW + P) + part;
-            const float4* q4 = reinterpret_cast<const float4*>(rows + j * ROW + 2 * P) + part;
-            float k[R], a[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int f = 0; f < fours; ++f) {
+            const float* rec = rec_s + (buf * FOURS + f) * REC;
+            const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(rec) + part;   // row r, its quarter i: rows[r * (P / 4) + DS_LANES * i]
+            const float4 c0 = *reinterpret_cast<const float4*>(rec + DS_ROWS * P), c1 = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 4);
+            const float4 beta = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 24);
+            const float4 d = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 8 + 4 * (part & 3));   // this lane's token's row
+            float2 v4[4];
 #pragma unroll
-            for (int i = 0; i < Q4; ++i) {
-                const float4 gg = g4[DS_LANES * i], kk = k4[DS_LANES * i];
-                const float ge[4] = {gg.x, gg.y, gg.z, gg.w}, ke[4] = {kk.x, kk.y, kk.z, kk.w};
+            for (int j = 0; j < 4; ++j) v4[j] = *reinterpret_cast<const float2*>(vs + (4 * f + j) * DS_COLS);
+            float sums[DS_EACH][8];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    k[4 * i + e] = ke[e];
-                    s[4 * i + e] *= ge[e];
-                    a[e] = fmaf(s[4 * i + e], ke[e], a[e]);
+            for (int x = 0; x < 8; ++x) {
+                unsigned long long acc[DS_EACH];
+#pragma unroll
+                for (int i = 0; i < Q4; ++i) {
+                    const ulonglong2 w = rows[x * (P / 4) + DS_LANES * i];
+#pragma unroll
+                    for (int c = 0; c < DS_EACH; ++c) {
+                        acc[c] = i == 0 ? mul_pair(s[c][0], w.x) : fma_pair(s[c][2 * i], w.x, acc[c]);
+                        acc[c] = fma_pair(s[c][2 * i + 1], w.y, acc[c]);
+                    }
                 }
+#pragma unroll
+                for (int c = 0; c < DS_EACH; ++c) sums[c][x] = sum_of_pair(acc[c]);
             }
-            float seen = (a[0] + a[1]) + (a[2] + a[3]);
-#pragma unroll
-            for (int o = 1; o < DS_LANES; o <<= 1) seen += __shfl_xor_sync(0xffffffffu, seen, o);
-            const float u = bs[j] * (vs[j * DS_COLS] - seen);
-            float b[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int i = 0; i < Q4; ++i) {
-                const float4 qq = q4[DS_LANES * i];
-                const float qe[4] = {qq.x, qq.y, qq.z, qq.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s[4 * i + e] = fmaf(k[4 * i + e], u, s[4 * i + e]);
-                    b[e] = fmaf(s[4 * i + e], qe[e], b[e]);
-                }
-            }
-            return (b[0] + b[1]) + (b[2] + b[3]);
-        };
-        for (int j0 = 0; j0 < n_here; j0 += DS_LANES) {
-            float y8[DS_LANES];
-            if (j0 + DS_LANES <= n_here) {
-#pragma unroll
-                for (int j = 0; j < DS_LANES; ++j) y8[j] = token(j0 + j);
-            } else {
-#pragma unroll
-                for (int j = 0; j < DS_LANES; ++j) y8[j] = j0 + j < n_here ? token(j0 + j) : 0.f;
-            }
-            // eight sums over eight lanes, halving: lane `part` ends with token j0 + part's
+            // eight sums over eight lanes, halving: lane `part` ends with sum `part`
 #pragma unroll
             for (int o = DS_LANES / 2; o > 0; o >>= 1) {
                 const bool upper = part & o;
 #pragma unroll
-                for (int j = 0; j < o; ++j) {
-                    const float mine = upper ? y8[j + o] : y8[j], theirs = upper ? y8[j] : y8[j + o];
-                    y8[j] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
+                for (int j = 0; j < o; ++j)
+#pragma unroll
+                    for (int c = 0; c < DS_EACH; ++c) {
+                        const float mine = upper ? sums[c][j + o] : sums[c][j], theirs = upper ? sums[c][j] : sums[c][j + o];
+                        sums[c][j] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
+                    }
+            }
+            float u[DS_EACH][4];
+#pragma unroll
+            for (int c = 0; c < DS_EACH; ++c) {
+                float left[4];   // v_i - S^T G_i k_i
+#pragma unroll
+                for (int j = 0; j < 4; ++j) left[j] = (c == 0 ? v4[j].x : v4[j].y) - __shfl_sync(0xffffffffu, sums[c][0], j, DS_LANES);
+                u[c][0] = beta.x * left[0];
+                u[c][1] = beta.y * fmaf(-c0.x, u[c][0], left[1]);
+                u[c][2] = beta.z * fmaf(-c0.z, u[c][1], fmaf(-c0.y, u[c][0], left[2]));
+                u[c][3] = beta.w * fmaf(-c1.y, u[c][2], fmaf(-c1.x, u[c][1], fmaf(-c0.w, u[c][0], left[3])));
+            }
+            unsigned long long uu[DS_EACH][4];
+#pragma unroll
+            for (int c = 0; c < DS_EACH; ++c)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) uu[c][j] = pair_of(u[c][j], u[c][j]);
+#pragma unroll
+            for (int i = 0; i < Q4; ++i) {
+                const ulonglong2 g = rows[12 * (P / 4) + DS_LANES * i];
+#pragma unroll
+                for (int c = 0; c < DS_EACH; ++c) {
+                    s[c][2 * i] = mul_pair(g.x, s[c][2 * i]);
+                    s[c][2 * i + 1] = mul_pair(g.y, s[c][2 * i + 1]);
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const ulonglong2 k = rows[(8 + j) * (P / 4) + DS_LANES * i];
+#pragma unroll
+                    for (int c = 0; c < DS_EACH; ++c) {
+                        s[c][2 * i] = fma_pair(k.x, uu[c][j], s[c][2 * i]);
+                        s[c][2 * i + 1] = fma_pair(k.y, uu[c][j], s[c][2 * i + 1]);
+                    }
                 }
             }
-            if (j0 + part < n_here && col < vdim) y[(size_t)(t0 + j0 + part) * ((size_t)heads * vdim) + (size_t)head * vdim + col] = y8[0];
+            const int t = t0 + DS_GROUP * f + (part & 3);
+            if (part >= 4 && t < len) {
+#pragma unroll
+                for (int c = 0; c < DS_EACH; ++c)
+                    if (col + c < vdim)
+                        y[(size_t)(begin + t) * ((size_t)heads * vdim) + (size_t)head * vdim + col + c] =
+                            fmaf(d.w, u[c][3], fmaf(d.z, u[c][2], fmaf(d.y, u[c][1], fmaf(d.x, u[c][0], sums[c][0]))));
+            }
         }
         if (more) stash(buf ^ 1);
     }
     if (column) {
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int d = 4 * (part + DS_LANES * (i / 4)) + i % 4;
-            if (d < dim) column[(size_t)d * vdim] = s[i];
-        }
+        for (int c = 0; c < DS_EACH; ++c)
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i) {
+                const int d = 4 * (part + DS_LANES * (i / 2)) + 2 * (i % 2);
+                const float2 both = unpair(s[c][i]);
+                if (col + c < vdim && d < dim) column[(size_t)d * vdim + c] = both.x;
+                if (col + c < vdim && d + 1 < dim) column[(size_t)(d + 1) * vdim + c] = both.y;
+            }
     }
 }
 
 template <typename T, int R, int TOKENS>
-static int launch_scan(const float* packed, const float* beta, const void* v, int v_stride, const int* cu_q, const int* slots, int n_seqs,
-                       float* state, long long slot_stride, long long s_offset, int n_tokens, int heads, int dim, int vdim, float* y,
-                       cudaStream_t stream) {
-    const size_t smem = (size_t)2 * TOKENS * (3 * DS_LANES * R + DS_COLS + 1) * sizeof(float);
-    cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<T, R, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+static int launch_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* z, int z_stride,
+                       const float* bias, const float* rate_log, const float* logit, int logit_stride, const int* cu_q, const int* slots,
+                       int n_seqs, int max_q_len, float* state, long long slot_stride, long long s_offset, int n_tokens, int heads, int groups,
+                       int dim, int vdim, float q_scale, float* packed, float* y, cudaStream_t stream) {
+    const int n_records = n_tokens / DS_GROUP + n_seqs;
+    const long long items = (long long)((max_q_len + DS_GROUP - 1) / DS_GROUP) * heads;
+    cudaError_t e = launch_pdl(delta_prepare_kernel<T, DS_LANES * R / 32>, dim3((unsigned)((items + 3) / 4), n_seqs), dim3(128), 0, stream,
+                               (const T*)q, q_stride, (const T*)k, k_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, n_records,
+                               heads, groups, dim, q_scale, packed);
     if (e != cudaSuccess) return (int)e;
-    return (int)launch_pdl(delta_scan_kernel<T, R, TOKENS>, dim3((vdim + DS_COLS - 1) / DS_COLS, heads, n_seqs), dim3(DS_WARPS * 32), smem,
-                           stream, packed, beta, (const T*)v, v_stride, cu_q, slots, state, slot_stride, s_offset, n_tokens, heads, dim, vdim, y);
+    const size_t smem = (size_t)2 * (TOKENS / DS_GROUP * record_floats(DS_LANES * R) + TOKENS * DS_COLS) * sizeof(float);
+    e = cudaFuncSetAttribute(delta_scan_kernel<T, R, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    // launched the ordinary way: blocks that started under the first kernel's tail would crowd onto the SMs it leaves first,
+    // and this kernel's few blocks are as fast as the SM they have to themselves
+    delta_scan_kernel<T, R, TOKENS><<<dim3((vdim + DS_COLS - 1) / DS_COLS, heads, n_seqs), dim3(DS_WARPS * 32), smem, stream>>>(
+        packed, (const T*)v, v_stride, cu_q, slots, state, slot_stride, s_offset, n_records, heads, dim, vdim, y);
+    return (int)cudaGetLastError();
 }
 
-// Floats per row of the packed form for a state of `dim` rows (0: not supported).
-QF_EXPORT int qf_delta_padded(int dim) { return dim <= 0 || dim > 256 ? 0 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+// Floats of a record of four tokens for a state of `dim` rows (0: not supported).
+static int padded_dim(int dim) { return dim <= 0 || dim > 256 ? 0 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+QF_EXPORT int qf_delta_record(int dim) { return padded_dim(dim) ? (int)record_floats(padded_dim(dim)) : 0; }
 
 // q, k: [T][groups * dim], v: [T][heads * vdim], activation dtype with row strides; z (the decays' pre-activations): float32
 // [T][heads * dim], logit (beta's): float32 [T][heads], with row strides; bias float32 [heads * dim], rate_log float32 [heads];
-// packed: float32 [heads][T][3][padded] and beta [heads][T], scratch; y: float32 [T][heads * vdim]; S in the slots' rows at s_offset.
+// packed: scratch of heads * (n_tokens / 4 + n_seqs) records; y: float32 [T][heads * vdim]; S in the slots' rows at s_offset.
 QF_EXPORT int qf_delta_scan(int is_bf16, const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
                             const float* z, int z_stride, const float* bias, const float* rate_log, const float* logit,
-                            int logit_stride, const int* cu_q, const int* slots, int n_seqs, float* state, long long slot_stride,
-                            long long s_offset, int n_tokens, int heads, int groups, int dim, int vdim, float q_scale, float* packed,
-                            float* beta, float* y, cudaStream_t stream) {
-    const int padded = qf_delta_padded(dim);
+                            int logit_stride, const int* cu_q, const int* slots, int n_seqs, int max_q_len, float* state,
+                            long long slot_stride, long long s_offset, int n_tokens, int heads, int groups, int dim, int vdim, float q_scale,
+                            float* packed, float* y, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
-    if (padded == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535) return (int)cudaErrorInvalidValue;
-    const unsigned blocks = (unsigned)(((long long)n_tokens * heads + 7) / 8);
-    cudaError_t e;
-    if (is_bf16)
-        e = launch_pdl(delta_prepare_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)q, q_stride, (const bf16*)k, k_stride, z,
-                       z_stride, bias, rate_log, logit, logit_stride, n_tokens, heads, groups, dim, padded, q_scale, packed, beta);
-    else
-        e = launch_pdl(delta_prepare_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)q, q_stride, (const float*)k, k_stride,
-                       z, z_stride, bias, rate_log, logit, logit_stride, n_tokens, heads, groups, dim, padded, q_scale, packed, beta);
-    if (e != cudaSuccess) return (int)e;
+    if (padded_dim(dim) == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535 || max_q_len <= 0 || heads > 65535 ||
+        ((uintptr_t)packed & 15))
+        return (int)cudaErrorInvalidValue;
 #define QF_DELTA_SCAN(R, TOKENS) (is_bf16 ? launch_scan<bf16, R, TOKENS>(QF_DELTA_ARGS) : launch_scan<float, R, TOKENS>(QF_DELTA_ARGS))
-#define QF_DELTA_ARGS packed, beta, v, v_stride, cu_q, slots, n_seqs, state, slot_stride, s_offset, n_tokens, heads, dim, vdim, y, stream
-    if (padded == 32) return QF_DELTA_SCAN(4, 32);
-    if (padded == 64) return QF_DELTA_SCAN(8, 32);
-    if (padded == 128) return QF_DELTA_SCAN(16, 32);
-    return QF_DELTA_SCAN(32, 16);
+#define QF_DELTA_ARGS q, q_stride, k, k_stride, v, v_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, slots, n_seqs, max_q_len, \
+                      state, slot_stride, s_offset, n_tokens, heads, groups, dim, vdim, q_scale, packed, y, stream
+    switch (padded_dim(dim)) {
+        case 32: return QF_DELTA_SCAN(4, 32);
+        case 64: return QF_DELTA_SCAN(8, 32);
+        case 128: return QF_DELTA_SCAN(16, 32);
+        default: return QF_DELTA_SCAN(32, 16);
+    }
 #undef QF_DELTA_ARGS
+#undef QF_DELTA_SCAN
 }
 
 // ------------------------------------------------------------------------------------------------------------------
@@ -381,7 +536,7 @@ QF_EXPORT int qf_delta_token(int is_bf16, const void* q, int q_stride, const voi
                              long long s_offset, int heads, int groups, int dim, int vdim, float q_scale, float* y, const void* norm,
                              float eps, const void* gate, int gate_stride, void* out, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
-    if (qf_delta_padded(dim) == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535 || (out && (vdim > 128 || !norm || !gate)))
+    if (padded_dim(dim) == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535 || (out && (vdim > 128 || !norm || !gate)))
         return (int)cudaErrorInvalidValue;
     if (dim <= 64) return is_bf16 ? token_columns<bf16, 4>(QF_TOKEN_ARGS) : token_columns<float, 4>(QF_TOKEN_ARGS);
     if (dim <= 128) return is_bf16 ? token_columns<bf16, 8>(QF_TOKEN_ARGS) : token_columns<float, 8>(QF_TOKEN_ARGS);

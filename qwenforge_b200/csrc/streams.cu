@@ -13,15 +13,16 @@
 // y is a row per token, or (dest, top) the sum of the `top` rows y[dest[t * top + k]], each times row_weight[that row] if given
 // (a feed-forward of routed experts leaves its chosen rows unsummed).
 //
-// A thread owns V neighbouring channels of a run of tokens of one sequence. The h of the tokens before its run are worked out
-// again from their streams (the old and the new streams are different buffers, so whoever owns those tokens has not changed
-// them); what lies before the step's first token comes from the sequence's state, float32 [taps - 1][width], zeros at a
-// sequence's start. Only a sequence's FIRST run reads the state, and the same threads replace it, having read it, by the
-// sequence's last taps - 1 values of h: no second kernel, and no order between blocks. A row's arithmetic is the same chain
-// of operations whatever the cut, the batch and the run.
+// A block takes a tile of tokens of one sequence and some of the channels, a thread one token's V neighbouring channels. The h of
+// the tokens before the tile are worked out again from their streams (the old and the new streams are different buffers, so
+// whoever owns those tokens has not changed them); what lies before the step's first token comes from the sequence's state,
+// float32 [taps - 1][width], zeros at a sequence's start. The tile's h meet in shared memory, where the convolution reads them.
+// Only a sequence's FIRST tile reads the state, and the same block replaces it, having read it, by the sequence's last taps - 1
+// values of h: no second kernel, and no order between blocks. A row's arithmetic is the same chain of operations whatever
+// the cut, the batch and the tile.
 #include "common.cuh"
 
-#define ST_THREADS 128
+#define ST_THREADS 256
 
 template <typename T> struct StreamsArgs {
     const float* src;           // old streams: element (t, s, c) at t * src_row + s * src_stream + c
@@ -80,12 +81,15 @@ template <> struct Channels<bf16, 4> {
     }
 };
 
-// NS: the most streams (a.n <= NS); HIST: the most inputs a convolution keeps (a.n_taps - 1 <= HIST), 0 without one; RUN >= HIST
-template <typename T, int V, int NS, int HIST, int RUN>
+// NS: the most streams (a.n <= NS); HIST: the most inputs a convolution keeps (a.n_taps - 1 <= HIST), 0 without one; ROWS: tokens
+// of a tile, the HIST before it included.
+template <typename T, int V, int NS, int HIST, int ROWS>
 __global__ void __launch_bounds__(ST_THREADS)
 streams_kernel(const StreamsArgs<T> a) {
     grid_launch_dependents();
+    constexpr int GROUPS = ST_THREADS / ROWS, OWN = ROWS - HIST;
     __shared__ float mix_s[NS * NS], out_s[NS], in_s[NS];
+    __shared__ __align__(16) float h_s[HIST > 0 ? ROWS : 1][HIST > 0 ? GROUPS * V : 1];
     // the coefficients are weights: fetched before the wait for the kernel before this one
     for (int i = threadIdx.x; i < NS * NS; i += ST_THREADS) {
         const int s = i / NS, r = i % NS;
@@ -95,13 +99,13 @@ streams_kernel(const StreamsArgs<T> a) {
         out_s[threadIdx.x] = (a.out_w && threadIdx.x < a.n) ? a.out_w[threadIdx.x] : 0.f;
         in_s[threadIdx.x] = threadIdx.x < a.n ? (a.in_w ? a.in_w[threadIdx.x] : 1.f) : 0.f;
     }
-    const int groups = a.width / V;
-    const long long item = (long long)blockIdx.x * ST_THREADS + threadIdx.x;
-    const int run = (int)(item / groups), c0 = (int)(item % groups) * V;
+    const int group = threadIdx.x % GROUPS, row = threadIdx.x / GROUPS;
+    const int c0 = (blockIdx.x * GROUPS + group) * V;
+    const bool in = c0 < a.width;
     float w[V], b[V], f[HIST > 0 ? HIST + 1 : 1][V];
 #pragma unroll
     for (int v = 0; v < V; ++v) w[v] = b[v] = 0.f;
-    if (a.weight) {
+    if (a.weight && in) {
         Channels<T, V>::load(a.weight + c0, w);
         Channels<T, V>::load(a.bias + c0, b);
     }
@@ -111,24 +115,14 @@ streams_kernel(const StreamsArgs<T> a) {
 #pragma unroll
             for (int v = 0; v < V; ++v) {
                 const int at = j - (HIST + 1 - a.n_taps);
-                f[j][v] = at >= 0 ? a.taps[(size_t)(c0 + v) * a.n_taps + at] : 0.f;
+                f[j][v] = (in && row >= HIST && at >= 0) ? a.taps[(size_t)(c0 + v) * a.n_taps + at] : 0.f;
             }
     }
     __syncthreads();
     grid_dependency_wait();
 
-    int begin = 0, len = a.rows ? a.n_rows : a.n_tokens, slot = -1;
-    if constexpr (HIST > 0) {
-        begin = a.cu_q[blockIdx.y];
-        len = a.cu_q[blockIdx.y + 1] - begin;
-        slot = a.slots[blockIdx.y];
-    }
-    const int first = run * RUN;
-    if (first >= len) return;
-    const int last = min(first + RUN, len);
-
     // h of token t (or u, without a norm); the new streams are stored on the way if asked
-    auto value = [&](int t, bool keep, float* h) {
+    auto value = [&](int t, bool keep, float (&h)[V]) {
         float x[NS][V], y[V];
         const float* xs = a.src + t * a.src_row + c0;
 #pragma unroll
@@ -141,13 +135,15 @@ streams_kernel(const StreamsArgs<T> a) {
             if (a.dest) {
 #pragma unroll
                 for (int v = 0; v < V; ++v) y[v] = 0.f;
-                for (int k = 0; k < a.top; ++k) {
-                    const int row = a.dest[(size_t)t * a.top + k];
-                    float part[V];
-                    Channels<T, V>::load(a.y + (size_t)row * a.width + c0, part);
-                    const float by = a.row_weight ? a.row_weight[row] : 1.f;
+                for (int k = 0; k < a.top; k += 2) {   // two rows asked for together
+                    const int r0 = a.dest[(size_t)t * a.top + k], r1 = k + 1 < a.top ? a.dest[(size_t)t * a.top + k + 1] : r0;
+                    float p0[V], p1[V];
+                    Channels<T, V>::load(a.y + (size_t)r0 * a.width + c0, p0);
+                    Channels<T, V>::load(a.y + (size_t)r1 * a.width + c0, p1);
+                    const float by0 = a.row_weight ? a.row_weight[r0] : 1.f;
+                    const float by1 = k + 1 < a.top ? (a.row_weight ? a.row_weight[r1] : 1.f) : 0.f;
 #pragma unroll
-                    for (int v = 0; v < V; ++v) y[v] = fmaf(by, part[v], y[v]);
+                    for (int v = 0; v < V; ++v) y[v] = fmaf(by1, p1[v], fmaf(by0, p0[v], y[v]));
                 }
             } else {
                 Channels<T, V>::load(a.y + (size_t)t * a.width + c0, y);
@@ -180,75 +176,80 @@ streams_kernel(const StreamsArgs<T> a) {
     };
 
     if constexpr (HIST == 0) {
-        for (int i = first; i < last; ++i) {
-            int t = i;
-            if (a.rows) {
-                t = a.rows[i];
-                if (t < 0 || t >= a.n_tokens) {
-                    if (c0 == 0) atomicOr(a.err, QF_ERR_ROW_RANGE);
-                    t = 0;
-                }
+        const int i = blockIdx.y * ROWS + row;
+        if (!in || i >= (a.rows ? a.n_rows : a.n_tokens)) return;
+        int t = i;
+        if (a.rows) {
+            t = a.rows[i];
+            if (t < 0 || t >= a.n_tokens) {
+                if (c0 == 0) atomicOr(a.err, QF_ERR_ROW_RANGE);
+                t = 0;
             }
-            float h[V];
-            value(t, !a.rows, h);
-            if (a.weight) Channels<T, V>::store(a.z + (size_t)i * a.width + c0, h);
-            else Channels<float, V>::store(a.u_out + (size_t)i * a.width + c0, h);
         }
+        float h[V];
+        value(t, !a.rows, h);
+        if (a.weight) Channels<T, V>::store(a.z + (size_t)i * a.width + c0, h);
+        else Channels<float, V>::store(a.u_out + (size_t)i * a.width + c0, h);
     } else {
-        float hist[HIST][V];
-        const int kept = a.n_taps - 1;
-        float* rows = slot >= 0 ? a.state + slot * a.slot_stride + a.offset + c0 : nullptr;
+        const int begin = a.cu_q[blockIdx.z], len = a.cu_q[blockIdx.z + 1] - begin, slot = a.slots[blockIdx.z];
+        const int first = blockIdx.y * OWN, kept = a.n_taps - 1;
+        if (first >= len) return;   // (the whole block)
+        float* rows = (slot >= 0 && in) ? a.state + slot * a.slot_stride + a.offset + c0 : nullptr;
+        const int at = first - HIST + row;   // this thread's token, counted from the sequence's first of the step
+        float h[V];
 #pragma unroll
-        for (int j = 0; j < HIST; ++j) {   // hist[j]: h of HIST - j tokens before the run
-            const int at = first - HIST + j, row = kept - (HIST - j);
-#pragma unroll
-            for (int v = 0; v < V; ++v) hist[j][v] = 0.f;
-            if (row < 0) continue;          // older than the filter reaches
-            if (at >= 0) value(begin + at, false, hist[j]);
-            else if (rows && first == 0) Channels<float, V>::load(rows + (size_t)row * a.width, hist[j]);
-        }
-        for (int i = first; i < last; ++i) {
-            float h[V], z[V];
-            value(begin + i, true, h);
-#pragma unroll
-            for (int v = 0; v < V; ++v) {
-                z[v] = 0.f;
-#pragma unroll
-                for (int j = 0; j < HIST; ++j) z[v] = fmaf(f[j][v], hist[j][v], z[v]);
-                z[v] = h[v] + fmaf(f[HIST][v], h[v], z[v]);
-#pragma unroll
-                for (int j = 0; j + 1 < HIST; ++j) hist[j][v] = hist[j + 1][v];
-                hist[HIST - 1][v] = h[v];
+        for (int v = 0; v < V; ++v) h[v] = 0.f;
+        if (in && at < len) {
+            if (at >= 0 && row >= HIST - kept) {
+                value(begin + at, row >= HIST, h);
+            } else if (at < 0 && rows && kept + at >= 0) {   // (before the step: the state's row, the newest last)
+                Channels<float, V>::load(rows + (size_t)(kept + at) * a.width, h);
             }
-            Channels<T, V>::store(a.z + (size_t)(begin + i) * a.width + c0, z);
         }
-        if (first == 0 && rows) {
-            // the sequence's last `kept` values: in the registers if it ends in this run, else worked out again
+        Channels<float, V>::store(&h_s[row][group * V], h);
+        __syncthreads();
+        if (row >= HIST && in && at < len) {
+            float z[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) z[v] = 0.f;
 #pragma unroll
             for (int j = 0; j < HIST; ++j) {
-                const int row = kept - (HIST - j);
-                if (row < 0) continue;
-                if (len > RUN) value(begin + len - (HIST - j), false, hist[j]);
-                Channels<float, V>::store(rows + (size_t)row * a.width, hist[j]);
+                float before[V];
+                Channels<float, V>::load(&h_s[row - HIST + j][group * V], before);
+#pragma unroll
+                for (int v = 0; v < V; ++v) z[v] = fmaf(f[j][v], before[v], z[v]);
             }
+#pragma unroll
+            for (int v = 0; v < V; ++v) z[v] = h[v] + fmaf(f[HIST][v], h[v], z[v]);
+            Channels<T, V>::store(a.z + (size_t)(begin + at) * a.width + c0, z);
+        }
+        if (first == 0 && rows && row < kept) {
+            // the sequence's last `kept` values: in shared memory if it ends in this tile, else worked out again
+            const int back = len - kept + row;
+            float last[V];
+            if (len <= OWN) Channels<float, V>::load(&h_s[HIST + back][group * V], last);
+            else value(begin + back, false, last);
+            Channels<float, V>::store(rows + (size_t)row * a.width, last);
         }
     }
 }
 
-template <typename T, int V, int NS, int HIST>
+template <typename T, int V, int NS, int HIST, int ROWS>
 static int launch_streams(const StreamsArgs<T>& a, int n_seqs, int max_q_len, cudaStream_t stream) {
-    constexpr int RUN = HIST > 8 ? 16 : HIST > 0 ? 8 : 2;
+    constexpr int OWN = ROWS - HIST, CHANNELS = ST_THREADS / ROWS * V;
     const long long longest = HIST > 0 ? max_q_len : (a.rows ? a.n_rows : a.n_tokens);
-    const long long items = (longest + RUN - 1) / RUN * (a.width / V);
-    const dim3 grid((unsigned)((items + ST_THREADS - 1) / ST_THREADS), HIST > 0 ? n_seqs : 1);
-    if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-    return (int)launch_pdl(streams_kernel<T, V, NS, HIST, RUN>, grid, dim3(ST_THREADS), 0, stream, a);
+    const long long tiles = (longest + OWN - 1) / OWN;
+    const dim3 grid((a.width + CHANNELS - 1) / CHANNELS, (unsigned)tiles, HIST > 0 ? n_seqs : 1);
+    if (tiles > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
+    return (int)launch_pdl(streams_kernel<T, V, NS, HIST, ROWS>, grid, dim3(ST_THREADS), 0, stream, a);
 }
 
 template <typename T, int V, int NS>
 static int launch_taps(const StreamsArgs<T>& a, int n_seqs, int max_q_len, cudaStream_t stream) {
-    if (!a.taps) return launch_streams<T, V, NS, 0>(a, n_seqs, max_q_len, stream);
-    return launch_streams<T, V, NS, 3>(a, n_seqs, max_q_len, stream);
+    if (!a.taps) return launch_streams<T, V, NS, 0, 4>(a, n_seqs, max_q_len, stream);
+    // one token per sequence: the three before it and itself, each a thread's
+    if (max_q_len == 1) return launch_streams<T, V, NS, 3, 4>(a, n_seqs, max_q_len, stream);
+    return launch_streams<T, V, NS, 3, 32>(a, n_seqs, max_q_len, stream);
 }
 
 template <typename T>
@@ -256,7 +257,7 @@ static int launch(const StreamsArgs<T>& a, int n_seqs, int max_q_len, cudaStream
     const uintptr_t all = (uintptr_t)a.src | (uintptr_t)a.dst | (uintptr_t)a.y | (uintptr_t)a.weight | (uintptr_t)a.bias | (uintptr_t)a.z |
                           (uintptr_t)a.u_out | (uintptr_t)a.state;
     const bool wide = a.width % 4 == 0 && all % 16 == 0 && (a.src_row | a.src_stream | a.slot_stride | a.offset) % 4 == 0;
-    if (a.taps && a.n_taps > 4) return launch_streams<T, 1, 8, 15>(a, n_seqs, max_q_len, stream);   // long filters: one form for all
+    if (a.taps && a.n_taps > 4) return launch_streams<T, 1, 8, 15, 32>(a, n_seqs, max_q_len, stream);   // long filters: one form for all
 #define QF_STREAMS(NS) return wide ? launch_taps<T, 4, NS>(a, n_seqs, max_q_len, stream) : launch_taps<T, 1, NS>(a, n_seqs, max_q_len, stream)
     if (a.n <= 2) QF_STREAMS(2);
     if (a.n <= 4) QF_STREAMS(4);

@@ -1849,24 +1849,26 @@ def _delta_args(what, q, k, v, z, bias, rate_log, logit, state, s_offset, n_head
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, rate_log: torch.Tensor,
                logit: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_heads: int,
-               n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor) -> None:
+               n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor, max_q_len: int = 0) -> None:
     """The gated delta rule with a decay per head and key channel, token after token of every sequence, float32 inside:
         q, k <- x / sqrt(sum(x^2) + 1e-6) per head (q also times q_scale);  g = exp(-exp(rate_log_h) softplus(z + bias));
         beta = sigmoid(logit);  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  y = S^T q.
     q, k: [T, groups * dim] (head h reads group h // (heads / groups)), v: [T, heads * vdim] in the activation dtype; z float32
     [T, heads * dim], logit float32 [T, heads]; rows may be strided; bias float32 [heads * dim], rate_log float32 [heads]; y float32
-    [T, heads * vdim]; S (dim x vdim per head) in `state` at s_offset as [heads, dim, vdim]."""
+    [T, heads * vdim]; S (dim x vdim per head) in `state` at s_offset as [heads, dim, vdim]. Four tokens at a time, written out as sums
+    over the state before them; `max_q_len`: the most tokens any sequence brings (0: not known)."""
     args = _delta_args("delta_scan", q, k, v, z, bias, rate_log, logit, state, s_offset, n_heads, n_groups, dim, vdim)
     n = q.shape[0]
     _dev("y", y, torch.float32)
     if y.shape != (n, n_heads * vdim):
         raise KernelError("delta_scan: y must be float32 [T, heads * vdim]")
-    lib = library("delta_rule")
-    padded = int(lib.qf_delta_padded(_I(dim)))
-    packed = torch.empty(n_heads * n * (3 * padded + 1), dtype=torch.float32, device=q.device)
-    _check(lib.qf_delta_scan(*args, _ptr(cu_q), _ptr(slots), _I(cu_q.numel() - 1), _ptr(state), _LL(state.stride(0)), _LL(s_offset), _I(n),
-                             _I(n_heads), _I(n_groups), _I(dim), _I(vdim), _F(q_scale), _ptr(packed),
-                             _ptr(packed[n_heads * n * 3 * padded:]), _ptr(y), _stream()), "delta_scan")
+    lib, n_seqs = library("delta_rule"), cu_q.numel() - 1
+    # records of four tokens, counted from each sequence's first token: sequence s starts at record cu_q[s] // 4 + s, so that
+    # the records of one never reach into the next one's
+    packed = torch.empty(n_heads * (n // 4 + n_seqs) * int(lib.qf_delta_record(_I(dim))), dtype=torch.float32, device=q.device)
+    _check(lib.qf_delta_scan(*args, _ptr(cu_q), _ptr(slots), _I(n_seqs), _I(max_q_len or n), _ptr(state), _LL(state.stride(0)),
+                             _LL(s_offset), _I(n), _I(n_heads), _I(n_groups), _I(dim), _I(vdim), _F(q_scale), _ptr(packed), _ptr(y),
+                             _stream()), "delta_scan")
 
 
 DELTA_FUSED_MAX_VDIM = 128   # value sizes up to which a single token's norm and gate ride on `delta_token`
