@@ -16,11 +16,13 @@
 //
 // which is the same recurrence, written out. `delta_prepare` works out all that does not depend on the state, a warp per
 // (head, four tokens): the unit vectors, the decays and their products, c, d and beta, packed as one record. `delta_scan` walks
-// every sequence's records in order. Eight lanes share two columns of S, the rows dealt out in fours, so a warp has eight columns
-// and a block of two warps sixteen (what a lane reads from shared memory serves both its columns: the shared memory's pace is
-// what bounds a block); a lane's part of S stays in registers, two rows to a register pair and one instruction, from the
-// sequence's first token of the step to its last. A column's eight sums (four for u, four for y) are formed together and reduced
-// together, each lane ending up with one of them. Records are staged through shared memory DS_TOKENS tokens at a time by asynchronous copies, the next
+// every sequence's records in order. LANES lanes share EACH columns of S, the rows dealt out in fours; a lane's part of S stays in
+// registers, two rows to a register pair and one instruction, from the sequence's first token of the step to its last. A
+// column's eight sums (four for u, four for y) are formed together and reduced together, each lane ending up with one of them.
+// What bounds the kernel is a warp's chain from one four to the next, so a lane has few rows (four; the more rows S has, the more
+// lanes share a column), and the rows of the next four are asked for before the sums of this one are; for tall states two
+// columns per lane, because a block is then bound by what it reads from shared memory.
+// Records are staged through shared memory 16 or 32 tokens at a time by asynchronous copies, the next
 // ones under way while these are worked on. Fours are counted from a sequence's first token of the step; the last one is
 // filled up with tokens that do nothing (g = 1, k = q = 0).
 //
@@ -29,10 +31,6 @@
 // if asked, the RMS norm per head, its weight and the sigmoid gate that follow.
 #include "mma.cuh"
 
-#define DS_LANES 8
-#define DS_WARPS 2
-#define DS_EACH 2                                       // columns of S per lane
-#define DS_COLS (DS_WARPS * 32 / DS_LANES * DS_EACH)    // and per block
 #define DELTA_LENGTH_EPS 1e-6f               // under the root of the unit vectors' length
 
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -190,33 +188,48 @@ delta_prepare_kernel(const T* __restrict__ q, int q_stride, const T* __restrict_
     if (lane < 4) tail[24 + lane] = t0 + lane < len ? 1.f / (1.f + expf(-raw_beta)) : 0.f;
 }
 
-// R rows of S per lane (a multiple of 4): padded = 8 * R. Lane l of a column has rows 4 * (l + 8 * i) .. + 3.
-template <typename T, int R, int TOKENS>
-__global__ void __launch_bounds__(DS_WARPS * 32)
+// A load that stays where it is written (see the scan of csrc/recurrent.cu).
+__device__ __forceinline__ float load_value(const float* p) {
+    float x;
+    asm volatile("ld.global.nc.f32 %0, [%1];" : "=f"(x) : "l"(p));
+    return x;
+}
+__device__ __forceinline__ float load_value(const bf16* p) {
+    unsigned short raw;
+    asm volatile("ld.global.nc.u16 %0, [%1];" : "=h"(raw) : "l"(p));
+    return __uint_as_float((unsigned)raw << 16);
+}
+
+// R rows of S per lane (a multiple of 4), padded = LANES * R. Lane l of a column has rows 4 * (l + LANES * i) .. + 3. A warp has
+// 32 / LANES * EACH columns, a block of WARPS warps COLS of them.
+template <typename T, int LANES, int EACH, int R, int WARPS, int TOKENS>
+__global__ void __launch_bounds__(WARPS * 32)
 delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int v_stride, const int* __restrict__ cu_q,
                   const int* __restrict__ slots, float* __restrict__ state, long long slot_stride, long long s_offset, int n_records,
                   int heads, int dim, int vdim, float* __restrict__ y) {
-    constexpr int P = DS_LANES * R, Q4 = R / 4, THREADS = DS_WARPS * 32, FOURS = TOKENS / DS_GROUP;
-    constexpr int REC = (int)record_floats(P);
+    constexpr int P = LANES * R, Q4 = R / 4, THREADS = WARPS * 32, FOURS = TOKENS / DS_GROUP, COLS = WARPS * 32 / LANES * EACH;
+    constexpr int REC = (int)record_floats(P), SUMS = 8 * EACH;
+    constexpr int SH = LANES / SUMS == 1 ? 0 : LANES / SUMS == 2 ? 1 : 2;   // after the reduction a lane has sum `part >> SH`
+    static_assert(LANES % SUMS == 0 && LANES / SUMS <= 4, "a sum per lane");
     extern __shared__ __align__(16) float ds_smem[];
     float* rec_s = ds_smem;                                // [2][FOURS][REC]
-    float* v_s = rec_s + 2 * FOURS * REC;                  // [2][TOKENS][DS_COLS]
+    float* v_s = rec_s + 2 * FOURS * REC;                  // [2][TOKENS][COLS]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, head = blockIdx.y, seq = blockIdx.z;
-    const int part = lane & (DS_LANES - 1), col_in = (warp * (32 / DS_LANES) + lane / DS_LANES) * DS_EACH, col = blockIdx.x * DS_COLS + col_in;
+    const int part = lane & (LANES - 1), col_in = (warp * (32 / LANES) + lane / LANES) * EACH, col = blockIdx.x * COLS + col_in;
     const int begin = cu_q[seq], len = cu_q[seq + 1] - begin, slot = slots[seq];
     if (len <= 0) return;
     float* column = slot >= 0 ? state + slot * slot_stride + s_offset + (long long)head * dim * vdim + col : nullptr;
-    unsigned long long s[DS_EACH][R / 2];   // rows in pairs
+    unsigned long long s[EACH][R / 2];   // rows in pairs
 #pragma unroll
-    for (int c = 0; c < DS_EACH; ++c)
+    for (int c = 0; c < EACH; ++c)
 #pragma unroll
         for (int i = 0; i < R / 2; ++i) {
-            const int d = 4 * (part + DS_LANES * (i / 2)) + 2 * (i % 2);
+            const int d = 4 * (part + LANES * (i / 2)) + 2 * (i % 2);
             const bool there = column && col + c < vdim;
             s[c][i] = pair_of(there && d < dim ? column[(size_t)d * vdim + c] : 0.f, there && d + 1 < dim ? column[(size_t)(d + 1) * vdim + c] : 0.f);
         }
-    constexpr int V_EACH = TOKENS * DS_COLS / THREADS;
-    T v_next[V_EACH];
+    constexpr int V_EACH = (TOKENS * COLS + THREADS - 1) / THREADS;
+    float v_next[V_EACH];
     const float* records = packed + ((size_t)head * n_records + first_record(begin, seq)) * REC;
     auto fetch = [&](int t0, int buf) {   // the records straight to shared memory, the values through registers
         const int fours = min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP);
@@ -226,13 +239,15 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
         cp_async_commit();
 #pragma unroll
         for (int u = 0; u < V_EACH; ++u) {
-            const int i = threadIdx.x + u * THREADS, j = t0 + i / DS_COLS, c = blockIdx.x * DS_COLS + i % DS_COLS;
-            v_next[u] = (j < len && c < vdim) ? v[(size_t)(begin + j) * v_stride + (size_t)head * vdim + c] : Num<T>::from_f(0.f);
+            const int i = threadIdx.x + u * THREADS, j = t0 + i / COLS, c = blockIdx.x * COLS + i % COLS;
+            v_next[u] = 0.f;
+            if (i < TOKENS * COLS && j < len && c < vdim) v_next[u] = load_value(v + (size_t)(begin + j) * v_stride + (size_t)head * vdim + c);
         }
     };
     auto stash = [&](int buf) {
 #pragma unroll
-        for (int u = 0; u < V_EACH; ++u) v_s[buf * TOKENS * DS_COLS + threadIdx.x + u * THREADS] = Num<T>::to_f(v_next[u]);
+        for (int u = 0; u < V_EACH; ++u)
+            if (threadIdx.x + u * THREADS < TOKENS * COLS) v_s[buf * TOKENS * COLS + threadIdx.x + u * THREADS] = v_next[u];
     };
     fetch(0, 0);
     stash(0);
@@ -242,95 +257,116 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
         __syncthreads();   // these records have arrived for everyone, and everyone is done with the other buffer
         const bool more = t0 + TOKENS < len;
         if (more) fetch(t0 + TOKENS, buf ^ 1);
-        const float* vs = v_s + buf * TOKENS * DS_COLS + col_in;
+        const float* vs = v_s + buf * TOKENS * COLS + col_in;
+        auto rows_of = [&](int f) { return reinterpret_cast<const ulonglong2*>(rec_s + (buf * FOURS + f) * REC) + part; };
+        ulonglong2 ahead[8][Q4];   // the rows of the eight sums: row x, its quarter i
+        {
+            const ulonglong2* rows = rows_of(0);
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+#pragma unroll
+                for (int i = 0; i < Q4; ++i) ahead[x][i] = rows[x * (P / 4) + LANES * i];
+        }
         for (int f = 0; f < fours; ++f) {
             const float* rec = rec_s + (buf * FOURS + f) * REC;
-            const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(rec) + part;   // row r, its quarter i: rows[r * (P / 4) + DS_LANES * i]
+            const ulonglong2* rows = rows_of(f);
+            float sums[SUMS];
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+#pragma unroll
+                for (int c = 0; c < EACH; ++c) {
+                    unsigned long long acc = mul_pair(s[c][0], ahead[x][0].x);
+                    acc = fma_pair(s[c][1], ahead[x][0].y, acc);
+#pragma unroll
+                    for (int i = 1; i < Q4; ++i) {
+                        acc = fma_pair(s[c][2 * i], ahead[x][i].x, acc);
+                        acc = fma_pair(s[c][2 * i + 1], ahead[x][i].y, acc);
+                    }
+                    sums[8 * c + x] = sum_of_pair(acc);
+                }
+            // what the second half needs, and the next four's rows, are on their way under the reduction
+            ulonglong2 g[Q4], k[4][Q4];
+#pragma unroll
+            for (int i = 0; i < Q4; ++i) {
+                g[i] = rows[12 * (P / 4) + LANES * i];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) k[j][i] = rows[(8 + j) * (P / 4) + LANES * i];
+            }
             const float4 c0 = *reinterpret_cast<const float4*>(rec + DS_ROWS * P), c1 = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 4);
             const float4 beta = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 24);
-            const float4 d = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 8 + 4 * (part & 3));   // this lane's token's row
-            float2 v4[4];
+            const float4 d = *reinterpret_cast<const float4*>(rec + DS_ROWS * P + 8 + 4 * ((part >> SH) & 3));   // this lane's token's row
+            float value[4][EACH];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) v4[j] = *reinterpret_cast<const float2*>(vs + (4 * f + j) * DS_COLS);
-            float sums[DS_EACH][8];
+            for (int j = 0; j < 4; ++j)
 #pragma unroll
-            for (int x = 0; x < 8; ++x) {
-                unsigned long long acc[DS_EACH];
+                for (int c = 0; c < EACH; ++c) value[j][c] = vs[(4 * f + j) * COLS + c];
+            {
+                const ulonglong2* next = rows_of(f + 1 < fours ? f + 1 : f);
 #pragma unroll
-                for (int i = 0; i < Q4; ++i) {
-                    const ulonglong2 w = rows[x * (P / 4) + DS_LANES * i];
+                for (int x = 0; x < 8; ++x)
 #pragma unroll
-                    for (int c = 0; c < DS_EACH; ++c) {
-                        acc[c] = i == 0 ? mul_pair(s[c][0], w.x) : fma_pair(s[c][2 * i], w.x, acc[c]);
-                        acc[c] = fma_pair(s[c][2 * i + 1], w.y, acc[c]);
+                    for (int i = 0; i < Q4; ++i) ahead[x][i] = next[x * (P / 4) + LANES * i];
+            }
+            // the sums over the lanes, halving the sums with the lanes while there is more than one
+#pragma unroll
+            for (int o = LANES / 2, n = SUMS / 2; o > 0; o >>= 1, n >>= 1) {
+                if (n > 0) {
+                    const bool upper = part & o;
+#pragma unroll
+                    for (int j = 0; j < n; ++j) {
+                        const float mine = upper ? sums[j + n] : sums[j], theirs = upper ? sums[j] : sums[j + n];
+                        sums[j] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
                     }
+                } else {
+                    sums[0] += __shfl_xor_sync(0xffffffffu, sums[0], o);
                 }
-#pragma unroll
-                for (int c = 0; c < DS_EACH; ++c) sums[c][x] = sum_of_pair(acc[c]);
             }
-            // eight sums over eight lanes, halving: lane `part` ends with sum `part`
+            float u[EACH][4];
 #pragma unroll
-            for (int o = DS_LANES / 2; o > 0; o >>= 1) {
-                const bool upper = part & o;
-#pragma unroll
-                for (int j = 0; j < o; ++j)
-#pragma unroll
-                    for (int c = 0; c < DS_EACH; ++c) {
-                        const float mine = upper ? sums[c][j + o] : sums[c][j], theirs = upper ? sums[c][j] : sums[c][j + o];
-                        sums[c][j] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
-                    }
-            }
-            float u[DS_EACH][4];
-#pragma unroll
-            for (int c = 0; c < DS_EACH; ++c) {
+            for (int c = 0; c < EACH; ++c) {
                 float left[4];   // v_i - S^T G_i k_i
 #pragma unroll
-                for (int j = 0; j < 4; ++j) left[j] = (c == 0 ? v4[j].x : v4[j].y) - __shfl_sync(0xffffffffu, sums[c][0], j, DS_LANES);
+                for (int j = 0; j < 4; ++j) left[j] = value[j][c] - __shfl_sync(0xffffffffu, sums[0], (8 * c + j) << SH, LANES);
                 u[c][0] = beta.x * left[0];
                 u[c][1] = beta.y * fmaf(-c0.x, u[c][0], left[1]);
                 u[c][2] = beta.z * fmaf(-c0.z, u[c][1], fmaf(-c0.y, u[c][0], left[2]));
                 u[c][3] = beta.w * fmaf(-c1.y, u[c][2], fmaf(-c1.x, u[c][1], fmaf(-c0.w, u[c][0], left[3])));
             }
-            unsigned long long uu[DS_EACH][4];
 #pragma unroll
-            for (int c = 0; c < DS_EACH; ++c)
+            for (int c = 0; c < EACH; ++c)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) uu[c][j] = pair_of(u[c][j], u[c][j]);
-#pragma unroll
-            for (int i = 0; i < Q4; ++i) {
-                const ulonglong2 g = rows[12 * (P / 4) + DS_LANES * i];
-#pragma unroll
-                for (int c = 0; c < DS_EACH; ++c) {
-                    s[c][2 * i] = mul_pair(g.x, s[c][2 * i]);
-                    s[c][2 * i + 1] = mul_pair(g.y, s[c][2 * i + 1]);
+                for (int i = 0; i < Q4; ++i) {
+                    s[c][2 * i] = mul_pair(g[i].x, s[c][2 * i]);
+                    s[c][2 * i + 1] = mul_pair(g[i].y, s[c][2 * i + 1]);
                 }
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const ulonglong2 k = rows[(8 + j) * (P / 4) + DS_LANES * i];
+            for (int j = 0; j < 4; ++j)
 #pragma unroll
-                    for (int c = 0; c < DS_EACH; ++c) {
-                        s[c][2 * i] = fma_pair(k.x, uu[c][j], s[c][2 * i]);
-                        s[c][2 * i + 1] = fma_pair(k.y, uu[c][j], s[c][2 * i + 1]);
+                for (int c = 0; c < EACH; ++c) {
+                    const unsigned long long uu = pair_of(u[c][j], u[c][j]);
+#pragma unroll
+                    for (int i = 0; i < Q4; ++i) {
+                        s[c][2 * i] = fma_pair(k[j][i].x, uu, s[c][2 * i]);
+                        s[c][2 * i + 1] = fma_pair(k[j][i].y, uu, s[c][2 * i + 1]);
                     }
                 }
-            }
-            const int t = t0 + DS_GROUP * f + (part & 3);
-            if (part >= 4 && t < len) {
+            const int sum = part >> SH, mine = sum >> 3, t = t0 + DS_GROUP * f + (sum & 3);   // mine: the column of this lane's sum
+            if ((sum & 4) && !(part & ((1 << SH) - 1)) && t < len && col + mine < vdim) {
+                float out = sums[0];
+                const float dj[4] = {d.x, d.y, d.z, d.w};
 #pragma unroll
-                for (int c = 0; c < DS_EACH; ++c)
-                    if (col + c < vdim)
-                        y[(size_t)(begin + t) * ((size_t)heads * vdim) + (size_t)head * vdim + col + c] =
-                            fmaf(d.w, u[c][3], fmaf(d.z, u[c][2], fmaf(d.y, u[c][1], fmaf(d.x, u[c][0], sums[c][0]))));
+                for (int j = 0; j < 4; ++j) out = fmaf(dj[j], EACH > 1 && mine ? u[EACH - 1][j] : u[0][j], out);
+                y[(size_t)(begin + t) * ((size_t)heads * vdim) + (size_t)head * vdim + col + mine] = out;
             }
         }
         if (more) stash(buf ^ 1);
     }
     if (column) {
 #pragma unroll
-        for (int c = 0; c < DS_EACH; ++c)
+        for (int c = 0; c < EACH; ++c)
 #pragma unroll
             for (int i = 0; i < R / 2; ++i) {
-                const int d = 4 * (part + DS_LANES * (i / 2)) + 2 * (i % 2);
+                const int d = 4 * (part + LANES * (i / 2)) + 2 * (i % 2);
                 const float2 both = unpair(s[c][i]);
                 if (col + c < vdim && d < dim) column[(size_t)d * vdim + c] = both.x;
                 if (col + c < vdim && d + 1 < dim) column[(size_t)(d + 1) * vdim + c] = both.y;
@@ -338,23 +374,24 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
     }
 }
 
-template <typename T, int R, int TOKENS>
+template <typename T, int LANES, int EACH, int R, int WARPS, int TOKENS>
 static int launch_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* z, int z_stride,
                        const float* bias, const float* rate_log, const float* logit, int logit_stride, const int* cu_q, const int* slots,
                        int n_seqs, int max_q_len, float* state, long long slot_stride, long long s_offset, int n_tokens, int heads, int groups,
                        int dim, int vdim, float q_scale, float* packed, float* y, cudaStream_t stream) {
+    constexpr int COLS = WARPS * 32 / LANES * EACH;
     const int n_records = n_tokens / DS_GROUP + n_seqs;
     const long long items = (long long)((max_q_len + DS_GROUP - 1) / DS_GROUP) * heads;
-    cudaError_t e = launch_pdl(delta_prepare_kernel<T, DS_LANES * R / 32>, dim3((unsigned)((items + 3) / 4), n_seqs), dim3(128), 0, stream,
+    cudaError_t e = launch_pdl(delta_prepare_kernel<T, LANES * R / 32>, dim3((unsigned)((items + 3) / 4), n_seqs), dim3(128), 0, stream,
                                (const T*)q, q_stride, (const T*)k, k_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, n_records,
                                heads, groups, dim, q_scale, packed);
     if (e != cudaSuccess) return (int)e;
-    const size_t smem = (size_t)2 * (TOKENS / DS_GROUP * record_floats(DS_LANES * R) + TOKENS * DS_COLS) * sizeof(float);
-    e = cudaFuncSetAttribute(delta_scan_kernel<T, R, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = (size_t)2 * (TOKENS / DS_GROUP * record_floats(LANES * R) + TOKENS * COLS) * sizeof(float);
+    e = cudaFuncSetAttribute(delta_scan_kernel<T, LANES, EACH, R, WARPS, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     // launched the ordinary way: blocks that started under the first kernel's tail would crowd onto the SMs it leaves first,
     // and this kernel's few blocks are as fast as the SM they have to themselves
-    delta_scan_kernel<T, R, TOKENS><<<dim3((vdim + DS_COLS - 1) / DS_COLS, heads, n_seqs), dim3(DS_WARPS * 32), smem, stream>>>(
+    delta_scan_kernel<T, LANES, EACH, R, WARPS, TOKENS><<<dim3((vdim + COLS - 1) / COLS, heads, n_seqs), dim3(WARPS * 32), smem, stream>>>(
         packed, (const T*)v, v_stride, cu_q, slots, state, slot_stride, s_offset, n_records, heads, dim, vdim, y);
     return (int)cudaGetLastError();
 }
@@ -375,14 +412,14 @@ QF_EXPORT int qf_delta_scan(int is_bf16, const void* q, int q_stride, const void
     if (padded_dim(dim) == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535 || max_q_len <= 0 || heads > 65535 ||
         ((uintptr_t)packed & 15))
         return (int)cudaErrorInvalidValue;
-#define QF_DELTA_SCAN(R, TOKENS) (is_bf16 ? launch_scan<bf16, R, TOKENS>(QF_DELTA_ARGS) : launch_scan<float, R, TOKENS>(QF_DELTA_ARGS))
+#define QF_DELTA_SCAN(...) (is_bf16 ? launch_scan<bf16, __VA_ARGS__>(QF_DELTA_ARGS) : launch_scan<float, __VA_ARGS__>(QF_DELTA_ARGS))
 #define QF_DELTA_ARGS q, q_stride, k, k_stride, v, v_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, slots, n_seqs, max_q_len, \
                       state, slot_stride, s_offset, n_tokens, heads, groups, dim, vdim, q_scale, packed, y, stream
     switch (padded_dim(dim)) {
-        case 32: return QF_DELTA_SCAN(4, 32);
-        case 64: return QF_DELTA_SCAN(8, 32);
-        case 128: return QF_DELTA_SCAN(16, 32);
-        default: return QF_DELTA_SCAN(32, 16);
+        case 32: return QF_DELTA_SCAN(8, 1, 4, 4, 32);
+        case 64: return QF_DELTA_SCAN(16, 1, 4, 4, 32);
+        case 128: return QF_DELTA_SCAN(32, 2, 4, 8, 32);
+        default: return QF_DELTA_SCAN(32, 2, 8, 8, 16);
     }
 #undef QF_DELTA_ARGS
 #undef QF_DELTA_SCAN

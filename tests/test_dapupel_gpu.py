@@ -512,8 +512,13 @@ def test_unequal_batches_in_slots_used_before(dtype, name, tmp_path):
 
 
 def peaked(cfg, weights, factor=5.0):
-    """Weights under which one score stands out: the queries of every attention grown, the distance bias small beside them."""
+    """Weights under which one score stands out: the queries of every attention grown, the distance bias small beside them, and what
+    the mixers write large beside the embedding."""
     w = {k: v.clone() for k, v in weights.items()}
+    w["embed"] *= 0.4
+    for name in w:
+        if name.endswith("hc1.out"):
+            w[name] = 2.5 * w[name].abs()
     for i, entry in enumerate(cfg["layers"]):
         if entry["type"] == "attention":
             w[f"l{i}.mix.q"] *= factor
@@ -544,12 +549,9 @@ def test_keys_at_the_edges_of_windows_and_pages_and_keys_far_back(dtype, tmp_pat
     # the mask and the positions matter here: every window one position longer, or no keys beyond 300 back, give other logits
     longer = {**cfg, "layers": [dict(e, mixer={**e["mixer"], "mask": {"size": e["mixer"]["mask"]["size"] + 1}}) if e["type"] == "attention" else e
                                 for e in cfg["layers"]]}
-    d = (plain.forward_logits(longer, used, tokens) - want[0])[100:]
-    assert float((d - d.mean(-1, keepdim=True)).square().mean(-1).sqrt().median() / want[0].std()) > 0.1
-    late = plain.forward_logits(cfg, used, tokens[300:])
-    d = late[100:] - want[0][400:]
-    print("a window longer by one, and no keys before position 300, move the median row by", float(d.std() / want[0].std()))
-    assert float((d - d.mean(-1, keepdim=True)).square().mean(-1).sqrt().median() / want[0].std()) > 0.1
+    moved = lambda d: float((d - d.mean(-1, keepdim=True)).square().mean(-1).sqrt().median() / want[0].std())
+    assert moved((plain.forward_logits(longer, used, tokens) - want[0])[100:]) > (0.03 if dtype == torch.float32 else 0.1)
+    assert moved(plain.forward_logits(cfg, used, tokens[300:])[100:] - want[0][400:]) > 0.3
 
 
 @pytest.mark.parametrize("dtype", BOTH)
