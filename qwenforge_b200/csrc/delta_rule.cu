@@ -19,10 +19,9 @@
 // every sequence's records in order. LANES lanes share EACH columns of S, the rows dealt out in fours; a lane's part of S stays in
 // registers, two rows to a register pair and one instruction, from the sequence's first token of the step to its last. A
 // column's eight sums (four for u, four for y) are formed together and reduced together, each lane ending up with one of them.
-// What bounds the kernel is a warp's chain from one four to the next, so a lane has few rows (four; the more rows S has, the more
-// lanes share a column), and the rows of the next four are asked for before the sums of this one are; for tall states two
-// columns per lane, because a block is then bound by what it reads from shared memory.
-// Records are staged through shared memory 16 or 32 tokens at a time by asynchronous copies, the next
+// What bounds the kernel is a warp's chain from one four to the next, so a lane has few rows (four or eight), and the rows of the
+// next four are asked for before the sums of this one are; two columns per lane where S is tall, because a block is then
+// bound by what it reads from shared memory. Records are staged through shared memory 16 or 32 tokens at a time by asynchronous copies, the next
 // ones under way while these are worked on. Fours are counted from a sequence's first token of the step; the last one is
 // filled up with tokens that do nothing (g = 1, k = q = 0).
 //
@@ -417,8 +416,8 @@ QF_EXPORT int qf_delta_scan(int is_bf16, const void* q, int q_stride, const void
                       state, slot_stride, s_offset, n_tokens, heads, groups, dim, vdim, q_scale, packed, y, stream
     switch (padded_dim(dim)) {
         case 32: return QF_DELTA_SCAN(8, 1, 4, 4, 32);
-        case 64: return QF_DELTA_SCAN(16, 1, 4, 4, 32);
-        case 128: return QF_DELTA_SCAN(32, 2, 4, 8, 32);
+        case 64: return QF_DELTA_SCAN(16, 1, 4, 2, 32);
+        case 128: return QF_DELTA_SCAN(16, 2, 8, 4, 32);
         default: return QF_DELTA_SCAN(32, 2, 8, 8, 16);
     }
 #undef QF_DELTA_ARGS

@@ -394,7 +394,7 @@ class ChannelDelta(Mixer):
         pieces.append(filled(t("g1")))
         self.proj_weight = torch.cat(pieces, dim=0).contiguous()
         self.conv_weight = torch.cat((t("q_conv"), t("k_conv"), t("v_conv")), dim=0).to(torch.float32).contiguous()
-        self.b_weight, self.a2, self.g2 = t("b_weight").contiguous(), t("a2").contiguous(), t("g2").contiguous()
+        self.b_weight, self.a2, self.g2 = filled(t("b_weight")).contiguous(), t("a2").contiguous(), t("g2").contiguous()
         self.rate_log, self.dt_bias = (t(k).to(torch.float32).contiguous() for k in ("rate_log", "dt_bias"))
         self.norm, self.o_weight = t("norm").contiguous(), t("o_weight")
         self.norm_heads = self.norm.repeat(self.n_heads).contiguous()      # the one weight [vdim] under every head
@@ -419,7 +419,7 @@ class ChannelDelta(Mixer):
         if runs_side_by_side(x):   # few rows: beta's product beside the one that feeds everything, the gates' beside the convolution
             main, side = fork(x)
             with torch.cuda.stream(side):
-                logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)
+                logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)[:, :h]
             proj = ops.linear_rows(x, self.proj_weight)
             join(main, side, logit)
             main, side = fork(proj)
@@ -428,7 +428,7 @@ class ChannelDelta(Mixer):
             conv()
             join(main, side, z, gate)
         else:
-            logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)
+            logit = ops.linear_rows(x, self.b_weight, out_dtype=torch.float32)[:, :h]
             proj = ops.linear_rows(x, self.proj_weight)                                  # [T, q | k | v | A1 h | G1 h]
             z, gate = self._gates(x, proj)
             conv()
