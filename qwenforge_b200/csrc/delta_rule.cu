@@ -21,7 +21,7 @@
 // column's eight sums (four for u, four for y) are formed together and reduced together, each lane ending up with one of them.
 // What bounds the kernel is a warp's chain from one four to the next, so a lane has few rows (four or eight), and the rows of the
 // next four are asked for before the sums of this one are; two columns per lane where S is tall, because a block is then
-// bound by what it reads from shared memory. Records are staged through shared memory 16 or 32 tokens at a time by asynchronous copies, the next
+// bound by what it reads from shared memory. Records are staged through shared memory 16 or 32 tokens at a time by bulk copies, the next
 // ones under way while these are worked on. Fours are counted from a sequence's first token of the step; the last one is
 // filled up with tokens that do nothing (g = 1, k = q = 0).
 //
@@ -205,7 +205,7 @@ template <typename T, int LANES, int EACH, int R, int WARPS, int TOKENS>
 __global__ void __launch_bounds__(WARPS * 32)
 delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int v_stride, const int* __restrict__ cu_q,
                   const int* __restrict__ slots, float* __restrict__ state, long long slot_stride, long long s_offset, int n_records,
-                  int heads, int dim, int vdim, float* __restrict__ y) {
+                  int heads, int dim, int vdim, float* __restrict__ y, int* err) {
     constexpr int P = LANES * R, Q4 = R / 4, THREADS = WARPS * 32, FOURS = TOKENS / DS_GROUP, COLS = WARPS * 32 / LANES * EACH;
     constexpr int REC = (int)record_floats(P), SUMS = 8 * EACH;
     constexpr int SH = LANES / SUMS == 1 ? 0 : LANES / SUMS == 2 ? 1 : 2;   // after the reduction a lane has sum `part >> SH`
@@ -213,6 +213,8 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
     extern __shared__ __align__(16) float ds_smem[];
     float* rec_s = ds_smem;                                // [2][FOURS][REC]
     float* v_s = rec_s + 2 * FOURS * REC;                  // [2][TOKENS][COLS]
+    float* y_s = v_s + 2 * TOKENS * COLS;                  // [2][TOKENS][COLS]
+    __shared__ __align__(8) uint64_t arrived[2];           // a tile's records are complete
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, head = blockIdx.y, seq = blockIdx.z;
     const int part = lane & (LANES - 1), col_in = (warp * (32 / LANES) + lane / LANES) * EACH, col = blockIdx.x * COLS + col_in;
     const int begin = cu_q[seq], len = cu_q[seq + 1] - begin, slot = slots[seq];
@@ -227,36 +229,62 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
             const bool there = column && col + c < vdim;
             s[c][i] = pair_of(there && d < dim ? column[(size_t)d * vdim + c] : 0.f, there && d + 1 < dim ? column[(size_t)(d + 1) * vdim + c] : 0.f);
         }
-    constexpr int V_EACH = (TOKENS * COLS + THREADS - 1) / THREADS;
-    float v_next[V_EACH];
+    if (threadIdx.x == 0) {
+        mbar_init(&arrived[0], 1);
+        mbar_init(&arrived[1], 1);
+    }
+    __syncthreads();
+    // a thread's values of a tile (and outputs): tokens token0, token0 + STEP, .. of column c_own
+    constexpr int STEP = THREADS / COLS, EACH_THREAD = TOKENS / STEP;
+    static_assert(THREADS % COLS == 0 && TOKENS % STEP == 0, "a tile's values in whole rounds");
+    const int token0 = threadIdx.x / COLS, c_own = threadIdx.x % COLS;
+    const bool column_there = blockIdx.x * COLS + c_own < vdim;
+    const T* v_own = v + (size_t)(begin + token0) * v_stride + (size_t)head * vdim + blockIdx.x * COLS + c_own;
+    float* y_own = y + (size_t)(begin + token0) * ((size_t)heads * vdim) + (size_t)head * vdim + blockIdx.x * COLS + c_own;
+    const size_t v_step = (size_t)STEP * v_stride, y_step = (size_t)STEP * heads * vdim;
+    float v_next[EACH_THREAD];
     const float* records = packed + ((size_t)head * n_records + first_record(begin, seq)) * REC;
-    auto fetch = [&](int t0, int buf) {   // the records straight to shared memory, the values through registers
-        const int fours = min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP);
-        const float* from = records + (size_t)(t0 / DS_GROUP) * REC;
-        float* to = rec_s + buf * FOURS * REC;
-        for (int i = threadIdx.x; i < fours * (REC / 4); i += THREADS) cp_async_16(to + 4 * i, from + 4 * i, true);
-        cp_async_commit();
+    auto fetch = [&](int t0, int buf) {   // the records by one bulk copy to shared memory, the values through registers
+        if (threadIdx.x == 0) {
+            const uint32_t bytes = (uint32_t)(min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP) * REC * sizeof(float));
+            mbar_expect_tx(&arrived[buf], bytes);
+            bulk_copy_g2s(rec_s + buf * FOURS * REC, records + (size_t)(t0 / DS_GROUP) * REC, bytes, &arrived[buf]);
+        }
+        const T* from = v_own + (size_t)t0 * v_stride;
 #pragma unroll
-        for (int u = 0; u < V_EACH; ++u) {
-            const int i = threadIdx.x + u * THREADS, j = t0 + i / COLS, c = blockIdx.x * COLS + i % COLS;
+        for (int u = 0; u < EACH_THREAD; ++u) {
             v_next[u] = 0.f;
-            if (i < TOKENS * COLS && j < len && c < vdim) v_next[u] = load_value(v + (size_t)(begin + j) * v_stride + (size_t)head * vdim + c);
+            if (column_there && t0 + token0 + u * STEP < len) v_next[u] = load_value(from + u * v_step);
         }
     };
     auto stash = [&](int buf) {
 #pragma unroll
-        for (int u = 0; u < V_EACH; ++u)
-            if (threadIdx.x + u * THREADS < TOKENS * COLS) v_s[buf * TOKENS * COLS + threadIdx.x + u * THREADS] = v_next[u];
+        for (int u = 0; u < EACH_THREAD; ++u) v_s[buf * TOKENS * COLS + threadIdx.x + u * THREADS] = v_next[u];
+    };
+    auto flush = [&](int t0, int buf) {   // a finished tile's outputs
+        float* to = y_own + (size_t)t0 * heads * vdim;
+#pragma unroll
+        for (int u = 0; u < EACH_THREAD; ++u)
+            if (column_there && t0 + token0 + u * STEP < len) to[u * y_step] = y_s[buf * TOKENS * COLS + threadIdx.x + u * THREADS];
     };
     fetch(0, 0);
     stash(0);
+    int t_last = 0, buf_last = 0;
     for (int t0 = 0, turn = 0; t0 < len; t0 += TOKENS, ++turn) {
         const int buf = turn & 1, fours = min(FOURS, (len - t0 + DS_GROUP - 1) / DS_GROUP);
-        cp_async_wait<0>();
-        __syncthreads();   // these records have arrived for everyone, and everyone is done with the other buffer
+        // these records have arrived for everyone, and everyone is done with the tile before
+        if (!__syncthreads_and(mbar_wait(&arrived[buf], (turn >> 1) & 1))) {
+            mbar_wait(&arrived[buf], (turn >> 1) & 1);   // (bounded too: nothing of this block's may still be under way when it ends)
+            if (threadIdx.x == 0) atomicOr(err, QF_ERR_COPY_TIMEOUT);
+            return;
+        }
         const bool more = t0 + TOKENS < len;
         if (more) fetch(t0 + TOKENS, buf ^ 1);
+        if (turn > 0) flush(t0 - TOKENS, buf ^ 1);
+        t_last = t0;
+        buf_last = buf;
         const float* vs = v_s + buf * TOKENS * COLS + col_in;
+        float* ys = y_s + buf * TOKENS * COLS + col_in;
         auto rows_of = [&](int f) { return reinterpret_cast<const ulonglong2*>(rec_s + (buf * FOURS + f) * REC) + part; };
         ulonglong2 ahead[8][Q4];   // the rows of the eight sums: row x, its quarter i
         {
@@ -349,17 +377,17 @@ delta_scan_kernel(const float* __restrict__ packed, const T* __restrict__ v, int
                         s[c][2 * i + 1] = fma_pair(k[j][i].y, uu, s[c][2 * i + 1]);
                     }
                 }
-            const int sum = part >> SH, mine = sum >> 3, t = t0 + DS_GROUP * f + (sum & 3);   // mine: the column of this lane's sum
-            if ((sum & 4) && !(part & ((1 << SH) - 1)) && t < len && col + mine < vdim) {
-                float out = sums[0];
-                const float dj[4] = {d.x, d.y, d.z, d.w};
+            const int sum = part >> SH, mine = sum >> 3;   // mine: the column of this lane's sum
+            float out = sums[0];
+            const float dj[4] = {d.x, d.y, d.z, d.w};
 #pragma unroll
-                for (int j = 0; j < 4; ++j) out = fmaf(dj[j], EACH > 1 && mine ? u[EACH - 1][j] : u[0][j], out);
-                y[(size_t)(begin + t) * ((size_t)heads * vdim) + (size_t)head * vdim + col + mine] = out;
-            }
+            for (int j = 0; j < 4; ++j) out = fmaf(dj[j], EACH > 1 && mine ? u[EACH - 1][j] : u[0][j], out);
+            if ((sum & 4) && !(part & ((1 << SH) - 1))) ys[(4 * f + (sum & 3)) * COLS + mine] = out;
         }
         if (more) stash(buf ^ 1);
     }
+    __syncthreads();
+    flush(t_last, buf_last);
     if (column) {
 #pragma unroll
         for (int c = 0; c < EACH; ++c)
@@ -377,7 +405,7 @@ template <typename T, int LANES, int EACH, int R, int WARPS, int TOKENS>
 static int launch_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* z, int z_stride,
                        const float* bias, const float* rate_log, const float* logit, int logit_stride, const int* cu_q, const int* slots,
                        int n_seqs, int max_q_len, float* state, long long slot_stride, long long s_offset, int n_tokens, int heads, int groups,
-                       int dim, int vdim, float q_scale, float* packed, float* y, cudaStream_t stream) {
+                       int dim, int vdim, float q_scale, float* packed, float* y, int* err, cudaStream_t stream) {
     constexpr int COLS = WARPS * 32 / LANES * EACH;
     const int n_records = n_tokens / DS_GROUP + n_seqs;
     const long long items = (long long)((max_q_len + DS_GROUP - 1) / DS_GROUP) * heads;
@@ -385,13 +413,13 @@ static int launch_scan(const void* q, int q_stride, const void* k, int k_stride,
                                (const T*)q, q_stride, (const T*)k, k_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, n_records,
                                heads, groups, dim, q_scale, packed);
     if (e != cudaSuccess) return (int)e;
-    const size_t smem = (size_t)2 * (TOKENS / DS_GROUP * record_floats(LANES * R) + TOKENS * COLS) * sizeof(float);
+    const size_t smem = (size_t)2 * (TOKENS / DS_GROUP * record_floats(LANES * R) + 2 * TOKENS * COLS) * sizeof(float);
     e = cudaFuncSetAttribute(delta_scan_kernel<T, LANES, EACH, R, WARPS, TOKENS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     // launched the ordinary way: blocks that started under the first kernel's tail would crowd onto the SMs it leaves first,
     // and this kernel's few blocks are as fast as the SM they have to themselves
     delta_scan_kernel<T, LANES, EACH, R, WARPS, TOKENS><<<dim3((vdim + COLS - 1) / COLS, heads, n_seqs), dim3(WARPS * 32), smem, stream>>>(
-        packed, (const T*)v, v_stride, cu_q, slots, state, slot_stride, s_offset, n_records, heads, dim, vdim, y);
+        packed, (const T*)v, v_stride, cu_q, slots, state, slot_stride, s_offset, n_records, heads, dim, vdim, y, err);
     return (int)cudaGetLastError();
 }
 
@@ -406,18 +434,18 @@ QF_EXPORT int qf_delta_scan(int is_bf16, const void* q, int q_stride, const void
                             const float* z, int z_stride, const float* bias, const float* rate_log, const float* logit,
                             int logit_stride, const int* cu_q, const int* slots, int n_seqs, int max_q_len, float* state,
                             long long slot_stride, long long s_offset, int n_tokens, int heads, int groups, int dim, int vdim, float q_scale,
-                            float* packed, float* y, cudaStream_t stream) {
+                            float* packed, float* y, int* err, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (padded_dim(dim) == 0 || vdim <= 0 || groups <= 0 || heads % groups || n_seqs > 65535 || max_q_len <= 0 || heads > 65535 ||
         ((uintptr_t)packed & 15))
         return (int)cudaErrorInvalidValue;
 #define QF_DELTA_SCAN(...) (is_bf16 ? launch_scan<bf16, __VA_ARGS__>(QF_DELTA_ARGS) : launch_scan<float, __VA_ARGS__>(QF_DELTA_ARGS))
 #define QF_DELTA_ARGS q, q_stride, k, k_stride, v, v_stride, z, z_stride, bias, rate_log, logit, logit_stride, cu_q, slots, n_seqs, max_q_len, \
-                      state, slot_stride, s_offset, n_tokens, heads, groups, dim, vdim, q_scale, packed, y, stream
+                      state, slot_stride, s_offset, n_tokens, heads, groups, dim, vdim, q_scale, packed, y, err, stream
     switch (padded_dim(dim)) {
         case 32: return QF_DELTA_SCAN(8, 1, 4, 4, 32);
         case 64: return QF_DELTA_SCAN(16, 1, 4, 2, 32);
-        case 128: return QF_DELTA_SCAN(16, 2, 8, 4, 32);
+        case 128: return QF_DELTA_SCAN(32, 2, 4, 4, 32);
         default: return QF_DELTA_SCAN(32, 2, 8, 8, 16);
     }
 #undef QF_DELTA_ARGS

@@ -1849,7 +1849,8 @@ def _delta_args(what, q, k, v, z, bias, rate_log, logit, state, s_offset, n_head
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, rate_log: torch.Tensor,
                logit: torch.Tensor, cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_heads: int,
-               n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor, max_q_len: int = 0) -> None:
+               n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor, max_q_len: int = 0,
+               err: Optional[torch.Tensor] = None) -> None:
     """The gated delta rule with a decay per head and key channel, token after token of every sequence, float32 inside:
         q, k <- x / sqrt(sum(x^2) + 1e-6) per head (q also times q_scale);  g = exp(-exp(rate_log_h) softplus(z + bias));
         beta = sigmoid(logit);  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  y = S^T q.
@@ -1868,7 +1869,7 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tenso
     packed = torch.empty(n_heads * (n // 4 + n_seqs) * int(lib.qf_delta_record(_I(dim))), dtype=torch.float32, device=q.device)
     _check(lib.qf_delta_scan(*args, _ptr(cu_q), _ptr(slots), _I(n_seqs), _I(max_q_len or n), _ptr(state), _LL(state.stride(0)),
                              _LL(s_offset), _I(n), _I(n_heads), _I(n_groups), _I(dim), _I(vdim), _F(q_scale), _ptr(packed), _ptr(y),
-                             _stream()), "delta_scan")
+                             _ptr(err if err is not None else _err_word_for(q.device)), _stream()), "delta_scan")
 
 
 DELTA_FUSED_MAX_VDIM = 128   # value sizes up to which a single token's norm and gate ride on `delta_token`

@@ -442,7 +442,7 @@ class ChannelDelta(Mixer):
         if single:
             ops.delta_token(*args, y=y)
         else:
-            ops.delta_scan(*args, y, max_q_len=ctx.max_q_len)
+            ops.delta_scan(*args, y, max_q_len=ctx.max_q_len, err=ctx.err)
         ops.gated_group_norm(y, gate, self.norm_heads, self.eps, out, h, h, "sigmoid", False)
         return ops.linear_rows(out, self.o_weight)
 

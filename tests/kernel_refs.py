@@ -583,7 +583,7 @@ def sigmoid_gate(x, gate):
     x.copy_((_f(x) * torch.sigmoid(_f(gate))).to(x.dtype))
 
 
-def delta_scan(q, k, v, z, bias, rate_log, logit, cu_q, slots, state, s_offset, n_heads, n_groups, dim, vdim, q_scale, y, max_q_len=0):
+def delta_scan(q, k, v, z, bias, rate_log, logit, cu_q, slots, state, s_offset, n_heads, n_groups, dim, vdim, q_scale, y, max_q_len=0, err=None):
     per, size = n_heads // n_groups, n_heads * dim * vdim
     unit = lambda x: x / torch.sqrt(x.square().sum(-1, keepdim=True) + 1e-6)
     spread = lambda x: unit(_f(x).view(x.shape[0], n_groups, dim)).repeat_interleave(per, dim=1)
