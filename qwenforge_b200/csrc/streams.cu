@@ -84,12 +84,12 @@ template <> struct Channels<bf16, 4> {
 // NS: the most streams (a.n <= NS); HIST: the most inputs a convolution keeps (a.n_taps - 1 <= HIST), 0 without one; ROWS: tokens
 // of a tile, the HIST before it included.
 template <typename T, int V, int NS, int HIST, int ROWS>
-__global__ void __launch_bounds__(ST_THREADS)
+__global__ void __launch_bounds__(ST_THREADS, NS <= 4 ? 4 : 2)
 streams_kernel(const StreamsArgs<T> a) {
     grid_launch_dependents();
     constexpr int GROUPS = ST_THREADS / ROWS, OWN = ROWS - HIST;
     __shared__ float mix_s[NS * NS], out_s[NS], in_s[NS];
-    __shared__ __align__(16) float h_s[HIST > 0 ? ROWS : 1][HIST > 0 ? GROUPS * V : 1];
+    __shared__ __align__(16) float h_s[2][HIST > 0 ? ROWS : 1][HIST > 0 ? GROUPS * V : 1];   // two tiles in turn
     // the coefficients are weights: fetched before the wait for the kernel before this one
     for (int i = threadIdx.x; i < NS * NS; i += ST_THREADS) {
         const int s = i / NS, r = i % NS;
@@ -102,7 +102,8 @@ streams_kernel(const StreamsArgs<T> a) {
     const int group = threadIdx.x % GROUPS, row = threadIdx.x / GROUPS;
     const int c0 = (blockIdx.x * GROUPS + group) * V;
     const bool in = c0 < a.width;
-    float w[V], b[V], f[HIST > 0 ? HIST + 1 : 1][V];
+    __shared__ __align__(16) float f_s[HIST + 1][HIST > 0 ? GROUPS * V : 1];   // the filter, a column per channel
+    float w[V], b[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) w[v] = b[v] = 0.f;
     if (a.weight && in) {
@@ -110,13 +111,10 @@ streams_kernel(const StreamsArgs<T> a) {
         Channels<T, V>::load(a.bias + c0, b);
     }
     if constexpr (HIST > 0) {
-#pragma unroll
-        for (int j = 0; j <= HIST; ++j)   // the oldest places of a shorter filter hold zeros
-#pragma unroll
-            for (int v = 0; v < V; ++v) {
-                const int at = j - (HIST + 1 - a.n_taps);
-                f[j][v] = (in && row >= HIST && at >= 0) ? a.taps[(size_t)(c0 + v) * a.n_taps + at] : 0.f;
-            }
+        for (int i = threadIdx.x; i < (HIST + 1) * GROUPS * V; i += ST_THREADS) {   // the oldest places of a shorter filter hold zeros
+            const int c = i / (HIST + 1), j = i % (HIST + 1), channel = blockIdx.x * GROUPS * V + c, at = j - (HIST + 1 - a.n_taps);
+            f_s[j][c] = (channel < a.width && at >= 0) ? a.taps[(size_t)channel * a.n_taps + at] : 0.f;
+        }
     }
     __syncthreads();
     grid_dependency_wait();
@@ -192,44 +190,48 @@ streams_kernel(const StreamsArgs<T> a) {
         else Channels<float, V>::store(a.u_out + (size_t)i * a.width + c0, h);
     } else {
         const int begin = a.cu_q[blockIdx.z], len = a.cu_q[blockIdx.z + 1] - begin, slot = a.slots[blockIdx.z];
-        const int first = blockIdx.y * OWN, kept = a.n_taps - 1;
-        if (first >= len) return;   // (the whole block)
+        const int kept = a.n_taps - 1;
         float* rows = (slot >= 0 && in) ? a.state + slot * a.slot_stride + a.offset + c0 : nullptr;
-        const int at = first - HIST + row;   // this thread's token, counted from the sequence's first of the step
-        float h[V];
+        for (int first = blockIdx.y * OWN, buf = 0; first < len; first += gridDim.y * OWN, buf ^= 1) {   // (the same for the whole block)
+            const int at = first - HIST + row;   // this thread's token, counted from the sequence's first of the step
+            float h[V];
 #pragma unroll
-        for (int v = 0; v < V; ++v) h[v] = 0.f;
-        if (in && at < len) {
-            if (at >= 0 && row >= HIST - kept) {
-                value(begin + at, row >= HIST, h);
-            } else if (at < 0 && rows && kept + at >= 0) {   // (before the step: the state's row, the newest last)
-                Channels<float, V>::load(rows + (size_t)(kept + at) * a.width, h);
+            for (int v = 0; v < V; ++v) h[v] = 0.f;
+            if (in && at < len) {
+                if (at >= 0 && row >= HIST - kept) {
+                    value(begin + at, row >= HIST, h);
+                } else if (at < 0 && rows && kept + at >= 0) {   // (before the step: the state's row, the newest last)
+                    Channels<float, V>::load(rows + (size_t)(kept + at) * a.width, h);
+                }
             }
-        }
-        Channels<float, V>::store(&h_s[row][group * V], h);
-        __syncthreads();
-        if (row >= HIST && in && at < len) {
-            float z[V];
+            Channels<float, V>::store(&h_s[buf][row][group * V], h);
+            __syncthreads();   // the tile's h are there; and nobody still reads the tile before the last
+            if (row >= HIST && in && at < len) {
+                float z[V];
 #pragma unroll
-            for (int v = 0; v < V; ++v) z[v] = 0.f;
+                for (int v = 0; v < V; ++v) z[v] = 0.f;
 #pragma unroll
-            for (int j = 0; j < HIST; ++j) {
-                float before[V];
-                Channels<float, V>::load(&h_s[row - HIST + j][group * V], before);
+                for (int j = 0; j < HIST; ++j) {
+                    float before[V], f[V];
+                    Channels<float, V>::load(&h_s[buf][row - HIST + j][group * V], before);
+                    Channels<float, V>::load(&f_s[j][group * V], f);
 #pragma unroll
-                for (int v = 0; v < V; ++v) z[v] = fmaf(f[j][v], before[v], z[v]);
+                    for (int v = 0; v < V; ++v) z[v] = fmaf(f[v], before[v], z[v]);
+                }
+                float f[V];
+                Channels<float, V>::load(&f_s[HIST][group * V], f);
+#pragma unroll
+                for (int v = 0; v < V; ++v) z[v] = h[v] + fmaf(f[v], h[v], z[v]);
+                Channels<T, V>::store(a.z + (size_t)(begin + at) * a.width + c0, z);
             }
-#pragma unroll
-            for (int v = 0; v < V; ++v) z[v] = h[v] + fmaf(f[HIST][v], h[v], z[v]);
-            Channels<T, V>::store(a.z + (size_t)(begin + at) * a.width + c0, z);
-        }
-        if (first == 0 && rows && row < kept) {
-            // the sequence's last `kept` values: in shared memory if it ends in this tile, else worked out again
-            const int back = len - kept + row;
-            float last[V];
-            if (len <= OWN) Channels<float, V>::load(&h_s[HIST + back][group * V], last);
-            else value(begin + back, false, last);
-            Channels<float, V>::store(rows + (size_t)row * a.width, last);
+            if (first == 0 && rows && row < kept) {
+                // the sequence's last `kept` values: in shared memory if it ends in this tile, else worked out again
+                const int back = len - kept + row;
+                float last[V];
+                if (len <= OWN) Channels<float, V>::load(&h_s[buf][HIST + back][group * V], last);
+                else value(begin + back, false, last);
+                Channels<float, V>::store(rows + (size_t)row * a.width, last);
+            }
         }
     }
 }
@@ -239,8 +241,15 @@ static int launch_streams(const StreamsArgs<T>& a, int n_seqs, int max_q_len, cu
     constexpr int OWN = ROWS - HIST, CHANNELS = ST_THREADS / ROWS * V;
     const long long longest = HIST > 0 ? max_q_len : (a.rows ? a.n_rows : a.n_tokens);
     const long long tiles = (longest + OWN - 1) / OWN;
-    const dim3 grid((a.width + CHANNELS - 1) / CHANNELS, (unsigned)tiles, HIST > 0 ? n_seqs : 1);
-    if (tiles > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
+    const int columns = (a.width + CHANNELS - 1) / CHANNELS;
+    long long down = tiles;
+    if (HIST > 0) {   // a block walks several tiles when there are more than the SMs hold at once: its coefficients stay
+        const long long held = (NS <= 4 ? 4ll : 2ll) * qf_sm_count() / ((long long)columns * n_seqs);
+        if (held >= 1 && down > held) down = (down + (down + held - 1) / held - 1) / ((down + held - 1) / held);
+        else if (held < 1) down = 1;
+    }
+    const dim3 grid(columns, (unsigned)down, HIST > 0 ? n_seqs : 1);
+    if (down > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
     return (int)launch_pdl(streams_kernel<T, V, NS, HIST, ROWS>, grid, dim3(ST_THREADS), 0, stream, a);
 }
 
