@@ -44,7 +44,7 @@ QF_EXPORT int qf_decode_advance(const int* sampled, int* token_ids, int* tok_pos
 }
 
 // The same step of the rows' state, and the NEXT step's first kernel with it: a block per row updates the row as above
-// and then copies the embedding of the row's next input token into the float32 stream `hidden[row]`, so that the next
+// and then copies the embedding of the row's next input token (times `scale`) into the float32 stream `hidden[row]`, so that the next
 // step starts at its first layer. All blocks read the cursor before any block can move it: the block that draws the
 // last ticket does that (and puts the ticket counter back to zero).
 template <typename T>
@@ -53,7 +53,7 @@ decode_advance_embed_kernel(const int* __restrict__ sampled, int* __restrict__ t
                             int* __restrict__ slots, int* __restrict__ steps, const int* __restrict__ budgets,
                             const int* __restrict__ stop_ids, int n_stop, int* __restrict__ out_tokens,
                             int* __restrict__ cursor, int max_steps, const T* __restrict__ table, int vocab, int width,
-                            float* __restrict__ hidden, int* __restrict__ ticket, int* err) {
+                            float scale, float* __restrict__ hidden, int* __restrict__ ticket, int* err) {
     grid_chain_entry();
     __shared__ int next_s, at_s;
     const int r = blockIdx.x, n_rows = gridDim.x;
@@ -86,7 +86,7 @@ decode_advance_embed_kernel(const int* __restrict__ sampled, int* __restrict__ t
     }
     const T* row = table + (size_t)id * width;
     float* dst = hidden + (size_t)r * width;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = bad ? 0.f : Num<T>::to_f(row[c]);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = bad ? 0.f : Num<T>::to_f(row[c]) * scale;
     if (threadIdx.x == 0) {
         __threadfence();
         if (atomicAdd(ticket, 1) == n_rows - 1) {
@@ -101,16 +101,16 @@ decode_advance_embed_kernel(const int* __restrict__ sampled, int* __restrict__ t
 QF_EXPORT int qf_decode_advance_embed(const int* sampled, int* token_ids, int* tok_pos, int* slots, int* steps,
                                       const int* budgets, const int* stop_ids, int n_stop, int* out_tokens, int* cursor,
                                       int max_steps, int n_rows, int is_bf16, const void* table, int vocab, int width,
-                                      float* hidden, int* ticket, int* err, cudaStream_t stream) {
+                                      float scale, float* hidden, int* ticket, int* err, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     int code;
     if (is_bf16)
         code = (int)launch_pdl(decode_advance_embed_kernel<bf16>, dim3(n_rows), dim3(128), 0, stream, sampled, token_ids, tok_pos, slots, steps, budgets,
                                                                      stop_ids, n_stop, out_tokens, cursor, max_steps,
-                                                                     (const bf16*)table, vocab, width, hidden, ticket, err);
+                                                                     (const bf16*)table, vocab, width, scale, hidden, ticket, err);
     else
         code = (int)launch_pdl(decode_advance_embed_kernel<float>, dim3(n_rows), dim3(128), 0, stream, sampled, token_ids, tok_pos, slots, steps, budgets,
                                                                       stop_ids, n_stop, out_tokens, cursor, max_steps,
-                                                                      (const float*)table, vocab, width, hidden, ticket, err);
+                                                                      (const float*)table, vocab, width, scale, hidden, ticket, err);
     return code;
 }

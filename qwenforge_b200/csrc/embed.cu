@@ -1,10 +1,10 @@
-// Row gathers: token embedding into the float32 residual stream, and the gather of the
+// Row gathers: token embedding (times a scale) into the float32 residual stream, and the gather of the
 // rows whose logits are wanted.
 #include "common.cuh"
 
 template <typename T>
 __global__ void embed_gather_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
-                                    int vocab, int width, int* err) {
+                                    int vocab, int width, float scale, int* err) {
     grid_chain_entry();
     const int t = blockIdx.x;
     int id = ids[t];
@@ -15,7 +15,7 @@ __global__ void embed_gather_kernel(const int* __restrict__ ids, const T* __rest
     }
     const T* row = table + (size_t)id * width;
     float* dst = out + (size_t)t * width;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = bad ? 0.f : Num<T>::to_f(row[c]);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = bad ? 0.f : Num<T>::to_f(row[c]) * scale;
 }
 
 // out[t] = table[ids[t]] + positions[tok_pos[t]]: token embedding plus a learned vector per absolute position, summed in
@@ -108,10 +108,10 @@ QF_EXPORT int qf_gather_rows_norm(int is_bf16, const float* hidden, const void* 
 }
 
 template <typename T>
-static int embed_launch(const int* ids, const void* table, float* out, int n_tokens, int vocab, int width, int* err,
+static int embed_launch(const int* ids, const void* table, float* out, int n_tokens, int vocab, int width, float scale, int* err,
                         cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    return (int)launch_pdl(embed_gather_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, ids, (const T*)table, out, vocab, width, err);
+    return (int)launch_pdl(embed_gather_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, ids, (const T*)table, out, vocab, width, scale, err);
 }
 
 template <typename T>
@@ -122,9 +122,9 @@ static int gather_launch(const float* hidden, const void* delta, const int* rows
 }
 
 QF_EXPORT int qf_embed_gather(int is_bf16, const int* ids, const void* table, float* out, int n_tokens, int vocab,
-                              int width, int* err, cudaStream_t stream) {
-    return is_bf16 ? embed_launch<bf16>(ids, table, out, n_tokens, vocab, width, err, stream)
-                   : embed_launch<float>(ids, table, out, n_tokens, vocab, width, err, stream);
+                              int width, float scale, int* err, cudaStream_t stream) {
+    return is_bf16 ? embed_launch<bf16>(ids, table, out, n_tokens, vocab, width, scale, err, stream)
+                   : embed_launch<float>(ids, table, out, n_tokens, vocab, width, scale, err, stream);
 }
 
 QF_EXPORT int qf_gather_rows(int is_bf16, const float* hidden, const void* delta, const int* rows, float* out,

@@ -54,20 +54,29 @@ __device__ __forceinline__ void moe_choose(const float* z_raw, const float* bias
 }
 
 // The choice among groups of neighbouring experts, with a correction that steers the choice and not the weights:
-//   s_e = sigmoid(z_e);  c_e = s_e + correction_e (the choice score);  the experts form `group_count` equal groups of
-//   neighbours, a group's score is the sum of its two largest c (of its one, in groups of one);  only experts of the
-//   `group_keep` groups with the largest scores can be chosen;  among them the `top` largest c;  weights s_e, divided by
-//   their sum with `renormalize`.  Ties go to the lower index.  (group_count 1: no groups.)
+//   s_e = sigmoid(z_e), or with `softmax_scores` the softmax over all experts;  c_e = s_e + correction_e (the choice score);  the
+//   experts form `count` equal groups of neighbours, a group's score is the sum of its `best` largest c (1 or 2; of its one, in
+//   groups of one);  only experts of the `keep` groups with the largest scores can be chosen;  among them the `top` largest c;
+//   weights s_e, divided by their sum with `renormalize`.  Ties go to the lower index.  (count 1: no groups.)
+// Softmax scores rise with their logits: where no correction and no sum of two enters, the choice compares the logits.
 struct MoeGroups {
     const float* correction;   // float32 [experts] or null
-    int count, keep;
+    int count, keep, best;
 };
 #define MOE_MAX_GROUPS 64
 
-__device__ __forceinline__ void moe_choose_grouped(const float* z_raw, const float* bias, int n_experts, int top, int renormalize,
-                                                   MoeGroups groups, int* chosen, float* weight) {
-    auto score = [&](int e) { return 1.0f / (1.0f + expf(-(bias ? z_raw[e] + bias[e] : z_raw[e]))); };
-    auto choice = [&](int e) { return groups.correction ? score(e) + groups.correction[e] : score(e); };
+__device__ __forceinline__ void moe_choose_grouped(const float* z_raw, const float* bias, int n_experts, int top, int softmax_scores,
+                                                   int renormalize, MoeGroups groups, int* chosen, float* weight) {
+    auto z = [&](int e) { return bias ? z_raw[e] + bias[e] : z_raw[e]; };
+    float top_z = -FLT_MAX, denom = 1.f;
+    if (softmax_scores) {
+        for (int e = 0; e < n_experts; ++e) top_z = fmaxf(top_z, z(e));
+        denom = 0.f;
+        for (int e = 0; e < n_experts; ++e) denom += expf(z(e) - top_z);
+    }
+    const bool by_logit = softmax_scores && !groups.correction && groups.best == 1;
+    auto score = [&](int e) { return softmax_scores ? expf(z(e) - top_z) / denom : 1.0f / (1.0f + expf(-z(e))); };
+    auto choice = [&](int e) { return by_logit ? z(e) : groups.correction ? score(e) + groups.correction[e] : score(e); };
     unsigned long long kept = ~0ull;
     const int size = n_experts / groups.count;
     if (groups.count > 1 && groups.keep < groups.count) {
@@ -83,7 +92,7 @@ __device__ __forceinline__ void moe_choose_grouped(const float* z_raw, const flo
                     second = c;
                 }
             }
-            group_score[g] = size > 1 ? first + second : first;
+            group_score[g] = size > 1 && groups.best > 1 ? first + second : first;
         }
         kept = 0ull;
         for (int k = 0; k < groups.keep; ++k) {
@@ -189,7 +198,7 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
     for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
         int chosen[MOE_MAX_TOP];
         float weight[MOE_MAX_TOP];
-        if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, renormalize, groups, chosen, weight);
+        if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, groups, chosen, weight);
         else moe_choose(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, chosen, weight);
         for (int k = 0; k < top; ++k) {
             const int pair = t * top + k;
@@ -250,7 +259,7 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, 
     int chosen[MOE_MAX_TOP], rank[MOE_MAX_TOP];
     float weight[MOE_MAX_TOP];
     if (t < n_tokens) {
-        if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, renormalize, groups, chosen, weight);
+        if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, groups, chosen, weight);
         else moe_choose(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, chosen, weight);
         for (int k = 0; k < top; ++k) rank[k] = atomicAdd(&counts[chosen[k]], 1);
     }
@@ -414,18 +423,18 @@ moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ dest, const 
 // is given, or x [n_tokens][width] and router [n_experts][width] (both bfloat16 or both float32), from which the kernel makes
 // the logits itself in shared memory (n_tokens * n_experts <= 8192).
 // bias: float32 [n_experts] added to the logits, or null.
-// correction (float32 [n_experts] or null), group_count, group_keep: the choice among groups of neighbouring experts
-// (`moe_choose_grouped`; sigmoid scores); group_count 0: the plain choice.
+// correction (float32 [n_experts] or null), group_count, group_keep, group_best: the choice among groups of neighbouring experts
+// (`moe_choose_grouped`); group_count 0: the plain choice.
 QF_EXPORT int qf_moe_plan_grouped(const float* logits, int n_tokens, int n_experts, int top, int softmax_scores, int renormalize,
                                   int* pair_expert, float* pair_weight, int* sorted_token, float* sorted_weight, int* dest,
                                   int* offsets, int* tile_group, int* tile_row0, int* n_tiles, int max_tiles, int tile_rows,
                                   const void* x, const void* router, int width, int x_is_bf16, const float* bias,
-                                  const float* correction, int group_count, int group_keep, cudaStream_t stream) {
+                                  const float* correction, int group_count, int group_keep, int group_best, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (group_count < 0 || group_count > MOE_MAX_GROUPS || (group_count > 0 && (n_experts % group_count || group_keep < 1 ||
-        group_keep > group_count || (long long)group_keep * (n_experts / group_count) < top || softmax_scores)))
+        group_keep > group_count || (long long)group_keep * (n_experts / group_count) < top || group_best < 1 || group_best > 2)))
         return (int)cudaErrorInvalidValue;
-    const MoeGroups groups = {correction, group_count, group_keep};
+    const MoeGroups groups = {correction, group_count, group_keep, group_best};
     if (top < 1 || top > MOE_MAX_TOP || top > n_experts || n_experts > 8192 || tile_rows <= 0) return (int)cudaErrorInvalidValue;
     if (!logits && !(x && router && (long long)n_tokens * n_experts <= 8192)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)(2 * n_experts + 1) * sizeof(int) + (logits ? 0 : (size_t)n_tokens * n_experts * sizeof(float));
@@ -442,7 +451,7 @@ QF_EXPORT int qf_moe_plan_biased(const float* logits, int n_tokens, int n_expert
                                  cudaStream_t stream) {
     return qf_moe_plan_grouped(logits, n_tokens, n_experts, top, softmax_scores, renormalize, pair_expert, pair_weight, sorted_token,
                                sorted_weight, dest, offsets, tile_group, tile_row0, n_tiles, max_tiles, tile_rows, x, router, width,
-                               x_is_bf16, bias, nullptr, 0, 0, stream);
+                               x_is_bf16, bias, nullptr, 0, 0, 2, stream);
 }
 
 QF_EXPORT int qf_moe_plan(const float* logits, int n_tokens, int n_experts, int top, int softmax_scores, int renormalize,
@@ -491,12 +500,12 @@ QF_EXPORT int qf_moe_plan_long_grouped(const float* logits, int n_tokens, int n_
                                        int renormalize, int* pair_expert, float* pair_weight, int* sorted_token,
                                        float* sorted_weight, int* dest, int* offsets, int* tile_group, int* tile_row0, int* n_tiles,
                                        int max_tiles, int tile_rows, int* expert_rows, const float* bias, const float* correction,
-                                       int group_count, int group_keep, cudaStream_t stream) {
+                                       int group_count, int group_keep, int group_best, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (group_count < 0 || group_count > MOE_MAX_GROUPS || (group_count > 0 && (n_experts % group_count || group_keep < 1 ||
-        group_keep > group_count || (long long)group_keep * (n_experts / group_count) < top || softmax_scores)))
+        group_keep > group_count || (long long)group_keep * (n_experts / group_count) < top || group_best < 1 || group_best > 2)))
         return (int)cudaErrorInvalidValue;
-    const MoeGroups groups = {correction, group_count, group_keep};
+    const MoeGroups groups = {correction, group_count, group_keep, group_best};
     if (top < 1 || top > MOE_MAX_TOP || top > n_experts || n_experts > 4096 || tile_rows <= 0 || !logits || !expert_rows)
         return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)(2 * n_experts + 1) * sizeof(int);
@@ -517,7 +526,7 @@ QF_EXPORT int qf_moe_plan_long_biased(const float* logits, int n_tokens, int n_e
                                       int max_tiles, int tile_rows, int* expert_rows, const float* bias, cudaStream_t stream) {
     return qf_moe_plan_long_grouped(logits, n_tokens, n_experts, top, softmax_scores, renormalize, pair_expert, pair_weight,
                                     sorted_token, sorted_weight, dest, offsets, tile_group, tile_row0, n_tiles, max_tiles, tile_rows,
-                                    expert_rows, bias, nullptr, 0, 0, stream);
+                                    expert_rows, bias, nullptr, 0, 0, 2, stream);
 }
 
 QF_EXPORT int qf_moe_plan_long(const float* logits, int n_tokens, int n_experts, int top, int softmax_scores, int renormalize,

@@ -704,3 +704,251 @@ QF_EXPORT int qf_rows_prepare(int is_bf16, void* x, int ld, int rows, int n_runs
         return (int)launch_pdl(rows_prepare_kernel<bf16>, dim3(rows, n_runs), dim3(128), 0, stream, (bf16*)x, ld, r[0], r[1], r[2], mix, eps);
     return (int)launch_pdl(rows_prepare_kernel<float>, dim3(rows, n_runs), dim3(128), 0, stream, (float*)x, ld, r[0], r[1], r[2], mix, eps);
 }
+
+// ------------------------------------------------------------------------------------------------------------------
+// Two RMS norms of one stream, for a layer whose two sublayers read norms of their own of the same x, with the two outputs of
+// the layer before on their way into it:
+//   hidden += (a + b) (each if given);  r = 1 / sqrt(mean(hidden^2) + eps);  out1 = hidden * r1 * w1;  out2 = hidden * r2 * w2
+// (either norm, or both, may be left out). b may be unsummed expert rows: with `dest`, row t of b is the sum of the `top` rows
+// b[dest[t * top + k]] (each times row_weight[that row], if given) in the order of k. With `rows`, output row i is the norm of
+// stream row rows[i] and the stream is left as it is (what an output head reads). Float32 inside. A TEAM of threads works on a
+// row (a warp for rows of up to 1,024 columns, a block beyond) and keeps up to KEEP groups of four columns per thread; which one,
+// and the order of its additions, depends on the width alone.
+#define PN_MAX_TOP 16
+template <typename T, int TEAM, int KEEP>
+__global__ void __launch_bounds__(256)
+pair_rms_norm_kernel(float* __restrict__ hidden, const T* __restrict__ a, const T* __restrict__ b, const int* __restrict__ dest, int top,
+                     const float* __restrict__ row_weight, const T* __restrict__ w1, float eps1, T* __restrict__ out1,
+                     const T* __restrict__ w2, float eps2, T* __restrict__ out2, const int* __restrict__ rows, int n_out, int n_in,
+                     int width, int* err) {
+    grid_chain_entry();
+    __shared__ float scratch[33];
+    const int lane = threadIdx.x % TEAM, team = threadIdx.x / TEAM;
+    const int i = blockIdx.x * (blockDim.x / TEAM) + team;
+    if (i >= n_out) return;   // (a block-wide team has a row of its own: all its threads leave together)
+    int t = rows ? rows[i] : i;
+    if (t < 0 || t >= n_in) {
+        if (lane == 0) atomicOr(err, QF_ERR_ROW_RANGE);
+        t = 0;
+    }
+    const int n4 = width / 4;
+    float* h = hidden + (size_t)t * width;
+    float4 v[KEEP], add[KEEP];
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+        const int c = lane + TEAM * u;
+        v[u] = c < n4 ? Vec4<float>::load(h + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        add[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (b && dest) {   // the token's expert rows: their places and weights first, then four rows at a time, in their order
+        int src[PN_MAX_TOP];
+        float w[PN_MAX_TOP];
+#pragma unroll
+        for (int k = 0; k < PN_MAX_TOP; ++k)
+            if (k < top) {
+                src[k] = dest[(size_t)t * top + k];
+                w[k] = row_weight ? row_weight[src[k]] : 1.f;
+            }
+#pragma unroll
+        for (int k = 0; k < PN_MAX_TOP; ++k)
+            if (k < top) {
+                const T* y = b + (size_t)src[k] * width;
+#pragma unroll
+                for (int u = 0; u < KEEP; ++u) {
+                    const int c = lane + TEAM * u;
+                    if (c < n4) {
+                        const float4 x = Vec4<T>::load(y + 4 * c);
+                        add[u].x += x.x * w[k];
+                        add[u].y += x.y * w[k];
+                        add[u].z += x.z * w[k];
+                        add[u].w += x.w * w[k];
+                    }
+                }
+            }
+    } else if (b) {
+#pragma unroll
+        for (int u = 0; u < KEEP; ++u) {
+            const int c = lane + TEAM * u;
+            if (c < n4) add[u] = Vec4<T>::load(b + (size_t)t * width + 4 * c);
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+        const int c = lane + TEAM * u;
+        if (c >= n4) continue;
+        if (a) {
+            const float4 x = Vec4<T>::load(a + (size_t)t * width + 4 * c);
+            add[u] = make_float4(x.x + add[u].x, x.y + add[u].y, x.z + add[u].z, x.w + add[u].w);
+        }
+        if (a || b) {
+            v[u] = make_float4(v[u].x + add[u].x, v[u].y + add[u].y, v[u].z + add[u].z, v[u].w + add[u].w);
+            if (!rows) Vec4<float>::store(h + 4 * c, v[u]);
+        }
+        ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    }
+    if (!w1 && !w2) return;
+    const float mean = (TEAM == 32 ? warp_sum(ss) : block_sum(ss, scratch)) / (float)width;
+    const float r1 = 1.0f / sqrtf(mean + eps1), r2 = 1.0f / sqrtf(mean + eps2);
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+        const int c = lane + TEAM * u;
+        if (c >= n4) continue;
+        if (w1) {
+            const float4 w = Vec4<T>::load(w1 + 4 * c);
+            Vec4<T>::store(out1 + (size_t)i * width + 4 * c, make_float4(v[u].x * r1 * w.x, v[u].y * r1 * w.y, v[u].z * r1 * w.z, v[u].w * r1 * w.w));
+        }
+        if (w2) {
+            const float4 w = Vec4<T>::load(w2 + 4 * c);
+            Vec4<T>::store(out2 + (size_t)i * width + 4 * c, make_float4(v[u].x * r2 * w.x, v[u].y * r2 * w.y, v[u].z * r2 * w.z, v[u].w * r2 * w.w));
+        }
+    }
+}
+
+// The same for any width and alignment: a block per row, an element at a time, what is pending summed twice where it is not stored.
+template <typename T>
+__global__ void __launch_bounds__(256)
+pair_rms_norm_any_kernel(float* __restrict__ hidden, const T* __restrict__ a, const T* __restrict__ b, const int* __restrict__ dest, int top,
+                         const float* __restrict__ row_weight, const T* __restrict__ w1, float eps1, T* __restrict__ out1,
+                         const T* __restrict__ w2, float eps2, T* __restrict__ out2, const int* __restrict__ rows, int n_in, int width,
+                         int* err) {
+    grid_chain_entry();
+    __shared__ float scratch[33];
+    const int i = blockIdx.x;
+    int t = rows ? rows[i] : i;
+    if (t < 0 || t >= n_in) {
+        if (threadIdx.x == 0) atomicOr(err, QF_ERR_ROW_RANGE);
+        t = 0;
+    }
+    float* h = hidden + (size_t)t * width;
+    auto pending = [&](int c) -> float {
+        float sum = 0.f;
+        if (b && dest) {
+            for (int k = 0; k < top; ++k) {
+                const int r = dest[(size_t)t * top + k];
+                sum += Num<T>::to_f(b[(size_t)r * width + c]) * (row_weight ? row_weight[r] : 1.f);
+            }
+        } else if (b) {
+            sum = Num<T>::to_f(b[(size_t)t * width + c]);
+        }
+        return a ? Num<T>::to_f(a[(size_t)t * width + c]) + sum : sum;
+    };
+    const bool any = a || b;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float x = any ? h[c] + pending(c) : h[c];
+        if (any && !rows) h[c] = x;
+        ss += x * x;
+    }
+    if (!w1 && !w2) return;
+    const float mean = block_sum(ss, scratch) / (float)width;
+    const float r1 = 1.0f / sqrtf(mean + eps1), r2 = 1.0f / sqrtf(mean + eps2);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {   // each thread re-reads the columns it wrote itself
+        const float x = any && rows ? h[c] + pending(c) : h[c];
+        if (w1) out1[(size_t)i * width + c] = Num<T>::from_f(x * r1 * Num<T>::to_f(w1[c]));
+        if (w2) out2[(size_t)i * width + c] = Num<T>::from_f(x * r2 * Num<T>::to_f(w2[c]));
+    }
+}
+
+template <typename T>
+static int pair_norm_launch(float* hidden, const void* a, const void* b, const int* dest, int top, const float* row_weight, const void* w1,
+                            float eps1, void* out1, const void* w2, float eps2, void* out2, const int* rows, int n_out, int n_in, int width,
+                            int* err, cudaStream_t stream) {
+    if (n_out <= 0) return 0;
+    const uintptr_t align = (uintptr_t)hidden | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out1 | (uintptr_t)out2;
+    if (width % 4 == 0 && width <= 4096 && align % 16 == 0 && top <= PN_MAX_TOP) {
+#define QF_PAIR_ARGS hidden, (const T*)a, (const T*)b, dest, top, row_weight, (const T*)w1, eps1, (T*)out1, (const T*)w2, eps2, (T*)out2, rows, \
+                     n_out, n_in, width, err
+        if (width <= 1024) {
+            const int per_block = n_out >= 2048 ? 8 : n_out >= 512 ? 2 : 1;
+            return (int)launch_pdl(pair_rms_norm_kernel<T, 32, 8>, dim3((n_out + per_block - 1) / per_block), dim3(32 * per_block), 0, stream, QF_PAIR_ARGS);
+        }
+        if (width <= 2048) return (int)launch_pdl(pair_rms_norm_kernel<T, 256, 2>, dim3(n_out), dim3(256), 0, stream, QF_PAIR_ARGS);
+        return (int)launch_pdl(pair_rms_norm_kernel<T, 256, 4>, dim3(n_out), dim3(256), 0, stream, QF_PAIR_ARGS);
+#undef QF_PAIR_ARGS
+    }
+    return (int)launch_pdl(pair_rms_norm_any_kernel<T>, dim3(n_out), dim3(256), 0, stream, hidden, (const T*)a, (const T*)b, dest, top, row_weight,
+                           (const T*)w1, eps1, (T*)out1, (const T*)w2, eps2, (T*)out2, rows, n_in, width, err);
+}
+
+// hidden float32 [n_in][width]; a, b (null where absent), w1, w2, out1, out2 share the activation type; dest, row_weight, rows: above.
+QF_EXPORT int qf_pair_rms_norm(int is_bf16, float* hidden, const void* a, const void* b, const int* dest, int top, const float* row_weight,
+                               const void* w1, float eps1, void* out1, const void* w2, float eps2, void* out2, const int* rows, int n_out,
+                               int n_in, int width, int* err, cudaStream_t stream) {
+    if ((dest && top < 1) || (!w1 != !out1) || (!w2 != !out2)) return (int)cudaErrorInvalidValue;
+    return is_bf16 ? pair_norm_launch<bf16>(hidden, a, b, dest, top, row_weight, w1, eps1, out1, w2, eps2, out2, rows, n_out, n_in, width, err, stream)
+                   : pair_norm_launch<float>(hidden, a, b, dest, top, row_weight, w1, eps1, out1, w2, eps2, out2, rows, n_out, n_in, width, err, stream);
+}
+
+// ------------------------------------------------------------------------------------------------------------------
+// The two maps of a differential attention brought together, per token and head:
+//   o = a1 - weight * a2;   out = gain * o / sqrt(mean(o^2) + eps)
+// x: [n_tokens][heads][2][pitch], the maps' attended values in the first vdim components; out: [n_tokens][heads * vdim].
+// A warp per (token, head); float32 inside.
+#define MD_MAX 8   // elements per lane: vdim up to 256 as pairs
+template <typename T, bool PAIRS>
+__global__ void __launch_bounds__(256)
+map_difference_kernel(const T* __restrict__ x, int pitch, float weight, float eps, float gain, T* __restrict__ out, long long items, int vdim) {
+    grid_chain_entry();
+    const int lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= items) return;
+    const T* a1 = x + item * 2 * pitch;
+    const T* a2 = a1 + pitch;
+    T* o = out + item * vdim;
+    float v[MD_MAX];
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < MD_MAX; ++u) {
+        const int c = PAIRS ? 64 * (u / 2) + 2 * lane + (u & 1) : 32 * u + lane;
+        if (PAIRS && (u & 1)) continue;
+        if constexpr (PAIRS) {
+            float2 p = make_float2(0.f, 0.f), q = make_float2(0.f, 0.f);
+            if (c < vdim) {
+                if constexpr (sizeof(T) == 2) {
+                    p = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a1 + c));
+                    q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a2 + c));
+                } else {
+                    p = *reinterpret_cast<const float2*>(a1 + c);
+                    q = *reinterpret_cast<const float2*>(a2 + c);
+                }
+            }
+            v[u] = p.x - weight * q.x;
+            v[u + 1] = p.y - weight * q.y;
+            ss += v[u] * v[u] + v[u + 1] * v[u + 1];
+        } else {
+            v[u] = c < vdim ? Num<T>::to_f(a1[c]) - weight * Num<T>::to_f(a2[c]) : 0.f;
+            ss += v[u] * v[u];
+        }
+    }
+    const float inv = gain / sqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+    for (int u = 0; u < MD_MAX; ++u) {
+        const int c = PAIRS ? 64 * (u / 2) + 2 * lane + (u & 1) : 32 * u + lane;
+        if (c >= vdim || (PAIRS && (u & 1))) continue;
+        if constexpr (PAIRS) {
+            if constexpr (sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(o + c) = __floats2bfloat162_rn(v[u] * inv, v[u + 1] * inv);
+            else *reinterpret_cast<float2*>(o + c) = make_float2(v[u] * inv, v[u + 1] * inv);
+        } else {
+            o[c] = Num<T>::from_f(v[u] * inv);
+        }
+    }
+}
+
+QF_EXPORT int qf_map_difference(int is_bf16, const void* x, int pitch, float weight, float eps, float gain, void* out, int n_tokens, int heads,
+                                int vdim, cudaStream_t stream) {
+    const long long items = (long long)n_tokens * heads;
+    if (items <= 0) return 0;
+    if (vdim <= 0 || vdim > 32 * MD_MAX || pitch < vdim) return (int)cudaErrorInvalidValue;
+    const int warps = items >= 4096 ? 8 : 2;
+    const dim3 grid((unsigned)((items + warps - 1) / warps)), block(32 * warps);
+    const bool pairs = vdim % 2 == 0 && pitch % 2 == 0 && ((uintptr_t)x | (uintptr_t)out) % 8 == 0;
+#define QF_DIFF(T, P) return (int)launch_pdl(map_difference_kernel<T, P>, grid, block, 0, stream, (const T*)x, pitch, weight, eps, gain, (T*)out, items, vdim)
+    if (is_bf16) {
+        if (pairs) QF_DIFF(bf16, true);
+        QF_DIFF(bf16, false);
+    }
+    if (pairs) QF_DIFF(float, true);
+    QF_DIFF(float, false);
+#undef QF_DIFF
+}

@@ -147,7 +147,7 @@ outer_state_scan_kernel(const T* __restrict__ q, int q_stride, const T* __restri
                         const int* __restrict__ cu_q, const int* __restrict__ slots, float* __restrict__ state,
                         long long slot_stride, long long s_offset, long long n_offset, int n_heads, int n_groups, int dim,
                         int vdim, float q_scale, float* __restrict__ y, float* __restrict__ nq, const float* __restrict__ bonus,
-                        const float* __restrict__ decay_bias, int decay_kind, float inv_tau) {
+                        const float* __restrict__ decay_bias, int decay_kind, float inv_tau, int gate_stride) {
     grid_chain_entry();
     extern __shared__ __align__(16) float scan_smem[];
     constexpr int THREADS = 32 * WARPS, PARTS = 2 * WARPS, padded = PARTS * ROWS;   // padded >= dim
@@ -214,8 +214,8 @@ outer_state_scan_kernel(const T* __restrict__ q, int q_stride, const T* __restri
                 v_next[u] = c < vdim ? load_early(v + (size_t)(t0 + j) * v_stride + head * vdim + c) : 1.f;
         }
         if (MODE == 0 && threadIdx.x < n_here) {
-            gate_next[0] = load_early(decay + (size_t)(t0 + threadIdx.x) * n_heads + head);
-            gate_next[1] = load_early(take + (size_t)(t0 + threadIdx.x) * n_heads + head);
+            gate_next[0] = load_early(decay + (size_t)(t0 + threadIdx.x) * gate_stride + head);
+            gate_next[1] = take ? load_early(take + (size_t)(t0 + threadIdx.x) * gate_stride + head) : 1.f;
         }
     };
     auto stash = [&]() {
@@ -351,7 +351,7 @@ template <typename T, int WARPS, int ROWS, int MODE>
 static int launch_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* decay,
                        const float* take, const int* cu_q, const int* slots, int n_seqs, float* state, long long slot_stride,
                        long long s_offset, long long n_offset, int n_heads, int n_groups, int dim, int vdim, float q_scale,
-                       float* y, float* nq, const float* bonus, const float* decay_bias, int decay_kind, float inv_tau,
+                       float* y, float* nq, const float* bonus, const float* decay_bias, int decay_kind, float inv_tau, int gate_stride,
                        cudaStream_t stream) {
     const int columns = vdim + (n_offset >= 0 ? 1 : 0);
     constexpr int PARTS = 2 * WARPS, padded = PARTS * ROWS;
@@ -361,11 +361,11 @@ static int launch_scan(const void* q, int q_stride, const void* k, int k_stride,
     return (int)launch_pdl(outer_state_scan_kernel<T, WARPS, ROWS, MODE>, dim3((columns + SCAN_COLS - 1) / SCAN_COLS, n_heads, n_seqs),
                            dim3(32 * WARPS), smem, stream, (const T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, decay,
                            take, cu_q, slots, state, slot_stride, s_offset, n_offset, n_heads, n_groups, dim, vdim, q_scale, y, nq, bonus, decay_bias,
-                           decay_kind, inv_tau);
+                           decay_kind, inv_tau, gate_stride);
 }
 
 #define QF_SCAN_ARGS q, q_stride, k, k_stride, v, v_stride, decay, take, cu_q, slots, n_seqs, state, slot_stride, s_offset, \
-                     n_offset, n_heads, n_groups, dim, vdim, q_scale, y, nq, bonus, decay_bias, decay_kind, inv_tau, stream
+                     n_offset, n_heads, n_groups, dim, vdim, q_scale, y, nq, bonus, decay_bias, decay_kind, inv_tau, gate_stride, stream
 // 2 * WARPS half warps of ROWS rows each cover `dim` rows
 #define QF_SCAN_CASE(WARPS, ROWS) \
     if (dim <= 2 * WARPS * ROWS)  \
@@ -373,6 +373,7 @@ static int launch_scan(const void* q, int q_stride, const void* k, int k_stride,
 
 // q, k: [T][groups * dim] with row strides; v: [T][heads * vdim]; decay, take: float32 [T][heads]; y: float32 [T][heads * vdim];
 // nq: float32 [T][heads] or null (then n_offset < 0). State pieces: S [heads][dim][vdim] at s_offset, n [heads][dim] at n_offset.
+// take null: nothing scales what a token adds, and `decay` is float32 [heads], the same for every token.
 QF_EXPORT int qf_outer_state_scan(int is_bf16, const void* q, int q_stride, const void* k, int k_stride, const void* v,
                                   int v_stride, const float* decay, const float* take, const int* cu_q, const int* slots,
                                   int n_seqs, float* state, long long slot_stride, long long s_offset, long long n_offset,
@@ -383,7 +384,7 @@ QF_EXPORT int qf_outer_state_scan(int is_bf16, const void* q, int q_stride, cons
     constexpr int MODE = 0;
     const float* bonus = nullptr;
     const float* decay_bias = nullptr;
-    const int decay_kind = 0;
+    const int decay_kind = 0, gate_stride = take ? n_heads : 0;
     const float inv_tau = 1.f;
     QF_SCAN_CASE(4, 4)
     QF_SCAN_CASE(8, 4)
@@ -400,6 +401,7 @@ static int scan_rows(int is_bf16, const void* q, int q_stride, const void* k, in
     const float* take = nullptr;
     float* nq = nullptr;
     const long long n_offset = -1;
+    const int gate_stride = n_heads;
     QF_SCAN_CASE(4, 4)
     QF_SCAN_CASE(8, 4)
     QF_SCAN_CASE(16, 4)

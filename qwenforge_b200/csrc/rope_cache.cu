@@ -400,6 +400,131 @@ QF_EXPORT int qf_rope_norm_cache_write(int is_bf16, const void* qkv, const void*
                                        eps, n_tokens, err, 0, 0, nullptr, nullptr, stream);
 }
 
+// Heads of several maps (a differential attention: every query head has `maps` queries and every key/value head `maps` keys, one
+// after the other in the head's row, over ONE value). The row of a token is [n_heads][maps][dim] queries, [kv_heads][maps][dim]
+// keys, [kv_heads][vdim] values. Each map is turned by itself: its first rot_dim components, component j with j + rot_dim / 2,
+// cosine and sine both times `amplitude`. In the cache a key/value head is one head of site.head_dim components: the keys of
+// its maps side by side, then zeros; and its value, then zeros. A query is written as a head of that size of its own with its
+// components where its map's keys lie and zeros elsewhere, so that its product with the cached row is the product with its own
+// map's key alone, and n_heads * maps plain query heads over kv_heads cached heads are the whole attention.
+// V components at a time (8: bfloat16 rows that 16-byte accesses can address, sizes and half the rotated part in whole eights; 1).
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+rope_maps_cache_kernel(const T* __restrict__ qkv, int qkv_stride, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+                       const int* __restrict__ slots, const float* __restrict__ inv_freq, int rot_dim, float amplitude, int n_heads,
+                       int maps, int dim, int vdim, T* __restrict__ q_out, KvSite<T> site, int write_cache, int n_tokens, int per_block,
+                       int* err) {
+    grid_chain_entry();
+    __shared__ float sin_s[RC_TOKENS][128], cos_s[RC_TOKENS][128];   // rot_dim <= 256
+    __shared__ int pos_s[RC_TOKENS];
+    __shared__ long long page_s[RC_TOKENS];   // element offset of the token's place in head 0 of its page, -1: nothing to write
+    const int D = site.head_dim, KVH = site.kv_heads, half = rot_dim / 2;
+    const int t0 = blockIdx.x * per_block, n_here = min(per_block, n_tokens - t0);
+    if (threadIdx.x < n_here) {
+        const int t = t0 + threadIdx.x, pos = tok_pos[t], slot = slots[tok_seq[t]];
+        pos_s[threadIdx.x] = pos;
+        long long offset = -1;
+        if (write_cache && slot >= 0) {
+            const int page = site.table[(long long)slot * site.table_stride + pos / QF_PAGE];
+            if (page < 0) atomicOr(err, QF_ERR_NO_PAGE);
+            else offset = (long long)page * site.page_elems + (long long)(pos % QF_PAGE) * D;
+        }
+        page_s[threadIdx.x] = offset;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < n_here * half; i += blockDim.x) {
+        const int k = i / half, j = i % half;
+        float s, c;
+        sincosf((float)pos_s[k] * inv_freq[j], &s, &c);
+        sin_s[k][j] = s * amplitude;
+        cos_s[k][j] = c * amplitude;
+    }
+    __syncthreads();
+    auto load = [&](const T* p, float (&v)[V]) {
+        if constexpr (V == 8) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(p);
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(h[e]);
+                v[2 * e] = f.x;
+                v[2 * e + 1] = f.y;
+            }
+        } else {
+            v[0] = Num<T>::to_f(p[0]);
+        }
+    };
+    auto store = [&](T* p, const float (&v)[V]) {
+        if constexpr (V == 8)
+            *reinterpret_cast<uint4*>(p) = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
+        else p[0] = Num<T>::from_f(v[0]);
+    };
+    // components c .. c + V - 1 of the map whose row starts at `src`, turned
+    auto turned = [&](const T* src, int k, int c, float (&v)[V]) {
+        load(src + c, v);
+        if (c >= rot_dim) return;
+        const bool first = c < half;
+        const int j = first ? c : c - half;
+        float other[V];
+        load(src + (first ? c + half : c - half), other);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float s = sin_s[k][j + e], cs = cos_s[k][j + e];
+            v[e] = first ? v[e] * cs - other[e] * s : v[e] * cs + other[e] * s;
+        }
+    };
+    const int groups = D / V, q_heads = n_heads * maps, per_token = (q_heads + 2 * KVH) * groups;
+    const int k_first = q_heads * dim, v_first = k_first + KVH * maps * dim;
+    for (int i = threadIdx.x; i < n_here * per_token; i += blockDim.x) {
+        const int k = i / per_token, item = i % per_token, t = t0 + k;
+        const int head = item / groups, c = (item % groups) * V;
+        const T* row = qkv + (size_t)t * qkv_stride;
+        float v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = 0.f;
+        if (head < q_heads) {
+            const int own = c - (head % maps) * dim;   // the component of the query's own map
+            if (own >= 0 && own < dim) turned(row + head * dim, k, own, v);
+            store(q_out + ((size_t)t * q_heads + head) * D + c, v);
+            continue;
+        }
+        const long long place = page_s[k];
+        if (place < 0) continue;
+        const int g = head - q_heads;
+        if (g < KVH) {
+            if (c < maps * dim) turned(row + k_first + g * maps * dim + c / dim * dim, k, c % dim, v);
+        } else if (c < vdim) {
+            load(row + v_first + (g - KVH) * vdim + c, v);
+        }
+        store(site.base + place + (long long)g * QF_PAGE * D + c, v);
+    }
+}
+
+// qkv: [n_tokens][qkv_stride] as above; q_out: [n_tokens][n_heads * maps * head_dim]; head_dim >= max(maps * dim, vdim).
+QF_EXPORT int qf_rope_maps_cache_write(int is_bf16, const void* qkv, int qkv_stride, const int* tok_seq, const int* tok_pos,
+                                       const int* slots, const float* inv_freq, int rot_dim, float amplitude, int n_heads, int maps,
+                                       int dim, int vdim, void* q_out, void* base, const int* table, long long page_elems,
+                                       int table_stride, int kv_heads, int head_dim, int write_cache, int n_tokens, int* err,
+                                       cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (!inv_freq) rot_dim = 0;
+    if (rot_dim < 0 || rot_dim > dim || (rot_dim & 1) || rot_dim > 256 || maps < 1 || maps * dim > head_dim || vdim > head_dim || kv_heads <= 0)
+        return (int)cudaErrorInvalidValue;
+    // (a token's arithmetic is the same whatever shares its block; few tokens get a block each)
+    const int per_block = n_tokens >= 64 * RC_TOKENS ? RC_TOKENS : 1;
+    const dim3 grid((n_tokens + per_block - 1) / per_block), block(256);
+    const bool vec = is_bf16 && head_dim % 8 == 0 && dim % 8 == 0 && vdim % 8 == 0 && rot_dim % 16 == 0 && qkv_stride % 8 == 0 &&
+                     page_elems % 8 == 0 && ((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)base) % 16 == 0;
+#define QF_MAPS(T, V)                                                                                                              \
+    return (int)launch_pdl(rope_maps_cache_kernel<T, V>, grid, block, 0, stream, (const T*)qkv, qkv_stride, tok_seq, tok_pos, slots, \
+                           inv_freq, rot_dim, amplitude, n_heads, maps, dim, vdim, (T*)q_out,                                      \
+                           KvSite<T>{(T*)base, table, page_elems, table_stride, kv_heads, head_dim}, write_cache, n_tokens, per_block, err)
+    if (vec) QF_MAPS(bf16, 8);
+    if (is_bf16) QF_MAPS(bf16, 1);
+    QF_MAPS(float, 1);
+#undef QF_MAPS
+}
+
 // Rows of whole blocks beside a cache: once the last position of a block of `pool` positions has been written, the block's
 // row in a second cache (`rows`: one row per block, addressed like positions) becomes the mean of the block's keys and the
 // mean of its values AS THE CACHE HOLDS THEM (float32 sums, divided by `pool`, rounded to the cache's type). A block of
@@ -476,19 +601,19 @@ QF_EXPORT int qf_pool_cache_write(int is_bf16, const int* cu_q, const int* tok_p
 }
 
 // The rotation angles of a step, once for all its layers: table[t][j] = (cos, sin) of tok_pos[t] * inv_freq[j], float32,
-// the same expression as in the kernels above.
+// the same expression as in the kernels above; both times `amplitude`.
 __global__ void rope_table_kernel(const int* __restrict__ tok_pos, const float* __restrict__ inv_freq, int n_tokens, int half,
-                                  float2* __restrict__ table) {
+                                  float amplitude, float2* __restrict__ table) {
     grid_chain_entry();
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n_tokens * half) return;
     float sn, c;
     sincosf((float)tok_pos[i / half] * inv_freq[i % half], &sn, &c);
-    table[i] = make_float2(c, sn);
+    table[i] = make_float2(c * amplitude, sn * amplitude);
 }
 
-QF_EXPORT int qf_rope_table(const int* tok_pos, const float* inv_freq, int n_tokens, int half, void* table, cudaStream_t stream) {
+QF_EXPORT int qf_rope_table(const int* tok_pos, const float* inv_freq, int n_tokens, int half, float amplitude, void* table, cudaStream_t stream) {
     if (n_tokens <= 0 || half <= 0) return 0;
     const long long total = (long long)n_tokens * half;
-    return (int)launch_pdl(rope_table_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, tok_pos, inv_freq, n_tokens, half, (float2*)table);
+    return (int)launch_pdl(rope_table_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, stream, tok_pos, inv_freq, n_tokens, half, amplitude, (float2*)table);
 }

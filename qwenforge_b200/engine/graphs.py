@@ -84,6 +84,7 @@ class DecodeGraph:
         # and a step starts at its first layer.
         lookup = getattr(model.embedding, "lookup_table", None)
         self.table = lookup() if lookup is not None else None
+        self.table_scale = model.embedding.lookup_scale() if self.table is not None else 1.0
         if self.table is not None:
             self.ctx.embedded = torch.zeros((rows, self.table.shape[1]), dtype=torch.float32, device=device)
             self.ticket = torch.zeros(1, **i32)
@@ -98,7 +99,7 @@ class DecodeGraph:
         if self.table is not None:
             ops.decode_advance_embed(self.sampled, self.token_ids, self.tok_pos, self.slots, self.steps, self.budgets,
                                      self.stop_ids, MAX_STOP_IDS, self.out_tokens, self.cursor, self.table,
-                                     self.ctx.embedded, self.ticket, self.model.err)
+                                     self.ctx.embedded, self.ticket, self.model.err, self.table_scale)
         else:
             ops.decode_advance(self.sampled, self.token_ids, self.tok_pos, self.slots, self.steps, self.budgets,
                                self.stop_ids, MAX_STOP_IDS, self.out_tokens, self.cursor)
@@ -118,7 +119,7 @@ class DecodeGraph:
         stops = list(stop_ids)[:MAX_STOP_IDS]
         self.stop_ids.copy_(torch.tensor(stops + [-1] * (MAX_STOP_IDS - len(stops)), dtype=torch.int32))
         if self.table is not None:   # the first step's rows; every later step's come from the step before it
-            ops.embed_gather(self.token_ids, self.table, self.ctx.embedded, self.model.err)
+            ops.embed_gather(self.token_ids, self.table, self.ctx.embedded, self.model.err, self.table_scale)
 
     def capture(self) -> None:
         """Two eager steps on a side stream (they size every scratch buffer), then the capture. The rows are all

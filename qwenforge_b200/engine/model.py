@@ -156,7 +156,7 @@ class Model:
         if ctx.want_rows is None:
             return None
         if isinstance(delta, Pending):
-            normed = delta.normed_rows(ctx.want_rows, self.final_norm, ctx.err)
+            normed = delta.normed_rows(hidden, ctx.want_rows, self.final_norm, ctx.err)
             if normed is not None:
                 return self.head.forward(normed)
             delta.add_to(hidden)

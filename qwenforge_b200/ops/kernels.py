@@ -115,8 +115,8 @@ class KvSiteArgs:
         self.head_dim = head_dim
 
 
-def embed_gather(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor) -> None:
-    """out[t] = float32(table[ids[t]]); ids int32 [T], table [V, W], out float32 [T, W]."""
+def embed_gather(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] = float32(table[ids[t]]) * scale; ids int32 [T], table [V, W], out float32 [T, W]."""
     _dev("ids", ids, torch.int32)
     _dev("table", table)
     _dev("out", out, torch.float32)
@@ -124,7 +124,7 @@ def embed_gather(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err:
     if out.shape != (n, width):
         raise KernelError(f"embed_gather: out is {tuple(out.shape)}, expected {(n, width)}")
     _check(library("embed").qf_embed_gather(_I(_is_bf16(table.dtype)), _ptr(ids), _ptr(table), _ptr(out), _I(n),
-                                            _I(vocab), _I(width), _ptr(err), _stream()), "embed_gather")
+                                            _I(vocab), _I(width), _F(scale), _ptr(err), _stream()), "embed_gather")
 
 
 def gather_rows(hidden: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor, out: torch.Tensor,
@@ -333,6 +333,47 @@ def _distance_bias(what: str, pair, n_heads: int, pool: int = 0):
 
 
 FAST_ATTENTION_HEAD_DIMS = (32, 64, 96, 128)
+
+
+def rope_maps_cache_write(qkv: torch.Tensor, tok_seq: torch.Tensor, tok_pos: torch.Tensor, slots: torch.Tensor,
+                          inv_freq: Optional[torch.Tensor], rot_dim: int, amplitude: float, n_heads: int, maps: int, dim: int, vdim: int,
+                          q_out: torch.Tensor, site: KvSiteArgs, write_cache: bool, err: torch.Tensor) -> None:
+    """`rope_cache_write` for heads of several maps (a differential attention). qkv [T, n_heads * maps * dim queries | kv_heads * maps *
+    dim keys | kv_heads * vdim values] (perhaps the first columns of wider rows); each map is turned by itself (split halves of its first
+    rot_dim components, cosine and sine times `amplitude`). A cached head of site.head_dim >= max(maps * dim, vdim) components holds the
+    keys of its maps side by side and its value, filled up with zeros; q_out [T, n_heads * maps * head_dim] holds one query head per
+    map, its components where its map's keys lie, zeros elsewhere."""
+    _rows("qkv", qkv)
+    _dev("q_out", q_out, qkv.dtype)
+    _dev("cache", site.storage, qkv.dtype)
+    for name, t in (("tok_seq", tok_seq), ("tok_pos", tok_pos), ("slots", slots)):
+        _dev(name, t, torch.int32)
+    n, d, kvh = qkv.shape[0], site.head_dim, site.kv_heads
+    if qkv.shape[1] < (n_heads + kvh) * maps * dim + kvh * vdim or q_out.shape != (n, n_heads * maps * d) or maps * dim > d or vdim > d:
+        raise KernelError("rope_maps_cache_write: qkv/q_out widths do not match the heads, their maps and the cached head")
+    if inv_freq is not None:
+        _dev("inv_freq", inv_freq, torch.float32)
+        if inv_freq.numel() * 2 != rot_dim or rot_dim > dim:
+            raise KernelError("rope_maps_cache_write: inv_freq must hold rot_dim / 2 frequencies, rot_dim at most dim")
+    _check(library("rope_cache").qf_rope_maps_cache_write(
+        _I(_is_bf16(qkv.dtype)), _ptr(qkv), _I(qkv.stride(0)), _ptr(tok_seq), _ptr(tok_pos), _ptr(slots), _ptr(inv_freq), _I(rot_dim),
+        _F(amplitude), _I(n_heads), _I(maps), _I(dim), _I(vdim), _ptr(q_out), _ptr(site.storage), _ptr(site.table), _LL(site.page_elems),
+        _I(site.table_stride), _I(kvh), _I(d), _I(1 if write_cache else 0), _I(n), _ptr(err), _stream()), "rope_maps_cache_write")
+
+
+MAP_DIFFERENCE_MAX_VDIM = 256
+
+
+def map_difference(x: torch.Tensor, pitch: int, weight: float, eps: float, gain: float, out: torch.Tensor, heads: int, vdim: int) -> None:
+    """The two maps of a differential attention brought together: x [T, heads * 2 * pitch] (the maps' attended values in the first vdim
+    components of each), out [T, heads * vdim] = gain * o / sqrt(mean(o^2) + eps) per head with o = a1 - weight * a2, float32 inside."""
+    _dev("x", x)
+    _dev("out", out, x.dtype)
+    n = x.shape[0]
+    if x.shape != (n, heads * 2 * pitch) or out.shape != (n, heads * vdim) or not 0 < vdim <= min(pitch, MAP_DIFFERENCE_MAX_VDIM):
+        raise KernelError(f"map_difference: x must be [T, heads * 2 * pitch], out [T, heads * vdim], vdim at most {MAP_DIFFERENCE_MAX_VDIM}")
+    _check(library("norm").qf_map_difference(_I(_is_bf16(x.dtype)), _ptr(x), _I(pitch), _F(weight), _F(eps), _F(gain), _ptr(out), _I(n),
+                                             _I(heads), _I(vdim), _stream()), "map_difference")
 
 
 def attention_prefill(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok_pos: torch.Tensor,
@@ -632,8 +673,8 @@ def decode_advance(sampled: torch.Tensor, token_ids: torch.Tensor, tok_pos: torc
 def decode_advance_embed(sampled: torch.Tensor, token_ids: torch.Tensor, tok_pos: torch.Tensor, slots: torch.Tensor,
                          steps: torch.Tensor, budgets: torch.Tensor, stop_ids: torch.Tensor, n_stop: int,
                          out_tokens: torch.Tensor, cursor: torch.Tensor, table: torch.Tensor, hidden: torch.Tensor,
-                         ticket: torch.Tensor, err: torch.Tensor) -> None:
-    """`decode_advance`, and the next step's embedding with it: hidden[r] = float32(table[the row's next input token]).
+                         ticket: torch.Tensor, err: torch.Tensor, scale: float = 1.0) -> None:
+    """`decode_advance`, and the next step's embedding with it: hidden[r] = float32(table[the row's next input token]) * scale.
     `ticket` is one int32 that is zero before the first call."""
     for name, t in (("sampled", sampled), ("token_ids", token_ids), ("tok_pos", tok_pos), ("slots", slots),
                     ("steps", steps), ("budgets", budgets), ("stop_ids", stop_ids), ("out_tokens", out_tokens),
@@ -649,7 +690,7 @@ def decode_advance_embed(sampled: torch.Tensor, token_ids: torch.Tensor, tok_pos
     _check(library("decode_state").qf_decode_advance_embed(
         _ptr(sampled), _ptr(token_ids), _ptr(tok_pos), _ptr(slots), _ptr(steps), _ptr(budgets), _ptr(stop_ids),
         _I(n_stop), _ptr(out_tokens), _ptr(cursor), _I(out_tokens.shape[0]), _I(n), _I(_is_bf16(table.dtype)),
-        _ptr(table), _I(table.shape[0]), _I(table.shape[1]), _ptr(hidden), _ptr(ticket), _ptr(err), _stream()),
+        _ptr(table), _I(table.shape[0]), _I(table.shape[1]), _F(scale), _ptr(hidden), _ptr(ticket), _ptr(err), _stream()),
         "decode_advance_embed")
 
 
@@ -1098,13 +1139,14 @@ class _TcQkvArgs(ctypes.Structure):
                 ("write_cache", _I)]
 
 
-def rope_table(tok_pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
-    """The rotation angles of a step's tokens, [tokens, rot_dim / 2, 2] float32 (cos, sin): made once, read by every layer."""
+def rope_table(tok_pos: torch.Tensor, inv_freq: torch.Tensor, amplitude: float = 1.0) -> torch.Tensor:
+    """The rotation angles of a step's tokens, [tokens, rot_dim / 2, 2] float32 (cos, sin), both times `amplitude`: made once, read
+    by every layer."""
     _dev("tok_pos", tok_pos, torch.int32)
     _dev("inv_freq", inv_freq, torch.float32)
     table = torch.empty((tok_pos.numel(), inv_freq.numel(), 2), dtype=torch.float32, device=tok_pos.device)
-    _check(library("rope_cache").qf_rope_table(_ptr(tok_pos), _ptr(inv_freq), _I(tok_pos.numel()), _I(inv_freq.numel()), _ptr(table),
-                                               _stream()), "rope_table")
+    _check(library("rope_cache").qf_rope_table(_ptr(tok_pos), _ptr(inv_freq), _I(tok_pos.numel()), _I(inv_freq.numel()),
+                                               _F(amplitude), _ptr(table), _stream()), "rope_table")
     return table
 
 
@@ -1386,21 +1428,20 @@ def moe_tile_rows(n_tokens: int, n_experts: int, top: int, weight: torch.Tensor)
 
 def moe_plan(logits: Optional[torch.Tensor], top: int, softmax_scores: bool = False, renormalize: bool = False,
              tile_rows: int = GROUP_TILE_ROWS, x: Optional[torch.Tensor] = None, router: Optional[torch.Tensor] = None,
-             bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, groups=None) -> MoePlan:
+             bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, groups=None,
+             group_best: int = 2) -> MoePlan:
     """Route: logits float32 [T, E] -> the `top` experts with the largest scores per token (sigmoid of the logit, or the
     softmax over the experts) and the sorted rows (see `MoePlan`), cut into tiles of `tile_rows`. Everything stays on the
     device. With `logits` None, the kernel makes the logits itself from `x` [T, W] and `router` [E, W] (float32 sums; for
     steps of few tokens, T * E <= MOE_FUSED_ROUTER_MAX). `bias` (float32 [E]) is added to the logits before the choice.
-    `correction` (float32 [E]) and `groups` = (count, keep), with sigmoid scores: the choice goes by score + correction, and
-    only among the experts of the `keep` best of `count` equal groups of neighbouring experts, a group's score being the sum
-    of its two largest choice scores; the weights are the scores without the correction."""
+    `correction` (float32 [E]) and `groups` = (count, keep): the choice goes by score + correction, and only among the experts of
+    the `keep` best of `count` equal groups of neighbouring experts, a group's score being the sum of its `group_best` (1 or 2)
+    largest choice scores; the weights are the scores without the correction."""
     if bias is not None:
         _dev("bias", bias, torch.float32)
     group_count, group_keep = (0, 0)
     if correction is not None or groups is not None:
         group_count, group_keep = (int(groups[0]), int(groups[1])) if groups is not None else (1, 1)
-        if softmax_scores:
-            raise KernelError("moe_plan: a correction or groups go with sigmoid scores")
         if correction is not None:
             _dev("correction", correction, torch.float32)
     if logits is not None:
@@ -1417,6 +1458,8 @@ def moe_plan(logits: Optional[torch.Tensor], top: int, softmax_scores: bool = Fa
         raise KernelError("moe_plan: bias must hold one float32 per expert")
     if correction is not None and correction.numel() != n_experts:
         raise KernelError("moe_plan: correction must hold one float32 per expert")
+    if group_best not in (1, 2):
+        raise KernelError(f"moe_plan: a group's score is its largest or the sum of its two largest scores, not of {group_best}")
     if group_count and (not 1 <= group_keep <= group_count <= 64 or n_experts % group_count or group_keep * (n_experts // group_count) < top):
         raise KernelError(f"moe_plan: {group_keep} of {group_count} groups over {n_experts} experts cannot yield {top} choices "
                           "(up to 64 equal groups)")
@@ -1427,7 +1470,7 @@ def moe_plan(logits: Optional[torch.Tensor], top: int, softmax_scores: bool = Fa
             _ptr(logits), _I(n_tokens), _I(n_experts), _I(top), _I(int(softmax_scores)), _I(int(renormalize)),
             _ptr(plan.pair_expert), _ptr(plan.pair_weight), _ptr(plan.sorted_token), _ptr(plan.sorted_weight), _ptr(plan.dest),
             _ptr(plan.offsets), _ptr(plan.tile_group), _ptr(plan.tile_row0), _ptr(plan.n_tiles), _I(plan.max_tiles),
-            _I(tile_rows), _ptr(expert_rows), _ptr(bias), _ptr(correction), _I(group_count), _I(group_keep), _stream())
+            _I(tile_rows), _ptr(expert_rows), _ptr(bias), _ptr(correction), _I(group_count), _I(group_keep), _I(group_best), _stream())
         if code == 1:
             raise KernelError(f"moe_plan: {top} of {n_experts} experts is not supported (top <= 16)")
         _check(code, "moe_plan")
@@ -1438,7 +1481,7 @@ def moe_plan(logits: Optional[torch.Tensor], top: int, softmax_scores: bool = Fa
                                       _ptr(plan.tile_group), _ptr(plan.tile_row0), _ptr(plan.n_tiles), _I(plan.max_tiles),
                                       _I(tile_rows), _ptr(x if logits is None else None), _ptr(router if logits is None else None),
                                       _I(width), _I(_is_bf16(x.dtype) if logits is None else 0), _ptr(bias), _ptr(correction),
-                                      _I(group_count), _I(group_keep), _stream())
+                                      _I(group_count), _I(group_keep), _I(group_best), _stream())
     if code == 1:
         raise KernelError(f"moe_plan: {top} of {n_experts} experts is not supported (top <= 16, experts <= 8192)")
     _check(code, "moe_plan")
@@ -1682,11 +1725,12 @@ def decay_gates(dt_pre: torch.Tensor, dt_bias: torch.Tensor, rate_log: torch.Ten
 OUTER_STATE_MAX_DIM = 256
 
 
-def outer_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, take: torch.Tensor,
+def outer_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, take: Optional[torch.Tensor],
                      cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_offset: int,
                      n_heads: int, n_groups: int, dim: int, vdim: int, q_scale: float, y: torch.Tensor,
                      nq: Optional[torch.Tensor]) -> None:
-    """The recurrence of a matrix state per head, token after token of every sequence, all float32 inside:
+    """The recurrence of a matrix state per head, token after token of every sequence, all float32 inside (`take` None: 1, and
+    `decay` float32 [heads], the same for every token):
         S <- decay_t S + take_t k_t v_t^T   (S: dim x vdim, kept in `state` at s_offset as [heads, dim, vdim]);  y_t = S^T (q_scale q_t)
     and, with `nq`, a vector n <- decay_t n + take_t k_t beside it (at n_offset, [heads, dim]) and nq_t = n . (q_scale q_t).
     q, k: [T, groups * dim] (head h reads group h // (heads / groups)), v: [T, heads * vdim], in the activation dtype, rows
@@ -1700,9 +1744,11 @@ def outer_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: t
     if dim > OUTER_STATE_MAX_DIM:
         raise KernelError(f"outer_state_scan: a state of {dim} rows per head exceeds the kernel's {OUTER_STATE_MAX_DIM}")
     for name, t in (("decay", decay), ("take", take)):
+        if t is None and name == "take":
+            continue
         _dev(name, t, torch.float32)
-        if t.shape != (n, n_heads):
-            raise KernelError(f"outer_state_scan: {name} must be float32 [T, heads]")
+        if t.shape != ((n, n_heads) if take is not None else (n_heads,)):
+            raise KernelError(f"outer_state_scan: {name} must be float32 [T, heads] (decay alone: [heads])")
     _dev("y", y, torch.float32)
     if y.shape != (n, n_heads * vdim):
         raise KernelError("outer_state_scan: y must be float32 [T, heads * vdim]")
@@ -2185,3 +2231,153 @@ def rows_prepare(x: torch.Tensor, runs, eps: float, mix=None) -> None:
     _check(library("norm").qf_rows_prepare(_I(_is_bf16(x.dtype)), _ptr(x), _I(x.stride(0)), _I(x.shape[0]), _I(n), col0, width, count,
                                            biases, weights, _I(mix_run), _ptr(other), _I(ldo), _I(size), _I(x_head), _I(other_head),
                                            _F(lam), _F(eps), _stream()), "rows_prepare")
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Two norms of one stream (csrc/norm.cu)
+PAIR_NORM_ROW_SUM_MAX = 16
+
+
+def pair_rms_norm(hidden: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torch.Tensor], weight1: Optional[torch.Tensor] = None,
+                  eps1: float = 0.0, out1: Optional[torch.Tensor] = None, weight2: Optional[torch.Tensor] = None, eps2: float = 0.0,
+                  out2: Optional[torch.Tensor] = None, b_rows: Optional[tuple] = None, rows: Optional[torch.Tensor] = None,
+                  err: Optional[torch.Tensor] = None) -> None:
+    """hidden += (a + b) (each if given), then two RMS norms of the same stream in one pass: out1 = rms(hidden) * weight1, out2 =
+    rms(hidden) * weight2 (either may be left out). hidden float32 [R, W]; a, b, weights and outs share the activation dtype.
+    `b_rows` = (dest int32 [R * top], top, row_weight float32 or None): b holds expert rows, and row t's share is the sum over k of
+    b[dest[t * top + k]] (times its row_weight), in the order of k. `rows` (int32): only those rows' norms, into outs of as many rows;
+    hidden is then left as it is."""
+    _dev("hidden", hidden, torch.float32)
+    n_in, width = hidden.shape
+    given = [t for t in (a, b, weight1, weight2) if t is not None]
+    if not given:
+        return
+    dtype = given[0].dtype
+    if a is not None:
+        _dev("a", a, dtype)
+        if a.shape != hidden.shape:
+            raise KernelError("pair_rms_norm: a and hidden differ in shape")
+    dest, top, row_weight = b_rows if b_rows is not None else (None, 1, None)
+    if b is not None:
+        _dev("b", b, dtype)
+        if dest is None and b.shape != hidden.shape:
+            raise KernelError("pair_rms_norm: b and hidden differ in shape")
+        if dest is not None:
+            _dev("dest", dest, torch.int32)
+            if dest.numel() != n_in * top or b.dim() != 2 or b.shape[1] != width:
+                raise KernelError("pair_rms_norm: dest must hold `top` rows of b per row of hidden")
+            if row_weight is not None:
+                _dev("row_weight", row_weight, torch.float32)
+    elif dest is not None:
+        raise KernelError("pair_rms_norm: rows to sum, and no b that holds them")
+    n_out = n_in
+    if rows is not None:
+        _dev("rows", rows, torch.int32)
+        n_out = rows.numel()
+    for name, w, out in (("1", weight1, out1), ("2", weight2, out2)):
+        if (w is None) != (out is None):
+            raise KernelError(f"pair_rms_norm: weight{name} goes with out{name}")
+        if w is not None:
+            _dev("weight" + name, w, dtype)
+            _dev("out" + name, out, dtype)
+            if w.shape != (width,) or out.shape != (n_out, width):
+                raise KernelError(f"pair_rms_norm: weight{name} must be [width], out{name} [rows, width]")
+    _check(library("norm").qf_pair_rms_norm(
+        _I(_is_bf16(dtype)), _ptr(hidden), _ptr(a), _ptr(b), _ptr(dest), _I(top), _ptr(row_weight), _ptr(weight1), _F(eps1), _ptr(out1),
+        _ptr(weight2), _F(eps2), _ptr(out2), _ptr(rows), _I(n_out), _I(n_in), _I(width),
+        _ptr(err if err is not None else _err_word_for(hidden.device)), _stream()), "pair_rms_norm")
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Retention (csrc/retention.cu)
+RETENTION_CHUNK = 64   # tokens of a chunk (RT_CHUNK): the decays' powers are given from 0 to this
+
+
+def _retention_args(what, q, k, v, gate, state, s_offset, n_heads, dim, vdim):
+    for name, t in (("q", q), ("k", k), ("v", v), ("gate", gate)):
+        if t is not None:
+            _rows(name, t, q.dtype)
+    _is_bf16(q.dtype)
+    n = q.shape[0]
+    if q.shape != (n, n_heads * dim) or k.shape != q.shape or v.shape != (n, n_heads * vdim) or (gate is not None and gate.shape != v.shape):
+        raise KernelError(f"{what}: q, k must be [T, heads * dim], v and the gate [T, heads * vdim]")
+    if state is not None:
+        _state(state, (s_offset, n_heads * dim * vdim))
+    return n
+
+
+def retention_chunks_take(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, state: torch.Tensor, s_offset: int, dim: int,
+                          vdim: int, rot_dim: int) -> bool:
+    """Whether `retention_chunks` takes these operands: bfloat16, sizes in whole eights up to 128, rows and states that 16-byte
+    accesses can address."""
+    return (q.is_cuda and q.dtype == torch.bfloat16 and bool(library("retention").qf_retention_chunks_take(_I(dim), _I(vdim), _I(rot_dim)))
+            and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v)) and gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0
+            and state.stride(0) % 4 == 0 and s_offset % 4 == 0 and state.data_ptr() % 16 == 0)
+
+
+def retention_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, angles: Optional[torch.Tensor], rot_dim: int,
+                     powers: torch.Tensor, k_scale: float, eps: float, cu_q: torch.Tensor, slots: torch.Tensor, max_q_len: int,
+                     state: torch.Tensor, s_offset: int, n_heads: int, dim: int, vdim: int, out: torch.Tensor) -> None:
+    """Retention over the tokens of a step, chunks of `RETENTION_CHUNK` tokens on the tensor cores (float32 products to rounding):
+        q, k turned (split halves of the first rot_dim components by `angles`, float32 [T, rot_dim / 2, 2] from `rope_table`), k * k_scale;
+        S <- decay_h S + k_t v_t^T;  o_t = S^T q_t;  out_t = o_t / sqrt(mean(o_t^2) + eps) * silu(gate_t)   per head.
+    q, k [T, heads * dim], v, gate [T, heads * vdim] (rows may be strided), out [T, heads * vdim]; powers float32 [heads,
+    RETENTION_CHUNK + 1]: every head's decay to the powers 0, 1, ...; S in `state` at s_offset as [heads, dim, vdim]. `max_q_len`: the
+    most tokens any sequence brings. bfloat16 only (`retention_chunks_take`)."""
+    n = _retention_args("retention_chunks", q, k, v, gate, state, s_offset, n_heads, dim, vdim)
+    _dev("powers", powers, torch.float32)
+    _dev("out", out, q.dtype)
+    if powers.shape != (n_heads, RETENTION_CHUNK + 1) or out.shape != (n, n_heads * vdim):
+        raise KernelError("retention_chunks: powers must be [heads, chunk + 1], out [T, heads * vdim]")
+    if rot_dim:
+        _dev("angles", angles, torch.float32)
+        if angles.shape != (n, rot_dim // 2, 2):
+            raise KernelError("retention_chunks: angles must be [T, rot_dim / 2, 2]")
+    if not retention_chunks_take(q, k, v, gate, state, s_offset, dim, vdim, rot_dim):
+        raise KernelError("retention_chunks: bfloat16 operands with sizes and strides in whole eights, up to 128 (retention_chunks_take)")
+    n_seqs = cu_q.numel() - 1
+    parts = torch.empty((n // RETENTION_CHUNK + n_seqs) * n_heads * dim * vdim, dtype=torch.float32, device=q.device)
+    _check(library("retention").qf_retention_chunks(
+        _ptr(q), _I(q.stride(0)), _ptr(k), _I(k.stride(0)), _ptr(v), _I(v.stride(0)), _ptr(gate), _I(gate.stride(0)),
+        _ptr(angles if rot_dim else q), _I(rot_dim), _ptr(powers), _F(k_scale), _F(eps), _ptr(cu_q), _ptr(slots), _I(n_seqs), _I(max_q_len),
+        _ptr(state), _LL(state.stride(0)), _LL(s_offset), _I(n_heads), _I(dim), _I(vdim), _ptr(parts), _ptr(out), _stream()), "retention_chunks")
+
+
+def retention_token(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, tok_pos: torch.Tensor,
+                    inv_freq: Optional[torch.Tensor], rot_dim: int, amplitude: float, decay: torch.Tensor, k_scale: float, eps: float,
+                    cu_q: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, s_offset: int, n_heads: int, dim: int, vdim: int,
+                    out: torch.Tensor) -> None:
+    """`retention_chunks` for a step of ONE token per sequence, both precisions and any sizes, the rotation formed inside from the
+    positions and `inv_freq` (cosine and sine times `amplitude`); decay float32 [heads]."""
+    n = _retention_args("retention_token", q, k, v, gate, state, s_offset, n_heads, dim, vdim)
+    _dev("decay", decay, torch.float32)
+    _dev("tok_pos", tok_pos, torch.int32)
+    _dev("out", out, q.dtype)
+    if n != cu_q.numel() - 1 or decay.numel() != n_heads or out.shape != (n, n_heads * vdim):
+        raise KernelError("retention_token: one token per sequence, decay [heads], out [T, heads * vdim]")
+    if rot_dim:
+        _dev("inv_freq", inv_freq, torch.float32)
+        if inv_freq.numel() * 2 != rot_dim:
+            raise KernelError("retention_token: inv_freq must hold rot_dim / 2 frequencies")
+    _check(library("retention").qf_retention_token(
+        _I(_is_bf16(q.dtype)), _ptr(q), _I(q.stride(0)), _ptr(k), _I(k.stride(0)), _ptr(v), _I(v.stride(0)), _ptr(gate), _I(gate.stride(0)),
+        _ptr(tok_pos), _ptr(inv_freq if rot_dim else None), _I(rot_dim), _F(amplitude), _ptr(decay), _F(k_scale), _F(eps), _ptr(cu_q),
+        _ptr(slots), _I(n), _ptr(state), _LL(state.stride(0)), _LL(s_offset), _I(n_heads), _I(dim), _I(vdim), _ptr(out), _stream()),
+        "retention_token")
+
+
+def retention_rows(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, angles: Optional[torch.Tensor], rot_dim: int, k_scale: float,
+                   n_heads: int, dim: int, vdim: int, rows: torch.Tensor) -> None:
+    """What `outer_state_scan` reads for a retention where the chunked kernels do not run: rows float32 [T, 2 * heads * dim + heads *
+    vdim] = [q turned | k turned, times k_scale | v]."""
+    n = _retention_args("retention_rows", q, k, v, None, None, 0, n_heads, dim, vdim)
+    _dev("rows", rows, torch.float32)
+    if rows.shape != (n, n_heads * (2 * dim + vdim)):
+        raise KernelError("retention_rows: rows must be [T, heads * (2 dim + vdim)]")
+    if rot_dim:
+        _dev("angles", angles, torch.float32)
+        if angles.shape != (n, rot_dim // 2, 2):
+            raise KernelError("retention_rows: angles must be [T, rot_dim / 2, 2]")
+    _check(library("retention").qf_retention_rows(
+        _I(_is_bf16(q.dtype)), _ptr(q), _I(q.stride(0)), _ptr(k), _I(k.stride(0)), _ptr(v), _I(v.stride(0)), _ptr(angles if rot_dim else None),
+        _I(rot_dim), _F(k_scale), _I(n), _I(n_heads), _I(dim), _I(vdim), _ptr(rows), _stream()), "retention_rows")

@@ -22,7 +22,8 @@ TIMED = ("embed_gather", "gather_rows", "add_rms_norm", "residual_add", "linear"
          "decay_gates", "gated_group_norm", "causal_conv_silu", "causal_conv", "add_dyt_norm", "add_dyt_norm_shift", "residual_add_pair", "stream_pair",
          "head_gate", "pool_cache_write", "add_rms_norm_scaled", "residual_add_scaled", "rms_norm_cols", "mix_rows", "bias_glu",
          "shift_mix", "channel_decay", "outer_state_scan_rows", "rows_prepare", "causal_conv_cached", "delta_scan", "delta_token",
-         "streams_norm", "rotate_heads", "sigmoid_gate")
+         "streams_norm", "rotate_heads", "sigmoid_gate", "pair_rms_norm", "map_difference", "rope_maps_cache_write", "rope_table",
+         "retention_chunks", "retention_token", "retention_rows")
 
 
 class KernelTimer:

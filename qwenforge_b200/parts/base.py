@@ -148,27 +148,45 @@ class Pending:
         """The float32 tensor that will be added (for diagnosis; not on the product path)."""
         raise NotImplementedError
 
-    def normed_rows(self, rows: torch.Tensor, norm: "Norm", err: torch.Tensor):
-        """The named tokens' rows of the finished stream under `norm`, where this can be had without resolving the whole
-        stream (what an output head reads); None otherwise."""
+    def normed_rows(self, hidden: torch.Tensor, rows: torch.Tensor, norm: "Norm", err: torch.Tensor):
+        """The named tokens' rows of the finished stream (`hidden` and what is pending) under `norm`, where this can be had
+        without resolving the whole stream (what an output head reads); None otherwise."""
         return None
 
 
 class PendingPair(Pending):
-    """The outputs of two sublayers that read the same input (a parallel layer): their sum goes into the stream, summed
-    with each other first. Either may be None."""
-    __slots__ = ("a", "b")
+    """The outputs of two sublayers that read the same stream (a parallel layer): their sum goes into the stream, summed
+    with each other first. Either may be None; the second may be a `RowSum` whose rows are still to be summed per token."""
+    __slots__ = ("a", "b", "rows")
 
     def __init__(self, a, b=None):
-        self.a, self.b = a, b
+        self.rows = (b.dest, b.top, b.row_weight) if isinstance(b, RowSum) else None
+        self.a, self.b = a, b.rows if isinstance(b, RowSum) else b
 
     def add_to(self, hidden: torch.Tensor) -> None:
         from .. import ops
-        ops.residual_add_pair(hidden, self.a, self.b)
+        if self.rows is not None:
+            ops.pair_rms_norm(hidden, self.a, self.b, b_rows=self.rows)
+        else:
+            ops.residual_add_pair(hidden, self.a, self.b)
 
     def value(self) -> torch.Tensor:
-        parts = [t.to(torch.float32) for t in (self.a, self.b) if t is not None]
+        b = self.b
+        if self.rows is not None:
+            dest, top, row_weight = self.rows
+            b = b.to(torch.float32) if row_weight is None else b.to(torch.float32) * row_weight[:, None]
+            b = b[dest.long()].view(-1, top, b.shape[1]).sum(1)
+        parts = [t.to(torch.float32) for t in (self.a, b) if t is not None]
         return parts[0] + parts[1] if len(parts) == 2 else parts[0]
+
+    def normed_rows(self, hidden, rows, norm, err):
+        rms = norm.fused_rms()
+        if rms is None or (self.a if self.a is not None else self.b).dtype != rms[0].dtype:
+            return None
+        from .. import ops
+        out = torch.empty((rows.numel(), hidden.shape[1]), dtype=rms[0].dtype, device=hidden.device)
+        ops.pair_rms_norm(hidden, self.a, self.b, rms[0], rms[1], out, b_rows=self.rows, rows=rows, err=err)
+        return out
 
 
 class PendingScaled(Pending):
@@ -274,7 +292,7 @@ class PendingStreams(Pending):
         hidden.copy_(self.total())
 
 
-    def normed_rows(self, rows, norm, err):
+    def normed_rows(self, hidden, rows, norm, err):
         fused = norm.elementwise() if hasattr(norm, "elementwise") else None
         if fused is None:
             return None
@@ -300,9 +318,13 @@ class Embedding(Part):
         raise NotImplementedError
 
     def lookup_table(self):
-        """The table [vocab, width] if this embedding is a plain row lookup (row id -> stream row, nothing added or
-        scaled), which the kernel that advances a decode graph's state may then do for the next step; else None."""
+        """The table [vocab, width] if this embedding is a plain row lookup (row id -> stream row times `lookup_scale()`,
+        nothing added), which the kernel that advances a decode graph's state may then do for the next step; else None."""
         return None
+
+    def lookup_scale(self) -> float:
+        """The factor on the looked-up rows."""
+        return 1.0
 
 
 class Norm(Part):

@@ -7,8 +7,9 @@ from __future__ import annotations
 
 import torch
 
+from .. import ops
 from ..cache import BundleNeed
-from .base import Norm, Part, Pending, PendingNormed, PendingPair, PendingScaled, PendingStreams
+from .base import Norm, Part, Pending, PendingNormed, PendingPair, PendingScaled, PendingStreams, RowSum, fork, join, runs_side_by_side
 from .registry import build_part, register_part
 
 
@@ -115,11 +116,13 @@ class SandwichBlock(Part):
 
 
 class ParallelBlock(Part):
-    """One norm that both sublayers read:  h = norm(x);  x += mixer(in(h)) + feed_forward(h).
-    Reads the layer spec's parts `norm`, `mixer` and, if the layer has them, `feed_forward` and `mixer_input` (a part of role
-    "mixer_input" that filters what the mixer reads and may keep a state of its own per sequence, such as a token shift;
-    the feed-forward reads h as it is). The two outputs stay pending as a pair: the next norm kernel of a block of this
-    kind adds their sum to the float32 stream on its way."""
+    """Two sublayers side by side:  h = norm(x);  x += mixer(in(h)) + feed_forward(h);  or, with a norm for each,
+    x += mixer(in(norm(x))) + feed_forward(feed_forward_norm(x)), both norms of the same x.
+    Reads the layer spec's parts `norm`, `mixer` and, if the layer has them, `feed_forward`, `feed_forward_norm` and `mixer_input` (a
+    part of role "mixer_input" that filters what the mixer reads and may keep a state of its own per sequence, such as a token
+    shift; the feed-forward reads its norm's output as it is). The two outputs stay pending as a pair: the next norm kernel of a block
+    of this kind adds their sum to the float32 stream on its way. In a block with two norms (plain RMS norms) that kernel makes both,
+    and sums a feed-forward's unsummed rows as well; the two sublayers of a step of few rows then run on two streams."""
 
     accepts_pending = (PendingPair,)
 
@@ -129,10 +132,15 @@ class ParallelBlock(Part):
         self.mixer = build_part("mixer", layer_spec.part("mixer"))
         self.mixer_input = build_part("mixer_input", layer_spec.part("mixer_input")) if "mixer_input" in layer_spec.parts else None
         self.feed_forward = build_part("feed_forward", layer_spec.part("feed_forward")) if "feed_forward" in layer_spec.parts else None
+        self.feed_forward_norm = build_part("norm", layer_spec.part("feed_forward_norm")) if "feed_forward_norm" in layer_spec.parts else None
         self.pair_norm = bool(getattr(self.norm, "takes_pair", False))   # its kernel adds two pending outputs on its way
+        # plain RMS norms: one kernel for what is pending and up to two norms
+        self.rms_norms = all(n is None or type(n).fused_rms is not Norm.fused_rms for n in (self.norm, self.feed_forward_norm))
+        if self.feed_forward_norm is not None and (self.feed_forward is None or self.mixer_input is not None or not self.rms_norms):
+            raise ValueError("parallel: a second norm goes with a feed-forward, with plain RMS norms and without a filter in front of the mixer")
 
     def sub_parts(self):
-        return [p for p in (self.norm, self.mixer_input, self.mixer, self.feed_forward) if p is not None]
+        return [p for p in (self.norm, self.mixer_input, self.mixer, self.feed_forward_norm, self.feed_forward) if p is not None]
 
     def cache_need(self):
         need = self.mixer.cache_need()
@@ -140,7 +148,36 @@ class ParallelBlock(Part):
             return need
         return BundleNeed((("input", self.mixer_input.cache_need()), ("mixer", need)))
 
+    def _forward_rms(self, hidden, delta, ctx, site, writes_cache):
+        """The layer with plain RMS norms (one or two) and nothing in front of the mixer."""
+        weight, eps = self.norm.fused_rms()
+        h1 = torch.empty(hidden.shape, dtype=weight.dtype, device=hidden.device)
+        second = {}
+        if self.feed_forward_norm is not None:
+            weight2, eps2 = self.feed_forward_norm.fused_rms()
+            second = {"weight2": weight2, "eps2": eps2, "out2": torch.empty_like(h1)}
+        if isinstance(delta, PendingPair):
+            ops.pair_rms_norm(hidden, delta.a, delta.b, weight, eps, h1, b_rows=delta.rows, **second)
+        else:
+            ops.pair_rms_norm(hidden, delta, None, weight, eps, h1, **second)
+        if self.feed_forward is None:
+            return PendingPair(self.mixer.forward(h1, ctx, site, writes_cache))
+        h2 = second.get("out2", h1)
+        # a feed-forward that leaves several rows per token hands them over unsummed: the next norm kernel adds them up
+        run = getattr(self.feed_forward, "forward_rows", None) or self.feed_forward.forward
+        if runs_side_by_side(h1):
+            main, side = fork(h2)
+            with torch.cuda.stream(side):
+                fed = run(h2, ctx)
+            mixed = self.mixer.forward(h1, ctx, site, writes_cache)
+            join(main, side, *((fed.rows, fed.dest, fed.row_weight) if isinstance(fed, RowSum) else (fed,)))
+        else:
+            mixed, fed = self.mixer.forward(h1, ctx, site, writes_cache), run(h2, ctx)
+        return PendingPair(mixed, fed)
+
     def forward(self, hidden, delta, ctx, site, writes_cache):
+        if self.rms_norms and self.mixer_input is None:
+            return self._forward_rms(hidden, delta, ctx, site, writes_cache)
         bundled = self.mixer_input is not None and self.mixer_input.cache_need() is not None
         if bundled and not writes_cache:
             raise ValueError("parallel: a layer whose mixer input keeps a state cannot read another entry's cache")
@@ -150,7 +187,7 @@ class ParallelBlock(Part):
             rider = self.mixer_input.rides_on_norm(hidden.shape[0], ctx, site["input"])
         extra = {} if rider is None else {"shift": rider}
         if isinstance(delta, PendingPair):
-            if self.pair_norm:
+            if self.pair_norm and delta.rows is None:
                 h = self.norm.forward(hidden, delta.a, delta.b, **extra)
             else:
                 delta.add_to(hidden)
@@ -211,7 +248,6 @@ class StreamsBlock(Part):
             if isinstance(delta, Pending):
                 delta.add_to(hidden)
             elif delta is not None:
-                from .. import ops
                 ops.residual_add(hidden, delta)
             delta = PendingStreams(hidden, self.n)
         at = lambda name: site.get(name) if site is not None else None

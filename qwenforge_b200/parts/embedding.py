@@ -10,12 +10,14 @@ from .registry import register_part
 
 
 class TokenEmbedding(Embedding):
-    """params: vocab_size, width. tensors: weight [vocab_size, width]."""
+    """params: vocab_size, width, and optionally scale (every row enters the stream times this factor, in float32).
+    tensors: weight [vocab_size, width]."""
 
     def __init__(self, spec):
         super().__init__(spec)
         self.vocab = int(self.params["vocab_size"])
         self.width = int(self.params["width"])
+        self.scale = float(self.params.get("scale", 1.0))
         self.weight = None
 
     def tensor_specs(self):
@@ -30,9 +32,12 @@ class TokenEmbedding(Embedding):
     def lookup_table(self):
         return self.weight
 
+    def lookup_scale(self):
+        return self.scale
+
     def forward(self, token_ids: torch.Tensor, ctx) -> torch.Tensor:
         hidden = torch.empty((token_ids.numel(), self.width), dtype=torch.float32, device=token_ids.device)
-        ops.embed_gather(token_ids, self.weight, hidden, ctx.err)
+        ops.embed_gather(token_ids, self.weight, hidden, ctx.err, self.scale)
         return hidden
 
 

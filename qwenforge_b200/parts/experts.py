@@ -16,10 +16,11 @@ Options, each a parameter of the spec:
                chosen experts' sum; with `gated` it is multiplied by sigmoid(s . h), one number per token
   gate         "none": the experts have no gate, expert(v) = D_e act(U_e v) with `activation` one of the library's (the square
                of relu, say); tensors up.<e>, down.<e> only, and the shared expert likewise
-  correction   a float32 number per expert that is added to the sigmoid score for the CHOICE only; the weights are the
+  correction   a float32 number per expert that is added to the score for the CHOICE only; the weights are the
                scores without it
   groups       (count, keep): the experts form `count` equal groups of neighbours, a group's score is the sum of its two
-               largest choice scores, and only experts of the `keep` best groups can be chosen
+               largest choice scores (`group_best` = 2, the default) or its largest one (1), and only experts of the `keep`
+               best groups can be chosen
 (score "softmax" with `renormalize` is the softmax over the chosen logits alone.)
 
 Routing, sorting by expert and the experts' products all stay on the device (`ops.moe_plan`, `ops.expert_linear`: one
@@ -63,8 +64,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: experts without a gate take one of the library's activations and the weight on the output")
         self.corrected = bool(p.get("correction", False))
         self.groups = tuple(int(g) for g in p["groups"]) if p.get("groups") else None
-        if (self.corrected or self.groups) and self.score != "sigmoid":
-            raise ValueError("routed_experts: a correction of the choice and groups of experts go with sigmoid scores")
+        self.group_best = int(p.get("group_best") or 2)
+        if self.group_best not in (1, 2):
+            raise ValueError("routed_experts: a group's score is its largest choice score (group_best 1) or the sum of its two largest (2)")
         if self.groups and (not 1 <= self.groups[1] <= self.groups[0] <= 64 or self.n_experts % self.groups[0]
                             or self.groups[1] * (self.n_experts // self.groups[0]) < self.top):
             raise ValueError(f"routed_experts: {self.groups[1]} of {self.groups[0]} groups over {self.n_experts} experts cannot "
@@ -162,7 +164,7 @@ class RoutedExperts(FeedForward):
         # (the large tile only where both products' operands allow it)
         tile_rows = min(ops.moe_tile_rows(n, self.n_experts, self.top, self.gate_up), ops.moe_tile_rows(n, self.n_experts, self.top, self.down))
         soft, renorm = self.score == "softmax", self.renormalize
-        choice = {"correction": self.correction, "groups": self.groups} if (self.corrected or self.groups) else {}
+        choice = {"correction": self.correction, "groups": self.groups, "group_best": self.group_best} if (self.corrected or self.groups) else {}
         if n * self.n_experts <= ops.MOE_FUSED_ROUTER_MAX:
             plan = ops.moe_plan(None, self.top, soft, renorm, tile_rows, x=x, router=self.router, bias=self.bias, **choice)   # few tokens: one launch
         else:

@@ -26,6 +26,13 @@ Two more kinds decay every ROW of S by a number of its own (a decay per head and
       S <- diag(a_t) S + k_t v_t^T;  y_t = S^T q_t (AFTER the token);  out = Wo (rms_per_head(y; n) * silu(Wg h)),
       the norm's weight [vdim] shared by the heads
 
+One decays by a number of its own per head, the same for every token:
+
+  retention
+      q = Wq h, k = Wk h in heads, both turned by position, k / sqrt(dim), v = Wv h;  S <- decay_h S + k_t v_t^T;  y_t = S^T q_t;
+      out = Wo (y / rms(y) per head * silu(Wg h)), the norm without a weight. With a fixed decay the recurrence can be written out
+      over a chunk of tokens (`ops.retention_chunks`, products on the tensor cores); single tokens take `ops.retention_token`
+
 And one corrects what the state already says about a key before it adds to it:
 
   channel_delta (the gated delta rule with a decay per head and key channel, `ops.delta_scan`, `ops.delta_token`)
@@ -36,8 +43,8 @@ And one corrects what the state already says about a key before it adds to it:
 
 The state lives in the sequence cache as ONE float32 row per sequence and schedule entry (`StateNeed`), zeroed when a
 sequence starts: [S | n | m] for the matrix memory, [S | the convolution's last taps - 1 inputs] for the state space,
-[S | the last token's h] for the time mixing, [S] for the gated linear attention, [S | the convolution's last inputs] for the
-delta rule.
+[S | the last token's h] for the time mixing, [S] for the gated linear attention and the retention, [S | the convolution's last
+inputs] for the delta rule.
 The gates' pre-activations are products with float32 results, and everything from there to the scan's output is
 float32 in both precisions; the other projections and the convolution carry the activation dtype.
 """
@@ -48,7 +55,7 @@ import torch
 from .. import ops
 from ..cache import StateNeed
 from .base import Mixer, TensorSpec, fork, join, runs_side_by_side
-from .registry import register_part
+from .registry import build_part, register_part
 
 
 class MatrixMemory(Mixer):
@@ -447,6 +454,90 @@ class ChannelDelta(Mixer):
         return ops.linear_rows(out, self.o_weight)
 
 
+class Retention(Mixer):
+    """params: hidden_size, num_heads, head_dim, value_dim, decay (one number per head), eps, position (PartSpec | None; component j
+    paired with j + half). tensors: q_weight, k_weight [H*dim, W], v_weight, g_weight [H*vdim, W], o_weight [W, H*vdim]."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.hidden, self.n_heads = int(p["hidden_size"]), int(p["num_heads"])
+        self.dim, self.vdim, self.eps = int(p["head_dim"]), int(p["value_dim"]), float(p["eps"])
+        self.decays = tuple(float(d) for d in p["decay"])
+        if len(self.decays) != self.n_heads:
+            raise ValueError(f"retention: {len(self.decays)} decays for {self.n_heads} heads")
+        if not 1 <= self.dim <= ops.OUTER_STATE_MAX_DIM or not 1 <= self.vdim <= 1024:
+            raise ValueError(f"retention: head_dim up to {ops.OUTER_STATE_MAX_DIM} and values of up to 1,024 are supported")
+        self.position = build_part("position", p["position"]) if p.get("position") is not None else None
+        if self.position is not None and getattr(self.position, "interleaved", True):
+            raise ValueError("retention: the position part pairs component j with j + half")
+        # (whole fours per slot: the kernels move four numbers of S at a time)
+        self.state_floats = -(-(self.n_heads * self.dim * self.vdim) // 4) * 4
+        self.proj_weight = self.o_weight = self.decay = self.powers = self.unit = None
+
+    def sub_parts(self):
+        return [self.position] if self.position is not None else []
+
+    def tensor_specs(self):
+        f, h, d, v, w = self.file_name, self.n_heads, self.dim, self.vdim, self.hidden
+        return [TensorSpec(f("q_weight"), (h * d, w)), TensorSpec(f("k_weight"), (h * d, w)), TensorSpec(f("v_weight"), (h * v, w)),
+                TensorSpec(f("g_weight"), (h * v, w)), TensorSpec(f("o_weight"), (w, h * v))]
+
+    def kernel_libraries(self, dtype):
+        return {"recurrent", "retention", "rope_cache"} | ({"gemm_f32"} if dtype == torch.float32 else {"skinny_gemm"})
+
+    def cache_need(self):
+        return StateNeed((self.state_floats,), torch.float32)
+
+    def bind(self, tensors, dtype, device):
+        t = lambda logical: tensors[self.file_name(logical)]
+        self.proj_weight = torch.cat((t("q_weight"), t("k_weight"), t("v_weight"), t("g_weight")), dim=0).contiguous()
+        self.o_weight = t("o_weight")
+        decay = torch.tensor(self.decays, dtype=torch.float64)
+        self.decay = decay.to(torch.float32).to(device)
+        # the powers of the decays that the chunked form multiplies with, formed in float64 and rounded once
+        self.powers = (decay[:, None] ** torch.arange(ops.RETENTION_CHUNK + 1, dtype=torch.float64)).to(torch.float32).contiguous().to(device)
+        self.unit = torch.ones(self.n_heads * self.vdim, dtype=dtype, device=device)
+
+    def step_weights(self):
+        return [self.proj_weight, self.o_weight]
+
+    def _angles(self, ctx):
+        """Cosine and sine of the step's tokens: made by the first layer of these frequencies, shared through the step's memo."""
+        if self.position is None:
+            return None
+        key = ("retention.angles", tuple(sorted((k, str(v)) for k, v in self.position.params.items())))
+        memo = ctx.step_memo if ctx.step_memo is not None else {}
+        if key not in memo:
+            memo[key] = ops.rope_table(ctx.tok_pos, self.position.fused_rotary()[0], self.position.amplitude)
+        return memo[key]
+
+    def forward(self, x, ctx, site, writes_cache):
+        if not writes_cache:
+            raise ValueError("retention: a recurrent state cannot be read from another schedule entry")
+        n, h, d, v = x.shape[0], self.n_heads, self.dim, self.vdim
+        inv_freq, rot_dim = self.position.fused_rotary() if self.position is not None else (None, 0)
+        proj = ops.linear_rows(x, self.proj_weight)                                  # [T, q | k | v | g]
+        q, k, value, gate = proj[:, :h * d], proj[:, h * d:2 * h * d], proj[:, 2 * h * d:2 * h * d + h * v], proj[:, 2 * h * d + h * v:]
+        out = torch.empty((n, h * v), dtype=x.dtype, device=x.device)
+        if ctx.is_decode and n == ctx.n_seqs:
+            amplitude = self.position.amplitude if self.position is not None else 1.0
+            ops.retention_token(q, k, value, gate, ctx.tok_pos, inv_freq, rot_dim, amplitude, self.decay, d ** -0.5, self.eps, ctx.cu_q,
+                                ctx.slots, site.storage, 0, h, d, v, out)
+        elif ops.retention_chunks_take(q, k, value, gate, site.storage, 0, d, v, rot_dim):
+            ops.retention_chunks(q, k, value, gate, self._angles(ctx), rot_dim, self.powers, d ** -0.5, self.eps, ctx.cu_q, ctx.slots,
+                                 ctx.max_q_len, site.storage, 0, h, d, v, out)
+        else:   # true float32 steps and sizes in no whole eights: the scan token by token
+            f32 = dict(dtype=torch.float32, device=x.device)
+            rows, y = torch.empty((n, h * (2 * d + v)), **f32), torch.empty((n, h * v), **f32)
+            ops.retention_rows(q, k, value, self._angles(ctx), rot_dim, d ** -0.5, h, d, v, rows)
+            ops.outer_state_scan(rows[:, :h * d], rows[:, h * d:2 * h * d], rows[:, 2 * h * d:], self.decay, None, ctx.cu_q, ctx.slots,
+                                 site.storage, 0, -1, h, h, d, v, 1.0, y, None)
+            ops.gated_group_norm(y, gate, self.unit, self.eps, out, h, h, "silu", False)
+        return ops.linear_rows(out, self.o_weight)
+
+
+register_part("mixer", "retention", Retention)
 register_part("mixer", "channel_delta", ChannelDelta)
 register_part("mixer", "matrix_memory", MatrixMemory)
 register_part("mixer", "time_mix", TimeMix)

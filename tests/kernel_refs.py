@@ -18,8 +18,8 @@ def _f(t):
     return t.to(torch.float64)
 
 
-def embed_gather(ids, table, out, err):
-    out.copy_(table[ids.long()].to(torch.float32))
+def embed_gather(ids, table, out, err, scale=1.0):
+    out.copy_(table[ids.long()].to(torch.float32) * scale)
 
 
 def gather_rows(hidden, delta, rows, out, err):
@@ -301,7 +301,7 @@ def scaled_swiglu(gate_up, row_scale, out):
 
 
 def moe_plan(logits, top, softmax_scores=False, renormalize=False, tile_rows=64, x=None, router=None, bias=None, correction=None,
-             groups=None):
+             groups=None, group_best=2):
     if logits is None:
         logits = (_f(x) @ _f(router).T)
     z = logits.to(torch.float32)
@@ -313,7 +313,7 @@ def moe_plan(logits, top, softmax_scores=False, renormalize=False, tile_rows=64,
         count, keep = groups if groups is not None else (1, 1)
         if keep < count:
             grouped = choice.view(z.shape[0], count, -1)
-            group_score = grouped.topk(min(2, grouped.shape[-1]), dim=-1).values.sum(-1)
+            group_score = grouped.topk(min(group_best, grouped.shape[-1]), dim=-1).values.sum(-1)
             kept = torch.zeros_like(group_score, dtype=torch.bool).scatter_(1, group_score.topk(keep, dim=-1).indices, True)
             choice = grouped.masked_fill(~kept[:, :, None], float("-inf")).reshape(z.shape)
         picked = torch.topk(choice, top, dim=-1).indices
@@ -508,7 +508,7 @@ def outer_state_scan(q, k, v, decay, take, cu_q, slots, state, s_offset, n_offse
             qt = (_f(q[t]) * q_scale).view(n_groups, dim).repeat_interleave(per, dim=0)
             kt = _f(k[t]).view(n_groups, dim).repeat_interleave(per, dim=0)
             vt = _f(v[t]).view(n_heads, vdim)
-            d, g = _f(decay[t])[:, None], _f(take[t])[:, None]
+            d, g = (_f(decay[t])[:, None], _f(take[t])[:, None]) if take is not None else (_f(decay)[:, None], torch.ones_like(_f(decay))[:, None])
             S = d[:, :, None] * S + g[:, :, None] * kt[:, :, None] * vt[:, None, :]
             y[t] = torch.einsum("hdv,hd->hv", S, qt).reshape(-1).float()
             if nq is not None:
@@ -715,3 +715,128 @@ ALL = dict(causal_conv_cached=causal_conv_cached, sigmoid_gate=sigmoid_gate, del
            embed_gather=embed_gather, gather_rows=gather_rows, gather_rows_norm=gather_rows_norm, add_rms_norm=add_rms_norm, gemm_f32=gemm_f32,
            linear=linear, rope_cache_write=rope_cache_write, attention_generic=attention_generic, swiglu=swiglu,
            sample=sample)
+
+
+# ---------------------------------------------------------------- heads of two maps, two norms of one stream, retention
+def _turn_halves(x, cos, sin):
+    """x [T, ..., D]; cos, sin [T, R/2]: component j of the first R turned with j + R/2."""
+    half = cos.shape[1]
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (half,)
+    c, s = cos.view(shape), sin.view(shape)
+    a, b = x[..., :half], x[..., half:2 * half]
+    return torch.cat((a * c - b * s, b * c + a * s, x[..., 2 * half:]), dim=-1)
+
+
+def rope_table(tok_pos, inv_freq, amplitude=1.0):
+    angle = (tok_pos.to(torch.float32).unsqueeze(-1) * inv_freq.to(torch.float32)).to(torch.float64)
+    return (torch.stack((angle.cos(), angle.sin()), dim=-1) * amplitude).to(torch.float32)
+
+
+def _angles_of(tok_pos, inv_freq, amplitude):
+    angle = (tok_pos.to(torch.float32).unsqueeze(-1) * inv_freq.to(torch.float32)).to(torch.float64)
+    return angle.cos() * amplitude, angle.sin() * amplitude
+
+
+def rope_maps_cache_write(qkv, tok_seq, tok_pos, slots, inv_freq, rot_dim, amplitude, n_heads, maps, dim, vdim, q_out, site, write_cache, err):
+    n, d, kvh = qkv.shape[0], site.head_dim, site.kv_heads
+    x = _f(qkv)
+    a, b = n_heads * maps * dim, kvh * maps * dim
+    q, k, v = x[:, :a].reshape(n, n_heads, maps, dim), x[:, a:a + b].reshape(n, kvh, maps, dim), x[:, a + b:a + b + kvh * vdim].reshape(n, kvh, vdim)
+    if inv_freq is not None and rot_dim > 0:
+        cos, sin = _angles_of(tok_pos, inv_freq, amplitude)
+        q, k = _turn_halves(q, cos, sin), _turn_halves(k, cos, sin)
+    wide = torch.zeros((n, n_heads, maps, d), dtype=torch.float64, device=qkv.device)
+    for m in range(maps):
+        wide[:, :, m, m * dim:(m + 1) * dim] = q[:, :, m]
+    q_out.copy_(wide.reshape(n, -1).to(q_out.dtype))
+    if not write_cache:
+        return
+    for t in range(n):
+        slot = int(slots[int(tok_seq[t])])
+        if slot < 0:
+            continue
+        pos = int(tok_pos[t])
+        page = int(site.table[slot, pos // PAGE])
+        assert page >= 0, "reference: write to a page that is not held"
+        rows = site.storage[page, :, :, pos % PAGE, :]
+        rows.zero_()
+        rows[0, :, :maps * dim] = k[t].reshape(kvh, maps * dim).to(rows.dtype)
+        rows[1, :, :vdim] = v[t].to(rows.dtype)
+
+
+def map_difference(x, pitch, weight, eps, gain, out, heads, vdim):
+    a = _f(x).view(x.shape[0], heads, 2, pitch)[..., :vdim]
+    o = a[:, :, 0] - weight * a[:, :, 1]
+    out.copy_((gain * o / torch.sqrt(o.square().mean(-1, keepdim=True) + eps)).reshape(out.shape).to(out.dtype))
+
+
+def pair_rms_norm(hidden, a, b, weight1=None, eps1=0.0, out1=None, weight2=None, eps2=0.0, out2=None, b_rows=None, rows=None, err=None):
+    total = torch.zeros(hidden.shape, dtype=torch.float64, device=hidden.device)
+    if b is not None:
+        y = _f(b)
+        if b_rows is not None:
+            dest, top, row_weight = b_rows
+            if row_weight is not None:
+                y = y * _f(row_weight)[:, None]
+            y = y[dest.long()].view(-1, top, y.shape[1]).sum(1)
+        total += y
+    if a is not None:
+        total += _f(a)
+    x = _f(hidden) + total
+    if rows is None:
+        hidden.copy_(x.to(torch.float32))
+        x = _f(hidden)
+    else:
+        x = x[rows.long()]
+    for weight, eps, out in ((weight1, eps1, out1), (weight2, eps2, out2)):
+        if weight is not None:
+            out.copy_(_rms(x, weight, eps).to(out.dtype))
+
+
+def retention_chunks_take(q, k, v, gate, state, s_offset, dim, vdim, rot_dim):
+    return q.dtype == torch.bfloat16
+
+
+def _retention(q, k, v, gate, cos, sin, decay, k_scale, eps, cu_q, slots, state, s_offset, n_heads, dim, vdim, out):
+    n, size = q.shape[0], n_heads * dim * vdim
+    qh, kh, vh = _f(q).reshape(n, n_heads, dim), _f(k).reshape(n, n_heads, dim), _f(v).reshape(n, n_heads, vdim)
+    if cos is not None:
+        qh, kh = _turn_halves(qh, cos, sin), _turn_halves(kh, cos, sin)
+    kh = kh * k_scale
+    for s in range(cu_q.numel() - 1):
+        slot = int(slots[s])
+        S = torch.zeros(n_heads, dim, vdim, dtype=torch.float64, device=q.device)
+        if slot >= 0:
+            S = _f(state[slot, s_offset:s_offset + size]).view(n_heads, dim, vdim).clone()
+        for t in range(int(cu_q[s]), int(cu_q[s + 1])):
+            S = _f(decay)[:, None, None] * S + kh[t][:, :, None] * vh[t][:, None, :]
+            o = torch.einsum("hdv,hd->hv", S, qh[t])
+            o = o / torch.sqrt(o.square().mean(-1, keepdim=True) + eps)
+            g = _f(gate[t])
+            out[t] = (o.reshape(-1) * g * torch.sigmoid(g)).to(out.dtype)
+        if slot >= 0:
+            state[slot, s_offset:s_offset + size] = S.reshape(-1).float()
+
+
+def retention_chunks(q, k, v, gate, angles, rot_dim, powers, k_scale, eps, cu_q, slots, max_q_len, state, s_offset, n_heads, dim, vdim, out):
+    cos, sin = (_f(angles[..., 0]), _f(angles[..., 1])) if rot_dim else (None, None)
+    _retention(q, k, v, gate, cos, sin, powers[:, 1], k_scale, eps, cu_q, slots, state, s_offset, n_heads, dim, vdim, out)
+
+
+def retention_token(q, k, v, gate, tok_pos, inv_freq, rot_dim, amplitude, decay, k_scale, eps, cu_q, slots, state, s_offset, n_heads, dim, vdim, out):
+    cos, sin = _angles_of(tok_pos, inv_freq, amplitude) if rot_dim else (None, None)
+    _retention(q, k, v, gate, cos, sin, decay, k_scale, eps, cu_q, slots, state, s_offset, n_heads, dim, vdim, out)
+
+
+def retention_rows(q, k, v, angles, rot_dim, k_scale, n_heads, dim, vdim, rows):
+    n = q.shape[0]
+    qh, kh = _f(q).reshape(n, n_heads, dim), _f(k).reshape(n, n_heads, dim)
+    if rot_dim:
+        cos, sin = _f(angles[..., 0]), _f(angles[..., 1])
+        qh, kh = _turn_halves(qh, cos, sin), _turn_halves(kh, cos, sin)
+    rows.copy_(torch.cat((qh.reshape(n, -1), kh.reshape(n, -1) * k_scale, _f(v)), dim=-1).to(torch.float32))
+
+
+ALL.update(rope_table=rope_table, rope_maps_cache_write=rope_maps_cache_write, map_difference=map_difference, pair_rms_norm=pair_rms_norm,
+           retention_chunks_take=retention_chunks_take, retention_chunks=retention_chunks, retention_token=retention_token,
+           retention_rows=retention_rows)
