@@ -7,6 +7,7 @@ decode at batch 1 and 64, and the same decode rate end to end through the Python
     python bench.py --design zebovik     # the same for the Zebovik presets (attention in blocks, mLSTM and Mamba-2 layers)
     python bench.py --design rarevik     # the same for the Rarevik presets (parallel layers, windows with pooled blocks, routed experts)
     python bench.py --design dapupel     # the Dapupel presets (several streams, latent attention, delta rule, experts) beside Rarevik's and Qwen2's
+    python bench.py --design lasonex     # the Lasonex presets (differential window attention, retention, experts in groups) beside Gatosun's, Rarevik's and Qwen2's
     python bench.py --design gatosun     # the same for the Gatosun presets (window attention beside time mixing, gated linear attention, experts in groups)
                                          # (prompt and decode rates, device times by kind of kernel), as one JSON line
 
@@ -47,7 +48,7 @@ def parse():
     p.add_argument("--workload", default=None, choices=sorted(WORKLOADS),
                    help="run only this named workload (3B: 16 unequal prompts then 256 steps; 7B: batch 64 to context "
                         "8192 at temperature 0.7) and print its line")
-    p.add_argument("--design", default=None, choices=["mefepel", "zebovik", "rarevik", "gatosun", "dapupel"],
+    p.add_argument("--design", default=None, choices=["mefepel", "zebovik", "rarevik", "gatosun", "dapupel", "lasonex"],
                    help="measure another design's prefill and decode beside the Qwen2 model of equal size (kernel by "
                         "kernel), instead of the default workload")
     p.add_argument("--no-workloads", action="store_true", help="leave the 3B and 7B workloads out of the default run's points")
@@ -364,9 +365,11 @@ DESIGN_PAIRS = {"mefepel": [("mefepel-0.5b", "qwen2.5-0.5b", None), ("mefepel-3b
                 "rarevik": [("rarevik-0.5b", "qwen2.5-0.5b", None), ("rarevik-3b", "qwen2.5-3b", None)],
                 "gatosun": [("gatosun-0.5b", "qwen2.5-0.5b", None), ("gatosun-3b", "qwen2.5-3b", None)],
                 "dapupel": [("dapupel-0.5b", "rarevik-0.5b", None), ("dapupel-0.5b", "qwen2.5-0.5b", None),
-                            ("dapupel-3b", "rarevik-3b", None), ("dapupel-3b", "qwen2.5-3b", None)]}
+                            ("dapupel-3b", "rarevik-3b", None), ("dapupel-3b", "qwen2.5-3b", None)],
+                "lasonex": [(f"lasonex-{size}", f"{other}-{size}", None) for size in ("0.5b", "3b") for other in ("gatosun", "rarevik", "qwen2.5")]}
 # what a kernel's label (ops/timing.py) counts as, so that like is laid beside like
-KERNEL_KINDS = (("streams_norm", "streams + norm + filter"), ("rotate_heads", "rotation of queries"), ("delta_", "recurrent scan"),
+KERNEL_KINDS = (("pair_rms_norm", "norms"), ("map_difference", "maps brought together"), ("rope_maps_cache_write", "rotation + cache write"),
+                ("rope_table", "rotation + cache write"), ("retention_", "recurrent scan"), ("streams_norm", "streams + norm + filter"), ("rotate_heads", "rotation of queries"), ("delta_", "recurrent scan"),
                 ("sigmoid_gate", "gates"), ("causal_conv_cached", "convolution + cache write"),
                 ("attention_prefill", "attention (prompt)"), ("attention_decode", "attention (decode)"),
                 ("attention_generic", "attention (plain)"), ("head_linear", "per-head products"),
