@@ -249,6 +249,141 @@ grouped_gemm_mma_kernel(GroupedArgs g) {
         }
 }
 
+// A step of up to 16 rows per group (decode steps): the work is fetching the groups' weights once, so the weights are the tall side
+// of the tensor-core tile (out^T = W a^T: 16 weight rows x 8 rows of A x 16 columns of K per mma) and a block keeps three slabs of
+// 128 columns of K of its 64 weight rows on their way, five times the bytes of the tile above, which is made for more rows.
+// GATED: the 64 weight rows are 32 gate rows and the 32 matching up rows; warp w takes 16 of both in every second slab step (w >> 1),
+// the halves of K are added through shared memory. Without a gate a warp takes 16 weight rows and all of K.
+#define GR_ROWS 16
+#define GR_BK 128
+#define GR_LD (GR_BK + 8)
+#define GR_STAGES 4
+#define GR_STAGE_ELEMS ((GG_BN + GR_ROWS) * GR_LD)
+template <bool GATED>
+__global__ void __launch_bounds__(128)
+grouped_rows_kernel(GroupedArgs g) {
+    grid_chain_entry();
+    extern __shared__ __align__(16) unsigned char gr_smem[];
+    bf16* stages = reinterpret_cast<bf16*>(gr_smem);   // [GR_STAGES][64 weight rows, then 16 rows of A][GR_LD]
+    int group, m0, m_end;
+    if (!grouped_tile<QF_GROUP_BM>(g, group, m0, m_end)) return;
+    m_end = min(m_end, m0 + GR_ROWS);
+    const bf16* A = (const bf16*)g.a;
+    const bf16* W = (const bf16*)g.w + (long long)group * g.w_group_stride;
+    bf16* C = (bf16*)g.c;
+    const int n0 = blockIdx.x * (GATED ? GG_BN / 2 : GG_BN), N = g.n, K = g.k;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int chunk = (threadIdx.x & 15) * 8, first = threadIdx.x >> 4;   // this thread's 16 bytes of a row, and its first row
+    long long a_row[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int gm = m0 + first + 8 * i;
+        a_row[i] = gm < m_end ? (g.a_rows ? g.a_rows[gm] : gm) : -1;
+    }
+    auto fetch = [&](int k0, int stage) {
+        bf16* w_s = stages + (size_t)stage * GR_STAGE_ELEMS;
+        bf16* a_s = w_s + GG_BN * GR_LD;
+        const bool k_ok = k0 + chunk < K;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int r = first + 8 * i, col = GATED ? n0 + (r & 31) : n0 + r;
+            const long long w_row = GATED ? (r < 32 ? col : (long long)N + col) : col;
+            const bool ok = k_ok && col < N;
+            cp_async_16(w_s + r * GR_LD + chunk, ok ? W + w_row * g.ldw + k0 + chunk : W, ok);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const bool ok = k_ok && a_row[i] >= 0;
+            cp_async_16(a_s + (first + 8 * i) * GR_LD + chunk, ok ? A + a_row[i] * g.lda + k0 + chunk : A, ok);
+        }
+    };
+    constexpr int TILES = GATED ? 2 : 1;   // 16-row tiles of weights per warp (gate and up)
+    float acc[TILES][2][4];
+#pragma unroll
+    for (int i = 0; i < TILES; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+    const int n_slabs = (K + GR_BK - 1) / GR_BK;
+    for (int s = 0; s < GR_STAGES - 1; ++s) {
+        if (s < n_slabs) fetch(s * GR_BK, s);
+        cp_async_commit();
+    }
+    for (int slab = 0; slab < n_slabs; ++slab) {
+        cp_async_wait<GR_STAGES - 2>();
+        __syncthreads();   // slab `slab` has arrived for everyone, and everyone is done with the buffer fetched next
+        if (slab + GR_STAGES - 1 < n_slabs) fetch((slab + GR_STAGES - 1) * GR_BK, (slab + GR_STAGES - 1) % GR_STAGES);
+        cp_async_commit();
+        const bf16* w_s = stages + (size_t)(slab % GR_STAGES) * GR_STAGE_ELEMS;
+        const bf16* a_s = w_s + GG_BN * GR_LD;
+#pragma unroll
+        for (int ks = 0; ks < GR_BK / 16; ks += GATED ? 2 : 1) {
+            const int k = 16 * (ks + (GATED ? warp >> 1 : 0));
+            uint32_t xf[4];   // the 16 rows of A as two column tiles
+            ldmatrix_x4(xf, a_s + (size_t)((lane >> 4) * 8 + (lane & 7)) * GR_LD + k + ((lane >> 3) & 1) * 8);
+#pragma unroll
+            for (int i = 0; i < TILES; ++i) {
+                const int row = GATED ? 32 * i + 16 * (warp & 1) : 16 * warp;
+                uint32_t wf[4];
+                ldmatrix_x4(wf, w_s + (size_t)(row + (lane & 15)) * GR_LD + k + (lane >> 4) * 8);
+                mma_bf16_16816(acc[i][0], wf, xf[0], xf[1]);
+                mma_bf16_16816(acc[i][1], wf, xf[2], xf[3]);
+            }
+        }
+    }
+    cp_async_wait<0>();
+    if (GATED) {
+        __syncthreads();   // the stages are free
+        float* half = reinterpret_cast<float*>(gr_smem);   // [2 warps][TILES * 8][32]
+        if (warp >= 2) {
+#pragma unroll
+            for (int i = 0; i < TILES; ++i)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) half[((warp - 2) * TILES * 8 + (i * 2 + j) * 4 + e) * 32 + lane] = acc[i][j][e];
+        }
+        __syncthreads();
+        if (warp >= 2) return;
+#pragma unroll
+        for (int i = 0; i < TILES; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[i][j][e] += half[(warp * TILES * 8 + (i * 2 + j) * 4 + e) * 32 + lane];
+    }
+    // element e of accumulator j: weight row (lane / 4) + 8 (e / 2), row 8 j + 2 (lane % 4) + e % 2 of A
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int gm = m0 + 8 * j + 2 * (lane & 3) + (e & 1), gn = n0 + 16 * (GATED ? warp & 1 : warp) + (lane >> 2) + 8 * (e >> 1);
+            if (gm >= m_end || gn >= N) continue;
+            float v = acc[0][j][e];
+            if (GATED) {
+                const float s = g.row_scale ? g.row_scale[gm] : 1.f;
+                float gate = s * v, up = s * acc[TILES - 1][j][e], slope = 1.f;
+                if (g.gate_limit > 0.f) {
+                    gate = fminf(gate, g.gate_limit);
+                    up = fminf(fmaxf(up, -g.gate_limit), g.gate_limit) + 1.0f;
+                    slope = g.gate_alpha;
+                }
+                v = gate / (1.0f + expf(-slope * gate)) * up;
+            } else if (g.act) {
+                v = activate(v, g.act - 1);
+            }
+            C[(long long)gm * g.ldc + gn] = __float2bfloat16_rn(v);
+        }
+}
+
+template <bool GATED>
+static int launch_rows(const GroupedArgs& g, cudaStream_t stream) {
+    const size_t smem = (size_t)GR_STAGES * GR_STAGE_ELEMS * sizeof(bf16);
+    cudaError_t e = cudaFuncSetAttribute(grouped_rows_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    const int cols = GATED ? GG_BN / 2 : GG_BN;
+    return (int)launch_pdl(grouped_rows_kernel<GATED>, dim3((g.n + cols - 1) / cols, g.max_tiles), dim3(128), smem, stream, g);
+}
+
 // The large tile: 128 x 128, eight warps as 2 x 4, warp (wy, wx) a quarter of 64 x 32 as 4 x 4 tiles of m16n8k16; slabs of
 // 32 columns of K, three in flight.
 #define GL_BM 128
@@ -356,20 +491,23 @@ static bool mma_takes(const GroupedArgs& g) {
 // operands only: see qf_grouped_gemm_large_takes). A, W and C share the activation dtype; a_rows: see the top.
 // gate_limit > 0 (gated products only): the clamped form of the gate with this limit and the slope gate_alpha.
 // act (products without a gate): 0 stores the sums, k + 1 stores activation k of them (the numbers of common.cuh).
+// most_rows (ragged): the most rows any group can have (0: not known); up to 16 take the kernel of few rows.
 QF_EXPORT int qf_grouped_gemm_act(int is_bf16, const void* a, long long lda, long long a_group_cols, const void* w,
                                   long long w_group_stride, long long ldw, void* c, long long ldc, long long c_group_cols,
                                   int rows, int n, int k, int n_groups, const int* tile_group, const int* tile_row0,
                                   const int* offsets, const int* n_tiles, int max_tiles, int tile_rows, const int* a_rows,
                                   int gated, const float* row_scale, float gate_limit, float gate_alpha, int act,
-                                  cudaStream_t stream) {
+                                  int most_rows, cudaStream_t stream) {
     if (rows <= 0 || n <= 0 || n_groups <= 0) return 0;
     if (act < 0 || act > 6 || (gated && act)) return (int)cudaErrorInvalidValue;
     GroupedArgs g{a, lda, a_group_cols, w, w_group_stride, ldw, c, ldc, c_group_cols, rows, n, k, n_groups,
                   tile_group, tile_row0, offsets, n_tiles, max_tiles, a_rows, row_scale, gate_limit, gate_alpha, act};
+    const bool few_rows = tile_group && tile_rows == QF_GROUP_BM && most_rows > 0 && most_rows <= GR_ROWS;
     if (gated) {  // n = columns of the result (half of a group's weight rows); the small tensor-core tile only
         if (!is_bf16 || !mma_takes(g) || (tile_group && tile_rows != QF_GROUP_BM)) return (int)cudaErrorInvalidValue;
         const dim3 grid((n + GG_BN / 2 - 1) / (GG_BN / 2), tile_group ? max_tiles : (rows + QF_GROUP_BM - 1) / QF_GROUP_BM, tile_group ? 1 : n_groups);
         if (grid.y == 0 || grid.y > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
+        if (few_rows) return launch_rows<true>(g, stream);
         return (int)launch_pdl(grouped_gemm_mma_kernel<true>, grid, dim3(128), 0, stream, g);
     }
     const bool large = tile_group ? tile_rows == GL_BM : (is_bf16 && mma_takes(g) && rows >= GL_MIN_ROWS);
@@ -385,6 +523,7 @@ QF_EXPORT int qf_grouped_gemm_act(int is_bf16, const void* a, long long lda, lon
     }
     const dim3 grid((n + GG_BN - 1) / GG_BN, tile_group ? max_tiles : (rows + QF_GROUP_BM - 1) / QF_GROUP_BM, tile_group ? 1 : n_groups);
     if (grid.y == 0 || grid.y > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
+    if (is_bf16 && mma_takes(g) && few_rows) return launch_rows<false>(g, stream);
     if (is_bf16 && mma_takes(g)) return (int)launch_pdl(grouped_gemm_mma_kernel<false>, grid, dim3(128), 0, stream, g);
     if (is_bf16) return (int)launch_pdl(grouped_gemm_plain_kernel<bf16>, grid, dim3(256), 0, stream, g);
     return (int)launch_pdl(grouped_gemm_plain_kernel<float>, grid, dim3(256), 0, stream, g);
@@ -397,7 +536,7 @@ QF_EXPORT int qf_grouped_gemm_gate(int is_bf16, const void* a, long long lda, lo
                                    int gated, const float* row_scale, float gate_limit, float gate_alpha, cudaStream_t stream) {
     return qf_grouped_gemm_act(is_bf16, a, lda, a_group_cols, w, w_group_stride, ldw, c, ldc, c_group_cols, rows, n, k, n_groups,
                                tile_group, tile_row0, offsets, n_tiles, max_tiles, tile_rows, a_rows, gated, row_scale, gate_limit,
-                               gate_alpha, 0, stream);
+                               gate_alpha, 0, 0, stream);
 }
 
 QF_EXPORT int qf_grouped_gemm(int is_bf16, const void* a, long long lda, long long a_group_cols, const void* w,

@@ -125,13 +125,77 @@ __device__ __forceinline__ void moe_choose_grouped(const float* z_raw, const flo
         for (int k = 0; k < top; ++k) weight[k] /= total;
 }
 
+// The same choice by a warp, a lane per expert (up to 32 of them): every lane learns its expert's place in the token's choice (0 the
+// best; -1: not chosen) and its weight. Ranks are counted by comparing with every other lane, so there is no chain of choices.
+// groups.count 0: the plain choice, by the logits.
+__device__ __forceinline__ int moe_choose_warp(float z, int n_experts, int top, int softmax_scores, int renormalize, MoeGroups groups,
+                                               float& weight) {
+    const int lane = threadIdx.x & 31;
+    const bool real = lane < n_experts;
+    float s;
+    if (softmax_scores) {
+        const float top_z = warp_max(real ? z : -FLT_MAX);
+        const float e = real ? expf(z - top_z) : 0.f;
+        s = e / warp_sum(e);
+    } else {
+        s = 1.0f / (1.0f + expf(-z));
+    }
+    float c = z;   // the choice score
+    if (groups.count > 0 && !(softmax_scores && !groups.correction && groups.best == 1))
+        c = groups.correction ? s + (real ? groups.correction[lane] : 0.f) : s;
+    bool allowed = real;
+    if (groups.count > 1 && groups.keep < groups.count) {
+        const int size = n_experts / groups.count, g = lane / size;
+        float first = -FLT_MAX, second = -FLT_MAX;
+        for (int i = 0; i < size; ++i) {
+            const float x = __shfl_sync(0xffffffffu, c, (g * size + i) & 31);
+            second = fmaxf(second, fminf(first, x));
+            first = fmaxf(first, x);
+        }
+        const float score = size > 1 && groups.best > 1 ? first + second : first;
+        int better = 0;
+        for (int o = 0; o < groups.count; ++o) {
+            const float x = __shfl_sync(0xffffffffu, score, o * size);
+            better += x > score || (x == score && o < g);
+        }
+        allowed = real && better < groups.keep;
+    }
+    const unsigned open = __ballot_sync(0xffffffffu, allowed);
+    int rank = 0;
+    for (int j = 0; j < n_experts; ++j) {
+        const float x = __shfl_sync(0xffffffffu, c, j);
+        rank += ((open >> j) & 1u) && (x > c || (x == c && j < lane));
+    }
+    const bool chosen = allowed && rank < top;
+    weight = renormalize ? s / warp_sum(chosen ? s : 0.f) : s;
+    return chosen ? rank : -1;
+}
+
+// Rows and tiles of up to 32 experts from their row counts: lane e gets its expert's first row and first tile; the totals in every lane.
+__device__ __forceinline__ void moe_scan_warp(int count, int tile_rows, int& row, int& tile, int& rows, int& tiles) {
+    const int lane = threadIdx.x & 31, t = (count + tile_rows - 1) / tile_rows;
+    int r_sum = count, t_sum = t;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, r_sum, o), b = __shfl_up_sync(0xffffffffu, t_sum, o);
+        if (lane >= o) {
+            r_sum += a;
+            t_sum += b;
+        }
+    }
+    row = r_sum - count;
+    tile = t_sum - t;
+    rows = __shfl_sync(0xffffffffu, r_sum, 31);
+    tiles = __shfl_sync(0xffffffffu, t_sum, 31);
+}
+
 // Scratch in pair order (pair = token * top + k): pair_expert, pair_weight. Results: dest [pairs] (the row of every pair),
 // and in row order sorted_token [pairs], sorted_weight float32 [pairs]; offsets [experts + 1]; tile_group, tile_row0
 // [max_tiles]; n_tiles [1].
 __global__ void __launch_bounds__(MOE_PLAN_THREADS)
 moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int softmax_scores, int renormalize,
-                int* __restrict__ pair_expert, float* __restrict__ pair_weight, int* __restrict__ sorted_token,
-                float* __restrict__ sorted_weight, int* __restrict__ dest, int* __restrict__ offsets,
+                int* pair_expert, float* pair_weight, int* __restrict__ sorted_token,
+                float* __restrict__ sorted_weight, int* dest, int* __restrict__ offsets,
                 int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ n_tiles, int max_tiles,
                 int tile_rows, const void* __restrict__ x, const void* __restrict__ router, int width, int x_is_bf16,
                 const float* __restrict__ bias, MoeGroups groups) {
@@ -195,20 +259,51 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
     }
     __syncthreads();
     // pass 1: choose, and take a rank among the expert's rows
-    for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
-        int chosen[MOE_MAX_TOP];
-        float weight[MOE_MAX_TOP];
-        if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, groups, chosen, weight);
-        else moe_choose(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, chosen, weight);
-        for (int k = 0; k < top; ++k) {
-            const int pair = t * top + k;
-            pair_expert[pair] = chosen[k];
-            dest[pair] = atomicAdd(&counts[chosen[k]], 1);        // for now: the pair's rank among its expert's rows
-            pair_weight[pair] = weight[k];
+    if (n_experts <= 32) {   // a warp per token
+        const int lane = threadIdx.x & 31;
+        for (int t = threadIdx.x >> 5; t < n_tokens; t += blockDim.x >> 5) {
+            const float z = lane < n_experts ? logits[(size_t)t * n_experts + lane] + (bias ? bias[lane] : 0.f) : 0.f;
+            float weight;
+            const int k = moe_choose_warp(z, n_experts, top, softmax_scores, renormalize, groups, weight);
+            if (k >= 0) {
+                const int pair = t * top + k;
+                pair_expert[pair] = lane;
+                dest[pair] = atomicAdd(&counts[lane], 1);        // for now: the pair's rank among its expert's rows
+                pair_weight[pair] = weight;
+            }
+        }
+    } else {
+        for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
+            int chosen[MOE_MAX_TOP];
+            float weight[MOE_MAX_TOP];
+            if (groups.count > 0) moe_choose_grouped(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, groups, chosen, weight);
+            else moe_choose(logits + (size_t)t * n_experts, bias, n_experts, top, softmax_scores, renormalize, chosen, weight);
+            for (int k = 0; k < top; ++k) {
+                const int pair = t * top + k;
+                pair_expert[pair] = chosen[k];
+                dest[pair] = atomicAdd(&counts[chosen[k]], 1);
+                pair_weight[pair] = weight[k];
+            }
         }
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
+    if (n_experts <= 32) {
+        if (threadIdx.x < 32) {
+            const int lane = threadIdx.x;
+            int row, tile, rows, tiles;
+            moe_scan_warp(lane < n_experts ? counts[lane] : 0, tile_rows, row, tile, rows, tiles);
+            if (lane < n_experts) {
+                offsets[lane] = row;
+                counts[lane] = row;
+                first_tile[lane] = tile;
+            }
+            if (lane == 0) {
+                offsets[n_experts] = rows;
+                first_tile[n_experts] = tiles;
+                n_tiles[0] = tiles < max_tiles ? tiles : max_tiles;
+            }
+        }
+    } else if (threadIdx.x == 0) {
         int row = 0, tile = 0;
         for (int e = 0; e < n_experts; ++e) {
             const int n = counts[e];
@@ -230,15 +325,12 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
             tile_row0[i] = row0 + (i - first_tile[e]) * tile_rows;
         }
     }
-    // pass 2: every pair's row (each thread finishes the pairs it made itself)
-    for (int t = threadIdx.x; t < n_tokens; t += blockDim.x) {
-        for (int k = 0; k < top; ++k) {
-            const int pair = t * top + k;
-            const int row = counts[pair_expert[pair]] + dest[pair];
-            dest[pair] = row;
-            sorted_token[row] = t;
-            sorted_weight[row] = pair_weight[pair];
-        }
+    // pass 2: every pair's row
+    for (int pair = threadIdx.x; pair < n_tokens * top; pair += blockDim.x) {
+        const int row = counts[pair_expert[pair]] + dest[pair];
+        dest[pair] = row;
+        sorted_token[row] = pair / top;
+        sorted_weight[row] = pair_weight[pair];
     }
 }
 
@@ -273,6 +365,81 @@ moe_route_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, 
             dest[pair] = base[chosen[k]] + rank[k];
             pair_weight[pair] = weight[k];
         }
+}
+
+// (1) by a warp per token, up to 32 experts; a block takes ROUTE_TOKENS tokens.
+#define ROUTE_TOKENS 16
+__global__ void __launch_bounds__(256)
+moe_route_warp_kernel(const float* __restrict__ logits, int n_tokens, int n_experts, int top, int softmax_scores, int renormalize,
+                      int* __restrict__ pair_expert, float* __restrict__ pair_weight, int* __restrict__ dest,
+                      int* __restrict__ expert_rows, const float* __restrict__ bias, MoeGroups groups) {
+    grid_chain_entry();
+    __shared__ int counts[32], base[32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (threadIdx.x < 32) counts[threadIdx.x] = 0;
+    __syncthreads();
+    constexpr int EACH = ROUTE_TOKENS / 8;
+    int place[EACH], rank[EACH];
+    float z[EACH], weight[EACH];
+#pragma unroll
+    for (int u = 0; u < EACH; ++u) {
+        const int t = blockIdx.x * ROUTE_TOKENS + warp * EACH + u;
+        z[u] = t < n_tokens && lane < n_experts ? logits[(size_t)t * n_experts + lane] + (bias ? bias[lane] : 0.f) : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < EACH; ++u) {
+        place[u] = moe_choose_warp(z[u], n_experts, top, softmax_scores, renormalize, groups, weight[u]);
+        if (blockIdx.x * ROUTE_TOKENS + warp * EACH + u >= n_tokens) place[u] = -1;
+        rank[u] = place[u] >= 0 ? atomicAdd(&counts[lane], 1) : 0;
+    }
+    __syncthreads();
+    if (threadIdx.x < n_experts) base[threadIdx.x] = counts[threadIdx.x] > 0 ? atomicAdd(&expert_rows[threadIdx.x], counts[threadIdx.x]) : 0;
+    __syncthreads();
+#pragma unroll
+    for (int u = 0; u < EACH; ++u) {
+        if (place[u] < 0) continue;
+        const int pair = (blockIdx.x * ROUTE_TOKENS + warp * EACH + u) * top + place[u];
+        pair_expert[pair] = lane;
+        dest[pair] = base[lane] + rank[u];
+        pair_weight[pair] = weight[u];
+    }
+}
+
+// (2) and (3) in one launch for up to 32 experts: every block works the experts' first rows out for itself, the first one also writes
+// the offsets and the tiles.
+__global__ void __launch_bounds__(256)
+moe_place_warp_kernel(const int* __restrict__ pair_expert, const float* __restrict__ pair_weight, const int* __restrict__ expert_rows,
+                      int n_experts, int* __restrict__ offsets, int* __restrict__ tile_group, int* __restrict__ tile_row0,
+                      int* __restrict__ n_tiles, int max_tiles, int tile_rows, int* __restrict__ dest, int* __restrict__ sorted_token,
+                      float* __restrict__ sorted_weight, int pairs, int top) {
+    grid_chain_entry();
+    __shared__ int first[32];
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x, n = lane < n_experts ? expert_rows[lane] : 0;
+        int row, tile, rows, tiles;
+        moe_scan_warp(n, tile_rows, row, tile, rows, tiles);
+        first[lane] = row;
+        if (blockIdx.x == 0) {
+            if (lane < n_experts) {
+                offsets[lane] = row;
+                for (int i = 0; i * tile_rows < n && tile + i < max_tiles; ++i) {
+                    tile_group[tile + i] = lane;
+                    tile_row0[tile + i] = row + i * tile_rows;
+                }
+            }
+            if (lane == 0) {
+                offsets[n_experts] = rows;
+                n_tiles[0] = tiles < max_tiles ? tiles : max_tiles;
+            }
+        }
+    }
+    __syncthreads();
+    const int pair = blockIdx.x * blockDim.x + threadIdx.x;
+    if (pair >= pairs) return;
+    const int row = first[pair_expert[pair]] + dest[pair];
+    dest[pair] = row;
+    sorted_token[row] = pair / top;
+    sorted_weight[row] = pair_weight[pair];
 }
 
 __global__ void __launch_bounds__(256)
@@ -495,7 +662,7 @@ QF_EXPORT int qf_moe_combine(int is_bf16, const void* y, const int* dest, const 
                                  nullptr, 0, stream);
 }
 
-// The plan of a long step by three launches (see moe_route_kernel). expert_rows: int32 [n_experts], zero before the call.
+// The plan of a long step by three launches (see moe_route_kernel), or two for up to 32 experts. expert_rows: int32 [n_experts], zero before the call.
 QF_EXPORT int qf_moe_plan_long_grouped(const float* logits, int n_tokens, int n_experts, int top, int softmax_scores,
                                        int renormalize, int* pair_expert, float* pair_weight, int* sorted_token,
                                        float* sorted_weight, int* dest, int* offsets, int* tile_group, int* tile_row0, int* n_tiles,
@@ -508,6 +675,15 @@ QF_EXPORT int qf_moe_plan_long_grouped(const float* logits, int n_tokens, int n_
     const MoeGroups groups = {correction, group_count, group_keep, group_best};
     if (top < 1 || top > MOE_MAX_TOP || top > n_experts || n_experts > 4096 || tile_rows <= 0 || !logits || !expert_rows)
         return (int)cudaErrorInvalidValue;
+    const int pairs = n_tokens * top;
+    if (n_experts <= 32) {
+        int code = (int)launch_pdl(moe_route_warp_kernel, dim3((n_tokens + ROUTE_TOKENS - 1) / ROUTE_TOKENS), dim3(256), 0, stream, logits, n_tokens,
+                                   n_experts, top, softmax_scores, renormalize, pair_expert, pair_weight, dest, expert_rows, bias, groups);
+        if (code) return code;
+        return (int)launch_pdl(moe_place_warp_kernel, dim3((pairs + 255) / 256), dim3(256), 0, stream, (const int*)pair_expert,
+                               (const float*)pair_weight, (const int*)expert_rows, n_experts, offsets, tile_group, tile_row0, n_tiles, max_tiles,
+                               tile_rows, dest, sorted_token, sorted_weight, pairs, top);
+    }
     const size_t smem = (size_t)(2 * n_experts + 1) * sizeof(int);
     int code = (int)launch_pdl(moe_route_kernel, dim3((n_tokens + 255) / 256), dim3(256), smem, stream, logits, n_tokens, n_experts,
                                top, softmax_scores, renormalize, pair_expert, pair_weight, dest, expert_rows, bias, groups);
@@ -515,7 +691,6 @@ QF_EXPORT int qf_moe_plan_long_grouped(const float* logits, int n_tokens, int n_
     code = (int)launch_pdl(moe_offsets_kernel, dim3(1), dim3(256), smem, stream, (const int*)expert_rows, n_experts, offsets,
                            tile_group, tile_row0, n_tiles, max_tiles, tile_rows);
     if (code) return code;
-    const int pairs = n_tokens * top;
     return (int)launch_pdl(moe_place_kernel, dim3((pairs + 255) / 256), dim3(256), 0, stream, (const int*)pair_expert,
                            (const float*)pair_weight, (const int*)offsets, dest, sorted_token, sorted_weight, pairs, top);
 }

@@ -711,71 +711,92 @@ QF_EXPORT int qf_rows_prepare(int is_bf16, void* x, int ld, int rows, int n_runs
 //   hidden += (a + b) (each if given);  r = 1 / sqrt(mean(hidden^2) + eps);  out1 = hidden * r1 * w1;  out2 = hidden * r2 * w2
 // (either norm, or both, may be left out). b may be unsummed expert rows: with `dest`, row t of b is the sum of the `top` rows
 // b[dest[t * top + k]] (each times row_weight[that row], if given) in the order of k. With `rows`, output row i is the norm of
-// stream row rows[i] and the stream is left as it is (what an output head reads). Float32 inside. A TEAM of threads works on a
-// row (a warp for rows of up to 1,024 columns, a block beyond) and keeps up to KEEP groups of four columns per thread; which one,
-// and the order of its additions, depends on the width alone.
-#define PN_MAX_TOP 16
-template <typename T, int TEAM, int KEEP>
-__global__ void __launch_bounds__(256)
+// stream row rows[i] and the stream is left as it is (what an output head reads). Float32 inside. A block works on a row and keeps up
+// to KEEP groups of four columns per thread; its size, and with it the order of its additions, depends on the width alone.
+// SUM: how many expert rows are summed (0: none, b is a plain output or absent; -1: any number, by a loop), known when the kernel is
+// chosen, so that a thread's loads of the stream, of a, of all of b's rows and of both weights are few and all on their way together.
+// The weights, which no kernel before this one writes, are asked for before the wait for it.
+template <typename T, int THREADS, int KEEP, int SUM>
+__global__ void __launch_bounds__(THREADS)
 pair_rms_norm_kernel(float* __restrict__ hidden, const T* __restrict__ a, const T* __restrict__ b, const int* __restrict__ dest, int top,
                      const float* __restrict__ row_weight, const T* __restrict__ w1, float eps1, T* __restrict__ out1,
-                     const T* __restrict__ w2, float eps2, T* __restrict__ out2, const int* __restrict__ rows, int n_out, int n_in,
-                     int width, int* err) {
-    grid_chain_entry();
+                     const T* __restrict__ w2, float eps2, T* __restrict__ out2, const int* __restrict__ rows, int n_in, int width, int* err) {
+    grid_launch_dependents();
     __shared__ float scratch[33];
-    const int lane = threadIdx.x % TEAM, team = threadIdx.x / TEAM;
-    const int i = blockIdx.x * (blockDim.x / TEAM) + team;
-    if (i >= n_out) return;   // (a block-wide team has a row of its own: all its threads leave together)
+    const int i = blockIdx.x, n4 = width / 4;
+    float4 g1[KEEP], g2[KEEP];
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+        const int c = threadIdx.x + THREADS * u;
+        g1[u] = w1 && c < n4 ? Vec4<T>::load(w1 + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        g2[u] = w2 && c < n4 ? Vec4<T>::load(w2 + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    grid_dependency_wait();
     int t = rows ? rows[i] : i;
     if (t < 0 || t >= n_in) {
-        if (lane == 0) atomicOr(err, QF_ERR_ROW_RANGE);
+        if (threadIdx.x == 0) atomicOr(err, QF_ERR_ROW_RANGE);
         t = 0;
     }
-    const int n4 = width / 4;
     float* h = hidden + (size_t)t * width;
+    constexpr int NS = SUM > 0 ? SUM : 1;
+    int src[NS];
+    float w[NS];
+    if constexpr (SUM > 0) {
+#pragma unroll
+        for (int k = 0; k < NS; ++k) src[k] = dest[(size_t)t * SUM + k];
+    }
     float4 v[KEEP], add[KEEP];
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
-        const int c = lane + TEAM * u;
+        const int c = threadIdx.x + THREADS * u;
         v[u] = c < n4 ? Vec4<float>::load(h + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        add[u] = make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    if (b && dest) {   // the token's expert rows: their places and weights first, then four rows at a time, in their order
-        int src[PN_MAX_TOP];
-        float w[PN_MAX_TOP];
+    auto plus = [](float4& sum, float4 x, float f) {
+        sum.x += x.x * f;
+        sum.y += x.y * f;
+        sum.z += x.z * f;
+        sum.w += x.w * f;
+    };
+    if constexpr (SUM > 0) {   // in the order of k
+        float4 x[NS][KEEP];
 #pragma unroll
-        for (int k = 0; k < PN_MAX_TOP; ++k)
-            if (k < top) {
-                src[k] = dest[(size_t)t * top + k];
-                w[k] = row_weight ? row_weight[src[k]] : 1.f;
+        for (int k = 0; k < NS; ++k) {
+            w[k] = row_weight ? row_weight[src[k]] : 1.f;
+#pragma unroll
+            for (int u = 0; u < KEEP; ++u) {
+                const int c = threadIdx.x + THREADS * u;
+                x[k][u] = c < n4 ? Vec4<T>::load(b + (size_t)src[k] * width + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
-#pragma unroll
-        for (int k = 0; k < PN_MAX_TOP; ++k)
-            if (k < top) {
-                const T* y = b + (size_t)src[k] * width;
-#pragma unroll
-                for (int u = 0; u < KEEP; ++u) {
-                    const int c = lane + TEAM * u;
-                    if (c < n4) {
-                        const float4 x = Vec4<T>::load(y + 4 * c);
-                        add[u].x += x.x * w[k];
-                        add[u].y += x.y * w[k];
-                        add[u].z += x.z * w[k];
-                        add[u].w += x.w * w[k];
-                    }
-                }
-            }
-    } else if (b) {
+        }
 #pragma unroll
         for (int u = 0; u < KEEP; ++u) {
-            const int c = lane + TEAM * u;
-            if (c < n4) add[u] = Vec4<T>::load(b + (size_t)t * width + 4 * c);
+            add[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int k = 0; k < NS; ++k) plus(add[u], x[k][u], w[k]);
+        }
+    } else if constexpr (SUM < 0) {
+#pragma unroll
+        for (int u = 0; u < KEEP; ++u) add[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < top; ++k) {
+            const int r = dest[(size_t)t * top + k];
+            const float f = row_weight ? row_weight[r] : 1.f;
+#pragma unroll
+            for (int u = 0; u < KEEP; ++u) {
+                const int c = threadIdx.x + THREADS * u;
+                if (c < n4) plus(add[u], Vec4<T>::load(b + (size_t)r * width + 4 * c), f);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int u = 0; u < KEEP; ++u) {
+            const int c = threadIdx.x + THREADS * u;
+            add[u] = b && c < n4 ? Vec4<T>::load(b + (size_t)t * width + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
     float ss = 0.f;
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
-        const int c = lane + TEAM * u;
+        const int c = threadIdx.x + THREADS * u;
         if (c >= n4) continue;
         if (a) {
             const float4 x = Vec4<T>::load(a + (size_t)t * width + 4 * c);
@@ -788,20 +809,14 @@ pair_rms_norm_kernel(float* __restrict__ hidden, const T* __restrict__ a, const 
         ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
     }
     if (!w1 && !w2) return;
-    const float mean = (TEAM == 32 ? warp_sum(ss) : block_sum(ss, scratch)) / (float)width;
+    const float mean = block_sum(ss, scratch) / (float)width;
     const float r1 = 1.0f / sqrtf(mean + eps1), r2 = 1.0f / sqrtf(mean + eps2);
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
-        const int c = lane + TEAM * u;
+        const int c = threadIdx.x + THREADS * u;
         if (c >= n4) continue;
-        if (w1) {
-            const float4 w = Vec4<T>::load(w1 + 4 * c);
-            Vec4<T>::store(out1 + (size_t)i * width + 4 * c, make_float4(v[u].x * r1 * w.x, v[u].y * r1 * w.y, v[u].z * r1 * w.z, v[u].w * r1 * w.w));
-        }
-        if (w2) {
-            const float4 w = Vec4<T>::load(w2 + 4 * c);
-            Vec4<T>::store(out2 + (size_t)i * width + 4 * c, make_float4(v[u].x * r2 * w.x, v[u].y * r2 * w.y, v[u].z * r2 * w.z, v[u].w * r2 * w.w));
-        }
+        if (w1) Vec4<T>::store(out1 + (size_t)i * width + 4 * c, make_float4(v[u].x * r1 * g1[u].x, v[u].y * r1 * g1[u].y, v[u].z * r1 * g1[u].z, v[u].w * r1 * g1[u].w));
+        if (w2) Vec4<T>::store(out2 + (size_t)i * width + 4 * c, make_float4(v[u].x * r2 * g2[u].x, v[u].y * r2 * g2[u].y, v[u].z * r2 * g2[u].z, v[u].w * r2 * g2[u].w));
     }
 }
 
@@ -850,22 +865,31 @@ pair_rms_norm_any_kernel(float* __restrict__ hidden, const T* __restrict__ a, co
     }
 }
 
+template <typename T, int THREADS, int KEEP>
+static int pair_norm_launch_keep(float* hidden, const void* a, const void* b, const int* dest, int top, const float* row_weight, const void* w1,
+                                 float eps1, void* out1, const void* w2, float eps2, void* out2, const int* rows, int n_out, int n_in, int width,
+                                 int* err, cudaStream_t stream) {
+#define QF_PAIR(SUM)                                                                                                                       \
+    return (int)launch_pdl(pair_rms_norm_kernel<T, THREADS, KEEP, SUM>, dim3(n_out), dim3(THREADS), 0, stream, hidden, (const T*)a, (const T*)b, \
+                           dest, top, row_weight, (const T*)w1, eps1, (T*)out1, (const T*)w2, eps2, (T*)out2, rows, n_in, width, err)
+    if (!b || !dest) QF_PAIR(0);
+    if (top == 1) QF_PAIR(1);
+    if (top == 2) QF_PAIR(2);
+    if (top == 4) QF_PAIR(4);
+    QF_PAIR(-1);
+#undef QF_PAIR
+}
+
 template <typename T>
 static int pair_norm_launch(float* hidden, const void* a, const void* b, const int* dest, int top, const float* row_weight, const void* w1,
                             float eps1, void* out1, const void* w2, float eps2, void* out2, const int* rows, int n_out, int n_in, int width,
                             int* err, cudaStream_t stream) {
     if (n_out <= 0) return 0;
     const uintptr_t align = (uintptr_t)hidden | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out1 | (uintptr_t)out2;
-    if (width % 4 == 0 && width <= 4096 && align % 16 == 0 && top <= PN_MAX_TOP) {
-#define QF_PAIR_ARGS hidden, (const T*)a, (const T*)b, dest, top, row_weight, (const T*)w1, eps1, (T*)out1, (const T*)w2, eps2, (T*)out2, rows, \
-                     n_out, n_in, width, err
-        if (width <= 1024) {
-            const int per_block = n_out >= 2048 ? 8 : n_out >= 512 ? 2 : 1;
-            return (int)launch_pdl(pair_rms_norm_kernel<T, 32, 8>, dim3((n_out + per_block - 1) / per_block), dim3(32 * per_block), 0, stream, QF_PAIR_ARGS);
-        }
-        if (width <= 2048) return (int)launch_pdl(pair_rms_norm_kernel<T, 256, 2>, dim3(n_out), dim3(256), 0, stream, QF_PAIR_ARGS);
-        return (int)launch_pdl(pair_rms_norm_kernel<T, 256, 4>, dim3(n_out), dim3(256), 0, stream, QF_PAIR_ARGS);
-#undef QF_PAIR_ARGS
+    if (width % 4 == 0 && width <= 4096 && align % 16 == 0) {
+        if (width <= 1024) return pair_norm_launch_keep<T, 128, 2>(hidden, a, b, dest, top, row_weight, w1, eps1, out1, w2, eps2, out2, rows, n_out, n_in, width, err, stream);
+        if (width <= 2048) return pair_norm_launch_keep<T, 256, 2>(hidden, a, b, dest, top, row_weight, w1, eps1, out1, w2, eps2, out2, rows, n_out, n_in, width, err, stream);
+        return pair_norm_launch_keep<T, 256, 4>(hidden, a, b, dest, top, row_weight, w1, eps1, out1, w2, eps2, out2, rows, n_out, n_in, width, err, stream);
     }
     return (int)launch_pdl(pair_rms_norm_any_kernel<T>, dim3(n_out), dim3(256), 0, stream, hidden, (const T*)a, (const T*)b, dest, top, row_weight,
                            (const T*)w1, eps1, (T*)out1, (const T*)w2, eps2, (T*)out2, rows, n_in, width, err);
@@ -935,11 +959,46 @@ map_difference_kernel(const T* __restrict__ x, int pitch, float weight, float ep
     }
 }
 
+// The same for bfloat16 heads that are whole 16 bytes wide: LANES = vdim / 8 lanes (a power of two up to 32) per head.
+__global__ void __launch_bounds__(256)
+map_difference_vec_kernel(const bf16* __restrict__ x, int pitch, float weight, float eps, float gain, bf16* __restrict__ out, long long items, int vdim) {
+    grid_chain_entry();
+    const int lanes = vdim / 8, at = threadIdx.x % lanes;
+    const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
+    const bool live = item < items;
+    const bf16* a1 = x + (live ? item : 0) * 2 * pitch + 8 * at;
+    const uint4 p = *reinterpret_cast<const uint4*>(a1), q = *reinterpret_cast<const uint4*>(a1 + pitch);
+    const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&p);
+    const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(&q);
+    float v[8];
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(p2[e]), g = __bfloat1622float2(q2[e]);
+        v[2 * e] = f.x - weight * g.x;
+        v[2 * e + 1] = f.y - weight * g.y;
+        ss += v[2 * e] * v[2 * e] + v[2 * e + 1] * v[2 * e + 1];
+    }
+    for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = gain / sqrtf(ss / (float)vdim + eps);
+    uint4 r;
+    __nv_bfloat162* r2 = reinterpret_cast<__nv_bfloat162*>(&r);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) r2[e] = __floats2bfloat162_rn(v[2 * e] * inv, v[2 * e + 1] * inv);
+    if (live) *reinterpret_cast<uint4*>(out + item * vdim + 8 * at) = r;
+}
+
 QF_EXPORT int qf_map_difference(int is_bf16, const void* x, int pitch, float weight, float eps, float gain, void* out, int n_tokens, int heads,
                                 int vdim, cudaStream_t stream) {
     const long long items = (long long)n_tokens * heads;
     if (items <= 0) return 0;
     if (vdim <= 0 || vdim > 32 * MD_MAX || pitch < vdim) return (int)cudaErrorInvalidValue;
+    const int lanes = vdim / 8;
+    if (is_bf16 && vdim % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 && pitch % 8 == 0 && ((uintptr_t)x | (uintptr_t)out) % 16 == 0) {
+        const int threads = items * lanes >= 64 * 1024 ? 256 : 64;
+        return (int)launch_pdl(map_difference_vec_kernel, dim3((unsigned)((items * lanes + threads - 1) / threads)), dim3(threads), 0, stream,
+                               (const bf16*)x, pitch, weight, eps, gain, (bf16*)out, items, vdim);
+    }
     const int warps = items >= 4096 ? 8 : 2;
     const dim3 grid((unsigned)((items + warps - 1) / warps)), block(32 * warps);
     const bool pairs = vdim % 2 == 0 && pitch % 2 == 0 && ((uintptr_t)x | (uintptr_t)out) % 8 == 0;

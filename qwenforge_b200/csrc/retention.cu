@@ -21,7 +21,7 @@
 #include "mma.cuh"
 
 #define RT_CHUNK 64
-#define RT_THREADS 128
+#define RT_THREADS 256
 #define RT_MAX_DIM 128
 #define RT_MAX_VDIM 128
 
@@ -176,44 +176,50 @@ retention_local_kernel(const bf16* __restrict__ k, int k_stride, const bf16* __r
 }
 
 // (2) The chain over a sequence's chunks: every chunk's record becomes the state BEFORE it, and the state after the last one goes
-// to the sequence's row. Four elements of S per thread; the records are read eight ahead.
-__global__ void __launch_bounds__(128)
+// to the sequence's row. Two elements of S per thread; the records are read sixteen ahead.
+#define RT_CARRY_THREADS 128
+__global__ void __launch_bounds__(RT_CARRY_THREADS)
 retention_carry_kernel(float* __restrict__ parts, const float* __restrict__ powers, const int* __restrict__ cu_q, const int* __restrict__ slots,
                        float* __restrict__ state, long long slot_stride, long long s_offset, int n_heads, int dim, int vdim) {
     grid_chain_entry();
     const int head = blockIdx.y, seq = blockIdx.z, size = dim * vdim;
-    const int at = (blockIdx.x * 128 + threadIdx.x) * 4;
+    const int at = (blockIdx.x * RT_CARRY_THREADS + threadIdx.x) * 2;
     const int len = cu_q[seq + 1] - cu_q[seq], slot = slots[seq];
     if (at >= size || len <= 0) return;
     const int chunks = (len + RT_CHUNK - 1) / RT_CHUNK;
     float* row = slot >= 0 ? state + slot * slot_stride + s_offset + (long long)head * size + at : nullptr;
-    float4 s = row ? *reinterpret_cast<const float4*>(row) : make_float4(0.f, 0.f, 0.f, 0.f);
+    float2 s = row ? *reinterpret_cast<const float2*>(row) : make_float2(0.f, 0.f);
     float* rec = parts + rt_record(cu_q, seq, 0, n_heads, head) * size + at;
     const long long pitch = (long long)n_heads * size;
     const float whole = powers[(size_t)head * (RT_CHUNK + 1) + RT_CHUNK];
     const float last = powers[(size_t)head * (RT_CHUNK + 1) + len - (chunks - 1) * RT_CHUNK];
-    constexpr int AHEAD = 8;
+    constexpr int AHEAD = 16;
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float4 own[AHEAD];
+        float2 own[AHEAD];
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u)
-            own[u] = c0 + u < chunks ? *reinterpret_cast<const float4*>(rec + (c0 + u) * pitch) : make_float4(0.f, 0.f, 0.f, 0.f);
+            own[u] = c0 + u < chunks ? *reinterpret_cast<const float2*>(rec + (c0 + u) * pitch) : make_float2(0.f, 0.f);
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
             if (c0 + u >= chunks) break;
-            *reinterpret_cast<float4*>(rec + (c0 + u) * pitch) = s;
+            *reinterpret_cast<float2*>(rec + (c0 + u) * pitch) = s;
             const float f = c0 + u == chunks - 1 ? last : whole;
-            s = make_float4(fmaf(f, s.x, own[u].x), fmaf(f, s.y, own[u].y), fmaf(f, s.z, own[u].z), fmaf(f, s.w, own[u].w));
+            s = make_float2(fmaf(f, s.x, own[u].x), fmaf(f, s.y, own[u].y));
         }
     }
-    if (row) *reinterpret_cast<float4*>(row) = s;
+    if (row) *reinterpret_cast<float2*>(row) = s;
 }
 
-// (3) A chunk's outputs. A warp owns 16 tokens; scores and outputs stay in its registers. First the part of the state before the
-// chunk (Q S0, S0 staged where the keys and values lie afterwards), then the scores under the decay and the causal mask, whose
-// accumulators are the left operand of the product with the values as they lie: accumulator column 2 q + e of eight tokens stands
-// for token 2 q + e, which the right operand's rows follow. Then the norm over a token's vdim components (four lanes hold a row), the
-// gate and the store. NV: eight-column tiles of the values that the registers hold.
+// (3) A chunk's outputs: the part of the state before it, Q S0 under the decay's powers, and the scores Q K^T under the decay and the
+// causal mask times the values; then the norm over a token's vdim components, the gate and the store. Warp w owns the 16 tokens
+// 16 (w % 4) onwards and one half (w / 4) of the value columns, whose sums stay in its registers; of the scores it makes every second
+// tile of eight keys, and the halves meet in shared memory, where S0 has been read by then. NV: eight-column tiles of the values
+// that a warp's registers hold.
+#define RT_PS (RT_CHUNK + 4)   // row stride of the scores in shared memory
+__host__ __device__ inline int rt_front(int dp, int vdim) {   // floats of the piece that holds S0 and then the scores
+    const int s0 = dp * rt_stride(vdim, 8);
+    return s0 > RT_CHUNK * RT_PS ? s0 : RT_CHUNK * RT_PS;
+}
 template <int NV>
 __global__ void __launch_bounds__(RT_THREADS)
 retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k, int k_stride, const bf16* __restrict__ v, int v_stride,
@@ -222,43 +228,55 @@ retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
                      const float* __restrict__ parts, bf16* __restrict__ out) {
     grid_chain_entry();
     extern __shared__ __align__(16) float rt_smem[];
+    __shared__ float norm_s[2][RT_CHUNK];
     const int head = blockIdx.y, seq = blockIdx.z;
     const int begin = cu_q[seq] + blockIdx.x * RT_CHUNK, end = cu_q[seq + 1];
     if (begin >= end) return;
     const int n = min(RT_CHUNK, end - begin), dp = rt_padded(dim);
-    const int qs = rt_stride(dp, 4), ss = rt_stride(vdim, 8), vs = rt_stride(vdim, 4);
-    float* q_s = rt_smem;                     // [RT_CHUNK][qs]
-    float* pow_s = q_s + RT_CHUNK * qs;       // [RT_CHUNK + 4]
-    float* s_s = pow_s + RT_CHUNK + 4;        // [dp][ss], then
-    float* k_s = s_s;                         // [RT_CHUNK][qs]
-    float* v_s = k_s + RT_CHUNK * qs;         // [RT_CHUNK][vs]
+    const int qs = rt_stride(dp, 4), ss = rt_stride(vdim, 8);
+    float* s_s = rt_smem;                     // [dp][ss], then the scores [RT_CHUNK][RT_PS]
+    float* q_s = s_s + rt_front(dp, vdim);    // [RT_CHUNK][qs]
+    float* k_s = q_s + RT_CHUNK * qs;         // [RT_CHUNK][qs]
+    float* v_s = k_s + RT_CHUNK * qs;         // [RT_CHUNK][ss]
+    float* pow_s = v_s + RT_CHUNK * ss;       // [RT_CHUNK + 1]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, r = lane >> 2, c4 = lane & 3;
     for (int i = threadIdx.x; i <= RT_CHUNK; i += RT_THREADS) pow_s[i] = powers[(size_t)head * (RT_CHUNK + 1) + i];
-    const float2* turn = angles + (size_t)begin * (rot_dim / 2);
-    stage_turned(q_s, qs, dp, q + (size_t)begin * q_stride + (size_t)head * dim, q_stride, n, dim, rot_dim, turn, 1.f, nullptr);
     {
         const float* s0 = parts + rt_record(cu_q, seq, blockIdx.x, n_heads, head) * dim * vdim;
         const int per_row = vdim / 4;
         for (int i = threadIdx.x; i < dp * per_row; i += RT_THREADS) {
             const int d = i / per_row, c = (i % per_row) * 4;
-            *reinterpret_cast<float4*>(s_s + (size_t)d * ss + c) =
-                d < dim ? *reinterpret_cast<const float4*>(s0 + (size_t)d * vdim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            cp_async_16(s_s + (size_t)d * ss + c, s0 + (d < dim ? (size_t)d * vdim + c : 0), d < dim);
         }
+        cp_async_commit();
     }
+    const float2* turn = angles + (size_t)begin * (rot_dim / 2);
+    stage_turned(q_s, qs, dp, q + (size_t)begin * q_stride + (size_t)head * dim, q_stride, n, dim, rot_dim, turn, 1.f, nullptr);
+    stage_turned(k_s, qs, dp, k + (size_t)begin * k_stride + (size_t)head * dim, k_stride, n, dim, rot_dim, turn, k_scale, nullptr);
+    stage_values(v_s, ss, v + (size_t)begin * v_stride + (size_t)head * vdim, v_stride, n, vdim);
+    cp_async_wait<0>();
     __syncthreads();
-    const int row0 = 16 * warp + r, row1 = row0 + 8;   // this lane's two tokens
-    const bool busy = 16 * warp < n;
-    float o[NV][4];
+    const int rows = warp & 3, half = warp >> 2;       // 16 tokens, and a half of the columns
+    const int row0 = 16 * rows + r, row1 = row0 + 8;   // this lane's two tokens
+    const int tiles = vdim / 8, first = half * ((tiles + 1) / 2), mine = half ? tiles - first : (tiles + 1) / 2, col0 = 8 * first;
+    const bool busy = 16 * rows < n;
+    float o[NV][4], s[4][4];
 #pragma unroll
     for (int t = 0; t < NV; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
+#pragma unroll
+    for (int t = 0; t < 4; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
     if (busy) {
         for (int d0 = 0; d0 < dp; d0 += 8) {
             const float* qa = q_s + (size_t)row0 * qs + d0 + c4;
             const Split a[4] = {split_tf32(qa[0]), split_tf32(qa[8 * qs]), split_tf32(qa[4]), split_tf32(qa[8 * qs + 4])};
-            const float* sb = s_s + (size_t)(d0 + c4) * ss + r;
+            const float* kb = k_s + (size_t)(8 * half + r) * qs + d0 + c4;
+#pragma unroll
+            for (int t = 0; t < 4; ++t)   // keys 16 t + 8 half onwards, up to this warp's own tokens
+                if (t <= rows) mma_split(s[t], a, split_tf32(kb[(size_t)16 * t * qs]), split_tf32(kb[(size_t)16 * t * qs + 4]));
+            const float* sb = s_s + (size_t)(d0 + c4) * ss + col0 + r;
 #pragma unroll
             for (int t = 0; t < NV; ++t)
-                if (8 * t < vdim) mma_split(o[t], a, split_tf32(sb[8 * t]), split_tf32(sb[4 * ss + 8 * t]));
+                if (t < mine) mma_split(o[t], a, split_tf32(sb[8 * t]), split_tf32(sb[4 * ss + 8 * t]));
         }
         const float f0 = pow_s[row0 + 1], f1 = pow_s[row1 + 1];
 #pragma unroll
@@ -269,59 +287,59 @@ retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
             o[t][3] *= f1;
         }
     }
-    __syncthreads();   // everyone has read S0: the keys and values take its place
-    stage_turned(k_s, qs, dp, k + (size_t)begin * k_stride + (size_t)head * dim, k_stride, n, dim, rot_dim, turn, k_scale, nullptr);
-    stage_values(v_s, vs, v + (size_t)begin * v_stride + (size_t)head * vdim, v_stride, n, vdim);
-    __syncthreads();
-    if (!busy) return;
-    const int last_tile = 2 * warp + 1;   // eight-token tiles of keys that this warp's tokens see: 0 .. last_tile
-    float s[8][4];
+    __syncthreads();   // everyone has read S0: the scores take its place
+    float* p_s = s_s;
+    if (busy) {
 #pragma unroll
-    for (int t = 0; t < 8; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
-    for (int d0 = 0; d0 < dp; d0 += 8) {
-        const float* qa = q_s + (size_t)row0 * qs + d0 + c4;
-        const Split a[4] = {split_tf32(qa[0]), split_tf32(qa[8 * qs]), split_tf32(qa[4]), split_tf32(qa[8 * qs + 4])};
-        const float* kb = k_s + (size_t)r * qs + d0 + c4;
+        for (int t = 0; t < 4; ++t) {
+            if (t > rows) continue;
+            const int j = 16 * t + 8 * half + 2 * c4;
 #pragma unroll
-        for (int t = 0; t < 8; ++t)
-            if (t <= last_tile) mma_split(s[t], a, split_tf32(kb[(size_t)8 * t * qs]), split_tf32(kb[(size_t)8 * t * qs + 4]));
-    }
-#pragma unroll
-    for (int t = 0; t < 8; ++t) {
-        if (t > last_tile) continue;
-        Split a[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? row0 : row1, j = 8 * t + 2 * c4 + (e & 1);
-            s[t][e] = i >= j ? s[t][e] * pow_s[i >= j ? i - j : 0] : 0.f;
+            for (int e = 0; e < 4; ++e) {
+                const int back = (e < 2 ? row0 : row1) - j - (e & 1);
+                s[t][e] = back >= 0 ? s[t][e] * pow_s[back >= 0 ? back : 0] : 0.f;
+            }
+            *reinterpret_cast<float2*>(p_s + row0 * RT_PS + j) = make_float2(s[t][0], s[t][1]);
+            *reinterpret_cast<float2*>(p_s + row1 * RT_PS + j) = make_float2(s[t][2], s[t][3]);
         }
-        a[0] = split_tf32(s[t][0]);
-        a[1] = split_tf32(s[t][2]);
-        a[2] = split_tf32(s[t][1]);
-        a[3] = split_tf32(s[t][3]);
-        const float* vb = v_s + (size_t)(8 * t + 2 * c4) * vs + r;
-#pragma unroll
-        for (int u = 0; u < NV; ++u)
-            if (8 * u < vdim) mma_half_split(o[u], a, vb[8 * u], vb[vs + 8 * u]);
     }
+    __syncthreads();
     float sum[2] = {0.f, 0.f};
+    if (busy) {
+        for (int t = 0; t <= 2 * rows + 1; ++t) {
+            const float* pa = p_s + row0 * RT_PS + 8 * t + c4;
+            const Split a[4] = {split_tf32(pa[0]), split_tf32(pa[8 * RT_PS]), split_tf32(pa[4]), split_tf32(pa[8 * RT_PS + 4])};
+            const float* vb = v_s + (size_t)(8 * t + c4) * ss + col0 + r;
 #pragma unroll
-    for (int t = 0; t < NV; ++t) {
-        sum[0] = fmaf(o[t][0], o[t][0], fmaf(o[t][1], o[t][1], sum[0]));
-        sum[1] = fmaf(o[t][2], o[t][2], fmaf(o[t][3], o[t][3], sum[1]));
+            for (int u = 0; u < NV; ++u)
+                if (u < mine) mma_half_split(o[u], a, vb[8 * u], vb[4 * ss + 8 * u]);
+        }
+#pragma unroll
+        for (int t = 0; t < NV; ++t) {
+            sum[0] = fmaf(o[t][0], o[t][0], fmaf(o[t][1], o[t][1], sum[0]));
+            sum[1] = fmaf(o[t][2], o[t][2], fmaf(o[t][3], o[t][3], sum[1]));
+        }
     }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
         sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+    }
+    if (c4 == 0) {
+        norm_s[half][row0] = sum[0];
+        norm_s[half][row1] = sum[1];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
         const int row = i ? row1 : row0;
         if (row >= n) continue;
-        const float inv = 1.0f / sqrtf(sum[i] / (float)vdim + eps);
-        const bf16* g = gate + (size_t)(begin + row) * gate_stride + (size_t)head * vdim + 2 * c4;
-        bf16* dst = out + (size_t)(begin + row) * n_heads * vdim + (size_t)head * vdim + 2 * c4;
+        const float inv = 1.0f / sqrtf((norm_s[0][row] + norm_s[1][row]) / (float)vdim + eps);
+        const bf16* g = gate + (size_t)(begin + row) * gate_stride + (size_t)head * vdim + col0 + 2 * c4;
+        bf16* dst = out + (size_t)(begin + row) * n_heads * vdim + (size_t)head * vdim + col0 + 2 * c4;
 #pragma unroll
         for (int t = 0; t < NV; ++t) {
-            if (8 * t >= vdim) continue;
+            if (t >= mine) continue;
             const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g + 8 * t));
             const float y0 = o[t][2 * i] * inv * (z.x / (1.f + expf(-z.x))), y1 = o[t][2 * i + 1] * inv * (z.y / (1.f + expf(-z.y)));
             *reinterpret_cast<__nv_bfloat162*>(dst + 8 * t) = __floats2bfloat162_rn(y0, y1);
@@ -356,12 +374,11 @@ QF_EXPORT int qf_retention_chunks(const void* q, int q_stride, const void* k, in
     e = launch_pdl(retention_local_kernel, grid, block, local_smem, stream, (const bf16*)k, k_stride, (const bf16*)v, v_stride,
                    (const float2*)angles, rot_dim, powers, k_scale, cu_q, n_heads, dim, vdim, parts);
     if (e != cudaSuccess) return (int)e;
-    e = launch_pdl(retention_carry_kernel, dim3((dim * vdim / 4 + 127) / 128, n_heads, n_seqs), dim3(128), 0, stream, parts, powers, cu_q, slots,
+    const int pairs = dim * vdim / 2;
+    e = launch_pdl(retention_carry_kernel, dim3((pairs + RT_CARRY_THREADS - 1) / RT_CARRY_THREADS, n_heads, n_seqs), dim3(RT_CARRY_THREADS), 0, stream, parts, powers, cu_q, slots,
                    state, slot_stride, s_offset, n_heads, dim, vdim);
     if (e != cudaSuccess) return (int)e;
-    const int qs = rt_stride(dp, 4);
-    const int front = dp * rt_stride(vdim, 8), back = RT_CHUNK * (qs + rt_stride(vdim, 4));
-    const size_t out_smem = (size_t)(RT_CHUNK * qs + RT_CHUNK + 4 + (front > back ? front : back)) * sizeof(float);
+    const size_t out_smem = (size_t)(rt_front(dp, vdim) + RT_CHUNK * (2 * rt_stride(dp, 4) + rt_stride(vdim, 8)) + RT_CHUNK + 1) * sizeof(float);
 #define QF_RETENTION(NV)                                                                                                              \
     {                                                                                                                                 \
         e = cudaFuncSetAttribute(retention_out_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem);              \
@@ -370,9 +387,9 @@ QF_EXPORT int qf_retention_chunks(const void* q, int q_stride, const void* k, in
                                (const bf16*)v, v_stride, (const bf16*)gate, gate_stride, (const float2*)angles, rot_dim, powers, k_scale, eps, \
                                cu_q, n_heads, dim, vdim, (const float*)parts, (bf16*)out);                                            \
     }
-    if (vdim <= 32) QF_RETENTION(4)
-    if (vdim <= 64) QF_RETENTION(8)
-    QF_RETENTION(16)
+    if (vdim <= 32) QF_RETENTION(2)
+    if (vdim <= 64) QF_RETENTION(4)
+    QF_RETENTION(8)
 #undef QF_RETENTION
 }
 

@@ -1365,7 +1365,7 @@ def _grouped(x, weight, out, a_group_cols, c_group_cols, rows, plan, a_rows=None
         _ptr(plan.tile_group if plan else None), _ptr(plan.tile_row0 if plan else None), _ptr(plan.offsets if plan else None),
         _ptr(plan.n_tiles if plan else None), _I(plan.max_tiles if plan else 0), _I(plan.tile_rows if plan else 0),
         _ptr(a_rows), _I(int(gated)), _ptr(row_scale), _F(limit), _F(alpha), _I(0 if activation is None else ACTIVATIONS[activation] + 1),
-        _stream())
+        _I(plan.n_tokens if plan else 0), _stream())   # (a token chooses an expert at most once)
     if code == 1:
         raise KernelError("grouped_gemm: the plan's tiles do not fit these operands (tiles of 128 rows need bfloat16 operands "
                           "whose K and strides are multiples of 8), or the grid is too large")
