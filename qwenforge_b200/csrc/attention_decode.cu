@@ -24,6 +24,9 @@
 // page is fetched once and read as both.
 // `bias_scale`, `bias_rate` (float32 per query head, or null): after the cap a score of the key `far` positions back loses
 // bias_scale[h] * ln(1 + bias_rate[h] * far), with the hardware's base-2 logarithm; compiled as a variant of its own.
+// `pairs`: query heads 2 i and 2 i + 1 are the two maps of one head of a differential attention. The output row then holds half as
+// many heads of pairs.width components, o / sqrt(mean(o^2) + eps) * gain with o = first - weight * second, formed from the float32
+// results where a row's runs come together; a variant of its own, not with sinks or fold_later.
 #include <algorithm>
 
 #include "tma.cuh"
@@ -105,14 +108,19 @@ decode_plan_kernel(const int* __restrict__ cu_q, const int* __restrict__ tok_pos
     for (int j = before + lane; j < n_pairs; j += 32) plan[j] = make_int4(-1, 0, 0, -1);
 }
 
-template <int D, int WARPS, bool TMA, bool BIASED>
+struct PairArgs {
+    float weight, eps, gain;
+    int width;
+};
+
+template <int D, int WARPS, bool TMA, bool BIASED, bool PAIRED>
 __global__ void __launch_bounds__(WARPS * 32)
 decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __restrict__ q, bf16* __restrict__ out,
                     const int* __restrict__ cu_q, const int4* __restrict__ plan, KvSite<bf16> site, int n_heads, int chunks, float scale_log2,
                     int window, int mask_block, float cap_in, float cap_out, int max_splits, int n_seqs, int fold_later, float* __restrict__ part_o,
                     float* __restrict__ part_ml, int* __restrict__ counters, int* err, unsigned long long* stamps,
                     const float* __restrict__ sinks, int shared_values, const float* __restrict__ bias_scale,
-                    const float* __restrict__ bias_rate) {
+                    const float* __restrict__ bias_rate, PairArgs pairs) {
     constexpr int DEC_WARPS = WARPS, DEC_THREADS = WARPS * 32;
     // measuring aid: if `stamps` is given, thread 0 leaves nanosecond time stamps of the block's phases in stamps[block][8]
     auto stamp = [&](int phase) {
@@ -152,12 +160,28 @@ decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __re
     const int tok = cu_q[seq];
     const int slot = record.w;
     const int q_width = n_heads * D;
-    bf16* out_row = out + (size_t)tok * q_width + (size_t)head0 * D;
+    bf16* out_row = PAIRED ? out + ((size_t)tok * n_heads + head0) / 2 * pairs.width : out + (size_t)tok * q_width + (size_t)head0 * D;
+    // both maps of a pair of rows to its one output row, a warp per pair; value(r, d): row r's attended component d, float32
+    auto bring_together = [&](auto value) {
+        for (int p = warp; p < n_g / 2; p += WARPS) {
+            float o[(D + 31) / 32], ss = 0.f;
+#pragma unroll
+            for (int u = 0; u < (D + 31) / 32; ++u) {
+                const int d = lane + 32 * u;
+                o[u] = d < pairs.width ? value(2 * p, d) - pairs.weight * value(2 * p + 1, d) : 0.f;
+                ss += o[u] * o[u];
+            }
+            const float inv = pairs.gain / sqrtf(warp_sum(ss) / (float)pairs.width + pairs.eps);
+#pragma unroll
+            for (int u = 0; u < (D + 31) / 32; ++u)
+                if (lane + 32 * u < pairs.width) out_row[(size_t)p * pairs.width + lane + 32 * u] = __float2bfloat16_rn(o[u] * inv);
+        }
+    };
 
     if (slot < 0) {  // padding entry: defined output (or a partial result that folds to zero), no cache access, no ticket
         grid_dependency_wait();
         if (split == 0 && !fold_later)
-            for (int i = threadIdx.x; i < n_g * D; i += DEC_THREADS) out_row[i] = __float2bfloat16_rn(0.f);
+            for (int i = threadIdx.x; i < (PAIRED ? n_g / 2 * pairs.width : n_g * D); i += DEC_THREADS) out_row[i] = __float2bfloat16_rn(0.f);
         if (split == 0 && fold_later && threadIdx.x < n_g) {
             float* ml = part_ml + (((size_t)seq * n_heads + head0 + threadIdx.x) * max_splits) * 2;
             ml[0] = QF_NEG_BIG;
@@ -442,6 +466,20 @@ decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __re
     stamp(5);
     // block result: row r: maximum max_w m_s[w][r], sum sum_w l_s[w][r], numerator sum_w (warp w's buffer)[r][:]
     const size_t part_row0 = ((size_t)seq * n_heads + head0) * max_splits;  // partial index of (row 0, split 0)
+    if constexpr (PAIRED) {
+        if (n_splits == 1) {
+            bring_together([&](int r, int d) -> float {
+                float num = 0.f, l = 0.f;
+#pragma unroll
+                for (int w = 0; w < DEC_WARPS; ++w) {
+                    num += reinterpret_cast<const float*>(smem_raw + (size_t)w * PAGE_BYTES)[r * OLD + d];
+                    l += l_s[w][r];
+                }
+                return l > 0.f ? num / l : 0.f;
+            });
+            return;
+        }
+    }
     for (int i = threadIdx.x; i < n_g * D; i += DEC_THREADS) {
         const int r = i / D, d = i % D;
         float num = 0.f;
@@ -559,11 +597,21 @@ decode_split_kernel(const __grid_constant__ CUtensorMap kv_map, const bf16* __re
                     den[x] = den[x] * keep + exp2f(s2 - m_new);
                 }
                 const float inv = den[x] > 0.f ? keep / den[x] : 0.f;
+                if constexpr (PAIRED) {   // float32, where every warp of the block finds both rows of its pairs
+                    const int i = i0 + x * DEC_THREADS;
+                    *reinterpret_cast<float4*>(reinterpret_cast<float*>(smem_raw) + i / D4 * OLD + i % D4 * 4) =
+                        make_float4(num[x].x * inv, num[x].y * inv, num[x].z * inv, num[x].w * inv);
+                    continue;
+                }
                 uint2 packed;
                 packed.x = pack_bf16(num[x].x * inv, num[x].y * inv);
                 packed.y = pack_bf16(num[x].z * inv, num[x].w * inv);
                 *reinterpret_cast<uint2*>(out_row + (size_t)(i0 + x * DEC_THREADS) * 4) = packed;
             }
+    }
+    if constexpr (PAIRED) {
+        __syncthreads();
+        bring_together([&](int r, int d) -> float { return reinterpret_cast<const float*>(smem_raw)[r * OLD + d]; });
     }
     stamp(7);
 }
@@ -582,7 +630,7 @@ template <int D>
 static int resident_blocks() {
     static int held = -1;
     if (held < 0) {
-        auto kernel = decode_split_kernel<D, decode_warps(D), decode_tma(D), false>;
+        auto kernel = decode_split_kernel<D, decode_warps(D), decode_tma(D), false, false>;
         int n = 0;
         if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem(D)) != cudaSuccess ||
             cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, kernel, decode_warps(D) * 32, decode_smem(D)) != cudaSuccess)
@@ -618,17 +666,17 @@ QF_EXPORT int qf_attention_decode_warps(int head_dim) {
     return head_dim == 32 || head_dim == 64 || head_dim == 96 || head_dim == 128 ? decode_warps(head_dim) : 0;
 }
 
-template <int D, bool BIASED>
+template <int D, bool BIASED, bool PAIRED>
 static int launch(const void* q, void* out, const int* cu_q, const int4* plan, void* base, const int* table,
                   long long page_elems, int table_stride, int kv_heads, int n_heads, int n_seqs, float scale, int window,
                   int n_splits, int fold_later, float* part_o, float* part_ml, int* counters, int* err,
                   unsigned long long* stamps, const float* sinks, int shared_values, int mask_block, float softcap,
-                  const float* bias_scale, const float* bias_rate, cudaStream_t stream) {
+                  const float* bias_scale, const float* bias_rate, PairArgs pairs, cudaStream_t stream) {
     constexpr int WARPS = decode_warps(D);
     constexpr bool TMA = decode_tma(D);
     const int G = n_heads / kv_heads, chunks = (G + 15) / 16;
     const size_t smem = decode_smem(D);
-    cudaError_t e = cudaFuncSetAttribute(decode_split_kernel<D, WARPS, TMA, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(decode_split_kernel<D, WARPS, TMA, BIASED, PAIRED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     KvSite<bf16> site{(bf16*)base, table, page_elems, table_stride, kv_heads, D};
     CUtensorMap kv_map = {};
@@ -638,10 +686,10 @@ static int launch(const void* q, void* out, const int* cu_q, const int4* plan, v
         if (!qf_make_map_bf16(&kv_map, base, 1ll << 31, D, D, QF_PAGE / 2)) return (int)cudaErrorNotSupported;
     }
     dim3 grid((unsigned)(plan_pairs(n_seqs, kv_heads, n_heads, D, n_splits) * kv_heads * chunks));
-    return (int)launch_pdl(decode_split_kernel<D, WARPS, TMA, BIASED>, grid, dim3(WARPS * 32), smem, stream, kv_map, (const bf16*)q,
+    return (int)launch_pdl(decode_split_kernel<D, WARPS, TMA, BIASED, PAIRED>, grid, dim3(WARPS * 32), smem, stream, kv_map, (const bf16*)q,
                            (bf16*)out, cu_q, plan, site, n_heads, chunks, scale * 1.4426950408889634f, window, mask_block,
                            softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, n_splits,
-                           n_seqs, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values, bias_scale, bias_rate);
+                           n_seqs, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values, bias_scale, bias_rate, pairs);
 }
 
 // How many 16-byte units a plan of this shape holds (what qf_attention_decode_plan writes and qf_attention_decode
@@ -679,16 +727,18 @@ static int decode_run(const void* q, void* out, const int* cu_q, const void* pla
                       long long page_elems, int table_stride, int kv_heads, int head_dim, int n_heads, int n_seqs,
                       float scale, int window, int n_splits, int fold_later, float* part_o, float* part_ml, int* counters,
                       int* err, unsigned long long* stamps, const float* sinks, int shared_values, cudaStream_t stream,
-                      int mask_block = 0, float softcap = 0.f, const float* bias_scale = nullptr, const float* bias_rate = nullptr) {
+                      int mask_block = 0, float softcap = 0.f, const float* bias_scale = nullptr, const float* bias_rate = nullptr, PairArgs pairs = {0.f, 0.f, 0.f, 0}) {
     if (n_seqs <= 0) return 0;
     if (kv_heads <= 0 || n_heads % kv_heads || n_splits < 1 || !plan || (fold_later && sinks)) return (int)cudaErrorInvalidValue;
+    if (pairs.width && (pairs.width < 0 || pairs.width > head_dim || (n_heads / kv_heads) % 2 || sinks || fold_later || bias_scale)) return (int)cudaErrorInvalidValue;
     if (fold_later ? (!part_o || !part_ml) : !out) return (int)cudaErrorInvalidValue;
 #define QF_DECODE_ARGS q, out, cu_q, (const int4*)plan, base, table, page_elems, table_stride, kv_heads, n_heads, n_seqs, scale, window, \
                        n_splits, fold_later, part_o, part_ml, counters, err, stamps, sinks, shared_values, mask_block, softcap,       \
-                       bias_scale, bias_rate, stream
-#define QF_CASE(DIM) \
-    case DIM:        \
-        return bias_scale ? launch<DIM, true>(QF_DECODE_ARGS) : launch<DIM, false>(QF_DECODE_ARGS);
+                       bias_scale, bias_rate, pairs, stream
+#define QF_CASE(DIM)                                                      \
+    case DIM:                                                             \
+        if (pairs.width) return launch<DIM, false, true>(QF_DECODE_ARGS); \
+        return bias_scale ? launch<DIM, true, false>(QF_DECODE_ARGS) : launch<DIM, false, false>(QF_DECODE_ARGS);
     switch (head_dim) {
         QF_CASE(32)
         QF_CASE(64)
@@ -743,6 +793,17 @@ QF_EXPORT int qf_attention_decode_biased(const void* q, void* out, const int* cu
     return decode_run(q, out, cu_q, plan, base, table, page_elems, table_stride, kv_heads, head_dim, n_heads, n_seqs, scale,
                       window, n_splits, fold_later, part_o, part_ml, counters, err, nullptr, sinks, shared_values, stream,
                       mask_block, softcap, bias_scale, bias_rate);
+}
+
+// And with the two maps of every head brought together: out [n_seqs][n_heads / 2 * width] (see `pairs` at the top of the file).
+QF_EXPORT int qf_attention_decode_paired(const void* q, void* out, const int* cu_q, const void* plan, void* base,
+                                         const int* table, long long page_elems, int table_stride, int kv_heads, int head_dim,
+                                         int n_heads, int n_seqs, float scale, int window, int n_splits, float* part_o, float* part_ml,
+                                         int* counters, int* err, float weight, float eps, float gain, int width, cudaStream_t stream) {
+    if (width <= 0) return (int)cudaErrorInvalidValue;
+    return decode_run(q, out, cu_q, plan, base, table, page_elems, table_stride, kv_heads, head_dim, n_heads, n_seqs, scale,
+                      window, n_splits, 0, part_o, part_ml, counters, err, nullptr, nullptr, 0, stream, 0, 0.f, nullptr, nullptr,
+                      PairArgs{weight, eps, gain, width});
 }
 
 // A measuring aid: the same launch, with every block's thread 0 writing nanosecond time stamps to stamps[block][8]:

@@ -16,8 +16,10 @@
 // in three launches: (1) every chunk's own part of S_n, all chunks at once; (2) the states before every chunk, a short chain of
 // one multiply-add per chunk and element of S; (3) every chunk's outputs, norm and gate, all chunks at once. No power of the decay
 // exceeds 1, so nothing has to be rescaled. The products run on the tensor cores as tf32 with float32 sums, every float32 operand
-// taken as the sum of two tf32 numbers (x = hi + lo to about 2^-22; hi hi + hi lo + lo hi), so they are float32 products to
+// taken as the sum of two tf32 numbers (x = hi + lo to about 2^-21; hi hi + hi lo + lo hi), so they are float32 products to
 // rounding; the values are bfloat16 numbers and need one.
+#include <type_traits>
+
 #include "mma.cuh"
 
 #define RT_CHUNK 64
@@ -25,18 +27,14 @@
 #define RT_MAX_DIM 128
 #define RT_MAX_VDIM 128
 
-__device__ __forceinline__ uint32_t to_tf32(float x) {
-    uint32_t y;
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(y) : "f"(x));
-    return y;
-}
 struct Split {
     uint32_t hi, lo;
 };
+// The leading eleven bits of x's significand, and the next eleven (both by cutting off: two logical operations and a subtraction).
 __device__ __forceinline__ Split split_tf32(float x) {
     Split s;
-    s.hi = to_tf32(x);
-    s.lo = to_tf32(x - __uint_as_float(s.hi));
+    s.hi = __float_as_uint(x) & 0xffffe000u;
+    s.lo = __float_as_uint(x - __uint_as_float(s.hi)) & 0xffffe000u;
     return s;
 }
 // D[16x8] += A[16x8] * B[8x8], tf32 operands, float32 accumulation.
@@ -59,8 +57,8 @@ __device__ __forceinline__ void mma_half_split(float (&d)[4], const Split (&a)[4
     mma_tf32(d, a[0].hi, a[1].hi, a[2].hi, a[3].hi, x0, x1);
 }
 
-__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {   // (through the read-only path: may run ahead of stores)
+    const uint4 raw = __ldg(reinterpret_cast<const uint4*>(p));
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -79,7 +77,8 @@ __device__ __forceinline__ void put8(float* p, const float (&v)[8]) {
 __device__ __forceinline__ void stage_turned(float* dst, int stride, int padded, const bf16* src, int src_stride, int n, int dim, int rot_dim,
                                              const float2* angles, float scale, const float* row_power) {
     const int half = rot_dim / 2, per_row = padded / 8;
-    for (int i = threadIdx.x; i < RT_CHUNK * per_row; i += blockDim.x) {
+#pragma unroll 2
+    for (int i = threadIdx.x; i < RT_CHUNK * per_row; i += RT_THREADS) {
         const int row = i / per_row, c = (i % per_row) * 8;
         float v[8];
 #pragma unroll
@@ -92,11 +91,13 @@ __device__ __forceinline__ void stage_turned(float* dst, int stride, int padded,
                 const int j = first ? c : c - half;
                 float other[8];
                 load8(p + (first ? c + half : c - half), other);
-                const float2* cs = angles + (size_t)row * half + j;
+                const float4* cs = reinterpret_cast<const float4*>(angles + (size_t)row * half + j);   // two pairs (cos, sin) each
+                const float sign = first ? -1.f : 1.f;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    const float2 a = cs[e];
-                    v[e] = first ? v[e] * a.x - other[e] * a.y : v[e] * a.x + other[e] * a.y;
+                for (int e = 0; e < 4; ++e) {
+                    const float4 a = __ldg(cs + e);
+                    v[2 * e] = fmaf(sign * other[2 * e], a.y, v[2 * e] * a.x);
+                    v[2 * e + 1] = fmaf(sign * other[2 * e + 1], a.w, v[2 * e + 1] * a.z);
                 }
             }
             const float f = row_power ? scale * row_power[n - 1 - row] : scale;
@@ -108,7 +109,8 @@ __device__ __forceinline__ void stage_turned(float* dst, int stride, int padded,
 }
 __device__ __forceinline__ void stage_values(float* dst, int stride, const bf16* src, int src_stride, int n, int vdim) {
     const int per_row = vdim / 8;
-    for (int i = threadIdx.x; i < RT_CHUNK * per_row; i += blockDim.x) {
+#pragma unroll 4
+    for (int i = threadIdx.x; i < RT_CHUNK * per_row; i += RT_THREADS) {
         const int row = i / per_row, c = (i % per_row) * 8;
         float v[8];
 #pragma unroll
@@ -214,14 +216,14 @@ retention_carry_kernel(float* __restrict__ parts, const float* __restrict__ powe
 // causal mask times the values; then the norm over a token's vdim components, the gate and the store. Warp w owns the 16 tokens
 // 16 (w % 4) onwards and one half (w / 4) of the value columns, whose sums stay in its registers; of the scores it makes every second
 // tile of eight keys, and the halves meet in shared memory, where S0 has been read by then. NV: eight-column tiles of the values
-// that a warp's registers hold.
+// that a warp's registers hold; FULL: both halves have all of them, so that no test stands between their loads and products.
 #define RT_PS (RT_CHUNK + 4)   // row stride of the scores in shared memory
 __host__ __device__ inline int rt_front(int dp, int vdim) {   // floats of the piece that holds S0 and then the scores
     const int s0 = dp * rt_stride(vdim, 8);
     return s0 > RT_CHUNK * RT_PS ? s0 : RT_CHUNK * RT_PS;
 }
-template <int NV>
-__global__ void __launch_bounds__(RT_THREADS)
+template <int NV, bool FULL>
+__global__ void __launch_bounds__(RT_THREADS, 2)
 retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k, int k_stride, const bf16* __restrict__ v, int v_stride,
                      const bf16* __restrict__ gate, int gate_stride, const float2* __restrict__ angles, int rot_dim,
                      const float* __restrict__ powers, float k_scale, float eps, const int* __restrict__ cu_q, int n_heads, int dim, int vdim,
@@ -265,18 +267,37 @@ retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
     for (int t = 0; t < NV; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
 #pragma unroll
     for (int t = 0; t < 4; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
-    if (busy) {
+    auto left = [&](int d0, Split (&a)[4]) {
+        const float* qa = q_s + (size_t)row0 * qs + d0 + c4;
+        a[0] = split_tf32(qa[0]);
+        a[1] = split_tf32(qa[8 * qs]);
+        a[2] = split_tf32(qa[4]);
+        a[3] = split_tf32(qa[8 * qs + 4]);
+    };
+    // keys 16 t + 8 half onwards, t up to this warp's own tokens
+    auto scores = [&](auto count) {
         for (int d0 = 0; d0 < dp; d0 += 8) {
-            const float* qa = q_s + (size_t)row0 * qs + d0 + c4;
-            const Split a[4] = {split_tf32(qa[0]), split_tf32(qa[8 * qs]), split_tf32(qa[4]), split_tf32(qa[8 * qs + 4])};
+            Split a[4];
+            left(d0, a);
             const float* kb = k_s + (size_t)(8 * half + r) * qs + d0 + c4;
 #pragma unroll
-            for (int t = 0; t < 4; ++t)   // keys 16 t + 8 half onwards, up to this warp's own tokens
-                if (t <= rows) mma_split(s[t], a, split_tf32(kb[(size_t)16 * t * qs]), split_tf32(kb[(size_t)16 * t * qs + 4]));
+            for (int t = 0; t < decltype(count)::value; ++t)
+                mma_split(s[t], a, split_tf32(kb[(size_t)16 * t * qs]), split_tf32(kb[(size_t)16 * t * qs + 4]));
+        }
+    };
+    if (busy) {
+        if (rows == 0) scores(std::integral_constant<int, 1>());
+        else if (rows == 1) scores(std::integral_constant<int, 2>());
+        else if (rows == 2) scores(std::integral_constant<int, 3>());
+        else scores(std::integral_constant<int, 4>());
+#pragma unroll 2
+        for (int d0 = 0; d0 < dp; d0 += 8) {
+            Split a[4];
+            left(d0, a);
             const float* sb = s_s + (size_t)(d0 + c4) * ss + col0 + r;
 #pragma unroll
             for (int t = 0; t < NV; ++t)
-                if (t < mine) mma_split(o[t], a, split_tf32(sb[8 * t]), split_tf32(sb[4 * ss + 8 * t]));
+                if (FULL || t < mine) mma_split(o[t], a, split_tf32(sb[8 * t]), split_tf32(sb[4 * ss + 8 * t]));
         }
         const float f0 = pow_s[row0 + 1], f1 = pow_s[row1 + 1];
 #pragma unroll
@@ -312,7 +333,7 @@ retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
             const float* vb = v_s + (size_t)(8 * t + c4) * ss + col0 + r;
 #pragma unroll
             for (int u = 0; u < NV; ++u)
-                if (u < mine) mma_half_split(o[u], a, vb[8 * u], vb[4 * ss + 8 * u]);
+                if (FULL || u < mine) mma_half_split(o[u], a, vb[8 * u], vb[4 * ss + 8 * u]);
         }
 #pragma unroll
         for (int t = 0; t < NV; ++t) {
@@ -329,19 +350,26 @@ retention_out_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
         norm_s[half][row0] = sum[0];
         norm_s[half][row1] = sum[1];
     }
+    uint32_t z_raw[2][NV];   // the gate's logits, on their way across the barrier
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int row = i ? row1 : row0;
+        const bf16* g = gate + (size_t)(begin + min(row, n - 1)) * gate_stride + (size_t)head * vdim + col0 + 2 * c4;
+#pragma unroll
+        for (int t = 0; t < NV; ++t) z_raw[i][t] = FULL || t < mine ? __ldg(reinterpret_cast<const unsigned*>(g + 8 * t)) : 0u;
+    }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         const int row = i ? row1 : row0;
         if (row >= n) continue;
         const float inv = 1.0f / sqrtf((norm_s[0][row] + norm_s[1][row]) / (float)vdim + eps);
-        const bf16* g = gate + (size_t)(begin + row) * gate_stride + (size_t)head * vdim + col0 + 2 * c4;
         bf16* dst = out + (size_t)(begin + row) * n_heads * vdim + (size_t)head * vdim + col0 + 2 * c4;
 #pragma unroll
         for (int t = 0; t < NV; ++t) {
-            if (t >= mine) continue;
-            const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g + 8 * t));
-            const float y0 = o[t][2 * i] * inv * (z.x / (1.f + expf(-z.x))), y1 = o[t][2 * i + 1] * inv * (z.y / (1.f + expf(-z.y)));
+            if (!FULL && t >= mine) continue;
+            const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&z_raw[i][t]));
+            const float y0 = o[t][2 * i] * inv * __fdividef(z.x, 1.f + expf(-z.x)), y1 = o[t][2 * i + 1] * inv * __fdividef(z.y, 1.f + expf(-z.y));
             *reinterpret_cast<__nv_bfloat162*>(dst + 8 * t) = __floats2bfloat162_rn(y0, y1);
         }
     }
@@ -381,9 +409,10 @@ QF_EXPORT int qf_retention_chunks(const void* q, int q_stride, const void* k, in
     const size_t out_smem = (size_t)(rt_front(dp, vdim) + RT_CHUNK * (2 * rt_stride(dp, 4) + rt_stride(vdim, 8)) + RT_CHUNK + 1) * sizeof(float);
 #define QF_RETENTION(NV)                                                                                                              \
     {                                                                                                                                 \
-        e = cudaFuncSetAttribute(retention_out_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem);              \
+        auto kernel = vdim == 16 * NV ? retention_out_kernel<NV, true> : retention_out_kernel<NV, false>;                            \
+        e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem);                                 \
         if (e != cudaSuccess) return (int)e;                                                                                          \
-        return (int)launch_pdl(retention_out_kernel<NV>, grid, block, out_smem, stream, (const bf16*)q, q_stride, (const bf16*)k, k_stride, \
+        return (int)launch_pdl(kernel, grid, block, out_smem, stream, (const bf16*)q, q_stride, (const bf16*)k, k_stride, \
                                (const bf16*)v, v_stride, (const bf16*)gate, gate_stride, (const float2*)angles, rot_dim, powers, k_scale, eps, \
                                cu_q, n_heads, dim, vdim, (const float*)parts, (bf16*)out);                                            \
     }
@@ -416,25 +445,47 @@ retention_token_kernel(const T* __restrict__ q, int q_stride, const T* __restric
     const int half = rot_dim / 2;
     const T* qh = q + (size_t)t * q_stride + (size_t)head * dim;
     const T* kh = k + (size_t)t * k_stride + (size_t)head * dim;
+    const int group = threadIdx.x % groups, r0 = threadIdx.x / groups;
+    float* S = slot >= 0 ? state + slot * slot_stride + s_offset + (long long)head * dim * vdim : nullptr;
+    constexpr int AHEAD = 8;
+    float s[AHEAD][COLS];   // rows d0, d0 + rb, ... of this thread's columns
+    auto load_rows = [&](int d0, int c) {
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u) {
+            const int d = d0 + u * rb;
+#pragma unroll
+            for (int e = 0; e < COLS; ++e) s[u][e] = 0.f;
+            if (S && d < dim) {
+                if constexpr (COLS == 4) {
+                    const float4 x = *reinterpret_cast<const float4*>(S + (size_t)d * vdim + c);
+                    s[u][0] = x.x;
+                    s[u][1] = x.y;
+                    s[u][2] = x.z;
+                    s[u][3] = x.w;
+                } else {
+                    s[u][0] = S[(size_t)d * vdim + c];
+                }
+            }
+        }
+    };
+    if (r0 < rb) load_rows(r0, group * COLS);   // the state's first rows are on their way while q and k are turned
     const float pos = (float)tok_pos[t], keep = decay[head];
     for (int i = threadIdx.x; i < dim; i += RK_THREADS) {
         float a = Num<T>::to_f(qh[i]), b = Num<T>::to_f(kh[i]);
         if (i < rot_dim) {
             const bool first = i < half;
             const int j = first ? i : i - half, other = first ? i + half : i - half;
-            float s, c;
-            sincosf(pos * inv_freq[j], &s, &c);
-            s *= first ? -amplitude : amplitude;
+            float sn, c;
+            sincosf(pos * inv_freq[j], &sn, &c);
+            sn *= first ? -amplitude : amplitude;
             c *= amplitude;
-            a = a * c + Num<T>::to_f(qh[other]) * s;
-            b = b * c + Num<T>::to_f(kh[other]) * s;
+            a = a * c + Num<T>::to_f(qh[other]) * sn;
+            b = b * c + Num<T>::to_f(kh[other]) * sn;
         }
         q_s[i] = a;
         k_s[i] = b * k_scale;
     }
     __syncthreads();
-    const int group = threadIdx.x % groups, r0 = threadIdx.x / groups;
-    float* S = slot >= 0 ? state + slot * slot_stride + s_offset + (long long)head * dim * vdim : nullptr;
     // (more column groups than threads: a thread takes several, one row group)
     for (int g = group; g < groups && r0 < rb; g += RK_THREADS) {
         const int c = g * COLS;
@@ -444,26 +495,8 @@ retention_token_kernel(const T* __restrict__ q, int q_stride, const T* __restric
             val[e] = Num<T>::to_f(v[(size_t)t * v_stride + (size_t)head * vdim + c + e]);
             acc[e] = 0.f;
         }
-        constexpr int AHEAD = 8;
         for (int d0 = r0; d0 < dim; d0 += rb * AHEAD) {
-            float s[AHEAD][COLS];
-#pragma unroll
-            for (int u = 0; u < AHEAD; ++u) {
-                const int d = d0 + u * rb;
-#pragma unroll
-                for (int e = 0; e < COLS; ++e) s[u][e] = 0.f;
-                if (S && d < dim) {
-                    if constexpr (COLS == 4) {
-                        const float4 x = *reinterpret_cast<const float4*>(S + (size_t)d * vdim + c);
-                        s[u][0] = x.x;
-                        s[u][1] = x.y;
-                        s[u][2] = x.z;
-                        s[u][3] = x.w;
-                    } else {
-                        s[u][0] = S[(size_t)d * vdim + c];
-                    }
-                }
-            }
+            if (g != group || d0 != r0) load_rows(d0, c);
 #pragma unroll
             for (int u = 0; u < AHEAD; ++u) {
                 const int d = d0 + u * rb;

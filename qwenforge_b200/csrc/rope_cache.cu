@@ -416,30 +416,9 @@ rope_maps_cache_kernel(const T* __restrict__ qkv, int qkv_stride, const int* __r
                        int* err) {
     grid_chain_entry();
     __shared__ float sin_s[RC_TOKENS][128], cos_s[RC_TOKENS][128];   // rot_dim <= 256
-    __shared__ int pos_s[RC_TOKENS];
     __shared__ long long page_s[RC_TOKENS];   // element offset of the token's place in head 0 of its page, -1: nothing to write
     const int D = site.head_dim, KVH = site.kv_heads, half = rot_dim / 2;
     const int t0 = blockIdx.x * per_block, n_here = min(per_block, n_tokens - t0);
-    if (threadIdx.x < n_here) {
-        const int t = t0 + threadIdx.x, pos = tok_pos[t], slot = slots[tok_seq[t]];
-        pos_s[threadIdx.x] = pos;
-        long long offset = -1;
-        if (write_cache && slot >= 0) {
-            const int page = site.table[(long long)slot * site.table_stride + pos / QF_PAGE];
-            if (page < 0) atomicOr(err, QF_ERR_NO_PAGE);
-            else offset = (long long)page * site.page_elems + (long long)(pos % QF_PAGE) * D;
-        }
-        page_s[threadIdx.x] = offset;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < n_here * half; i += blockDim.x) {
-        const int k = i / half, j = i % half;
-        float s, c;
-        sincosf((float)pos_s[k] * inv_freq[j], &s, &c);
-        sin_s[k][j] = s * amplitude;
-        cos_s[k][j] = c * amplitude;
-    }
-    __syncthreads();
     auto load = [&](const T* p, float (&v)[V]) {
         if constexpr (V == 8) {
             const uint4 raw = *reinterpret_cast<const uint4*>(p);
@@ -459,44 +438,85 @@ rope_maps_cache_kernel(const T* __restrict__ qkv, int qkv_stride, const int* __r
             *reinterpret_cast<uint4*>(p) = make_uint4(pack2(v[0], v[1]), pack2(v[2], v[3]), pack2(v[4], v[5]), pack2(v[6], v[7]));
         else p[0] = Num<T>::from_f(v[0]);
     };
-    // components c .. c + V - 1 of the map whose row starts at `src`, turned
-    auto turned = [&](const T* src, int k, int c, float (&v)[V]) {
-        load(src + c, v);
-        if (c >= rot_dim) return;
-        const bool first = c < half;
-        const int j = first ? c : c - half;
-        float other[V];
-        load(src + (first ? c + half : c - half), other);
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-            const float s = sin_s[k][j + e], cs = cos_s[k][j + e];
-            v[e] = first ? v[e] * cs - other[e] * s : v[e] * cs + other[e] * s;
-        }
-    };
     const int groups = D / V, q_heads = n_heads * maps, per_token = (q_heads + 2 * KVH) * groups;
     const int k_first = q_heads * dim, v_first = k_first + KVH * maps * dim;
-    for (int i = threadIdx.x; i < n_here * per_token; i += blockDim.x) {
-        const int k = i / per_token, item = i % per_token, t = t0 + k;
-        const int head = item / groups, c = (item % groups) * V;
-        const T* row = qkv + (size_t)t * qkv_stride;
-        float v[V];
+    // Item i of the block: V components from c on of a query, a cached head's keys or its values; `at`: where they come from in the
+    // token's row (-1: zeros), `own`: their place in their map (-1: not turned).
+    struct Item {
+        int k, head, c, at, own;
+    };
+    auto item_of = [&](int i) -> Item {
+        Item it;
+        it.k = i / per_token;
+        const int item = i % per_token;
+        it.head = item / groups;
+        it.c = (item % groups) * V;
+        it.at = it.own = -1;
+        if (it.head < q_heads) {
+            const int own = it.c - (it.head % maps) * dim;
+            if (own >= 0 && own < dim) {
+                it.own = own;
+                it.at = it.head * dim + own;
+            }
+        } else if (it.head < q_heads + KVH) {
+            if (it.c < maps * dim) {
+                it.own = it.c % dim;
+                it.at = k_first + (it.head - q_heads) * maps * dim + it.c;
+            }
+        } else if (it.c < vdim) {
+            it.at = v_first + (it.head - q_heads - KVH) * vdim + it.c;
+        }
+        return it;
+    };
+    auto fetch = [&](const Item& it, float (&v)[V], float (&other)[V]) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) v[e] = 0.f;
-        if (head < q_heads) {
-            const int own = c - (head % maps) * dim;   // the component of the query's own map
-            if (own >= 0 && own < dim) turned(row + head * dim, k, own, v);
-            store(q_out + ((size_t)t * q_heads + head) * D + c, v);
-            continue;
+        for (int e = 0; e < V; ++e) v[e] = other[e] = 0.f;
+        if (it.at < 0) return;
+        const T* src = qkv + (size_t)(t0 + it.k) * qkv_stride + it.at;
+        load(src, v);
+        if (it.own >= 0 && it.own < rot_dim) load(it.own < half ? src + half : src - half, other);
+    };
+    auto finish = [&](const Item& it, float (&v)[V], const float (&other)[V]) {
+        if (it.own >= 0 && it.own < rot_dim) {
+            const bool first = it.own < half;
+            const int j = first ? it.own : it.own - half;
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                const float s = sin_s[it.k][j + e], cs = cos_s[it.k][j + e];
+                v[e] = first ? v[e] * cs - other[e] * s : v[e] * cs + other[e] * s;
+            }
         }
-        const long long place = page_s[k];
-        if (place < 0) continue;
-        const int g = head - q_heads;
-        if (g < KVH) {
-            if (c < maps * dim) turned(row + k_first + g * maps * dim + c / dim * dim, k, c % dim, v);
-        } else if (c < vdim) {
-            load(row + v_first + (g - KVH) * vdim + c, v);
+        if (it.head < q_heads) store(q_out + ((size_t)(t0 + it.k) * q_heads + it.head) * D + it.c, v);
+        else if (page_s[it.k] >= 0) store(site.base + page_s[it.k] + (long long)(it.head - q_heads) * QF_PAGE * D + it.c, v);
+    };
+    const int total = n_here * per_token;
+    float v[V], other[V];
+    Item it = item_of(threadIdx.x);
+    if (threadIdx.x < total) fetch(it, v, other);   // the first item is on its way while the angles are formed
+    if (threadIdx.x < n_here) {
+        const int t = t0 + threadIdx.x, pos = tok_pos[t], slot = slots[tok_seq[t]];
+        long long offset = -1;
+        if (write_cache && slot >= 0) {
+            const int page = site.table[(long long)slot * site.table_stride + pos / QF_PAGE];
+            if (page < 0) atomicOr(err, QF_ERR_NO_PAGE);
+            else offset = (long long)page * site.page_elems + (long long)(pos % QF_PAGE) * D;
         }
-        store(site.base + place + (long long)g * QF_PAGE * D + c, v);
+        page_s[threadIdx.x] = offset;
+    }
+    for (int i = threadIdx.x; i < n_here * half; i += blockDim.x) {
+        const int k = i / half, j = i % half;
+        float s, c;
+        sincosf((float)tok_pos[t0 + k] * inv_freq[j], &s, &c);
+        sin_s[k][j] = s * amplitude;
+        cos_s[k][j] = c * amplitude;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < total; i += blockDim.x) {
+        if (i != (int)threadIdx.x) {
+            it = item_of(i);
+            fetch(it, v, other);
+        }
+        finish(it, v, other);
     }
 }
 

@@ -508,14 +508,17 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok
                      slots: torch.Tensor, site: KvSiteArgs, n_heads: int, n_seqs: int, scale: float, window: int,
                      n_splits: int, scratch: DecodeScratch, err: torch.Tensor, plan: Optional[torch.Tensor] = None,
                      fold_later: bool = False, sinks: Optional[torch.Tensor] = None, shared_values: bool = False,
-                     chunk: int = 0, softcap: float = 0.0, distance_bias: Optional[tuple] = None) -> None:
+                     chunk: int = 0, softcap: float = 0.0, distance_bias: Optional[tuple] = None,
+                     pairs: Optional[tuple] = None) -> None:
     """Split-K flash decoding: ONE new token per sequence over its cache; bfloat16, head sizes 32/64/96/128.
     `n_splits` is the most blocks that share one (sequence, kv head); `plan` (attention_decode_plan with the same
     shape, made in this step; made here when absent) says how many of them each sequence gets. With `fold_later` the
     kernel stops at the runs' partial results in `scratch` and writes no `out` (which may be None): `fold_project`
     folds them on its way into the output projection. `sinks`, `shared_values`, `chunk`, `softcap`, `distance_bias`: as in
     `attention_generic` (sinks not with `fold_later`; a given `plan` must have been made with the same `chunk`; the cap
-    with the hardware's approximate tanh)."""
+    with the hardware's approximate tanh). `pairs` = (weight, eps, gain, vdim): heads 2 i and 2 i + 1 are the two maps of one head
+    (an even group; none of the other options), out [n_seqs, n_heads / 2 * vdim] takes them brought together as `map_difference`
+    does, from the float32 results."""
     _dev("q", q, torch.bfloat16)
     if sinks is not None:
         _dev("sinks", sinks, torch.float32)
@@ -528,7 +531,11 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok
     if d not in FAST_ATTENTION_HEAD_DIMS:
         raise KernelError(f"attention_decode: head_dim {d} has no tensor-core kernel (have {FAST_ATTENTION_HEAD_DIMS}); "
                           "use attention_generic")
-    if q.shape != (n_seqs, n_heads * d) or (not fold_later and out.shape != q.shape):
+    if pairs is not None:
+        if (n_heads // site.kv_heads) % 2 or not 0 < pairs[3] <= d or out.shape != (n_seqs, n_heads // 2 * pairs[3]) or fold_later \
+                or sinks is not None or shared_values or chunk or softcap or distance_bias is not None:
+            raise KernelError("attention_decode: pairs go with an even group of heads, out [n_seqs, n_heads / 2 * vdim], and no other option")
+    if q.shape != (n_seqs, n_heads * d) or (not fold_later and pairs is None and out.shape != q.shape):
         raise KernelError("attention_decode: wants exactly one token per sequence, q [n_seqs, n_heads * head_dim]")
     if not 1 <= n_splits <= 128:
         raise KernelError(f"attention_decode: n_splits {n_splits} outside 1..128")
@@ -539,6 +546,13 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor, tok
     partials = n_splits > 1 or fold_later
     if partials:
         scratch.ensure(n_seqs, n_heads, n_splits, d, n_counters)
+    if pairs is not None:
+        _check(library("attention_decode").qf_attention_decode_paired(
+            _ptr(q), _ptr(out), _ptr(cu_q), _ptr(plan), _ptr(site.storage), _ptr(site.table), _LL(site.page_elems), _I(site.table_stride),
+            _I(site.kv_heads), _I(d), _I(n_heads), _I(n_seqs), _F(scale), _I(window), _I(n_splits), _ptr(scratch.part_o if partials else None),
+            _ptr(scratch.part_ml if partials else None), _ptr(scratch.counters if partials else None), _ptr(err), _F(pairs[0]), _F(pairs[1]),
+            _F(pairs[2]), _I(pairs[3]), _stream()), "attention_decode")
+        return
     by, rate = _distance_bias("attention_decode", distance_bias, n_heads)
     _check(library("attention_decode").qf_attention_decode_biased(
         _ptr(q), _ptr(None if fold_later else out), _ptr(cu_q), _ptr(plan), _ptr(site.storage), _ptr(site.table),

@@ -82,19 +82,22 @@ class DifferentialAttention(GqaAttention):
         args = ops.KvSiteArgs(site.storage, site.table, self.n_kv, self.head_dim)
         ops.rope_maps_cache_write(qkv, ctx.tok_seq, ctx.tok_pos, ctx.slots, inv_freq, rot_dim, amplitude, self.pairs, MAPS, self.map_dim,
                                   self.value_dim, q, args, writes_cache, ctx.err)
-        attended = torch.empty_like(q)
+        out = torch.empty((n, self.pairs * self.value_dim), dtype=x.dtype, device=x.device)
         fast = ctx.attention == "auto" and x.dtype == torch.bfloat16 and self.head_dim in ops.FAST_ATTENTION_HEAD_DIMS
+        if fast and ctx.is_decode and n == ctx.n_seqs:   # single tokens: the maps meet inside the attention kernel
+            ops.attention_decode(q, out, ctx.cu_q, ctx.tok_pos, ctx.slots, args, self.n_heads, ctx.n_seqs, self.scale, self.window,
+                                 self.decode_splits(ctx), ctx.decode_scratch, ctx.err, self.decode_plan(ctx),
+                                 pairs=(self.map_weight, self.eps, 1.0 - self.offset, self.value_dim))
+            return ops.linear_rows(out, self.o_weight)
+        attended = torch.empty_like(q)
         common = (q, attended, ctx.cu_q, ctx.tok_pos, ctx.slots, args, self.n_heads, ctx.n_seqs)
-        if fast and ctx.is_decode and n == ctx.n_seqs:
-            ops.attention_decode(*common, self.scale, self.window, self.decode_splits(ctx), ctx.decode_scratch, ctx.err, self.decode_plan(ctx))
-        elif fast:
+        if fast:
             least = TC_PREFILL_MIN_TOKENS.get(self.head_dim)
             run = ops.attention_prefill_tc if least is not None and n >= least and ctx.max_q_len >= 128 else ops.attention_prefill
             run(*common, ctx.max_q_len, self.scale, self.window, ctx.err, max_kv_len=ctx.max_kv_len)
         else:
             ops.attention_generic(*common, ctx.max_q_len, self.scale, self.window, ctx.err, scratch=ctx.decode_scratch,
                                   max_kv_len=ctx.max_kv_len)
-        out = torch.empty((n, self.pairs * self.value_dim), dtype=x.dtype, device=x.device)
         ops.map_difference(attended, self.head_dim, self.map_weight, self.eps, 1.0 - self.offset, out, self.pairs, self.value_dim)
         return ops.linear_rows(out, self.o_weight)
 

@@ -186,6 +186,33 @@ def test_two_maps_brought_together(dtype, heads, vdim, pitch):
         close(out, want, dtype, f"{n} tokens", f32=2e-6)
 
 
+@pytest.mark.parametrize("kv,pairs,size,vdim", [(2, 7, 64, 64), (1, 20, 32, 30), (2, 2, 96, 80), (4, 4, 128, 128), (1, 3, 128, 70)])
+def test_single_tokens_with_the_maps_brought_together(kv, pairs, size, vdim):
+    """The decode kernel's own combination (one run per sequence and several, groups beyond one tile of heads, a padding entry) against
+    the plain attention and combination in float64."""
+    from qwenforge_b200 import ops
+    g = torch.Generator().manual_seed(size + vdim)
+    heads = 2 * pairs * kv
+    for lengths, window, splits in (([130, 5, 640], 0, 4), ([700, 64, 65], 0, 1), ([700, 300, 1], 200, 3)):
+        site = Site(ops, torch.bfloat16, kv, size, slots=4, pages=48, per_slot=12)
+        site.storage.copy_(rand(g, *site.storage.shape, dtype=torch.bfloat16))
+        site.storage[:, 1, :, :, vdim:] = 0
+        table = torch.randperm(48, generator=g).to(torch.int32).view(4, 12).to(DEV)
+        args = ops.KvSiteArgs(site.storage, table, kv, size)
+        b = Batch([2, 0, 3, -1], [(n - 1, 1) for n in lengths] + [(0, 1)])
+        q = rand(g, 4, heads * size, dtype=torch.bfloat16)
+        scratch, err = ops.DecodeScratch(torch.device(DEV)), ints([0])
+        out = torch.full((4, heads // 2 * vdim), 9.0, dtype=torch.bfloat16, device=DEV)
+        for _ in range(2):   # (the second call meets the ticket counters as the first left them)
+            ops.attention_decode(q, out, b.cu_q, b.tok_pos, b.slots, args, heads, 4, 0.2, window, splits, scratch, err, pairs=(0.6, 1e-4, 0.7, vdim))
+        wide = torch.empty(4, heads * size, dtype=torch.float64, device=DEV)
+        refs.attention_generic(q, wide, b.cu_q, b.tok_pos, b.slots, args, heads, 4, 1, 0.2, window, None)
+        want = torch.empty(4, heads // 2 * vdim, dtype=torch.float64, device=DEV)
+        refs.map_difference(wide, size, 0.6, 1e-4, 0.7, want, heads // 2, vdim)
+        close(out[:3], want[:3], torch.bfloat16, f"{lengths} {splits}", bf16=1.5e-2)
+        assert int(err) == 0 and float(out[3].abs().max()) == 0
+
+
 def retention_case(g, n, heads, dim, vdim, dtype):
     width = heads * (2 * dim + 2 * vdim)
     proj = rand(g, n, width + (-width) % 8, dtype=dtype)
