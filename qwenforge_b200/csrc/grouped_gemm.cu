@@ -250,28 +250,28 @@ grouped_gemm_mma_kernel(GroupedArgs g) {
 }
 
 // A step of up to 16 rows per group (decode steps): the work is fetching the groups' weights once, so the weights are the tall side
-// of the tensor-core tile (out^T = W a^T: 16 weight rows x 8 rows of A x 16 columns of K per mma) and a block keeps three slabs of
-// 128 columns of K of its 64 weight rows on their way, five times the bytes of the tile above, which is made for more rows.
-// GATED: the 64 weight rows are 32 gate rows and the 32 matching up rows; warp w takes 16 of both in every second slab step (w >> 1),
-// the halves of K are added through shared memory. Without a gate a warp takes 16 weight rows and all of K.
+// of the tensor-core tile (out^T = W a^T: 16 weight rows x 8 rows of A x 16 columns of K per mma), a block has 32 weight rows, so that
+// the blocks spread evenly over the SMs, and STAGES - 1 slabs of 128 columns of K are on their way: as many as the blocks that share
+// an SM leave room for. GATED: the 32 rows are 16 gate rows and the 16 matching up rows. The block's four warps share the rows and the
+// steps of K; the parts of K are added through shared memory in the order of the warps.
 #define GR_ROWS 16
+#define GR_WROWS 32
 #define GR_BK 128
 #define GR_LD (GR_BK + 8)
-#define GR_STAGES 4
-#define GR_STAGE_ELEMS ((GG_BN + GR_ROWS) * GR_LD)
-template <bool GATED>
+#define GR_STAGE_ELEMS ((GR_WROWS + GR_ROWS) * GR_LD)
+template <bool GATED, int STAGES>
 __global__ void __launch_bounds__(128)
 grouped_rows_kernel(GroupedArgs g) {
     grid_chain_entry();
     extern __shared__ __align__(16) unsigned char gr_smem[];
-    bf16* stages = reinterpret_cast<bf16*>(gr_smem);   // [GR_STAGES][64 weight rows, then 16 rows of A][GR_LD]
+    bf16* stages = reinterpret_cast<bf16*>(gr_smem);   // [STAGES][32 weight rows, then 16 rows of A][GR_LD]
     int group, m0, m_end;
     if (!grouped_tile<QF_GROUP_BM>(g, group, m0, m_end)) return;
     m_end = min(m_end, m0 + GR_ROWS);
     const bf16* A = (const bf16*)g.a;
     const bf16* W = (const bf16*)g.w + (long long)group * g.w_group_stride;
     bf16* C = (bf16*)g.c;
-    const int n0 = blockIdx.x * (GATED ? GG_BN / 2 : GG_BN), N = g.n, K = g.k;
+    const int n0 = blockIdx.x * (GATED ? GR_WROWS / 2 : GR_WROWS), N = g.n, K = g.k;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int chunk = (threadIdx.x & 15) * 8, first = threadIdx.x >> 4;   // this thread's 16 bytes of a row, and its first row
     long long a_row[2];
@@ -282,12 +282,12 @@ grouped_rows_kernel(GroupedArgs g) {
     }
     auto fetch = [&](int k0, int stage) {
         bf16* w_s = stages + (size_t)stage * GR_STAGE_ELEMS;
-        bf16* a_s = w_s + GG_BN * GR_LD;
+        bf16* a_s = w_s + GR_WROWS * GR_LD;
         const bool k_ok = k0 + chunk < K;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int r = first + 8 * i, col = GATED ? n0 + (r & 31) : n0 + r;
-            const long long w_row = GATED ? (r < 32 ? col : (long long)N + col) : col;
+        for (int i = 0; i < GR_WROWS / 8; ++i) {
+            const int r = first + 8 * i, col = GATED ? n0 + (r & 15) : n0 + r;
+            const long long w_row = GATED ? (r < 16 ? col : (long long)N + col) : col;
             const bool ok = k_ok && col < N;
             cp_async_16(w_s + r * GR_LD + chunk, ok ? W + w_row * g.ldw + k0 + chunk : W, ok);
         }
@@ -297,66 +297,69 @@ grouped_rows_kernel(GroupedArgs g) {
             cp_async_16(a_s + (first + 8 * i) * GR_LD + chunk, ok ? A + a_row[i] * g.lda + k0 + chunk : A, ok);
         }
     };
-    constexpr int TILES = GATED ? 2 : 1;   // 16-row tiles of weights per warp (gate and up)
+    constexpr int TILES = GATED ? 2 : 1;        // 16-row tiles of weights per warp: a gate tile and its up tile, or one
+    constexpr int SPLIT = GATED ? 4 : 2;        // warps that share a tile's steps of K
+    const int tile = GATED ? 0 : warp & 1, part = GATED ? warp : warp >> 1;
     float acc[TILES][2][4];
 #pragma unroll
     for (int i = 0; i < TILES; ++i)
 #pragma unroll
         for (int j = 0; j < 2; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
     const int n_slabs = (K + GR_BK - 1) / GR_BK;
-    for (int s = 0; s < GR_STAGES - 1; ++s) {
+    for (int s = 0; s < STAGES - 1; ++s) {
         if (s < n_slabs) fetch(s * GR_BK, s);
         cp_async_commit();
     }
     for (int slab = 0; slab < n_slabs; ++slab) {
-        cp_async_wait<GR_STAGES - 2>();
+        cp_async_wait<STAGES - 2>();
         __syncthreads();   // slab `slab` has arrived for everyone, and everyone is done with the buffer fetched next
-        if (slab + GR_STAGES - 1 < n_slabs) fetch((slab + GR_STAGES - 1) * GR_BK, (slab + GR_STAGES - 1) % GR_STAGES);
+        if (slab + STAGES - 1 < n_slabs) fetch((slab + STAGES - 1) * GR_BK, (slab + STAGES - 1) % STAGES);
         cp_async_commit();
-        const bf16* w_s = stages + (size_t)(slab % GR_STAGES) * GR_STAGE_ELEMS;
-        const bf16* a_s = w_s + GG_BN * GR_LD;
+        const bf16* w_s = stages + (size_t)(slab % STAGES) * GR_STAGE_ELEMS;
+        const bf16* a_s = w_s + GR_WROWS * GR_LD;
 #pragma unroll
-        for (int ks = 0; ks < GR_BK / 16; ks += GATED ? 2 : 1) {
-            const int k = 16 * (ks + (GATED ? warp >> 1 : 0));
+        for (int ks = 0; ks < GR_BK / 16; ks += SPLIT) {
+            const int k = 16 * (ks + part);
             uint32_t xf[4];   // the 16 rows of A as two column tiles
             ldmatrix_x4(xf, a_s + (size_t)((lane >> 4) * 8 + (lane & 7)) * GR_LD + k + ((lane >> 3) & 1) * 8);
 #pragma unroll
             for (int i = 0; i < TILES; ++i) {
-                const int row = GATED ? 32 * i + 16 * (warp & 1) : 16 * warp;
                 uint32_t wf[4];
-                ldmatrix_x4(wf, w_s + (size_t)(row + (lane & 15)) * GR_LD + k + (lane >> 4) * 8);
+                ldmatrix_x4(wf, w_s + (size_t)(16 * (GATED ? i : tile) + (lane & 15)) * GR_LD + k + (lane >> 4) * 8);
                 mma_bf16_16816(acc[i][0], wf, xf[0], xf[1]);
                 mma_bf16_16816(acc[i][1], wf, xf[2], xf[3]);
             }
         }
     }
     cp_async_wait<0>();
-    if (GATED) {
-        __syncthreads();   // the stages are free
-        float* half = reinterpret_cast<float*>(gr_smem);   // [2 warps][TILES * 8][32]
-        if (warp >= 2) {
-#pragma unroll
-            for (int i = 0; i < TILES; ++i)
-#pragma unroll
-                for (int j = 0; j < 2; ++j)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) half[((warp - 2) * TILES * 8 + (i * 2 + j) * 4 + e) * 32 + lane] = acc[i][j][e];
-        }
-        __syncthreads();
-        if (warp >= 2) return;
+    __syncthreads();   // the stages are free
+    float* parts = reinterpret_cast<float*>(gr_smem);   // [4 warps][TILES * 8][32]
+    if (part > 0) {
 #pragma unroll
         for (int i = 0; i < TILES; ++i)
 #pragma unroll
             for (int j = 0; j < 2; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) acc[i][j][e] += half[(warp * TILES * 8 + (i * 2 + j) * 4 + e) * 32 + lane];
+                for (int e = 0; e < 4; ++e) parts[((warp * TILES + i) * 8 + j * 4 + e) * 32 + lane] = acc[i][j][e];
+    }
+    __syncthreads();
+    if (part > 0) return;
+#pragma unroll
+    for (int p = 1; p < SPLIT; ++p) {
+        const int from = GATED ? p : tile + 2 * p;
+#pragma unroll
+        for (int i = 0; i < TILES; ++i)
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[i][j][e] += parts[((from * TILES + i) * 8 + j * 4 + e) * 32 + lane];
     }
     // element e of accumulator j: weight row (lane / 4) + 8 (e / 2), row 8 j + 2 (lane % 4) + e % 2 of A
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int gm = m0 + 8 * j + 2 * (lane & 3) + (e & 1), gn = n0 + 16 * (GATED ? warp & 1 : warp) + (lane >> 2) + 8 * (e >> 1);
+            const int gm = m0 + 8 * j + 2 * (lane & 3) + (e & 1), gn = n0 + 16 * tile + (lane >> 2) + 8 * (e >> 1);
             if (gm >= m_end || gn >= N) continue;
             float v = acc[0][j][e];
             if (GATED) {
@@ -375,13 +378,22 @@ grouped_rows_kernel(GroupedArgs g) {
         }
 }
 
+template <bool GATED, int STAGES>
+static int launch_rows_staged(const GroupedArgs& g, int col_blocks, cudaStream_t stream) {
+    const size_t smem = (size_t)STAGES * GR_STAGE_ELEMS * sizeof(bf16);
+    cudaError_t e = cudaFuncSetAttribute(grouped_rows_kernel<GATED, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    return (int)launch_pdl(grouped_rows_kernel<GATED, STAGES>, dim3(col_blocks, g.max_tiles), dim3(128), smem, stream, g);
+}
+
+// The stages by how many blocks with work an SM gets: all of them are to be resident at once.
 template <bool GATED>
 static int launch_rows(const GroupedArgs& g, cudaStream_t stream) {
-    const size_t smem = (size_t)GR_STAGES * GR_STAGE_ELEMS * sizeof(bf16);
-    cudaError_t e = cudaFuncSetAttribute(grouped_rows_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    const int cols = GATED ? GG_BN / 2 : GG_BN;
-    return (int)launch_pdl(grouped_rows_kernel<GATED>, dim3((g.n + cols - 1) / cols, g.max_tiles), dim3(128), smem, stream, g);
+    const int cols = GATED ? GR_WROWS / 2 : GR_WROWS, col_blocks = (g.n + cols - 1) / cols;
+    const long long busy = (long long)col_blocks * (g.rows < g.n_groups ? g.rows : g.n_groups), sms = qf_sm_count() > 0 ? qf_sm_count() : 1;
+    if (busy <= 2 * sms) return launch_rows_staged<GATED, 6>(g, col_blocks, stream);
+    if (busy <= 4 * sms) return launch_rows_staged<GATED, 4>(g, col_blocks, stream);
+    return launch_rows_staged<GATED, 3>(g, col_blocks, stream);
 }
 
 // The large tile: 128 x 128, eight warps as 2 x 4, warp (wy, wx) a quarter of 64 x 32 as 4 x 4 tiles of m16n8k16; slabs of

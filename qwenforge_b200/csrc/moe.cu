@@ -16,9 +16,12 @@
 // whatever the block's atomics gave; no result depends on it, since a row of a product is computed alone.
 #include <float.h>
 
-#include "common.cuh"
+#include "mma.cuh"
 
 #define MOE_PLAN_THREADS 1024
+// Whether the plan's block makes the router's logits on the tensor cores: few tokens and experts, rows in whole steps of K.
+__host__ __device__ inline bool plan_on_tiles(int n_tokens, int n_experts, int width) { return n_tokens <= 32 && n_experts <= 32 && width % 16 == 0; }
+#define PLAN_HELD 512     // pairs that the plan keeps in shared memory
 #define MOE_MAX_TOP 16
 
 // One token's choice: the `top` experts with the largest scores (the larger logit is the larger score; ties go to the
@@ -199,68 +202,132 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
                 int* __restrict__ tile_group, int* __restrict__ tile_row0, int* __restrict__ n_tiles, int max_tiles,
                 int tile_rows, const void* __restrict__ x, const void* __restrict__ router, int width, int x_is_bf16,
                 const float* __restrict__ bias, MoeGroups groups) {
-    grid_chain_entry();
+    grid_launch_dependents();
     extern __shared__ int shared[];
     int* counts = shared;                   // [experts]: rows per expert, then every expert's first row
     int* first_tile = shared + n_experts;   // [experts + 1]
     for (int e = threadIdx.x; e < n_experts; e += blockDim.x) counts[e] = 0;
-    if (x) {  // the router's product first: z[t][e] = sum_c x[t][c] * router[e][c], a warp per logit, kept in shared memory
-        float* logits_out = reinterpret_cast<float*>(shared + 2 * n_experts + 1);
-        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-        for (int i = warp; i < n_tokens * n_experts; i += n_warps) {
-            const int t = i / n_experts, e = i % n_experts;
-            float sum = 0.f;
-            if (x_is_bf16) {
-                const bf16* xr = (const bf16*)x + (size_t)t * width;
-                const bf16* rr = (const bf16*)router + (size_t)e * width;
-                if (width % 8 == 0 && (((uintptr_t)x | (uintptr_t)router) & 15) == 0) {
-                    // eight elements per load, and no load waits for a sum: a lane's loads are all on their way at once
-                    const uint4* xv = reinterpret_cast<const uint4*>(xr);
-                    const uint4* rv = reinterpret_cast<const uint4*>(rr);
-                    // four steps of a lane at a time, all their loads asked for before the first product (zeros beyond the
-                    // row's end add nothing): the sums run in the same order as one step after the other
-                    for (int c0 = lane; c0 < width / 8; c0 += 4 * 32) {
-                        uint4 a[4], b[4];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const bool wide = x && x_is_bf16 && width % 8 == 0 && (((uintptr_t)x | (uintptr_t)router) & 15) == 0;
+    if (x) {  // the router's product first: z[t][e] = sum_c x[t][c] * router[e][c], kept in shared memory
+        float* logits_out = reinterpret_cast<float*>(shared + (2 * n_experts + 1 + 3) / 4 * 4);
+        if (wide && plan_on_tiles(n_tokens, n_experts, width)) {
+            // Tiles of 16 tokens x 8 experts on the tensor cores (float32 sums), the block's warps dealing out K in steps of 16 columns;
+            // their partial sums are added in the warps' order. One SM fetches every row once: that is what a logit per warp lacked.
+            // The router's weights, which no kernel before this one writes, are asked for before the wait for it.
+            float* part = logits_out + (n_tokens * n_experts + 3) / 4 * 4;   // [n_warps][128]
+            const int steps = width / 16, g = lane >> 2, q = 2 * (lane & 3);
+            constexpr int AHEAD = 4;
+            uint32_t b[AHEAD][2];
+            auto router_steps = [&](int e0, int s0) {
+                const bf16* rr = (const bf16*)router + (size_t)min(e0 + g, n_experts - 1) * width + q;
 #pragma unroll
-                        for (int u = 0; u < 4; ++u) {
-                            const int c = c0 + 32 * u;
-                            a[u] = b[u] = make_uint4(0u, 0u, 0u, 0u);
-                            if (c < width / 8) {
-                                a[u] = xv[c];
-                                b[u] = rv[c];
-                            }
+                for (int u = 0; u < AHEAD; ++u) {
+                    const int s = s0 + u * n_warps;
+                    b[u][0] = s < steps ? *reinterpret_cast<const uint32_t*>(rr + 16 * s) : 0u;
+                    b[u][1] = s < steps ? *reinterpret_cast<const uint32_t*>(rr + 16 * s + 8) : 0u;
+                }
+            };
+            router_steps(0, warp);
+            grid_dependency_wait();
+            for (int t0 = 0; t0 < n_tokens; t0 += 16)
+                for (int e0 = 0; e0 < n_experts; e0 += 8) {
+                    const bf16* x0 = (const bf16*)x + (size_t)min(t0 + g, n_tokens - 1) * width + q;
+                    const bf16* x1 = (const bf16*)x + (size_t)min(t0 + g + 8, n_tokens - 1) * width + q;
+                    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+                    for (int s0 = warp; s0 < steps; s0 += AHEAD * n_warps) {
+                        if (t0 + e0 > 0 || s0 != warp) router_steps(e0, s0);
+                        uint32_t a[AHEAD][4];
+#pragma unroll
+                        for (int u = 0; u < AHEAD; ++u) {
+                            const int s = s0 + u * n_warps;
+                            const bool ok = s < steps;
+                            a[u][0] = ok ? *reinterpret_cast<const uint32_t*>(x0 + 16 * s) : 0u;
+                            a[u][1] = ok ? *reinterpret_cast<const uint32_t*>(x1 + 16 * s) : 0u;
+                            a[u][2] = ok ? *reinterpret_cast<const uint32_t*>(x0 + 16 * s + 8) : 0u;
+                            a[u][3] = ok ? *reinterpret_cast<const uint32_t*>(x1 + 16 * s + 8) : 0u;
                         }
 #pragma unroll
-                        for (int u = 0; u < 4; ++u) {
-                            if (c0 + 32 * u >= width / 8) break;
-                            const __nv_bfloat162* a2 = reinterpret_cast<const __nv_bfloat162*>(&a[u]);
-                            const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&b[u]);
+                        for (int u = 0; u < AHEAD; ++u) mma_bf16_16816(acc, a[u], b[u][0], b[u][1]);
+                    }
+                    __syncthreads();   // the tile before has been added up
+                    *reinterpret_cast<float4*>(part + warp * 128 + 4 * lane) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+                    __syncthreads();
+                    // eight threads per logit, each a run of warps
+                    const int i = threadIdx.x >> 3, each = n_warps / 8, from = (threadIdx.x & 7) * each;
+                    float z = 0.f;
+                    for (int w = from; w < from + each; ++w) z += part[w * 128 + i];
 #pragma unroll
-                            for (int j = 0; j < 4; ++j) {
-                                const float2 af = __bfloat1622float2(a2[j]), bf = __bfloat1622float2(b2[j]);
-                                sum = fmaf(af.x, bf.x, sum);
-                                sum = fmaf(af.y, bf.y, sum);
-                            }
+                    for (int o = 1; o < 8; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+                    const int t = t0 + (i >> 4) + 8 * ((i >> 1) & 1), e = e0 + 2 * ((i >> 2) & 3) + (i & 1);
+                    if ((threadIdx.x & 7) == 0 && t < n_tokens && e < n_experts) logits_out[t * n_experts + e] = bias ? z + bias[e] : z;
+                }
+        } else if (wide) {
+            grid_dependency_wait();
+            for (int i = warp; i < n_tokens * n_experts; i += n_warps) {   // a warp per logit, eight elements per load, four loads ahead
+                const uint4* xv = reinterpret_cast<const uint4*>((const bf16*)x + (size_t)(i / n_experts) * width);
+                const uint4* rv = reinterpret_cast<const uint4*>((const bf16*)router + (size_t)(i % n_experts) * width);
+                float sum = 0.f;
+                for (int c0 = lane; c0 < width / 8; c0 += 4 * 32) {
+                    uint4 a[4], b[4];
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        const int c = c0 + 32 * u;
+                        a[u] = b[u] = make_uint4(0u, 0u, 0u, 0u);   // (zeros beyond the row's end add nothing)
+                        if (c < width / 8) {
+                            a[u] = xv[c];
+                            b[u] = rv[c];
                         }
                     }
-                } else {
-                    for (int c = lane; c < width; c += 32) sum = fmaf(__bfloat162float(xr[c]), __bfloat162float(rr[c]), sum);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        const __nv_bfloat162* a2 = reinterpret_cast<const __nv_bfloat162*>(&a[u]);
+                        const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&b[u]);
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) {
+                            const float2 af = __bfloat1622float2(a2[j]), bf = __bfloat1622float2(b2[j]);
+                            sum = fmaf(af.x, bf.x, sum);
+                            sum = fmaf(af.y, bf.y, sum);
+                        }
+                    }
                 }
-            } else {
-                const float* xr = (const float*)x + (size_t)t * width;
-                const float* rr = (const float*)router + (size_t)e * width;
-                for (int c = lane; c < width; c += 32) sum = fmaf(xr[c], rr[c], sum);
+                sum = warp_sum(sum);
+                if (lane == 0) logits_out[i] = bias ? sum + bias[i % n_experts] : sum;
             }
-            sum = warp_sum(sum);
-            if (lane == 0) logits_out[i] = bias ? sum + bias[e] : sum;   // the bias once, here: the choice reads shared memory only
+        } else {
+            grid_dependency_wait();
+            for (int i = warp; i < n_tokens * n_experts; i += n_warps) {   // a warp per logit
+                const int t = i / n_experts, e = i % n_experts;
+                float sum = 0.f;
+                if (x_is_bf16) {
+                    const bf16* xr = (const bf16*)x + (size_t)t * width;
+                    const bf16* rr = (const bf16*)router + (size_t)e * width;
+                    for (int c = lane; c < width; c += 32) sum = fmaf(__bfloat162float(xr[c]), __bfloat162float(rr[c]), sum);
+                } else {
+                    const float* xr = (const float*)x + (size_t)t * width;
+                    const float* rr = (const float*)router + (size_t)e * width;
+                    for (int c = lane; c < width; c += 32) sum = fmaf(xr[c], rr[c], sum);
+                }
+                sum = warp_sum(sum);
+                if (lane == 0) logits_out[i] = bias ? sum + bias[e] : sum;
+            }
         }
         logits = logits_out;
         bias = nullptr;
+    } else {
+        grid_dependency_wait();
     }
     __syncthreads();
-    // pass 1: choose, and take a rank among the expert's rows
+    // pass 1: choose, and take a rank among the expert's rows; few pairs stay in shared memory on their way to the second pass
+    __shared__ int held_expert[PLAN_HELD], held_rank[PLAN_HELD];
+    __shared__ float held_weight[PLAN_HELD];
+    int* experts_out = n_tokens * top <= PLAN_HELD ? pair_expert : nullptr;
+    if (n_tokens * top <= PLAN_HELD) {
+        pair_expert = held_expert;
+        pair_weight = held_weight;
+    }
+    int* rank_of = n_tokens * top <= PLAN_HELD ? held_rank : dest;
     if (n_experts <= 32) {   // a warp per token
-        const int lane = threadIdx.x & 31;
         for (int t = threadIdx.x >> 5; t < n_tokens; t += blockDim.x >> 5) {
             const float z = lane < n_experts ? logits[(size_t)t * n_experts + lane] + (bias ? bias[lane] : 0.f) : 0.f;
             float weight;
@@ -268,7 +335,7 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
             if (k >= 0) {
                 const int pair = t * top + k;
                 pair_expert[pair] = lane;
-                dest[pair] = atomicAdd(&counts[lane], 1);        // for now: the pair's rank among its expert's rows
+                rank_of[pair] = atomicAdd(&counts[lane], 1);     // the pair's rank among its expert's rows
                 pair_weight[pair] = weight;
             }
         }
@@ -281,7 +348,7 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
             for (int k = 0; k < top; ++k) {
                 const int pair = t * top + k;
                 pair_expert[pair] = chosen[k];
-                dest[pair] = atomicAdd(&counts[chosen[k]], 1);
+                rank_of[pair] = atomicAdd(&counts[chosen[k]], 1);
                 pair_weight[pair] = weight[k];
             }
         }
@@ -289,7 +356,6 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
     __syncthreads();
     if (n_experts <= 32) {
         if (threadIdx.x < 32) {
-            const int lane = threadIdx.x;
             int row, tile, rows, tiles;
             moe_scan_warp(lane < n_experts ? counts[lane] : 0, tile_rows, row, tile, rows, tiles);
             if (lane < n_experts) {
@@ -327,7 +393,8 @@ moe_plan_kernel(const float* logits, int n_tokens, int n_experts, int top, int s
     }
     // pass 2: every pair's row
     for (int pair = threadIdx.x; pair < n_tokens * top; pair += blockDim.x) {
-        const int row = counts[pair_expert[pair]] + dest[pair];
+        const int row = counts[pair_expert[pair]] + rank_of[pair];
+        if (experts_out) experts_out[pair] = pair_expert[pair];
         dest[pair] = row;
         sorted_token[row] = pair / top;
         sorted_weight[row] = pair_weight[pair];
@@ -604,7 +671,13 @@ QF_EXPORT int qf_moe_plan_grouped(const float* logits, int n_tokens, int n_exper
     const MoeGroups groups = {correction, group_count, group_keep, group_best};
     if (top < 1 || top > MOE_MAX_TOP || top > n_experts || n_experts > 8192 || tile_rows <= 0) return (int)cudaErrorInvalidValue;
     if (!logits && !(x && router && (long long)n_tokens * n_experts <= 8192)) return (int)cudaErrorInvalidValue;
-    const size_t smem = (size_t)(2 * n_experts + 1) * sizeof(int) + (logits ? 0 : (size_t)n_tokens * n_experts * sizeof(float));
+    const size_t logits_floats = (size_t)((long long)n_tokens * n_experts + 3) / 4 * 4;
+    const size_t smem = (size_t)((2 * n_experts + 1 + 3) / 4 * 4) * sizeof(int) +
+                        (logits ? 0 : logits_floats * sizeof(float) + (plan_on_tiles(n_tokens, n_experts, width) ? MOE_PLAN_THREADS / 32 * 128 * sizeof(float) : 0));
+    if (smem > 40 * 1024) {   // (the kernel has six KB of its own beside it)
+        cudaError_t e = cudaFuncSetAttribute(moe_plan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
     return (int)launch_pdl(moe_plan_kernel, dim3(1), dim3(MOE_PLAN_THREADS), smem, stream, logits, n_tokens, n_experts, top,
                            softmax_scores, renormalize, pair_expert, pair_weight, sorted_token, sorted_weight, dest, offsets,
                            tile_group, tile_row0, n_tiles, max_tiles, tile_rows, logits ? nullptr : x, router, width, x_is_bf16, bias,
