@@ -48,8 +48,7 @@ class ClampedGlu(FeedForward):
 
     def forward(self, x, ctx):
         act = torch.empty((x.shape[0], self.inter), dtype=x.dtype, device=x.device)
-        if not (self.limit > 0 and ops.gated_rows(x, self.gate_up_weight, act, clamp=(self.limit, self.alpha))):   # few rows: the gate in the product
-            ops.clamped_glu(ops.linear_rows(x, self.gate_up_weight), self.limit, self.alpha, act)
+        ops.clamped_glu(ops.linear_rows(x, self.gate_up_weight), self.limit, self.alpha, act)
         return ops.linear_rows(act, self.down_weight)
 
 
